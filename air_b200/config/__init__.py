@@ -3,6 +3,7 @@ from .bivizen_config import BivizenConfig
 from .tomodra_config import TomodraConfig
 from .pefivik_config import PefivikConfig
 from .tabopel_config import TabopelConfig
+from .dafotar_config import DafotarConfig
 from . import architectures  # registers the known architectures
 import json
 import os

@@ -6,6 +6,7 @@ from __future__ import annotations
 from ..parts.registry import register_architecture
 from ..parts.spec import BlockSpec, ModelSpec, PartSpec, RunStep
 from .bivizen_config import BivizenConfig
+from .dafotar_config import DafotarConfig
 from .model_config import Qwen2Config
 from .pefivik_config import PefivikConfig
 from .tabopel_config import TabopelConfig
@@ -266,3 +267,54 @@ def tabopel_spec(config: TabopelConfig) -> ModelSpec:
 
 
 register_architecture("Tabopel", TabopelConfig, tabopel_spec)
+
+
+def dafotar_spec(config: DafotarConfig) -> ModelSpec:
+    """Dafotar: several residual streams side by side, read, mixed and written by learned numbers per sub-layer
+    (hyper-connections), with layer norms that have a bias, and a causal convolution per channel whose output is added to
+    what a mixer reads.  The mixer is grouped-query attention inside a sliding window with normalised queries and keys, a
+    learned factor per head on the scores and values that are rotated by their position and turned back where they are
+    summed (a layer may read the keys and values that an earlier layer keeps), or mLSTM, a matrix memory with
+    exponential gates.  The feed-forward is a dense gated one with the rectifier.  The token table is the output matrix.
+    Tensors: embed, l<i>.norm1, norm1.b, norm2, norm2.b, hc1.{in,out,mix}, hc2.{in,out,mix}, canon1, l<i>.mix.*,
+    l<i>.mlp.*, final.norm, final.norm.b."""
+    e = config.width
+    norm = PartSpec("layer", {"size": e, "eps": config.eps, "tensor": "", "bias": ".b"})
+    # pages are kept as long as the widest window among the layers that read them needs them
+    keep = {}
+    for i, l in enumerate(config.layers):
+        if l.type == "attention":
+            keep.setdefault(i if l.kv_from is None else l.kv_from, []).append(l.window)
+    layers, order = [], []
+    for i, l in enumerate(config.layers):
+        if l.type == "attention":
+            def turned(dims):
+                return PartSpec("rope_live", {"rotary_dim": dims if l.rot_base else 0, "theta": l.rot_base or 1.0,
+                                              "pairing": "half"})
+            windows = keep[i if l.kv_from is None else l.kv_from]
+            mixer = PartSpec("normed_attention", {
+                "hidden": e, "heads": l.heads, "kv_heads": l.kv_heads, "head_dim": l.dim, "v_dim": l.vdim,
+                "scale": l.scale, "window": l.window, "eps": config.eps, "qk_norm": "head", "head_temp": True,
+                "position": turned(l.rot_dims), "value_position": turned(l.vdim), "borrows": l.kv_from is not None,
+                "keep": None if None in windows else max(windows)})
+        else:
+            mixer = PartSpec("mlstm", {"hidden": e, "heads": l.heads, "head_dim": l.dim, "v_dim": l.vdim,
+                                       "gate_cap": l.gate_cap, "eps": config.eps})
+        parts = {"mixer_norm": norm, "mixer": mixer}
+        names = {"mixer_norm": "norm1", "mixer": "mix.", "mixer_streams": "hc1.", "feed_forward_norm": "norm2",
+                 "feed_forward": "mlp.", "feed_forward_streams": "hc2.", "mixer_filter": "canon1"}
+        if config.taps:
+            parts["mixer_filter"] = PartSpec("residual_conv", {"size": e, "taps": config.taps})
+        if l.ff:
+            parts["feed_forward_norm"] = norm
+            parts["feed_forward"] = PartSpec("reglu", {"hidden": e, "intermediate": l.ff})
+        layers.append(BlockSpec(kind="streams", prefix=f"l{i}.", parts=parts, names=names,
+                                params={"streams": config.streams}))
+        order.append(RunStep(i, cache_from=l.kv_from))
+    return ModelSpec(
+        architecture=config.architecture, hidden_size=e, vocab_size=config.vocab, max_positions=config.max_positions,
+        layers=tuple(layers), order=tuple(order), final_norm=norm, embedding_name="embed", final_norm_prefix="final.norm",
+        output_name=None, eos_token_id=config.eos_token_id)
+
+
+register_architecture("Dafotar", DafotarConfig, dafotar_spec)

@@ -109,7 +109,15 @@ AIR_API int air_trace_set_attention_prepare(unsigned long long* buffer) { return
 //   the norm is taken over ALL heads of q at once (and all heads of k): x / sqrt(mean over H dk (x^2) + eps) * w with
 //   w of that whole size (q_w [H dk], k_w [G dk]).
 //
+//   q_scale [H] multiplies the heads of q behind norm and rotation (a factor per head on the scores).  v_freq [v_rot / 2]
+//   rotates the first v_rot elements of every head of v as well, in the same pairing, before it is written (no magnitude).
+//   Without write_kv proj holds q alone and nothing is written to the pages (a layer that reads another layer's keys).
+//
 // One block per token, one warp per head of q or k; a lane holds up to QKN_PAIRS pairs of its head.
+//
+// turn_heads_kernel  rotates the first `rot` elements of every head of x [T, H, n] by sign * position * freq[j], in place:
+//                    values that were rotated by their own positions and summed over positions are turned back by the
+//                    query's.
 namespace air {
 
 constexpr int QKN_PAIRS = 4;      // head sizes up to 64 * QKN_PAIRS
@@ -121,8 +129,9 @@ qk_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __
                          int pairing, float magnitude, const int* __restrict__ positions,
                          const int* __restrict__ token_seq, const int* __restrict__ block_table, int max_blocks,
                          TO* __restrict__ q_out, TO* __restrict__ cache, int H, int G, int dk, int dv, int P,
-                         int* status, const float* __restrict__ bias, int whole) {
-    __shared__ float cs[128], sn[128], scratch[32];
+                         int* status, const float* __restrict__ bias, int whole, const float* __restrict__ q_scale,
+                         const double* __restrict__ v_freq, int v_rot, int write_kv) {
+    __shared__ float cs[128], sn[128], vcs[128], vsn[128], scratch[32];
     pdl_enter(TR_QK_NORMED_PREPARE);
     const int t = blockIdx.x;
     const int slot = token_seq[t];
@@ -136,22 +145,33 @@ qk_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __
         cs[j] = (float)c * magnitude;
         sn[j] = (float)s * magnitude;
     }
-    const int page = block_table[(size_t)slot * max_blocks + pos / P];
+    const int vhalf = v_rot / 2;
+    if (write_kv)
+        for (int j = threadIdx.x; j < vhalf; j += blockDim.x) {
+            double s, c;
+            sincos((double)pos * v_freq[j], &s, &c);
+            vcs[j] = (float)c;
+            vsn[j] = (float)s;
+        }
     TO* kdst = nullptr;
     TO* vdst = nullptr;
-    if (page < 0) {
-        if (threadIdx.x == 0 && status) atomicExch(status, 2);
-    } else {
-        TO* base = cache + (size_t)page * G * P * (dk + dv);
-        kdst = base + (size_t)(pos % P) * dk;
-        vdst = base + (size_t)G * P * dk + (size_t)(pos % P) * dv;
+    if (write_kv) {
+        const int page = block_table[(size_t)slot * max_blocks + pos / P];
+        if (page < 0) {
+            if (threadIdx.x == 0 && status) atomicExch(status, 2);
+        } else {
+            TO* base = cache + (size_t)page * G * P * (dk + dv);
+            kdst = base + (size_t)(pos % P) * dk;
+            vdst = base + (size_t)G * P * dk + (size_t)(pos % P) * dv;
+        }
     }
+    const int heads = write_kv ? H + G : H;
     __syncthreads();
     float whole_q = 1.f, whole_k = 1.f;
     if (whole && q_w) {      // one scale for all heads of q and one for all heads of k
         // (four loads of a thread under way at once: the sums are a chain of latencies otherwise)
         float sq = 0.f, sk = 0.f;
-        const int n = (H + G) * dk, step = blockDim.x;
+        const int n = heads * dk, step = blockDim.x;
         for (int i0 = threadIdx.x; i0 < n; i0 += 4 * step) {
             float v[4];
 #pragma unroll
@@ -170,7 +190,7 @@ qk_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __
     }
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int pairs = dk / 2;
-    for (int head = warp; head < H + G; head += warps) {
+    for (int head = warp; head < heads; head += warps) {
         const float* x = in + (size_t)head * dk;
         const float* hb = bias ? bias + (size_t)head * dk : nullptr;
         const float* w = head < H ? q_w : k_w;
@@ -209,6 +229,10 @@ qk_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __
                 u = ru;
                 v = rv;
             }
+            if (q_scale && head < H) {
+                u *= q_scale[head];
+                v *= q_scale[head];
+            }
             if (dst) {
                 dst[ia[c]] = from_float<TO>(u);
                 dst[ib[c]] = from_float<TO>(v);
@@ -216,10 +240,49 @@ qk_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __
         }
     }
     const int vcol = (H + G) * dk;
-    if (vdst)
-        for (int idx = threadIdx.x; idx < G * dv; idx += blockDim.x)
-            vdst[(size_t)(idx / dv) * P * dv + idx % dv] =
-                from_float<TO>(in[vcol + idx] + (bias ? bias[vcol + idx] : 0.f));
+    if (!vdst) return;
+    // v: one item per pair of rotated elements and per element behind them
+    const int per_head = dv - vhalf;
+    for (int idx = threadIdx.x; idx < G * per_head; idx += blockDim.x) {
+        const int g = idx / per_head, j = idx % per_head;
+        const int i0 = j >= vhalf ? j + vhalf : pairing == 0 ? j : 2 * j, i1 = pairing == 0 ? i0 + vhalf : i0 + 1;
+        const int col = vcol + g * dv;
+        TO* dst = vdst + (size_t)g * P * dv;
+        const float a = in[col + i0] + (bias ? bias[col + i0] : 0.f);
+        if (j >= vhalf) {
+            dst[i0] = from_float<TO>(a);
+            continue;
+        }
+        const float b = in[col + i1] + (bias ? bias[col + i1] : 0.f);
+        dst[i0] = from_float<TO>(a * vcs[j] - b * vsn[j]);
+        dst[i1] = from_float<TO>(b * vcs[j] + a * vsn[j]);
+    }
+}
+
+template <typename TX>
+__global__ void __launch_bounds__(256)
+turn_heads_kernel(TX* __restrict__ x, const double* __restrict__ freq, int rot, int pairing, double sign,
+                  const int* __restrict__ positions, const int* __restrict__ token_seq, int H, int n) {
+    __shared__ float cs[128], sn[128];
+    pdl_enter(TR_TURN);
+    const int t = blockIdx.x;
+    if (token_seq[t] < 0) return;
+    const int half = rot / 2;
+    for (int j = threadIdx.x; j < half; j += blockDim.x) {
+        double s, c;
+        sincos(sign * (double)positions[t] * freq[j], &s, &c);
+        cs[j] = (float)c;
+        sn[j] = (float)s;
+    }
+    __syncthreads();
+    for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
+        const int h = idx / half, j = idx % half;
+        TX* row = x + ((size_t)t * H + h) * n;
+        const int i0 = pairing == 0 ? j : 2 * j, i1 = pairing == 0 ? j + half : 2 * j + 1;
+        const float a = to_float(row[i0]), b = to_float(row[i1]);
+        row[i0] = from_float<TX>(a * cs[j] - b * sn[j]);
+        row[i1] = from_float<TX>(b * cs[j] + a * sn[j]);
+    }
 }
 
 }  // namespace air
@@ -228,14 +291,25 @@ AIR_API int air_qk_normed_prepare(const float* proj, int ld, const float* q_w, c
                                   const double* freq, int rot, int pairing, float magnitude, const int* positions,
                                   const int* token_seq, const int* block_table, int max_blocks, void* q_out,
                                   void* cache, int out_dtype, int T, int H, int G, int dk, int dv, int P, int* status,
-                                  const float* bias, int whole, cudaStream_t stream) {
+                                  const float* bias, int whole, const float* q_scale, const double* v_freq, int v_rot,
+                                  int write_kv, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (v_rot < 0 || v_rot > dv || (v_rot & 1) || v_rot > 256 || (v_rot > 0 && !v_freq)) return AIR_ERR_BAD_ARGUMENT;
     if (rot < 0 || rot > dk || (rot & 1) || (dk & 1) || rot > 256 || dk > 64 * air::QKN_PAIRS || (rot > 0 && !freq) ||
-        pairing < 0 || pairing > 1 || (!q_w) != (!k_w))
+        pairing < 0 || pairing > 1 || (write_kv && (!q_w) != (!k_w)))
         return AIR_ERR_BAD_ARGUMENT;
     AIR_DISPATCH(out_dtype, TO, return air::launch(air::qk_normed_prepare_kernel<TO>, T, 256, 0, stream, proj, ld, q_w,
                                                    k_w, eps, freq, rot, pairing, magnitude, positions, token_seq,
                                                    block_table, max_blocks, (TO*)q_out, (TO*)cache, H, G, dk, dv, P,
-                                                   status, bias, whole));
+                                                   status, bias, whole, q_scale, v_freq, v_rot, write_kv));
+    return 0;
+}
+
+AIR_API int air_turn_heads(void* x, int dtype, const double* freq, int rot, int pairing, int back, const int* positions,
+                           const int* token_seq, int T, int H, int n, cudaStream_t stream) {
+    if (T <= 0 || rot == 0) return 0;
+    if (rot < 0 || rot > n || (rot & 1) || rot > 256 || !freq || pairing < 0 || pairing > 1) return AIR_ERR_BAD_ARGUMENT;
+    AIR_DISPATCH(dtype, TX, return air::launch(air::turn_heads_kernel<TX>, T, 256, 0, stream, (TX*)x, freq, rot, pairing,
+                                               back ? -1.0 : 1.0, positions, token_seq, H, n));
     return 0;
 }

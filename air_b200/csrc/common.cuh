@@ -46,7 +46,7 @@ enum TraceId { TR_EMBED = 1, TR_NORM, TR_ROPE, TR_SILU, TR_CONVERT, TR_TABLE, TR
                TR_ATT_PREFILL, TR_GEMM_F32, TR_GEMM_TC, TR_SAMPLE, TR_CONV, TR_SCAN, TR_GATED, TR_QKV_PREPARE,
                TR_GLU, TR_SCALED_NORM, TR_POST_NORM, TR_QK_NORMED_PREPARE, TR_LATENT_PREPARE, TR_MOE_ROUTE, TR_MOE_SORT,
                TR_GROUPED_GEMM, TR_GATHER_KEYS, TR_MASKED_SOFTMAX, TR_ATT_GROUPED, TR_POLYNORM, TR_STREAM_ADD,
-               TR_HEAD_GATE, TR_SANDWICH_NORM, TR_RELU2 };
+               TR_HEAD_GATE, TR_SANDWICH_NORM, TR_RELU2, TR_STREAM_NORM, TR_RESIDUAL_CONV, TR_MLSTM, TR_TURN };
 
 __device__ __forceinline__ void pdl_enter(int id = 0) {
     pdl_trigger();
@@ -117,6 +117,18 @@ __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
     return v;
+}
+
+// The gated activation of a feed-forward: g' * sigmoid(alpha * g') * (u' + shift) with g' = min(g, limit) and
+// u' = clamp(u, -limit, limit) where limit > 0; with alpha < 0 the rectifier stands in the sigmoid form's place:
+// max(g', 0) * (u' + shift).
+__device__ __forceinline__ float gated_activation(float g, float u, float alpha, float limit, float shift) {
+    if (limit > 0.f) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+    }
+    if (alpha < 0.f) return fmaxf(g, 0.f) * (u + shift);
+    return g / (1.f + expf(-alpha * g)) * (u + shift);
 }
 
 // Sum over a block of up to 1024 threads; every thread gets the result.  The order of

@@ -723,10 +723,14 @@ __global__ void qkv_rope_store_vec4_many_kernel(const TI* __restrict__ qkv, int 
     }
 }
 
-// ---------------------------------------------------------------- SiLU(gate) * up
+// ---------------------------------------------------------------- SiLU(gate) * up, or (RELU) max(gate, 0) * up
 // in [T, 2I]: blocks of `block` gate columns and `block` up columns in turn (block = I: all gate
 // columns, then all up columns).  out [T, I].
-template <typename TI, typename TO>
+template <bool RELU> __device__ __forceinline__ float glu_gate(float g) {
+    return RELU ? fmaxf(g, 0.f) : g / (1.f + expf(-g));
+}
+
+template <typename TI, typename TO, bool RELU>
 __global__ void silu_mul_kernel(const TI* __restrict__ in, TO* __restrict__ out, int I, int block, size_t total) {
     pdl_enter(TR_SILU);
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -736,11 +740,11 @@ __global__ void silu_mul_kernel(const TI* __restrict__ in, TO* __restrict__ out,
         const size_t at = t * 2 * I + (size_t)(i / block) * 2 * block + i % block;
         const float g = to_float(in[at]);
         const float u = to_float(in[at + block]);
-        out[idx] = from_float<TO>(g / (1.f + expf(-g)) * u);
+        out[idx] = from_float<TO>(glu_gate<RELU>(g) * u);
     }
 }
 
-template <typename TI, typename TO>
+template <typename TI, typename TO, bool RELU>
 __global__ void silu_mul_vec4_kernel(const TI* __restrict__ in, TO* __restrict__ out, int I, int block,
                                      size_t total4) {
     pdl_enter(TR_SILU);
@@ -754,12 +758,13 @@ __global__ void silu_mul_vec4_kernel(const TI* __restrict__ in, TO* __restrict__
         load4(in + at, g);
         load4(in + at + block, u);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) y[e] = g[e] / (1.f + expf(-g[e])) * u[e];
+        for (int e = 0; e < 4; ++e) y[e] = glu_gate<RELU>(g[e]) * u[e];
         store4(out + t * I + i, y);
     }
 }
 
 // Eight bfloat16 at a time (16-byte accesses), for I % 8 == 0 and block % 8 == 0.
+template <bool RELU>
 __global__ void __launch_bounds__(256, 4) silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ in,
                                                                  __nv_bfloat16* __restrict__ out, int I, int block,
                                                                  size_t total8) {
@@ -800,8 +805,11 @@ __global__ void __launch_bounds__(256, 4) silu_mul_bf16x8_kernel(const __nv_bflo
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const float2 g = __bfloat1622float2(g2[e]), u = __bfloat1622float2(u2[e]);
-                    o2[e] = __floats2bfloat162_rn(__fdividef(g.x, 1.f + __expf(-g.x)) * u.x,
-                                                  __fdividef(g.y, 1.f + __expf(-g.y)) * u.y);
+                    if (RELU)
+                        o2[e] = __floats2bfloat162_rn(fmaxf(g.x, 0.f) * u.x, fmaxf(g.y, 0.f) * u.y);
+                    else
+                        o2[e] = __floats2bfloat162_rn(__fdividef(g.x, 1.f + __expf(-g.x)) * u.x,
+                                                      __fdividef(g.y, 1.f + __expf(-g.y)) * u.y);
                 }
                 *reinterpret_cast<uint4*>(out + to[k]) = ov;
             }
@@ -965,29 +973,37 @@ AIR_API int air_qkv_rope_store(const void* qkv, int in_dtype, int parts, const v
     return (int)cudaGetLastError();
 }
 
-AIR_API int air_silu_mul(const void* in, int in_dtype, void* out, int out_dtype, int T, int I, int block,
-                         cudaStream_t stream) {
+template <bool RELU>
+static int launch_silu_mul(const void* in, int in_dtype, void* out, int out_dtype, int T, int I, int block,
+                           cudaStream_t stream) {
     const size_t total = (size_t)T * I;
-    if (total == 0) return 0;
-    if (block <= 0 || I % block) return AIR_ERR_BAD_ARGUMENT;
     if (in_dtype == AIR_BF16 && out_dtype == AIR_BF16 && I % 8 == 0 && block % 8 == 0) {
         const size_t n = total / 8;
         const size_t want = (n + 511) / 512;               // 256 threads, two groups each
         const int blocks = (int)(want < 148 * 32 ? want : 148 * 32);
-        return launch(silu_mul_bf16x8_kernel, blocks, 256, 0, stream, (const __nv_bfloat16*)in, (__nv_bfloat16*)out, I,
-                      block, n);
+        return launch(silu_mul_bf16x8_kernel<RELU>, blocks, 256, 0, stream, (const __nv_bfloat16*)in,
+                      (__nv_bfloat16*)out, I, block, n);
     }
     AIR_DISPATCH(in_dtype, TI, AIR_DISPATCH(out_dtype, TO, {
         if (I % 4 == 0 && block % 4 == 0) {
             const size_t n = total / 4;
             const int blocks = (int)((n + 255) / 256 < 148 * 32 ? (n + 255) / 256 : 148 * 32);
-            return launch(silu_mul_vec4_kernel<TI, TO>, blocks, 256, 0, stream, (const TI*)in, (TO*)out, I, block, n);
+            return launch(silu_mul_vec4_kernel<TI, TO, RELU>, blocks, 256, 0, stream, (const TI*)in, (TO*)out, I, block, n);
         } else {
             const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-            return launch(silu_mul_kernel<TI, TO>, blocks, 256, 0, stream, (const TI*)in, (TO*)out, I, block, total);
+            return launch(silu_mul_kernel<TI, TO, RELU>, blocks, 256, 0, stream, (const TI*)in, (TO*)out, I, block, total);
         }
     }));
     return (int)cudaGetLastError();
+}
+
+// relu: max(gate, 0) * up instead of SiLU(gate) * up
+AIR_API int air_silu_mul(const void* in, int in_dtype, void* out, int out_dtype, int T, int I, int block, int relu,
+                         cudaStream_t stream) {
+    if (T <= 0 || I <= 0) return 0;
+    if (block <= 0 || I % block) return AIR_ERR_BAD_ARGUMENT;
+    return relu ? launch_silu_mul<true>(in, in_dtype, out, out_dtype, T, I, block, stream)
+                : launch_silu_mul<false>(in, in_dtype, out, out_dtype, T, I, block, stream);
 }
 
 AIR_API int air_convert(const void* in, int in_dtype, void* out, int out_dtype, long long n,

@@ -50,7 +50,7 @@ struct TcArgs {
     int prefetch;       // further k-tiles of W that a block asks into L2 before its predecessor has ended
     int* status;
     // EPI_SILU computes g' * sigmoid(act_alpha * g') * (u' + act_shift) with g' = min(gate, act_limit) and
-    // u' = clamp(up, -act_limit, act_limit) where act_limit > 0: (1, 0, 0) is SiLU(gate) * up.
+    // u' = clamp(up, -act_limit, act_limit) where act_limit > 0: (1, 0, 0) is SiLU(gate) * up; act_alpha < 0: max(g', 0) * (u' + act_shift).
     float act_alpha, act_limit, act_shift;
 };
 
@@ -239,12 +239,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 float y[8];
 #pragma unroll
                                 for (int e = 0; e < 8; ++e) {
-                                    float g = __uint_as_float(gate[j + e]), u = __uint_as_float(up[j + e]);
-                                    if (args.act_limit > 0.f) {
-                                        g = fminf(g, args.act_limit);
-                                        u = fminf(fmaxf(u, -args.act_limit), args.act_limit);
-                                    }
-                                    y[e] = g / (1.f + expf(-args.act_alpha * g)) * (u + args.act_shift);
+                                    y[e] = gated_activation(__uint_as_float(gate[j + e]), __uint_as_float(up[j + e]),
+                                                            args.act_alpha, args.act_limit, args.act_shift);
                                 }
                                 store4(out + c + j, *(const float(*)[4])&y[0]);
                                 store4(out + c + j + 4, *(const float(*)[4])&y[4]);

@@ -44,7 +44,7 @@ struct TsArgs {
     int ss_tiles;
     float eps;
     // SILU computes g' * sigmoid(act_alpha * g') * (u' + act_shift) with g' = min(gate, act_limit) and
-    // u' = clamp(up, -act_limit, act_limit) where act_limit > 0: (1, 0, 0) is SiLU(gate) * up.
+    // u' = clamp(up, -act_limit, act_limit) where act_limit > 0: (1, 0, 0) is SiLU(gate) * up; act_alpha < 0: max(g', 0) * (u' + act_shift).
     float act_alpha, act_limit, act_shift;
 };
 
@@ -246,13 +246,8 @@ gemm_tc_small_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_con
 #pragma unroll
                     for (int t = 0; t < NT; ++t)
                         if (t < args.T) {
-                            float g = gate[t], u = up[t];
-                            if (args.act_limit > 0.f) {
-                                g = fminf(g, args.act_limit);
-                                u = fminf(fmaxf(u, -args.act_limit), args.act_limit);
-                            }
-                            out[(size_t)t * (args.N / 2)] =
-                                __float2bfloat16_rn(g / (1.f + expf(-args.act_alpha * g)) * (u + args.act_shift));
+                            out[(size_t)t * (args.N / 2)] = __float2bfloat16_rn(
+                                gated_activation(gate[t], up[t], args.act_alpha, args.act_limit, args.act_shift));
                         }
                 }
             } else {

@@ -39,7 +39,16 @@ _SIGNATURES = {
                       c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "air_qk_normed_prepare": [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_float, c_void_p,
                               c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                              c_int, c_void_p, c_void_p, c_int, c_void_p],
+                              c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
+    "air_turn_heads": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "air_stream_norm": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_void_p, c_void_p,
+                        c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float,
+                        c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+    "air_residual_conv": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                          c_void_p],
+    "air_mlstm_step": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                       c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                       c_float, c_float, c_void_p],
     "air_latent_prepare": [c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                            c_void_p, c_void_p],
@@ -140,7 +149,7 @@ TRACE_NAMES = {1: "embedding", 2: "add_rmsnorm", 3: "qkv_rope_store", 4: "silu_m
                12: "gemm_tc", 13: "sample", 14: "short_conv", 15: "linear_scan", 16: "gated_rmsnorm",
                17: "qkv_prepare", 18: "glu", 19: "scaled_norm", 20: "post_norm", 21: "qk_normed_prepare",
                22: "latent_prepare", 23: "moe_route", 24: "moe_sort", 25: "grouped_gemm", 26: "gather_keys", 27: "masked_softmax", 28: "grouped_attention", 29: "polynorm", 30: "stream_add", 31: "head_gate",
-               32: "normed_add_norm", 33: "relu2"}
+               32: "normed_add_norm", 33: "relu2", 34: "stream_norm", 35: "residual_conv", 36: "mlstm", 37: "turn_heads"}
 
 
 def set_trace(buffer: Optional[torch.Tensor]) -> None:
@@ -365,9 +374,9 @@ def qkv_rope_store(qkv, bias, table, positions, token_seq, block_table, q_out, c
     return q_out
 
 
-def silu_mul(gate_up, out, block=None):
+def silu_mul(gate_up, out, block=None, relu=False):
     """out[t, i] = silu(gate[t, i]) * up[t, i], where gate_up [T, 2I] holds blocks of `block` gate
-    columns and `block` up columns in turn (default: all gate columns, then all up columns)."""
+    columns and `block` up columns in turn (default: all gate columns, then all up columns); relu: max(gate, 0) * up."""
     T, I = out.shape
     block = I if block is None else block
     if block <= 0 or I % block:
@@ -375,7 +384,7 @@ def silu_mul(gate_up, out, block=None):
     _req(gate_up, "gate_up", _FLOATS, (T, 2 * I))
     _req(out, "out", _FLOATS)
     _check(_get("air_silu_mul")(gate_up.data_ptr(), _DT[gate_up.dtype], out.data_ptr(), _DT[out.dtype], T, I,
-                                block, _stream()), "silu_mul")
+                                block, 1 if relu else 0, _stream()), "silu_mul")
     return out
 
 
@@ -573,23 +582,32 @@ def post_norm(h, alpha, a, b, b_row_scale, weight, eps, out):
 
 
 def qk_normed_prepare(proj, q_weight, k_weight, eps, freq, pairing, magnitude, positions, token_seq, block_table, q_out,
-                      cache, kv_heads, v_dim, page_tokens, status=None, bias=None, whole=False):
+                      cache, kv_heads, v_dim, page_tokens, status=None, bias=None, whole=False, q_scale=None, v_freq=None,
+                      write_kv=True):
     """From the fused projection proj (float32 [T, (H + G) dk + G dv]: q, k, v per token) to q_out [T, H, dk] and
     the pages (keys [G, P, dk], then values [G, P, dv]).  q and k heads are normalised (x / sqrt(mean(x^2) + eps) * w,
     w float32 [dk]: q_weight for q, k_weight for k; None: no norm), then their first 2 * len(freq) elements are
     rotated by position * freq[j] (freq float64), pair j = (2j, 2j + 1) where pairing == "neighbours", (j, j + rot/2)
     where "half"; cos and sin are multiplied by magnitude.  bias (float32 [W]) is added to q, k and v first.  whole: the
     norm is taken over all heads of q at once (and over all heads of k), with weights [H * dk] and [G * dk].  proj may be
-    a band of columns of a wider matrix."""
+    a band of columns of a wider matrix.  q_scale (float32 [H]) multiplies the finished heads of q.  v_freq (float64): the
+    first 2 * len(v_freq) elements of every head of v are rotated too before they are written, in the same pairing.
+    write_kv False: proj is q alone [T, H dk], and nothing is written to the pages."""
     T, H, dk = q_out.shape
     G, dv, P = int(kv_heads), int(v_dim), int(page_tokens)
-    W = (H + G) * dk + G * dv
+    W = (H + G) * dk + G * dv if write_kv else H * dk
     pp, ld = _columns(proj, "proj")
     if tuple(proj.shape) != (T, W):
         raise KernelError(f"qk_normed_prepare: proj {tuple(proj.shape)}, wanted {(T, W)}")
     for name, w, heads in (("q_weight", q_weight, H), ("k_weight", k_weight, G)):
         if w is not None:
             _req(w, name, (torch.float32,), (heads * dk if whole else dk,))
+    if q_scale is not None:
+        _req(q_scale, "q_scale", (torch.float32,), (H,))
+    v_rot = 0
+    if v_freq is not None:
+        _req(v_freq, "v_freq", (torch.float64,))
+        v_rot = 2 * v_freq.numel()
     if bias is not None:
         _req(bias, "bias", (torch.float32,), (W,))
     rot = 0
@@ -609,8 +627,122 @@ def qk_normed_prepare(proj, q_weight, k_weight, eps, freq, pairing, magnitude, p
         pp, ld, _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(freq), rot,
         1 if pairing == "neighbours" else 0, float(magnitude), positions.data_ptr(), token_seq.data_ptr(),
         block_table.data_ptr(), block_table.shape[1], q_out.data_ptr(), cache.data_ptr(), _DT[q_out.dtype], T, H, G, dk,
-        dv, P, _ptr(status), _ptr(bias), 1 if whole else 0, _stream()), "qk_normed_prepare")
+        dv, P, _ptr(status), _ptr(bias), 1 if whole else 0, _ptr(q_scale), _ptr(v_freq), v_rot, 1 if write_kv else 0,
+        _stream()), "qk_normed_prepare")
     return q_out
+
+
+def turn_heads(x, freq, pairing, positions, token_seq, back=False):
+    """x [T, H, n] in place: the first 2 * len(freq) elements of every head are rotated by positions[t] * freq[j] (freq
+    float64; pair j = (j, j + rot/2) where pairing is "half", (2j, 2j + 1) where "neighbours"), backwards with back."""
+    T, H, n = x.shape
+    _req(x, "x", _FLOATS)
+    _req(freq, "freq", (torch.float64,))
+    _req(positions, "positions", _I32, (T,))
+    _req(token_seq, "token_seq", _I32, (T,))
+    _check(_get("air_turn_heads")(x.data_ptr(), _DT[x.dtype], freq.data_ptr(), 2 * freq.numel(),
+                                  1 if pairing == "neighbours" else 0, 1 if back else 0, positions.data_ptr(),
+                                  token_seq.data_ptr(), T, H, n, _stream()), "turn_heads")
+    return x
+
+
+STREAMS_MAX = 16
+
+
+def stream_norm(h, streams, weight, bias, eps, out, term=None, mix=None, out_weights=None, read=None, h_out=None, rows=None,
+                center=True, conv=None):
+    """Residual streams x_0 .. x_(S-1): h float32 [S, T, E], or [T, E] where all streams are still equal (or S = 1).
+    x'_t = sum_s mix[s, t] x_s + out_weights[t] * term (mix None: x_t; term None: nothing is added; term [T, E] or partial
+    sums [parts, T, E]); written to h_out [S, T, E] (which may be h) where given.  u = sum_t read[t] x'_t (read None: the
+    plain sum); out = norm(u) * weight + bias with norm(u) = (u - mean) / sqrt(var + eps), or u / sqrt(mean(u^2) + eps)
+    without center; bias may be None; weight None (and out None): only the streams are completed.  rows: out[r] is that of
+    row rows[r].  conv = (weight [taps, E], state [slots, taps - 1, E] or None, token_seq [T]): every row is its request's
+    only token of the step, and a causal convolution over time is added to the row (see residual_conv)."""
+    S, E = int(streams), h.shape[-1]
+    T = h.shape[-2]
+    _req(h, "h", (torch.float32,), (T, E) if h.dim() == 2 else (S, T, E))
+    if h_out is not None:
+        _req(h_out, "h_out", (torch.float32,), (T, E) if S == 1 and h_out.dim() == 2 else (S, T, E))
+        if rows is not None:
+            raise KernelError("stream_norm: chosen rows are read only")
+        if h_out.data_ptr() == h.data_ptr() and h_out.dim() != h.dim():
+            raise KernelError("stream_norm: equal streams that are one tensor cannot be completed in place")
+    parts = 1
+    if term is not None:
+        parts = 1 if term.dim() == 2 else term.shape[0]
+        _req(term, "term", (torch.float32,), (T, E) if term.dim() == 2 else (parts, T, E))
+    for name, v, shape in (("mix", mix, (S, S)), ("out_weights", out_weights, (S,)), ("read", read, (S,)),
+                           ("weight", weight, (E,)), ("bias", bias, (E,))):
+        if v is not None:
+            _req(v, name, (torch.float32,), shape)
+    R = T if rows is None else rows.shape[0]
+    if rows is not None:
+        _req(rows, "rows", _I32)
+    if weight is not None:
+        _req(out, "out", _FLOATS, (R, E))
+    cw = cs = ct = None
+    taps = 0
+    if conv is not None:
+        cw, cs, ct = conv
+        taps = cw.shape[0]
+        _req(cw, "conv weight", (torch.float32,), (taps, E))
+        if taps > 1:
+            _req(cs, "conv state", (torch.float32,), (None, taps - 1, E))
+        _req(ct, "token_seq", _I32, (T,))
+    _check(_get("air_stream_norm")(
+        h.data_ptr(), 0 if h.dim() == 2 else T * E, _ptr(h_out), T * E, _ptr(term), parts, T * E, _ptr(mix),
+        _ptr(out_weights), _ptr(read), S, _ptr(weight), _ptr(bias), _ptr(out) if weight is not None else None,
+        _DT[out.dtype] if weight is not None else 0, _ptr(rows), R, E, 1 if center else 0, float(eps), _ptr(cw),
+        _ptr(cs) if taps > 1 else None, _ptr(ct), taps, _stream()), "stream_norm")
+    return out
+
+
+def residual_conv(h, weight, state, out, q_start, slots, max_tokens):
+    """out[t] = h[t] + sum_j weight[j] * h[t - taps + 1 + j] over the tokens of every entry of the batch (rows q_start[e] ..
+    q_start[e + 1], state row slots[e]), channel by channel; inputs before the portion come from state
+    [slots, taps - 1, E] (oldest first; zeros at a request's start), whose place the portion's last inputs take.
+    h float32 [T, E]; weight float32 [taps, E]; out [T, E]; max_tokens: the longest portion (it sizes the grid)."""
+    T, E = h.shape
+    taps = weight.shape[0]
+    _req(h, "h", (torch.float32,))
+    _req(weight, "weight", (torch.float32,), (taps, E))
+    if taps > 1:
+        _req(state, "state", (torch.float32,), (None, taps - 1, E))
+    _req(out, "out", _FLOATS, (T, E))
+    _req(q_start, "q_start", _I32)
+    _req(slots, "slots", _I32)
+    _check(_get("air_residual_conv")(h.data_ptr(), weight.data_ptr(), _ptr(state) if taps > 1 else None, out.data_ptr(),
+                                     _DT[out.dtype], q_start.data_ptr(), slots.data_ptr(), slots.shape[0], E, taps,
+                                     int(max_tokens), _stream()), "residual_conv")
+    return out
+
+
+def mlstm_step(proj, columns, i_bias, f_bias, weight, S, n, m, out, q_start, slots, cap, q_scale, eps):
+    """mLSTM's matrix memory (see mlstm.cu) for every entry of the batch, token after token, one block per head and
+    entry.  proj float32 [T, W]; columns: where q, k, v, g (the heads side by side), i and f (a logit per head) start in it;
+    i_bias, f_bias float32 [H]; weight float32 [H * dv]; the states S [slots, H, d, dv], n [slots, H, d], m [slots, H];
+    out [T, H * dv]: every head's read-out normalised, weighted and gated."""
+    slots_n, H, d, dv = S.shape
+    T = out.shape[0]
+    pp, ld = _columns(proj, "proj")
+    need = {"q": H * d, "k": H * d, "v": H * dv, "g": H * dv, "i": H, "f": H}
+    for c, width in need.items():
+        if columns[c] + width > proj.shape[1]:
+            raise KernelError(f"mlstm_step: projection {c} does not fit")
+    _req(i_bias, "i_bias", (torch.float32,), (H,))
+    _req(f_bias, "f_bias", (torch.float32,), (H,))
+    _req(weight, "weight", (torch.float32,), (H * dv,))
+    _req(S, "S", (torch.float32,))
+    _req(n, "n", (torch.float32,), (slots_n, H, d))
+    _req(m, "m", (torch.float32,), (slots_n, H))
+    _req(out, "out", _FLOATS, (proj.shape[0], H * dv))
+    _req(q_start, "q_start", _I32)
+    _req(slots, "slots", _I32)
+    _check(_get("air_mlstm_step")(
+        pp, ld, *(int(columns[c]) for c in "qkvgif"), i_bias.data_ptr(), f_bias.data_ptr(), weight.data_ptr(), S.data_ptr(),
+        n.data_ptr(), m.data_ptr(), out.data_ptr(), _DT[out.dtype], q_start.data_ptr(), slots.data_ptr(), slots.shape[0],
+        H, d, dv, float(cap), float(q_scale), float(eps), _stream()), "mlstm_step")
+    return out
 
 
 def latent_prepare(proj, c_weight, eps, freq, positions, token_seq, block_table, q_plain, q_full, cache, owns,
@@ -1256,6 +1388,7 @@ EPI_F32, EPI_BF16, EPI_SILU, EPI_PARTIAL, EPI_RELU2 = 0, 1, 2, 3, 4
 
 
 SILU = (1.0, 0.0, 0.0)      # the gated activation of EPI_SILU as (alpha, limit, shift): see gemm_tc
+RELU = (-1.0, 0.0, 0.0)     # max(gate, 0) * up
 
 
 def gemm_tc(a, w, out, bn, epi, splits=1, status=None, max_blocks=0, force_rows_as_m=False, row_ss=None, eps=0.0,
@@ -1266,7 +1399,8 @@ def gemm_tc(a, w, out, bn, epi, splits=1, status=None, max_blocks=0, force_rows_
     add_prenorm).
     epi EPI_F32: out float32 [M,N]; EPI_BF16: out bfloat16 [M,N]; EPI_SILU: w holds gate and up rows
     interleaved in blocks of bn/2, out bfloat16 [M,N/2] = silu(gate)*up, or with act = (alpha, limit, shift)
-    g * sigmoid(alpha * g) * (u + shift) where g = min(gate, limit), u = clamp(up, -limit, limit) if limit > 0;
+    g * sigmoid(alpha * g) * (u + shift) where g = min(gate, limit), u = clamp(up, -limit, limit) if limit > 0
+    (alpha < 0: max(g, 0) * (u + shift));
     EPI_RELU2: out bfloat16 [M,N] = max(product, 0)^2; EPI_PARTIAL: out float32
     [splits,M,N] partial sums over parts of k.  With up to 64 rows and bn 128 or 256 the product runs with the
     weights as the M side of the instruction (gemm_tc_small.cu) unless force_rows_as_m."""

@@ -1,0 +1,295 @@
+// Row-wise operations of layers that carry several residual streams side by side (hyper-connections), of layer norms with
+// a bias, and of a convolution over time that is added to its own input.
+//
+//   stream_norm_kernel    with the streams x_0 .. x_(S-1) [T, E] (S = 1: an ordinary residual stream) and the output y of
+//                         the sub-layer before (float32 [T, E], or the partial sums [parts, T, E] of a split product, added
+//                         in order):
+//                           x'_t = sum_s mix[s, t] x_s + out_t y     (without mix: x_t; without out: y as it is)
+//                           u    = sum_t read_t x'_t                 (without read: the plain sum)
+//                           row  = norm(u) * w + b
+//                         where norm is (u - mean) / sqrt(var + eps), var the mean of the squared deviations, or (center 0)
+//                         u / sqrt(mean(u^2) + eps), and b may be absent.  x' is written when h_out is given; with `rows` the
+//                         kernel reads row rows[r] of everything and writes row r.  The streams may all be one tensor
+//                         (stream stride 0: they start out equal).  Everything is 32-bit; the row is written in its own type.
+//                         With conv (a step in which every row is its request's only token) the row becomes
+//                         row + sum_j cw[j] in_(t - taps + 1 + j) before it is written, the earlier inputs coming from
+//                         the request's state, which is moved on by one token.
+//   residual_conv_kernel  y_t = h_t + sum_j cw[j] h_(t - taps + 1 + j) over the tokens of each entry of the batch: the same
+//                         convolution for portions of any length.
+//
+// cw is [taps, E] (the last row multiplies the token itself), the state [slots, taps - 1, E], oldest input first, zeros at
+// a request's start.
+#include "common.cuh"
+
+namespace air {
+
+struct StreamNormArgs {
+    const float* x; size_t x_stride;       // stream s at x + s * x_stride
+    float* h_out; size_t h_stride;         // may be x itself (a thread reads its columns of all streams before it writes)
+    const float* y; int y_parts; size_t part_stride;
+    const float* mix;                      // [S, S], from row s to column t
+    const float* out_w;                    // [S]
+    const float* read;                     // [S]
+    const float* w; const float* b;        // [E]
+    void* out;
+    const int* rows;
+    const float* conv_w; float* conv_state; const int* token_seq; int taps;
+    int S, E, center;
+    float eps;
+};
+
+constexpr int STREAMS_MAX = 16;
+
+// N columns of all streams of a row: mixed, written, and folded into u.  NS: the number of streams (0: p.S of them).
+template <int NS, int N>
+__device__ __forceinline__ void stream_columns(const StreamNormArgs& p, size_t src, int i, const float* coef, float (&u)[N]) {
+    constexpr int M = NS ? NS : STREAMS_MAX;
+    const int S = NS ? NS : p.S;
+    auto ld = [](const float* q, float (&v)[N]) {
+        if constexpr (N == 4) load4(q, v);
+        else v[0] = *q;
+    };
+    auto st = [](float* q, const float (&v)[N]) {
+        if constexpr (N == 4) store4(q, v);
+        else *q = v[0];
+    };
+    float x[M][N], y[N];
+#pragma unroll
+    for (int s = 0; s < M; ++s)
+        if (s < S) {
+            if (s == 0 || p.x_stride) ld(p.x + s * p.x_stride + src + i, x[s]);
+            else {
+#pragma unroll
+                for (int j = 0; j < N; ++j) x[s][j] = x[0][j];
+            }
+        }
+    if (p.y) {
+        ld(p.y + src + i, y);
+#pragma unroll 4
+        for (int q = 1; q < p.y_parts; ++q) {
+            float t[N];
+            ld(p.y + q * p.part_stride + src + i, t);
+#pragma unroll
+            for (int j = 0; j < N; ++j) y[j] += t[j];
+        }
+    }
+    const float *mix = coef, *out_w = coef + S * S, *read = out_w + S;
+#pragma unroll
+    for (int j = 0; j < N; ++j) u[j] = 0.f;
+#pragma unroll
+    for (int t = 0; t < M; ++t) {
+        if (t >= S) break;
+        float v[N];
+        if (p.mix) {
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[j] = 0.f;
+#pragma unroll
+            for (int s = 0; s < M; ++s)
+                if (s < S) {
+                    const float m = mix[s * S + t];
+#pragma unroll
+                    for (int j = 0; j < N; ++j) v[j] = fmaf(m, x[s][j], v[j]);
+                }
+        } else {
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[j] = x[t][j];
+        }
+        if (p.y) {
+            const float o = out_w[t];
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[j] = fmaf(o, y[j], v[j]);
+        }
+        if (p.h_out) st(p.h_out + t * p.h_stride + src + i, v);
+        const float r = read[t];
+#pragma unroll
+        for (int j = 0; j < N; ++j) u[j] = fmaf(r, v[j], u[j]);
+    }
+}
+
+template <typename TO, int NS, int N>
+__global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormArgs p) {
+    __shared__ float scratch[32];
+    __shared__ float coef[STREAMS_MAX * STREAMS_MAX + 2 * STREAMS_MAX];
+    extern __shared__ __align__(16) float urow[];
+    pdl_enter(TR_STREAM_NORM);
+    const int r = blockIdx.x, E = p.E, S = NS ? NS : p.S;
+    const size_t src = (size_t)(p.rows ? p.rows[r] : r) * E;
+    for (int i = threadIdx.x; i < S * S + 2 * S; i += blockDim.x) {
+        const int k = i - S * S;
+        coef[i] = k < 0 ? (p.mix ? p.mix[i] : 0.f) : k < S ? (p.out_w ? p.out_w[k] : 1.f) : (p.read ? p.read[k - S] : 1.f);
+    }
+    __syncthreads();
+    float sum = 0.f;
+    const int step = blockDim.x * N;
+    for (int i = threadIdx.x * N; i < E; i += step) {
+        float u[N];
+        stream_columns<NS, N>(p, src, i, coef, u);
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+            urow[i + j] = u[j];
+            sum += p.center ? u[j] : u[j] * u[j];
+        }
+    }
+    if (!p.w) return;
+    float mean = 0.f, var;
+    if (p.center) {
+        mean = block_sum(sum, scratch) / (float)E;
+        sum = 0.f;
+        for (int i = threadIdx.x * N; i < E; i += step)
+#pragma unroll
+            for (int j = 0; j < N; ++j) {
+                const float d = urow[i + j] - mean;
+                sum = fmaf(d, d, sum);
+            }
+    }
+    var = block_sum(sum, scratch) / (float)E;
+    const float scale = 1.f / sqrtf(var + p.eps);
+    TO* out = (TO*)p.out + (size_t)r * E;
+    const int slot = p.conv_w ? p.token_seq[r] : -1;
+    for (int i = threadIdx.x * N; i < E; i += step) {
+        float v[N], wv[N], bv[N];
+        if constexpr (N == 4) load4(p.w + i, wv);
+        else wv[0] = p.w[i];
+        if (p.b) {
+            if constexpr (N == 4) load4(p.b + i, bv);
+            else bv[0] = p.b[i];
+        }
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+            v[j] = (urow[i + j] - mean) * scale * wv[j];
+            if (p.b) v[j] += bv[j];
+        }
+        if (slot >= 0) {
+            const int keep = p.taps - 1;
+            float* st = p.conv_state + (size_t)slot * keep * E + i;
+            float acc[N];
+#pragma unroll
+            for (int j = 0; j < N; ++j) acc[j] = v[j];
+            for (int k = 0; k <= keep; ++k) {
+#pragma unroll
+                for (int j = 0; j < N; ++j) {
+                    const float in = k < keep ? st[(size_t)k * E + j] : v[j];
+                    acc[j] = fmaf(p.conv_w[(size_t)k * E + i + j], in, acc[j]);
+                    if (k > 0) st[(size_t)(k - 1) * E + j] = in;
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[j] = acc[j];
+        }
+        if constexpr (N == 4) store4(out + i, v);
+        else out[i] = from_float<TO>(v[0]);
+    }
+}
+
+// grid (column blocks, entries, chunks of `chunk` tokens, at least taps - 1); a thread takes N columns.  The thread of a
+// column in an entry's first chunk is the only one that reads or writes that column's state.
+template <typename TO, int N>
+__global__ void __launch_bounds__(128)
+residual_conv_kernel(const float* __restrict__ h, const float* __restrict__ w, float* __restrict__ state,
+                     TO* __restrict__ y, const int* __restrict__ q_start, const int* __restrict__ slots, int E, int taps,
+                     int chunk) {
+    pdl_enter(TR_RESIDUAL_CONV);
+    const int i = (blockIdx.x * 128 + threadIdx.x) * N, e = blockIdx.y;
+    const int slot = slots[e];
+    if (i >= E || slot < 0) return;
+    const int q0 = q_start[e], n = q_start[e + 1] - q0, keep = taps - 1;
+    const int t0 = blockIdx.z * chunk, t1 = min(n, t0 + chunk);
+    if (t0 >= n) return;
+    auto ld = [](const float* q, float (&v)[N]) {
+        if constexpr (N == 4) load4(q, v);
+        else v[0] = *q;
+    };
+    const float* in = h + (size_t)q0 * E + i;
+    float* st = state + (size_t)slot * keep * E + i;
+    for (int t = t0; t < t1; ++t) {
+        float cur[N], acc[N], v[N], wv[N];
+        ld(in + (size_t)t * E, cur);
+        ld(w + (size_t)keep * E + i, wv);
+#pragma unroll
+        for (int j = 0; j < N; ++j) acc[j] = fmaf(wv[j], cur[j], cur[j]);
+        for (int k = 0; k < keep; ++k) {
+            const int back = t - keep + k;
+            ld(back >= 0 ? in + (size_t)back * E : st + (size_t)(keep + back) * E, v);
+            ld(w + (size_t)k * E + i, wv);
+#pragma unroll
+            for (int j = 0; j < N; ++j) acc[j] = fmaf(wv[j], v[j], acc[j]);
+        }
+        if constexpr (N == 4) store4(y + (size_t)(q0 + t) * E + i, acc);
+        else y[(size_t)(q0 + t) * E + i] = from_float<TO>(acc[0]);
+    }
+    if (blockIdx.z == 0)
+        for (int k = 0; k < keep; ++k) {       // the entry's last taps - 1 inputs (older ones were in the state already)
+            float v[N];
+            const int at = n - keep + k;
+            ld(at >= 0 ? in + (size_t)at * E : st + (size_t)(keep + at) * E, v);
+            if constexpr (N == 4) store4(st + (size_t)k * E, v);
+            else st[(size_t)k * E] = v[0];
+        }
+}
+
+}  // namespace air
+
+AIR_API int air_stream_norm(const float* x, long long x_stride, float* h_out, long long h_stride, const float* y, int y_parts,
+                            long long part_stride, const float* mix, const float* out_w, const float* read, int S,
+                            const float* w, const float* b, void* out, int out_dtype, const int* rows, int R, int E,
+                            int center, float eps, const float* conv_w, float* conv_state, const int* token_seq, int taps,
+                            cudaStream_t stream) {
+    if (R <= 0) return 0;
+    if (!x || S < 1 || S > air::STREAMS_MAX || E <= 0 || (y && y_parts < 1) || (w && !out) || (conv_w && (taps < 1 || rows || !token_seq)) ||
+        (conv_w && taps > 1 && !conv_state))
+        return AIR_ERR_BAD_ARGUMENT;
+    const size_t smem = sizeof(float) * (size_t)E;
+    if (smem > 200 * 1024) return AIR_ERR_BAD_ARGUMENT;
+    air::StreamNormArgs p;
+    p.x = x; p.x_stride = (size_t)x_stride; p.h_out = h_out; p.h_stride = (size_t)h_stride; p.y = y; p.y_parts = y_parts;
+    p.part_stride = (size_t)part_stride; p.mix = mix; p.out_w = out_w; p.read = read; p.S = S; p.w = w; p.b = b; p.out = out;
+    p.rows = rows; p.E = E; p.center = center; p.eps = eps; p.conv_w = conv_w; p.conv_state = conv_state;
+    p.token_seq = token_seq; p.taps = taps;
+    auto al = [](const void* q) { return ((uintptr_t)q & 15) == 0; };
+    const bool vec = E % 4 == 0 && x_stride % 4 == 0 && h_stride % 4 == 0 && part_stride % 4 == 0 && al(x) && al(h_out) &&
+                     al(y) && al(w) && al(b) && al(out);
+    // few rows: one access of a thread per row, all of a row's loads under way at once
+    const int items = vec ? E / 4 : E;
+    int threads = items >= 256 ? 256 : (items + 31) / 32 * 32;
+    if (R <= 256) threads = items >= 1024 ? 1024 : (items + 31) / 32 * 32;
+    AIR_DISPATCH(out_dtype, TO, {
+        auto go = [&](auto kernel) {
+            if (smem > 44 * 1024) {
+                cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+                if (err != cudaSuccess) return (int)err;
+            }
+            return air::launch(kernel, R, threads, smem, stream, p);
+        };
+        if (!vec) return go(air::stream_norm_kernel<TO, 0, 1>);
+        switch (S) {
+            case 1: return go(air::stream_norm_kernel<TO, 1, 4>);
+            case 2: return go(air::stream_norm_kernel<TO, 2, 4>);
+            case 3: return go(air::stream_norm_kernel<TO, 3, 4>);
+            case 4: return go(air::stream_norm_kernel<TO, 4, 4>);
+            default: return go(air::stream_norm_kernel<TO, 0, 1>);
+        }
+    });
+    return 0;
+}
+
+AIR_API int air_residual_conv(const float* h, const float* w, float* state, void* y, int out_dtype, const int* q_start,
+                              const int* slots, int entries, int E, int taps, int max_tokens, cudaStream_t stream) {
+    if (entries <= 0 || E <= 0) return 0;
+    if (taps < 1 || (taps > 1 && !state) || entries > 65535) return AIR_ERR_BAD_ARGUMENT;
+    const int chunk = taps - 1 > 16 ? taps - 1 : 16;
+    const int chunks = (max_tokens + chunk - 1) / chunk < 1 ? 1 : (max_tokens + chunk - 1) / chunk;
+    if (chunks > 65535) return AIR_ERR_BAD_ARGUMENT;
+    const bool vec = E % 4 == 0 && (((uintptr_t)h | (uintptr_t)w | (uintptr_t)state | (uintptr_t)y) & 15) == 0;
+    const int items = vec ? E / 4 : E;
+    const dim3 grid((items + 127) / 128, entries, chunks);
+    AIR_DISPATCH(out_dtype, TO, {
+        if (vec)
+            return air::launch(air::residual_conv_kernel<TO, 4>, grid, 128, 0, stream, h, w, state, (TO*)y, q_start, slots,
+                               E, taps, chunk);
+        return air::launch(air::residual_conv_kernel<TO, 1>, grid, 128, 0, stream, h, w, state, (TO*)y, q_start, slots, E,
+                           taps, chunk);
+    });
+    return 0;
+}
+
+AIR_API int air_trace_set_stream_ops(unsigned long long* buffer) { return air::set_trace_here(buffer); }

@@ -84,9 +84,10 @@ class Model:
             and getattr(self.embedder, "graph_safe", False)
 
     def cache_needs(self):
-        """Per run of the order list: the needs of the layer's mixer, or nothing for a run that
-        reads another run's cache; behind the runs, what the embedding keeps per request."""
-        return [self.blocks[run.layer].cache_needs() if run.cache_from is None else ()
+        """Per run of the order list: the needs of the layer's mixer, or for a run that reads another run's cache what
+        it keeps all the same (usually nothing); behind the runs, what the embedding keeps per request."""
+        return [self.blocks[run.layer].cache_needs() if run.cache_from is None
+                else tuple(getattr(self.blocks[run.layer], "borrowing_needs", tuple)())
                 for run in self.spec.order] + [tuple(self.embedder.cache_needs())]
 
     def weight_bytes(self) -> int:
@@ -123,14 +124,17 @@ class Model:
             owner = i if run.cache_from is None else run.cache_from
             if run.add_embedding or run.add_row is not None:
                 # what the run adds to the stream ahead of its layer: the stream is completed first
-                Norm.add_delta(h, pending)
+                h = Norm.add_delta(h, pending)
                 pending = None
                 row = None if run.add_row is None else self.stream_tables[run.add_row[0]][run.add_row[1]]
                 ops.stream_add(h, again[0] if run.add_embedding else None, row)
+            kept = cache.views(i) if run.cache_from is not None else ()
             h, pending = self.blocks[run.layer].forward(h, pending, ctx, cache.views(owner),
-                                                        owns_cache=run.cache_from is None)
+                                                        owns_cache=run.cache_from is None,
+                                                        **({"kept": kept} if kept else {}))
             if self.tap is not None:
-                self.tap.append(Norm.add_delta(h.clone(), pending))
+                x = Norm.add_delta(h.clone(), pending)
+                self.tap.append(x if x.dim() == 2 else x.sum(0))      # (several streams: their sum)
         R = ctx.logit_rows.shape[0]
         if R == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=rt.device)

@@ -21,6 +21,8 @@ other parts of its block are.
                     forward(x, ctx, cache, owns_cache) -> [T, hidden], or float32 [parts, T, hidden]
                     partial sums, or None after adding its output into ctx.residual itself
   FeedForward       forward(x, ctx) -> as a mixer
+  RowFilter         what stands between a norm and the part that reads its rows: forward(x, ctx, view) -> rows in the
+                    compute dtype from float32 rows; may keep a state per request (cache_needs)
   Block             forward(h, pending, ctx, cache, owns_cache) -> (h, pending): an arrangement of
                     parts around the residual stream; `pending` is a delta in the sense above
   Embedding         forward(ctx, cache, copies) -> the stream's first rows from the step's token ids; may keep a
@@ -257,6 +259,17 @@ class NormedSum:
     eps: float
 
 
+@dataclass
+class StreamSum:
+    """What a sub-layer of a block with several residual streams hands on (hyper-connections): the streams
+    x_0 .. x_(S-1) become x'_t = sum_s mix[s, t] x_s + out[t] * term, with term float32 [T, hidden] or partial sums
+    [parts, T, hidden], mix float32 [S, S], out float32 [S].  A form of a norm's `delta` for a stream h [S, T, hidden], or
+    h [T, hidden] while all streams are still equal."""
+    term: torch.Tensor
+    mix: torch.Tensor
+    out: torch.Tensor
+
+
 class Part:
     # True if forward() only launches work on the current stream from device data (no host
     # reads of the batch or of a result), so that a decode step can be captured in a CUDA graph.
@@ -292,9 +305,16 @@ class Norm(Part):
 
     @staticmethod
     def add_delta(h: torch.Tensor, delta) -> torch.Tensor:
-        """h += delta for every form of delta that a part may hand on (see the module's text)."""
+        """h += delta for every form of delta that a part may hand on (see the module's text); returns h, or for a
+        StreamSum the completed streams [S, T, hidden] (h itself unless its streams were still one tensor)."""
         if delta is not None:
             from ..csrc import ops
+            if isinstance(delta, StreamSum):
+                S = delta.out.shape[0]
+                full = h if h.dim() == 3 else torch.empty((S,) + tuple(h.shape), dtype=h.dtype, device=h.device)
+                ops.stream_norm(h, S, None, None, 0.0, None, term=delta.term, mix=delta.mix, out_weights=delta.out,
+                                h_out=full)
+                return full
             if isinstance(delta, ScaledSum):
                 ops.scaled_norm(h, delta.terms, None, 0.0, None)
             elif isinstance(delta, GatedSum):
@@ -329,6 +349,20 @@ class Embedding(Part):
         return ()
 
     def forward(self, ctx, cache, copies: int = 1):
+        raise NotImplementedError
+
+
+class RowFilter(Part):
+    """Rows on their way from a norm (float32) to the part behind it (compute dtype).  single_tokens(ctx, cache): what
+    the norm's kernel needs to apply the filter itself in a step in which every row is its request's only token, or None."""
+
+    def cache_needs(self) -> Tuple[CacheNeed, ...]:
+        return ()
+
+    def single_tokens(self, ctx, cache):
+        return None
+
+    def forward(self, x, ctx, cache):
         raise NotImplementedError
 
 

@@ -1,7 +1,7 @@
 """How the parts of one layer stand around the residual stream."""
 from __future__ import annotations
 
-from .registry import register_block, MIXERS, FEED_FORWARDS, NORMS
+from .registry import register_block, MIXERS, FEED_FORWARDS, NORMS, ROW_FILTERS
 from .spec import BlockSpec
 
 
@@ -27,6 +27,11 @@ class Block:
     def cache_needs(self):
         """What the layer keeps per request (CacheNeed objects); forward() receives their views as `cache`,
         in the same order."""
+        return ()
+
+    def borrowing_needs(self):
+        """What a run of the layer keeps for itself although it reads another run's cache.  Where this is not empty,
+        forward() of such a run receives the views as `kept`, beside the other run's as `cache`."""
         return ()
 
     @property
@@ -286,3 +291,99 @@ class PostNormBlock(Block):
             x = self.ff_norm.forward(h, self.feed_forward.forward(x, ctx) if self.feed_forward is not None else None)
         ctx.shared[self.ROWS] = x
         return h, None
+
+
+@register_block("streams")
+class StreamsBlock(Block):
+    """Several residual streams x_0 .. x_(S-1) instead of one (hyper-connections).  For each of the two sub-layers, with its
+    learned numbers read [S], mix [S, S] and out [S]:
+
+        u = sum_s read[s] x_s;   y = sub-layer(norm(u));   x_t = sum_s mix[s, t] x_s + out[t] y   (all at once)
+
+    Roles: mixer_norm, mixer, and feed_forward_norm with feed_forward (a layer may lack these two); mixer_filter (optional):
+    a row filter between the first norm and the mixer.  The norms are of a kind that offers forward_streams.  spec.names
+    gives with mixer_streams and feed_forward_streams the prefixes of the tensors in [S], mix [S, S] (from, to) and out [S];
+    the parameter streams is S.
+
+    The streams are float32 [S, T, hidden] ([T, hidden] until the first of them differ).  A sub-layer's output is handed on
+    as a StreamSum, so that ONE kernel completes the streams, folds them for the next sub-layer and normalises; in a step of
+    single tokens that kernel applies the filter as well.  What a request keeps: the mixer's needs, then the filter's; a run
+    that reads another run's cache keeps the filter's state itself."""
+
+    def __init__(self, spec: BlockSpec):
+        super().__init__(spec)
+        self.streams = int(spec.params["streams"])
+        from ..config.model_config import ConfigError
+        from ..csrc import ops
+        if not (1 <= self.streams <= ops.STREAMS_MAX):
+            raise ConfigError("unsupported", f"block 'streams': {self.streams} streams (1 to {ops.STREAMS_MAX})")
+        self.mixer_norm = NORMS.get(spec.part("mixer_norm").kind)(spec.part("mixer_norm"), spec.name("mixer_norm"))
+        self.mixer = MIXERS.get(spec.part("mixer").kind)(spec.part("mixer"), spec.name("mixer"))
+        self.filter = self.ff_norm = self.feed_forward = None
+        if "mixer_filter" in spec.parts:
+            self.filter = ROW_FILTERS.get(spec.part("mixer_filter").kind)(spec.part("mixer_filter"),
+                                                                          spec.name("mixer_filter"))
+        if "feed_forward" in spec.parts:
+            self.ff_norm = NORMS.get(spec.part("feed_forward_norm").kind)(spec.part("feed_forward_norm"),
+                                                                          spec.name("feed_forward_norm"))
+            self.feed_forward = FEED_FORWARDS.get(spec.part("feed_forward").kind)(spec.part("feed_forward"),
+                                                                                  spec.name("feed_forward"))
+
+    def parts(self):
+        return tuple(p for p in (self.mixer_norm, self.filter, self.mixer, self.ff_norm, self.feed_forward)
+                     if p is not None)
+
+    def _stream_names(self):
+        return [self.spec.name("mixer_streams")] + ([self.spec.name("feed_forward_streams")] if self.feed_forward else [])
+
+    def tensor_specs(self):
+        from ..weights.loader import TensorSpec
+        S = self.streams
+        return super().tensor_specs() + [
+            TensorSpec(name + n, shape, init="uniform", std=1.0 / S if n == "mix" else 1.0, wide=True)
+            for name in self._stream_names() for n, shape in (("in", (S,)), ("out", (S,)), ("mix", (S, S)))]
+
+    def load(self, tensors, rt):
+        super().load(tensors, rt)
+        import torch
+        f32 = lambda n: tensors[n].to(torch.float32).contiguous()
+        # per sub-layer: (read, mix, out)
+        self.numbers = [(f32(p + "in"), f32(p + "mix"), f32(p + "out")) for p in self._stream_names()]
+
+    def cache_needs(self):
+        return tuple(self.mixer.cache_needs()) + self.borrowing_needs()
+
+    def borrowing_needs(self):
+        return tuple(self.filter.cache_needs()) if self.filter is not None else ()
+
+    @staticmethod
+    def _handed_on(y, numbers):
+        import torch
+        from ..csrc import ops
+        from .base import GatedSum, NormedSum, ScaledSum, StreamSum
+        if y is None or isinstance(y, (GatedSum, ScaledSum, NormedSum, StreamSum)):
+            raise ops.KernelError("streams: the sub-layer must return its output as a tensor or as partial sums")
+        if y.dtype != torch.float32:
+            y = ops.convert(y, torch.empty(y.shape, dtype=torch.float32, device=y.device))
+        return StreamSum(y, numbers[1], numbers[2])
+
+    def forward(self, h, pending, ctx, cache, owns_cache=True, kept=()):
+        import torch
+        ctx.residual = None          # the sub-layers' outputs go to all streams: the parts return them
+        first = self.numbers[0]
+        mine = len(self.mixer.cache_needs())
+        if self.filter is None:
+            h, x = self.mixer_norm.forward_streams(h, pending, first[0])
+        else:
+            views = tuple(cache[mine:]) if owns_cache else tuple(kept)
+            conv = self.filter.single_tokens(ctx, views)
+            h, x = self.mixer_norm.forward_streams(h, pending, first[0], conv=conv,
+                                                   dtype=None if conv is not None else torch.float32)
+            if conv is None:
+                x = self.filter.forward(x, ctx, views)
+        pending = self._handed_on(self.mixer.forward(x, ctx, tuple(cache[:mine]), owns_cache), first)
+        if self.feed_forward is None:
+            return h, pending
+        second = self.numbers[1]
+        h, x = self.ff_norm.forward_streams(h, pending, second[0])
+        return h, self._handed_on(self.feed_forward.forward(x, ctx), second)

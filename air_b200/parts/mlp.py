@@ -52,6 +52,7 @@ class SwiGLU(FeedForward):
 
     graph_safe = True
 
+    ACT = ops.SILU          # the gated activation (ops.gemm_tc)
     # what follows the prefix in the names of the three matrices
     NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
 
@@ -86,17 +87,26 @@ class SwiGLU(FeedForward):
                 and (self.gate_up.small(x) or fused_gate_up_pays(x.shape[0], self.gate_up.out_features))):
             # few rows or many: the tcgen05 product with SiLU(gate) * up in its epilogue (the 2 I wide
             # intermediate is never written)
-            act = self.gate_up.silu_mul(x)
+            act = self.gate_up.silu_mul(x, act=self.ACT)
         else:
             gu = self.gate_up(x, torch.float32 if self.rt.is_fp32 else self.rt.dtype)
             act = torch.empty((x.shape[0], self.intermediate), dtype=self.rt.dtype, device=x.device)
-            ops.silu_mul(gu, act, block=self.block)
+            ops.silu_mul(gu, act, block=self.block, relu=self.ACT is ops.RELU)
         if self.down.small(act):
             return self.down.partial(act)
         residual = getattr(ctx, "residual", None)
         if self.down.adds_into(act, residual):
             return self.down.add_into(act, residual)
         return self.down(act, torch.float32)
+
+
+@register_feed_forward("reglu")
+class ReGLU(SwiGLU):
+    """down(max(gate(x), 0) * up(x)): a gated feed-forward with the rectifier in SiLU's place.  params: hidden, intermediate.
+    Tensors: <prefix>gate, up [intermediate, hidden], down [hidden, intermediate].  Everything else is SwiGLU's."""
+
+    ACT = ops.RELU
+    NAMES = {"gate": "gate", "up": "up", "down": "down"}
 
 
 @register_feed_forward("clamped_glu")

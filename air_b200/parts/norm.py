@@ -1,11 +1,11 @@
-"""RMSNorm fused with the residual addition that precedes it."""
+"""Norms fused with the residual addition that precedes them."""
 from __future__ import annotations
 
 import torch
 
 from ..csrc import ops
 from ..weights.loader import TensorSpec
-from .base import GatedSum, Norm, NormedSum, PreNormed, ScaledSum
+from .base import GatedSum, Norm, NormedSum, PreNormed, ScaledSum, StreamSum
 from .registry import register_norm
 
 
@@ -123,3 +123,59 @@ class PostRMSNorm(Norm):
         out = None if self.rt.is_fp32 else torch.empty(h.shape, dtype=self.rt.dtype, device=h.device)
         ops.post_norm(h, self.alpha, a, b, gate, self.weight, self.eps, out)
         return h if out is None else out
+
+
+@register_norm("layer")
+class LayerNorm(Norm):
+    """(x - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations.  params: size, eps; tensor and bias:
+    what follows the prefix in the names of w and b ("weight" and "bias" unless given).  Tensors: <prefix><tensor>,
+    <prefix><bias> [size].  32-bit.
+
+    Besides an ordinary residual stream it serves several that stand side by side (forward_streams): one kernel completes
+    the streams with what the sub-layer before handed on, folds them into the row that the next one reads and normalises
+    that.  Without weights for the reading (forward) the row is the sum of the streams."""
+
+    graph_safe = True
+
+    def _names(self):
+        return self.prefix + self.spec.get("tensor", "weight"), self.prefix + self.spec.get("bias", "bias")
+
+    def tensor_specs(self):
+        w, b = self._names()
+        return [TensorSpec(w, (self.spec["size"],), init="one_plus_normal", wide=True),
+                TensorSpec(b, (self.spec["size"],), wide=True)]
+
+    def load(self, tensors, rt):
+        super().load(tensors, rt)
+        w, b = self._names()
+        self.weight, self.bias = tensors[w].to(torch.float32).contiguous(), tensors[b].to(torch.float32).contiguous()
+        self.eps = float(self.spec["eps"])
+
+    def forward(self, h, delta, rows=None):
+        if isinstance(delta, StreamSum) or h.dim() == 3:
+            return self.forward_streams(h, delta, None, rows=rows)[1]
+        n = h.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, h.shape[1]), dtype=self.rt.dtype, device=h.device)
+        if isinstance(delta, (ScaledSum, GatedSum, NormedSum)) or (delta is not None and delta.dtype != torch.float32):
+            if rows is not None:
+                h = h.clone()
+            self.add_delta(h, delta)
+            delta = None
+        return ops.stream_norm(h, 1, self.weight, self.bias, self.eps, out, term=delta,
+                               h_out=h if delta is not None and rows is None else None, rows=rows)
+
+    def forward_streams(self, h, delta, read, rows=None, dtype=None, conv=None):
+        """(the streams, the normalised rows): delta is a StreamSum (or None), read float32 [S] the weights with which the
+        streams are read (None: their sum).  dtype: of the rows, the compute dtype unless given.  conv: see
+        ops.stream_norm.  With rows the streams are left as they are."""
+        S = delta.out.shape[0] if delta is not None else (h.shape[0] if h.dim() == 3 else read.shape[0])
+        n, E = (h.shape[-2] if rows is None else rows.shape[0]), h.shape[-1]
+        out = torch.empty((n, E), dtype=dtype or self.rt.dtype, device=h.device)
+        if delta is None:
+            return h, ops.stream_norm(h, S, self.weight, self.bias, self.eps, out, read=read, rows=rows, conv=conv)
+        full = None
+        if rows is None:
+            full = h if h.dim() == 3 else torch.empty((S,) + tuple(h.shape), dtype=torch.float32, device=h.device)
+        ops.stream_norm(h, S, self.weight, self.bias, self.eps, out, term=delta.term, mix=delta.mix, out_weights=delta.out,
+                        read=read, h_out=full, rows=rows, conv=conv)
+        return (h if full is None else full), out

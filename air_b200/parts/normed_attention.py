@@ -35,14 +35,22 @@ class NormedAttention(PortionAttention, Mixer):
       * conv > 1 puts a causal convolution over time of `conv` taps on every channel of q, k and v, right behind the
         projection (no activation); its last conv - 1 inputs are a state of the request;
       * softcap > 0 turns a score s into softcap * tanh(s / softcap);
-      * out_gate multiplies the heads' outputs, element by element, by sigmoid(Wg x) ahead of the output projection.
+      * out_gate multiplies the heads' outputs, element by element, by sigmoid(Wg x) ahead of the output projection;
+      * head_temp multiplies head h's scores by a learned number temp_h (it rides on the normalised queries);
+      * value_position rotates the values by their position before they are kept (an encoding of kind rope_live over the
+        first part of a value) and turns every head's sum over values back by the query's position, ahead of the gate:
+        what a head returns then depends on how far away the values stand;
+      * a layer that borrows reads the keys and values that another layer's run keeps (RunStep.cache_from): it has no
+        projections or norms of keys and values; `keep` is the widest window among the layers that read one layer's
+        pages, which live as long.
 
     params: hidden, heads, kv_heads, head_dim, v_dim, scale, window, chunk (at most one of the two), qk_norm (False,
-    True or "head", "whole"), sink (False, True or "learned", "zero"), eps, position, qkv_bias, conv, softcap, out_gate.
+    True or "head", "whole"), sink (False, True or "learned", "zero"), eps, position, qkv_bias, conv, softcap, out_gate,
+    head_temp, value_position, borrows, keep.
     Tensors: <prefix>q [heads*head_dim, hidden], k [kv_heads*head_dim, hidden], v [kv_heads*v_dim, hidden],
     q.norm, k.norm [head_dim] where qk_norm ([heads*head_dim] and [kv_heads*head_dim] where "whole"), sink [heads] where
     the sink is learned, o [hidden, heads*v_dim]; q.b, k.b, v.b where qkv_bias; q.conv, k.conv, v.conv [channels, conv]
-    where conv; g [heads*v_dim, hidden] where out_gate.
+    where conv; g [heads*v_dim, hidden] where out_gate; temp [heads] where head_temp.
 
     q, k and v are one product; one kernel then normalises, rotates and writes keys and values to the pages; pages of a
     chunk that no later query can see go back to the pool.  Prompt portions attend through matrix products over their
@@ -68,6 +76,8 @@ class NormedAttention(PortionAttention, Mixer):
         self.sink_learned = self.sink and sink != "zero"
         if norm not in (False, True, None, "head", "whole") or sink not in (False, True, None, "learned", "zero"):
             raise ConfigError("data_error", f"normed_attention: qk_norm {norm!r}, sink {sink!r}")
+        self.head_temp, self.borrows = bool(p.get("head_temp", False)), bool(p.get("borrows", False))
+        self.keep = p.get("keep", self.window) if self.window else None
         self.qkv_bias, self.out_gate = bool(p.get("qkv_bias", False)), bool(p.get("out_gate", False))
         self.taps, self.softcap = int(p.get("conv") or 0), float(p.get("softcap") or 0.0)
         if self.taps > 16:
@@ -79,8 +89,12 @@ class NormedAttention(PortionAttention, Mixer):
         if self.head_dim % 2 or max(self.head_dim, self.v_dim) > 256:
             raise ConfigError("unsupported", f"attention: head sizes {self.head_dim} / {self.v_dim}: the kernels take "
                                              "even key sizes, and sizes up to 256")
-        pos = p["position"]
+        if self.borrows and (self.qkv_bias or self.taps or self.norm_whole or self.out_gate):
+            raise ConfigError("unsupported", "normed_attention: a layer that borrows keys and values takes queries with a "
+                                             "norm per head or none, without bias, convolution or output gate")
+        pos, vpos = p["position"], p.get("value_position")
         self.position = POSITION_ENCODINGS.get(pos.kind)(pos)
+        self.value_position = None if vpos is None else POSITION_ENCODINGS.get(vpos.kind)(vpos)
 
     def tiles_fit(self) -> bool:
         """Whether this layer's attention runs on the dense decoder's tile kernels (see the class's text)."""
@@ -117,14 +131,15 @@ class NormedAttention(PortionAttention, Mixer):
         return (self.heads + self.kv_heads) * self.head_dim + self.kv_heads * self.v_dim
 
     def cache_needs(self):
-        pages = PagedKV(self.kv_heads, self.head_dim, self.window, self.v_dim, self.chunk)
+        pages = PagedKV(self.kv_heads, self.head_dim, self.keep, self.v_dim, self.chunk)
         return (pages, SlotState((self.channels, self.taps - 1))) if self.taps > 1 else (pages,)
 
     def tensor_specs(self):
         p, e = self.prefix, self.hidden
-        specs = [TensorSpec(p + "q", (self.heads * self.head_dim, e)),
-                 TensorSpec(p + "k", (self.kv_heads * self.head_dim, e)),
-                 TensorSpec(p + "v", (self.kv_heads * self.v_dim, e))]
+        specs = [TensorSpec(p + "q", (self.heads * self.head_dim, e))]
+        if not self.borrows:
+            specs += [TensorSpec(p + "k", (self.kv_heads * self.head_dim, e)),
+                      TensorSpec(p + "v", (self.kv_heads * self.v_dim, e))]
         rows = {"q": self.heads * self.head_dim, "k": self.kv_heads * self.head_dim, "v": self.kv_heads * self.v_dim}
         if self.qkv_bias:
             specs += [TensorSpec(p + n + ".b", (rows[n],), wide=True) for n in "qkv"]
@@ -132,7 +147,9 @@ class NormedAttention(PortionAttention, Mixer):
             specs += [TensorSpec(p + n + ".conv", (rows[n], self.taps), wide=True, std=0.3) for n in "qkv"]
         if self.qk_norm:
             specs += [TensorSpec(p + n + ".norm", (rows[n] if self.norm_whole else self.head_dim,),
-                                 init="one_plus_normal", wide=True) for n in "qk"]
+                                 init="one_plus_normal", wide=True) for n in ("q" if self.borrows else "qk")]
+        if self.head_temp:
+            specs.append(TensorSpec(p + "temp", (self.heads,), init="one_plus_normal", wide=True))
         if self.sink_learned:
             specs.append(TensorSpec(p + "sink", (self.heads,), std=1.0, wide=True))
         if self.out_gate:
@@ -143,7 +160,7 @@ class NormedAttention(PortionAttention, Mixer):
     def load(self, tensors, rt):
         super().load(tensors, rt)
         p = self.prefix
-        ws = [tensors[p + n] for n in ("qkvg" if self.out_gate else "qkv")]
+        ws = [tensors[p + n] for n in ("q" if self.borrows else "qkvg" if self.out_gate else "qkv")]
         if len({w.dtype for w in ws}) != 1:
             raise ValueError(f"{p}: the projections are stored in different precisions")
         self.proj = Linear(torch.cat(ws, dim=0).contiguous(), rt.status)
@@ -151,7 +168,8 @@ class NormedAttention(PortionAttention, Mixer):
         self.q_weight = self.k_weight = self.sinks = None
         if self.qk_norm:
             self.q_weight = tensors[p + "q.norm"].to(torch.float32).contiguous()
-            self.k_weight = tensors[p + "k.norm"].to(torch.float32).contiguous()
+            self.k_weight = None if self.borrows else tensors[p + "k.norm"].to(torch.float32).contiguous()
+        self.temp = tensors[p + "temp"].to(torch.float32).contiguous() if self.head_temp else None
         if self.sink_learned:
             self.sinks = tensors[p + "sink"].to(torch.float32).contiguous()
         elif self.sink:
@@ -166,10 +184,20 @@ class NormedAttention(PortionAttention, Mixer):
             raise ConfigError("unsupported", "normed_attention takes a position encoding that gives 64-bit frequencies")
         if self.position.rotary_dim > self.head_dim:
             raise ConfigError("data_error", "normed_attention: the rotated part is larger than a head")
+        self.v_freq = None
+        if self.value_position is not None:
+            v = self.value_position
+            v.load(tensors, rt)
+            if not hasattr(v, "frequencies64") or v.magnitude != 1.0 or v.pairing != self.position.pairing:
+                raise ConfigError("unsupported", "normed_attention: values are rotated with 64-bit frequencies, in the "
+                                                 "keys' pairing")
+            if v.rotary_dim > self.v_dim:
+                raise ConfigError("data_error", "normed_attention: the rotated part is larger than a value")
+            self.v_freq = v.frequencies64()
 
     def forward(self, x, ctx, cache, owns_cache=True):
-        if not owns_cache:
-            raise ops.KernelError("normed_attention: a run that reads another run's keys and values is not offered")
+        if owns_cache == self.borrows:
+            raise ops.KernelError("normed_attention: the layer and the run list disagree on whose keys the layer reads")
         pages = cache[0]
         T, H, G, dk, dv = x.shape[0], self.heads, self.kv_heads, self.head_dim, self.v_dim
         rt = self.rt
@@ -191,13 +219,19 @@ class NormedAttention(PortionAttention, Mixer):
         pos = self.position
         ops.qk_normed_prepare(proj, self.q_weight, self.k_weight, self.eps, pos.frequencies64(), pos.pairing,
                               pos.magnitude, ctx.positions, ctx.token_seq, bt, q, kv, G, dv, P, status=ctx.status,
-                              bias=self.bias, whole=self.norm_whole)
+                              bias=self.bias, whole=self.norm_whole, q_scale=self.temp, v_freq=self.v_freq,
+                              write_kv=owns_cache)
         out = torch.empty((T, H, dv), dtype=rt.dtype, device=x.device)
         gate = full[:, C:] if self.out_gate else None
+        late_gate, gate = (gate, None) if self.v_freq is not None else (None, gate)      # a gate comes behind the turn back
         plan = ctx.plans.get(TiledAttention.plan_key(self)) if self.tiles_fit() and not ctx.all_decode else None
         if plan is not None:
             self.attend_tiles(q, pages.kv, bt, ctx, out, plan, gate)
         else:
             self.attend(q, kv, bt, ctx, out, kv_heads=G, page_tokens=P, gate=gate,
                         pages=pages.kv if pages.kv.dim() == 5 else None)
+        if self.v_freq is not None:
+            ops.turn_heads(out, self.v_freq, pos.pairing, ctx.positions, ctx.token_seq, back=True)
+            if late_gate is not None:
+                ops.sigmoid_gate(out.view(T, H * dv), late_gate, ctx.token_seq)
         return self.o.f32_sums(out.view(T, H * dv))

@@ -286,3 +286,62 @@ class Retention(_StateMixer):
                         self.decays, state.state, o, ctx.q_start, ctx.slots, ctx.token_seq, positions=ctx.positions,
                         freq=self.freq, k_scale=d ** -0.5)
         return self._finish(o, proj, ctx)
+
+
+@register_mixer("mlstm")
+class MLSTM(_StateMixer):
+    """The matrix memory of xLSTM.  q = W_q x * head_dim^-1/2, k = W_k x (heads x head_dim), v = W_v x (heads x v_dim); per
+    head the logarithms of an input gate i = c tanh((W_i x + b_i) / c) and of a forget gate
+    f = log sigmoid(c tanh((W_f x + b_f) / c)), c = gate_cap; per head and token, with the state S, n and m zero at first
+
+        m' = max(f + m, i);   S = exp(f + m - m') S + exp(i - m') k v^T;   n likewise with k alone;
+        o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
+
+    then each head's o / sqrt(mean(o^2) + eps), all heads times norm, times sigmoid(W_g x), and the output projection.
+    S, n and m are the request's state, 32-bit; the gates, the recurrence, the norm and the read-out are 32-bit.
+
+    params: hidden, heads, head_dim, v_dim, gate_cap, eps.  Tensors: <prefix>q, k [heads*head_dim, hidden]; v, g
+    [heads*v_dim, hidden]; i, f [heads, hidden]; i.b, f.b [heads]; norm [heads*v_dim]; o [hidden, heads*v_dim]."""
+
+    def __init__(self, spec, prefix=""):
+        super().__init__(spec, prefix)
+        p = spec.params
+        self.hidden, self.heads, self.head_dim, self.v_dim = p["hidden"], p["heads"], p["head_dim"], p["v_dim"]
+        self.cap, self.eps = float(p["gate_cap"]), float(p["eps"])
+        if not (self.cap > 0.0):
+            raise ConfigError("data_error", "mlstm: gate_cap must be positive")
+
+    def cache_needs(self):
+        H, d, dv = self.heads, self.head_dim, self.v_dim
+        return (SlotState((H, d, dv)), SlotState((H, d)), SlotState((H,)))
+
+    def tensor_specs(self):
+        p, e, H, d, dv = self.prefix, self.hidden, self.heads, self.head_dim, self.v_dim
+        return [TensorSpec(p + "q", (H * d, e)), TensorSpec(p + "k", (H * d, e)), TensorSpec(p + "v", (H * dv, e)),
+                TensorSpec(p + "g", (H * dv, e)), TensorSpec(p + "i", (H, e)), TensorSpec(p + "f", (H, e)),
+                TensorSpec(p + "i.b", (H,), wide=True), TensorSpec(p + "f.b", (H,), init="one_plus_normal", wide=True),
+                TensorSpec(p + "norm", (H * dv,), init="one_plus_normal", wide=True), TensorSpec(p + "o", (e, H * dv))]
+
+    def load(self, tensors, rt):
+        super().load(tensors, rt)
+        p = self.prefix
+        # (rows of zeros fill the matrix up to a multiple of 8, which the tensor-core kernels want)
+        rows = self.heads * (2 * self.head_dim + 2 * self.v_dim + 2)
+        pad = -rows % 8
+        if pad:
+            tensors = dict(tensors, **{p + "pad": torch.zeros((pad, self.hidden), dtype=tensors[p + "q"].dtype,
+                                                              device=tensors[p + "q"].device)})
+        self._project(tensors, ["q", "k", "v", "g", "i", "f"] + (["pad"] if pad else []), rt)
+        f32 = lambda n: tensors[p + n].to(torch.float32).contiguous()
+        self.i_bias, self.f_bias, self.norm_weight = f32("i.b"), f32("f.b"), f32("norm")
+        self.o = Linear(tensors[p + "o"], rt.status)
+
+    def forward(self, x, ctx, cache, owns_cache=True):
+        memory, key_sum, level = cache
+        T = x.shape[0]
+        proj = self.proj.f32(x)
+        y = torch.empty((T, self.heads * self.v_dim), dtype=self.rt.dtype, device=x.device)
+        ops.mlstm_step(proj, {n: at for n, (at, _) in self.columns.items()}, self.i_bias, self.f_bias, self.norm_weight,
+                       memory.state, key_sum.state, level.state, y, ctx.q_start, ctx.slots, self.cap,
+                       self.head_dim ** -0.5, self.eps)
+        return self.o.f32_sums(y)

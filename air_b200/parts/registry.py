@@ -39,6 +39,7 @@ NORMS = _Registry("norm")
 POSITION_ENCODINGS = _Registry("position encoding")
 BLOCKS = _Registry("block arrangement")
 EMBEDDINGS = _Registry("embedding")
+ROW_FILTERS = _Registry("row filter")
 
 
 def register_mixer(kind, cls=None):
@@ -63,6 +64,10 @@ def register_block(kind, cls=None):
 
 def register_embedding(kind, cls=None):
     return EMBEDDINGS.register(kind, cls)
+
+
+def register_row_filter(kind, cls=None):
+    return ROW_FILTERS.register(kind, cls)
 
 
 class Architecture(NamedTuple):
