@@ -13,6 +13,19 @@
 //
 //   mlstm_step_kernel    one block per (head, entry) does all of it, token after token: the road of single next tokens (one
 //                        launch behind the projections, the state read and written once) and of short portions.
+//
+// Longer portions are cut into chunks of ML_C tokens, counted from the portion's start.  With the decays a_t and weights
+// b_t of the recurrence (they depend on the gates alone), P(s, t) = a_(s+1) .. a_t (products, not differences of sums of
+// logarithms, so that a forgotten stretch costs no digits), W[t, s] = (q_t . k_s) b_s P(s, t) for s <= t inside a chunk and
+// A_t = a_first .. a_t, a chunk's read-outs are W V + A (Q S_chunk) and n . q = row sum of W + A (q . n_chunk), with S_chunk
+// and n_chunk the states ahead of the chunk: 32-bit products on the CUDA cores, rows of different chunks side by side.
+//
+//   mlstm_gates_kernel   a, b and exp(-m) of every token: block (head, portion); m by a parallel scan of the maps
+//                        m -> max(F + m, M) (64-bit sums), 256 tokens at a time
+//   mlstm_states_kernel  the states ahead of every chunk: block (tile of 32 x 64 of S, head, portion), the tile in
+//                        registers, chunk after chunk: S <- (product of the chunk's a) S + sum_s b_s P(s, end) k_s v_s^T
+//   mlstm_outputs_kernel block (chunk, head, 128 columns of v): the read-outs; where a head's v fits one block also the norm,
+//                        the weight and the gate, else mlstm_finish_kernel does those
 #include "common.cuh"
 
 namespace air {
@@ -128,6 +141,380 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(const MlstmArgs 
     if (tid == 0) p.m[(size_t)slot * p.H + h] = m;
 }
 
+// ------------------------------------------------------------------ longer portions
+constexpr int ML_C = 64;                   // tokens of a chunk
+constexpr int ML_TD = 32, ML_TV = 64;      // the tile of S that a block of mlstm_states_kernel holds
+constexpr int ML_OV = 128;                 // columns of v per block of mlstm_outputs_kernel
+constexpr int ML_KS = 64;                  // key channels staged at a time there
+constexpr int ML_LD = ML_KS + 4, ML_LV = ML_OV + 4;
+
+struct MlstmChunkArgs {
+    MlstmArgs p;
+    const int* portions;                   // [L, 4]: first row, tokens, slot, first chunk
+    const int* chunks;                     // [N, 2]: first row, tokens
+    float* gates;                          // [3, H, T]: a, b, exp(-m)
+    float* chunk_S; float* chunk_n;        // [N, H, d, dv], [N, H, d]: the states ahead of every chunk
+    float* o;                              // [T, H, dv] read-outs where a head's v takes several blocks, else null
+    int T, vec;                            // vec: proj's rows and columns allow 16-byte accesses
+};
+
+__global__ void __launch_bounds__(256) mlstm_gates_kernel(const MlstmChunkArgs c) {
+    __shared__ double wF[8], wM[8], mt[257];
+    pdl_enter(TR_MLSTM);
+    const MlstmArgs& p = c.p;
+    const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int row0 = c.portions[blockIdx.y * 4], cnt = c.portions[blockIdx.y * 4 + 1], slot = c.portions[blockIdx.y * 4 + 2];
+    const float ib = p.ib[h], fb = p.fb[h];
+    double carry = (double)p.m[(size_t)slot * p.H + h];
+    float *ga = c.gates + (size_t)h * c.T, *gb = ga + (size_t)p.H * c.T, *ge = gb + (size_t)p.H * c.T;
+    for (int t0 = 0; t0 < cnt; t0 += 256) {
+        const int t = t0 + tid;
+        // a place behind the portion's end leaves m as it is: F = 0, M far below
+        float lf = 0.f, li = -1e30f;
+        if (t < cnt) {
+            const float* row = p.proj + (size_t)(row0 + t) * p.ld;
+            li = ml_capped(row[p.ci + h] + ib, p.cap);
+            lf = ml_log_sigmoid(ml_capped(row[p.cf + h] + fb, p.cap));
+        }
+        double F = lf, M = li;
+#pragma unroll
+        for (int off = 1; off < 32; off <<= 1) {
+            const double F0 = __shfl_up_sync(0xffffffffu, F, off), M0 = __shfl_up_sync(0xffffffffu, M, off);
+            if (lane >= off) {
+                M = fmax(M0 + F, M);
+                F = F0 + F;
+            }
+        }
+        if (lane == 31) { wF[warp] = F; wM[warp] = M; }
+        if (tid == 0) mt[0] = carry;
+        __syncthreads();
+        double m = carry;
+        for (int w = 0; w < warp; ++w) m = fmax(wF[w] + m, wM[w]);
+        m = fmax(F + m, M);
+        mt[tid + 1] = m;
+        __syncthreads();
+        if (t < cnt) {
+            ga[row0 + t] = expf((float)((double)lf + mt[tid] - m));
+            gb[row0 + t] = expf((float)((double)li - m));
+            ge[row0 + t] = expf(-(float)m);
+        }
+        carry = mt[256];
+        __syncthreads();
+    }
+    if (tid == 0) p.m[(size_t)slot * p.H + h] = (float)carry;
+}
+
+__device__ __forceinline__ void ml_cp16(void* smem, const void* gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem)
+                 : "memory");
+}
+__device__ __forceinline__ void ml_cp4(void* smem, const void* gmem) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem)
+                 : "memory");
+}
+
+// `rows` x COLS numbers from src (row stride ld, `width` columns of it exist, `live` rows exist) to dst (row stride DLD) by
+// cp.async, zeros where there are none; NT threads.  vec: 16-byte pieces (everything a multiple of 4 numbers).
+template <int COLS, int DLD, int NT>
+__device__ __forceinline__ void ml_stage(float* dst, const float* src, size_t ld, int rows, int live, int width, int vec) {
+    if (vec) {
+        constexpr int P4 = COLS / 4;
+        for (int i = threadIdx.x; i < rows * P4; i += NT) {
+            const int r = i / P4, c = i % P4 * 4;
+            float* to = dst + r * DLD + c;
+            if (r < live && c < width) ml_cp16(to, src + (size_t)r * ld + c);
+            else *reinterpret_cast<float4*>(to) = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    } else {
+        for (int i = threadIdx.x; i < rows * COLS; i += NT) {
+            const int r = i / COLS, c = i % COLS;
+            float* to = dst + r * DLD + c;
+            if (r < live && c < width) ml_cp4(to, src + (size_t)r * ld + c);
+            else *to = 0.f;
+        }
+    }
+}
+
+constexpr size_t ML_STATES_SMEM = sizeof(float) * (2 * ML_C * (ML_TD + ML_TV) + ML_C + 1);
+
+// 128 threads, 4 x 4 numbers of the tile each.
+__global__ void __launch_bounds__(128) mlstm_states_kernel(const MlstmChunkArgs c) {
+    extern __shared__ __align__(16) float smem[];
+    float* const sk[2] = {smem, smem + ML_C * ML_TD};
+    float* const sv[2] = {smem + 2 * ML_C * ML_TD, smem + 2 * ML_C * ML_TD + ML_C * ML_TV};
+    float* const se = smem + 2 * ML_C * (ML_TD + ML_TV);
+    pdl_enter(TR_MLSTM);
+    const MlstmArgs& p = c.p;
+    const int d = p.d, dv = p.dv, tid = threadIdx.x, h = blockIdx.y;
+    const int tiles_v = (dv + ML_TV - 1) / ML_TV;
+    const int r0 = blockIdx.x / tiles_v * ML_TD, v0 = blockIdx.x % tiles_v * ML_TV;
+    const int* po = c.portions + blockIdx.z * 4;
+    const int row0 = po[0], cnt = po[1], slot = po[2], chunk0 = po[3];
+    const int ty = tid >> 4, tx = tid & 15;
+    const bool has_n = v0 == 0 && tid < ML_TD && r0 + tid < d;
+    float acc[4][4], nacc = 0.f;
+    float* S = p.S + ((size_t)slot * p.H + h) * d * dv;
+    float* nn = p.n + ((size_t)slot * p.H + h) * d;
+    const bool v4 = dv % 4 == 0 && v0 + tx * 4 < dv;       // (then the four columns exist and lie on 16 bytes)
+    auto at = [&](float* base, int i) { return base + (size_t)(r0 + ty * 4 + i) * dv + v0 + tx * 4; };
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            acc[i][j] = (r0 + ty * 4 + i < d && v0 + tx * 4 + j < dv) ? at(S, i)[j] : 0.f;
+    if (has_n) nacc = nn[r0 + tid];
+    auto stage = [&](int t0, int b) {
+        const float* src = p.proj + (size_t)(row0 + t0) * p.ld;
+        ml_stage<ML_TD, ML_TD, 128>(sk[b], src + p.ck + h * d + r0, p.ld, ML_C, cnt - t0, d - r0, c.vec);
+        ml_stage<ML_TV, ML_TV, 128>(sv[b], src + p.cv + h * dv + v0, p.ld, ML_C, cnt - t0, dv - v0, c.vec);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    const float *ga = c.gates + (size_t)h * c.T + row0, *gb = ga + (size_t)p.H * c.T;
+    stage(0, 0);
+    int b = 0;
+    for (int t0 = 0, ch = chunk0; t0 < cnt; t0 += ML_C, ++ch, b ^= 1) {
+        // the states ahead of this chunk
+        float* cs = c.chunk_S + ((size_t)ch * p.H + h) * d * dv;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            if (r0 + ty * 4 + i >= d) continue;
+            if (v4) *reinterpret_cast<float4*>(at(cs, i)) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+            else
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (v0 + tx * 4 + j < dv) at(cs, i)[j] = acc[i][j];
+        }
+        if (has_n) c.chunk_n[((size_t)ch * p.H + h) * d + r0 + tid] = nacc;
+        if (tid < 32) {      // b_s P(s, end) for the chunk's tokens and the product of all its a, by one warp, two tokens a lane
+            const int s = t0 + 2 * tid;
+            const float a0 = s < cnt ? ga[s] : 1.f, a1 = s + 1 < cnt ? ga[s + 1] : 1.f;
+            float prod = a0 * a1;                              // becomes the product from this lane's tokens to the end
+#pragma unroll
+            for (int off = 1; off < 32; off <<= 1) {
+                const float up = __shfl_down_sync(0xffffffffu, prod, off);
+                if (tid + off < 32) prod *= up;
+            }
+            float behind = __shfl_down_sync(0xffffffffu, prod, 1);
+            if (tid == 31) behind = 1.f;
+            se[2 * tid] = (s < cnt ? gb[s] : 0.f) * (a1 * behind);
+            se[2 * tid + 1] = (s + 1 < cnt ? gb[s + 1] : 0.f) * behind;
+            if (tid == 0) se[ML_C] = prod;
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (t0 + ML_C < cnt) stage(t0 + ML_C, b ^ 1);
+        for (int i = tid; i < ML_C * ML_TD; i += 128) sk[b][i] *= se[i / ML_TD];
+        const float all = se[ML_C];
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[i][j] *= all;
+#pragma unroll 8
+        for (int s = 0; s < ML_C; ++s) {
+            float k[4], v[4];
+            load4(&sk[b][s * ML_TD + ty * 4], k);
+            load4(&sv[b][s * ML_TV + tx * 4], v);
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(k[i], v[j], acc[i][j]);
+        }
+        if (has_n) {
+            float part[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+            for (int s = 0; s < ML_C; s += 4)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) part[j] += sk[b][(s + j) * ML_TD + tid];
+            nacc = fmaf(nacc, all, (part[0] + part[1]) + (part[2] + part[3]));
+        }
+        // (the next round's barrier stands between these reads and the copies into this buffer after next; se is
+        // written by warp 0 again before that barrier, so everyone must have read `all`: it has, ahead of the second one)
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (r0 + ty * 4 + i < d && v0 + tx * 4 + j < dv) at(S, i)[j] = acc[i][j];
+    if (has_n) nn[r0 + tid] = nacc;
+}
+
+// acc[i][j] += sum_k A[4 ty + i][k] B[k][4 tx + j (j < 4), 64 + 4 tx + j - 4]: A [64, ML_LD], B [64, ML_LV], 64 values of k
+__device__ __forceinline__ void ml_product(float (&acc)[4][8], const float* A, const float* B, int ty, int tx) {
+#pragma unroll 2
+    for (int k0 = 0; k0 < 64; k0 += 4) {
+        float a[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) load4(A + (4 * ty + i) * ML_LD + k0, a[i]);
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            float b0[4], b1[4];
+            load4(B + (k0 + kk) * ML_LV + 4 * tx, b0);
+            load4(B + (k0 + kk) * ML_LV + 64 + 4 * tx, b1);
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    acc[i][j] = fmaf(a[i][kk], b0[j], acc[i][j]);
+                    acc[i][4 + j] = fmaf(a[i][kk], b1[j], acc[i][4 + j]);
+                }
+        }
+    }
+}
+
+constexpr size_t ML_OUT_SMEM = sizeof(float) * (3 * 64 * ML_LD + 64 * ML_LV + 3 * 64 + ML_KS);
+
+template <typename TO>
+__global__ void __launch_bounds__(256, 2) mlstm_outputs_kernel(const MlstmChunkArgs c) {
+    extern __shared__ __align__(16) float smem[];
+    float *sq = smem, *sk = sq + 64 * ML_LD, *sw = sk + 64 * ML_LD, *sb = sw + 64 * ML_LD;
+    float *sa = sb + 64 * ML_LV, *sA = sa + 64, *sinv = sA + 64, *sn = sinv + 64;
+    pdl_enter(TR_MLSTM);
+    const MlstmArgs& p = c.p;
+    const int ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * ML_OV, tid = threadIdx.x, d = p.d, dv = p.dv;
+    const int row0 = c.chunks[2 * ch], cnt = c.chunks[2 * ch + 1];
+    const int ty = tid >> 4, tx = tid & 15;
+    const float *ga = c.gates + (size_t)h * c.T + row0, *gb = ga + (size_t)p.H * c.T, *ge = gb + (size_t)p.H * c.T;
+    const float* src = p.proj + (size_t)row0 * p.ld;
+    const float* S = c.chunk_S + ((size_t)ch * p.H + h) * d * dv;
+    const float* nn = c.chunk_n + ((size_t)ch * p.H + h) * d;
+    auto stage = [&](int k0) {
+        ml_stage<ML_KS, ML_LD, 256>(sq, src + p.cq + h * d + k0, p.ld, 64, cnt, d - k0, c.vec);
+        ml_stage<ML_KS, ML_LD, 256>(sk, src + p.ck + h * d + k0, p.ld, 64, cnt, d - k0, c.vec);
+        ml_stage<ML_OV, ML_LV, 256>(sb, S + (size_t)k0 * dv + v0, dv, 64, d - k0, dv - v0, dv % 4 == 0);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (tid < ML_KS) sn[tid] = k0 + tid < d ? nn[k0 + tid] : 0.f;
+    };
+    stage(0);
+    if (tid < 64) sa[tid] = tid < cnt ? ga[tid] : 1.f;
+    __syncthreads();
+    if (tid < 64) {          // b_s P(s, t) in the place of W[t, s]
+        float w = tid < cnt ? gb[tid] : 0.f;
+        for (int t = 0; t < 64; ++t) {
+            if (t > tid) w *= sa[t];
+            sw[t * ML_LD + tid] = t < tid ? 0.f : w;
+        }
+    } else if (tid == 64) {  // A_t
+        float w = 1.f;
+        for (int t = 0; t < 64; ++t) {
+            w *= sa[t];
+            sA[t] = w;
+        }
+    }
+    float acc[4][8], w[4][4], qn = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[i][j] = 0.f;
+    }
+    for (int k0 = 0; k0 < d; k0 += ML_KS) {
+        if (k0) {
+            __syncthreads();                               // the last slab has been used
+            stage(k0);
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        // w[i][j] += q_(4 ty + i) . k_(tx + 16 j)
+#pragma unroll 4
+        for (int k = 0; k < ML_KS; k += 4) {
+            float a[4][4], b[4][4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) load4(sq + (4 * ty + i) * ML_LD + k, a[i]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) load4(sk + (tx + 16 * j) * ML_LD + k, b[j]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int kk = 0; kk < 4; ++kk) w[i][j] = fmaf(a[i][kk], b[j][kk], w[i][j]);
+        }
+        ml_product(acc, sq, sb, ty, tx);
+        // a quarter of q_t . n for row t = tid / 4
+        const float* qr = sq + (tid >> 2) * ML_LD + (tid & 3) * 16;
+        const float* nr = sn + (tid & 3) * 16;
+#pragma unroll
+        for (int k = 0; k < 16; ++k) qn = fmaf(qr[k], nr[k], qn);
+    }
+    __syncthreads();
+    // the values take the last slab's place
+    ml_stage<ML_OV, ML_LV, 256>(sb, src + p.cv + h * dv + v0, p.ld, 64, cnt, dv - v0, c.vec);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float A = sA[4 * ty + i];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[i][j] *= A;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) sw[(4 * ty + i) * ML_LD + tx + 16 * j] *= w[i][j];
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    {
+        const int t = tid >> 2;
+        const float* wr = sw + t * ML_LD + (tid & 3) * 16;
+        float sum = sA[t] * qn;
+#pragma unroll
+        for (int k = 0; k < 16; ++k) sum += wr[k];
+        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+        if ((tid & 3) == 0)       // (q's scale multiplies both read-outs, here)
+            sinv[t] = p.q_scale / (fmaxf(fabsf(sum * p.q_scale), t < cnt ? ge[t] : 1.f) + 1e-6f);
+    }
+    ml_product(acc, sw, sb, ty, tx);
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = 4 * ty + i;
+        const float inv = sinv[t];
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            acc[i][j] *= inv;
+            ss = fmaf(acc[i][j], acc[i][j], ss);
+        }
+        auto column = [&](int j) { return v0 + (j < 4 ? 4 * tx + j : 64 + 4 * tx + j - 4); };
+        if (c.o) {
+            if (t < cnt)
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    if (column(j) < dv) c.o[((size_t)(row0 + t) * p.H + h) * dv + column(j)] = acc[i][j];
+            continue;
+        }
+        // (columns beyond dv are zeros: they add nothing to the sum)
+#pragma unroll
+        for (int off = 1; off < 16; off <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+        if (t >= cnt) continue;
+        const float scale = 1.f / sqrtf(ss / (float)dv + p.eps);
+        const float* gr = src + (size_t)t * p.ld + p.cg + h * dv;
+        TO* y = (TO*)p.y + ((size_t)(row0 + t) * p.H + h) * dv;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int col = column(j);
+            if (col < dv) y[col] = from_float<TO>(acc[i][j] * scale * p.w[h * dv + col] / (1.f + expf(-gr[col])));
+        }
+    }
+}
+
+// One warp per (token of a portion, head): the norm, the weight and the gate.
+template <typename TO>
+__global__ void __launch_bounds__(128) mlstm_finish_kernel(const MlstmChunkArgs c) {
+    pdl_enter(TR_MLSTM);
+    const MlstmArgs& p = c.p;
+    const int row0 = c.chunks[2 * blockIdx.x], cnt = c.chunks[2 * blockIdx.x + 1], h = blockIdx.y, lane = threadIdx.x & 31;
+    for (int t = threadIdx.x >> 5; t < cnt; t += 4) {
+        const size_t at = ((size_t)(row0 + t) * p.H + h) * p.dv;
+        float ss = 0.f;
+        for (int i = lane; i < p.dv; i += 32) ss = fmaf(c.o[at + i], c.o[at + i], ss);
+        const float scale = 1.f / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
+        const float* gr = p.proj + (size_t)(row0 + t) * p.ld + p.cg + h * p.dv;
+        for (int i = lane; i < p.dv; i += 32)
+            ((TO*)p.y)[at + i] = from_float<TO>(c.o[at + i] * scale * p.w[h * p.dv + i] / (1.f + expf(-gr[i])));
+    }
+}
+
 }  // namespace air
 
 AIR_API int air_mlstm_step(const float* proj, int ld, int cq, int ck, int cv, int cg, int ci, int cf, const float* ib,
@@ -150,6 +537,43 @@ AIR_API int air_mlstm_step(const float* proj, int ld, int cq, int ck, int cv, in
             return air::launch(kernel, dim3(H, entries), air::ML_THREADS, smem, stream, p);
         };
         return vec ? go(air::mlstm_step_kernel<TO, 4>) : go(air::mlstm_step_kernel<TO, 1>);
+    });
+    return 0;
+}
+
+// Portions of several tokens (see the file's head): portions int32 [L, 4] = (first row, tokens, slot, first chunk) and
+// chunks int32 [N, 2] = (first row, tokens), a portion's chunks of 64 tokens one after the other.  Scratch: gates float32
+// [3, H, T], chunk_S [N, H, d, dv], chunk_n [N, H, d], and o [T, H, dv] where dv > 128.
+AIR_API int air_mlstm_portions(const float* proj, int ld, int cq, int ck, int cv, int cg, int ci, int cf, const float* ib,
+                               const float* fb, const float* w, float* S, float* n, float* m, void* y, int out_dtype,
+                               const int* portions, int L, const int* chunks, int N, float* gates, float* chunk_S,
+                               float* chunk_n, float* o, int T, int H, int d, int dv, float cap, float q_scale, float eps,
+                               cudaStream_t stream) {
+    if (L <= 0 || N <= 0) return 0;
+    const int v_blocks = (dv + air::ML_OV - 1) / air::ML_OV;
+    if (H <= 0 || H > 65535 || d <= 0 || dv <= 0 || L > 65535 || v_blocks > 65535 || !(cap > 0.f) || !gates || !chunk_S ||
+        !chunk_n || (v_blocks > 1 && !o) || (((uintptr_t)chunk_S | (uintptr_t)S) & 15))
+        return AIR_ERR_BAD_ARGUMENT;
+    const int vec = ((ld | cq | ck | cv | d | dv) & 3) == 0 && ((uintptr_t)proj & 15) == 0;
+    air::MlstmChunkArgs c;
+    c.p = air::MlstmArgs{proj, ld, cq, ck, cv, cg, ci, cf, ib, fb, w, S, n, m, y, nullptr, nullptr, H, d, dv, cap, q_scale, eps};
+    c.portions = portions; c.chunks = chunks; c.gates = gates; c.chunk_S = chunk_S; c.chunk_n = chunk_n;
+    c.o = v_blocks > 1 ? o : nullptr; c.T = T; c.vec = vec;
+    int rc = air::launch(air::mlstm_gates_kernel, dim3(H, L), 256, 0, stream, c);
+    if (rc) return rc;
+    const int tiles = ((d + air::ML_TD - 1) / air::ML_TD) * ((dv + air::ML_TV - 1) / air::ML_TV);
+    cudaError_t err = cudaFuncSetAttribute(air::mlstm_states_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                           (int)air::ML_STATES_SMEM);
+    if (err != cudaSuccess) return (int)err;
+    rc = air::launch(air::mlstm_states_kernel, dim3(tiles, H, L), 128, air::ML_STATES_SMEM, stream, c);
+    if (rc) return rc;
+    AIR_DISPATCH(out_dtype, TO, {
+        auto kernel = air::mlstm_outputs_kernel<TO>;
+        err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)air::ML_OUT_SMEM);
+        if (err != cudaSuccess) return (int)err;
+        rc = air::launch(kernel, dim3(N, H, v_blocks), 256, air::ML_OUT_SMEM, stream, c);
+        if (rc || v_blocks == 1) return rc;
+        return air::launch(air::mlstm_finish_kernel<TO>, dim3(N, H), 128, 0, stream, c);
     });
     return 0;
 }

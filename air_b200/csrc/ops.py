@@ -49,6 +49,9 @@ _SIGNATURES = {
     "air_mlstm_step": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
                        c_float, c_float, c_void_p],
+    "air_mlstm_portions": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                           c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p],
     "air_latent_prepare": [c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                            c_void_p, c_void_p],
@@ -717,18 +720,13 @@ def residual_conv(h, weight, state, out, q_start, slots, max_tokens):
     return out
 
 
-def mlstm_step(proj, columns, i_bias, f_bias, weight, S, n, m, out, q_start, slots, cap, q_scale, eps):
-    """mLSTM's matrix memory (see mlstm.cu) for every entry of the batch, token after token, one block per head and
-    entry.  proj float32 [T, W]; columns: where q, k, v, g (the heads side by side), i and f (a logit per head) start in it;
-    i_bias, f_bias float32 [H]; weight float32 [H * dv]; the states S [slots, H, d, dv], n [slots, H, d], m [slots, H];
-    out [T, H * dv]: every head's read-out normalised, weighted and gated."""
+def _mlstm(proj, columns, i_bias, f_bias, weight, S, n, m, out):
     slots_n, H, d, dv = S.shape
-    T = out.shape[0]
     pp, ld = _columns(proj, "proj")
     need = {"q": H * d, "k": H * d, "v": H * dv, "g": H * dv, "i": H, "f": H}
     for c, width in need.items():
         if columns[c] + width > proj.shape[1]:
-            raise KernelError(f"mlstm_step: projection {c} does not fit")
+            raise KernelError(f"mlstm: projection {c} does not fit")
     _req(i_bias, "i_bias", (torch.float32,), (H,))
     _req(f_bias, "f_bias", (torch.float32,), (H,))
     _req(weight, "weight", (torch.float32,), (H * dv,))
@@ -736,12 +734,44 @@ def mlstm_step(proj, columns, i_bias, f_bias, weight, S, n, m, out, q_start, slo
     _req(n, "n", (torch.float32,), (slots_n, H, d))
     _req(m, "m", (torch.float32,), (slots_n, H))
     _req(out, "out", _FLOATS, (proj.shape[0], H * dv))
+    return (pp, ld, *(int(columns[c]) for c in "qkvgif"), i_bias.data_ptr(), f_bias.data_ptr(), weight.data_ptr(),
+            S.data_ptr(), n.data_ptr(), m.data_ptr(), out.data_ptr(), _DT[out.dtype]), (H, d, dv)
+
+
+def mlstm_step(proj, columns, i_bias, f_bias, weight, S, n, m, out, q_start, slots, cap, q_scale, eps):
+    """mLSTM's matrix memory (see mlstm.cu) for every entry of the batch (slots[e] < 0: skipped), token after token, one
+    block per head and entry.  proj float32 [T, W]; columns: where q, k, v, g (the heads side by side), i and f (a logit per
+    head) start in it; i_bias, f_bias float32 [H]; weight float32 [H * dv]; the states S [slots, H, d, dv], n [slots, H, d],
+    m [slots, H]; out [T, H * dv]: every head's read-out normalised, weighted and gated."""
+    args, (H, d, dv) = _mlstm(proj, columns, i_bias, f_bias, weight, S, n, m, out)
     _req(q_start, "q_start", _I32)
     _req(slots, "slots", _I32)
-    _check(_get("air_mlstm_step")(
-        pp, ld, *(int(columns[c]) for c in "qkvgif"), i_bias.data_ptr(), f_bias.data_ptr(), weight.data_ptr(), S.data_ptr(),
-        n.data_ptr(), m.data_ptr(), out.data_ptr(), _DT[out.dtype], q_start.data_ptr(), slots.data_ptr(), slots.shape[0],
-        H, d, dv, float(cap), float(q_scale), float(eps), _stream()), "mlstm_step")
+    _check(_get("air_mlstm_step")(*args, q_start.data_ptr(), slots.data_ptr(), slots.shape[0], H, d, dv, float(cap),
+                                  float(q_scale), float(eps), _stream()), "mlstm_step")
+    return out
+
+
+MLSTM_CHUNK = 64
+
+
+def mlstm_portions(proj, columns, i_bias, f_bias, weight, S, n, m, out, portions, chunks, cap, q_scale, eps):
+    """The same for portions of several tokens, in chunks whose rows are computed side by side: portions int32 [L, 4] =
+    (first row, tokens, slot, first chunk), chunks int32 [N, 2] = (first row, tokens), a portion's chunks of MLSTM_CHUNK
+    tokens (the last one shorter) one after the other.  Rows of other entries are left alone."""
+    global launches
+    args, (H, d, dv) = _mlstm(proj, columns, i_bias, f_bias, weight, S, n, m, out)
+    T, dev = proj.shape[0], proj.device
+    _req(portions, "portions", _I32, (None, 4))
+    _req(chunks, "chunks", _I32, (None, 2))
+    L, N = portions.shape[0], chunks.shape[0]
+    gates = torch.empty((3, H, T), dtype=torch.float32, device=dev)
+    chunk_S = torch.empty((N, H, d, dv), dtype=torch.float32, device=dev)
+    chunk_n = torch.empty((N, H, d), dtype=torch.float32, device=dev)
+    o = torch.empty((T, H, dv), dtype=torch.float32, device=dev) if dv > 128 else None
+    _check(_get("air_mlstm_portions")(*args, portions.data_ptr(), L, chunks.data_ptr(), N, gates.data_ptr(),
+                                      chunk_S.data_ptr(), chunk_n.data_ptr(), _ptr(o), T, H, d, dv, float(cap),
+                                      float(q_scale), float(eps), _stream()), "mlstm_portions")
+    launches += 2 if o is None else 3
     return out
 
 

@@ -40,35 +40,30 @@ struct StreamNormArgs {
 
 constexpr int STREAMS_MAX = 16;
 
-// N columns of all streams of a row: mixed, written, and folded into u.  NS: the number of streams (0: p.S of them).
+template <int N> __device__ __forceinline__ void load_columns(const float* q, float (&v)[N]) {
+    if constexpr (N == 4) load4(q, v);
+    else v[0] = *q;
+}
+template <int N> __device__ __forceinline__ void store_columns(float* q, const float (&v)[N]) {
+    if constexpr (N == 4) store4(q, v);
+    else *q = v[0];
+}
+
+// N columns of all streams of a row: mixed, written, and folded into u.  NS: the number of streams, all at compile-time
+// indices; 0: p.S of them, in a loop.
 template <int NS, int N>
 __device__ __forceinline__ void stream_columns(const StreamNormArgs& p, size_t src, int i, const float* coef, float (&u)[N]) {
-    constexpr int M = NS ? NS : STREAMS_MAX;
     const int S = NS ? NS : p.S;
-    auto ld = [](const float* q, float (&v)[N]) {
-        if constexpr (N == 4) load4(q, v);
-        else v[0] = *q;
-    };
-    auto st = [](float* q, const float (&v)[N]) {
-        if constexpr (N == 4) store4(q, v);
-        else *q = v[0];
-    };
-    float x[M][N], y[N];
-#pragma unroll
-    for (int s = 0; s < M; ++s)
-        if (s < S) {
-            if (s == 0 || p.x_stride) ld(p.x + s * p.x_stride + src + i, x[s]);
-            else {
-#pragma unroll
-                for (int j = 0; j < N; ++j) x[s][j] = x[0][j];
-            }
-        }
+    constexpr int UN = NS ? NS : 1;
+    float x[NS ? NS : STREAMS_MAX][N], y[N];
+#pragma unroll UN
+    for (int s = 0; s < S; ++s) load_columns<N>(p.x + s * p.x_stride + src + i, x[s]);
     if (p.y) {
-        ld(p.y + src + i, y);
+        load_columns<N>(p.y + src + i, y);
 #pragma unroll 4
-        for (int q = 1; q < p.y_parts; ++q) {
+        for (int q = 1; q < p.y_parts; ++q) {                                        // (loads ahead, sums in order)
             float t[N];
-            ld(p.y + q * p.part_stride + src + i, t);
+            load_columns<N>(p.y + q * p.part_stride + src + i, t);
 #pragma unroll
             for (int j = 0; j < N; ++j) y[j] += t[j];
         }
@@ -76,33 +71,22 @@ __device__ __forceinline__ void stream_columns(const StreamNormArgs& p, size_t s
     const float *mix = coef, *out_w = coef + S * S, *read = out_w + S;
 #pragma unroll
     for (int j = 0; j < N; ++j) u[j] = 0.f;
-#pragma unroll
-    for (int t = 0; t < M; ++t) {
-        if (t >= S) break;
+#pragma unroll UN
+    for (int t = 0; t < S; ++t) {
         float v[N];
-        if (p.mix) {
 #pragma unroll
-            for (int j = 0; j < N; ++j) v[j] = 0.f;
+        for (int j = 0; j < N; ++j) v[j] = p.mix ? 0.f : x[t][j];
+        if (p.mix)
+#pragma unroll UN
+            for (int s = 0; s < S; ++s)
 #pragma unroll
-            for (int s = 0; s < M; ++s)
-                if (s < S) {
-                    const float m = mix[s * S + t];
+                for (int j = 0; j < N; ++j) v[j] = fmaf(mix[s * S + t], x[s][j], v[j]);
+        if (p.y)
 #pragma unroll
-                    for (int j = 0; j < N; ++j) v[j] = fmaf(m, x[s][j], v[j]);
-                }
-        } else {
+            for (int j = 0; j < N; ++j) v[j] = fmaf(out_w[t], y[j], v[j]);
+        if (p.h_out) store_columns<N>(p.h_out + t * p.h_stride + src + i, v);
 #pragma unroll
-            for (int j = 0; j < N; ++j) v[j] = x[t][j];
-        }
-        if (p.y) {
-            const float o = out_w[t];
-#pragma unroll
-            for (int j = 0; j < N; ++j) v[j] = fmaf(o, y[j], v[j]);
-        }
-        if (p.h_out) st(p.h_out + t * p.h_stride + src + i, v);
-        const float r = read[t];
-#pragma unroll
-        for (int j = 0; j < N; ++j) u[j] = fmaf(r, v[j], u[j]);
+        for (int j = 0; j < N; ++j) u[j] = fmaf(read[t], v[j], u[j]);
     }
 }
 

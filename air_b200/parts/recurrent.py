@@ -2,12 +2,13 @@
 token updates and reads (linear attention with gates), and the short convolutions in front of it."""
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from ..config.model_config import ConfigError
 from ..csrc import ops
 from ..weights.loader import TensorSpec
-from .base import Mixer, SlotState
+from .base import HostBatch, Mixer, Plan, SlotState
 from .linear import Linear
 from .registry import register_mixer
 
@@ -300,6 +301,9 @@ class MLSTM(_StateMixer):
     then each head's o / sqrt(mean(o^2) + eps), all heads times norm, times sigmoid(W_g x), and the output projection.
     S, n and m are the request's state, 32-bit; the gates, the recurrence, the norm and the read-out are 32-bit.
 
+    Single tokens and portions of fewer than PORTION tokens take one kernel, token after token; longer portions are cut into
+    chunks whose rows are computed side by side from the states ahead of them (csrc/mlstm.cu).
+
     params: hidden, heads, head_dim, v_dim, gate_cap, eps.  Tensors: <prefix>q, k [heads*head_dim, hidden]; v, g
     [heads*v_dim, hidden]; i, f [heads, hidden]; i.b, f.b [heads]; norm [heads*v_dim]; o [hidden, heads*v_dim]."""
 
@@ -314,6 +318,28 @@ class MLSTM(_StateMixer):
     def cache_needs(self):
         H, d, dv = self.heads, self.head_dim, self.v_dim
         return (SlotState((H, d, dv)), SlotState((H, d)), SlotState((H,)))
+
+    PORTION = 16
+
+    def plan_key(self):
+        return ("mlstm.chunks", self.PORTION)
+
+    def plan(self, batch: HostBatch) -> Plan:
+        """portions [L, 4] = (first row, tokens, slot, first chunk) of the entries of at least PORTION tokens, chunks [N, 2]
+        = (first row, tokens) of theirs; short_slots: the slot of every other entry, -1 for the portions."""
+        portions, chunks, short_slots = [], [], []
+        for i, n in enumerate(batch.counts):
+            if n < self.PORTION:
+                short_slots.append(batch.slots[i])
+                continue
+            short_slots.append(-1)
+            first = batch.q_start[i]
+            portions.append((first, n, batch.slots[i], len(chunks)))
+            chunks += [(first + at, min(ops.MLSTM_CHUNK, n - at)) for at in range(0, n, ops.MLSTM_CHUNK)]
+        return Plan(arrays={"portions": np.asarray(portions, dtype=np.int32).reshape(-1, 4),
+                            "chunks": np.asarray(chunks, dtype=np.int32).reshape(-1, 2),
+                            "short_slots": np.asarray(short_slots, dtype=np.int32)},
+                    values={"long": bool(portions), "short": len(portions) < len(batch.counts)})
 
     def tensor_specs(self):
         p, e, H, d, dv = self.prefix, self.hidden, self.heads, self.head_dim, self.v_dim
@@ -338,10 +364,16 @@ class MLSTM(_StateMixer):
 
     def forward(self, x, ctx, cache, owns_cache=True):
         memory, key_sum, level = cache
-        T = x.shape[0]
         proj = self.proj.f32(x)
-        y = torch.empty((T, self.heads * self.v_dim), dtype=self.rt.dtype, device=x.device)
-        ops.mlstm_step(proj, {n: at for n, (at, _) in self.columns.items()}, self.i_bias, self.f_bias, self.norm_weight,
-                       memory.state, key_sum.state, level.state, y, ctx.q_start, ctx.slots, self.cap,
-                       self.head_dim ** -0.5, self.eps)
+        y = torch.empty((x.shape[0], self.heads * self.v_dim), dtype=self.rt.dtype, device=x.device)
+        args = (proj, {n: at for n, (at, _) in self.columns.items()}, self.i_bias, self.f_bias, self.norm_weight,
+                memory.state, key_sum.state, level.state, y)
+        numbers = (self.cap, self.head_dim ** -0.5, self.eps)
+        plan = ctx.plans.get(self.plan_key())
+        if plan is None or not plan.long:
+            ops.mlstm_step(*args, ctx.q_start, ctx.slots, *numbers)
+        else:
+            if plan.short:
+                ops.mlstm_step(*args, ctx.q_start, plan.short_slots, *numbers)
+            ops.mlstm_portions(*args, plan.portions, plan.chunks, *numbers)
         return self.o.f32_sums(y)

@@ -64,7 +64,8 @@ def input_convolution(h, w):
     y = h.copy()
     for j in range(taps):
         back = taps - 1 - j
-        y[back:] += w[:, j] * h[:len(h) - back]
+        if back < len(h):
+            y[back:] += w[:, j] * h[:len(h) - back]
     return y
 
 
