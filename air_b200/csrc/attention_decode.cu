@@ -260,7 +260,8 @@ template <int D, int CHUNK>
 __global__ void decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                       const int* __restrict__ token_seq, __nv_bfloat16* __restrict__ out, int H,
                                       int splits, const float* __restrict__ sink, const float* __restrict__ gate,
-                                      int ldg) {
+                                      int ldg, const TurnBack turn) {
+    __shared__ float row[D];
     pdl_enter(TR_ATT_COMBINE);
     const int t = blockIdx.y, h = blockIdx.x;
     const size_t base = ((size_t)t * H + h) * splits;
@@ -301,9 +302,21 @@ __global__ void decode_combine_kernel(const float* __restrict__ part_o, const fl
             ll = ll * keep + exp2f(s2 - top);
             acc *= keep;
         }
+        if (turn.freq) {
+            row[col] = acc / ll;
+            continue;
+        }
         // (a gate per output element: the logit's sigmoid multiplies as the row is written)
         const float g = gate && slot >= 0 ? 1.f / (1.f + expf(-gate[(size_t)t * ldg + h * D + col])) : 1.f;
         if (slot >= 0) out[((size_t)t * H + h) * D + col] = __float2bfloat16_rn(acc / ll * g);
+    }
+    if (turn.freq) {         // the whole row first, then its elements turned back in pairs
+        __syncthreads();
+        if (slot < 0) return;
+        for (int col = threadIdx.x; col < D; col += blockDim.x) {
+            const float g = gate ? 1.f / (1.f + expf(-gate[(size_t)t * ldg + h * D + col])) : 1.f;
+            out[((size_t)t * H + h) * D + col] = __float2bfloat16_rn(turned_back(row, col, turn, turn.positions[t]) * g);
+        }
     }
 }
 
@@ -311,16 +324,16 @@ __global__ void decode_combine_kernel(const float* __restrict__ part_o, const fl
 template <int D>
 int launch_combine(const float* part_o, const float* part_ml, const int* token_seq, __nv_bfloat16* out, int T, int H,
                    int splits, cudaStream_t stream, const float* sink = nullptr, const float* gate = nullptr,
-                   int ldg = 0) {
+                   int ldg = 0, const TurnBack& turn = TurnBack{nullptr, 0, 0, nullptr}) {
     const int threads = D >= 128 ? 128 : 64;
     if (splits <= 8)
         return launch(decode_combine_kernel<D, 8>, dim3(H, T), threads, 0, stream, part_o, part_ml, token_seq, out, H,
-                      splits, sink, gate, ldg);
+                      splits, sink, gate, ldg, turn);
     if (splits <= 16)
         return launch(decode_combine_kernel<D, 16>, dim3(H, T), threads, 0, stream, part_o, part_ml, token_seq, out, H,
-                      splits, sink, gate, ldg);
+                      splits, sink, gate, ldg, turn);
     return launch(decode_combine_kernel<D, 32>, dim3(H, T), threads, 0, stream, part_o, part_ml, token_seq, out, H,
-                  splits, sink, gate, ldg);
+                  splits, sink, gate, ldg, turn);
 }
 
 template <int D>
@@ -387,12 +400,15 @@ AIR_API int air_decode_combine(const float* part_o, const float* part_ml, const 
 // sigmoid(gate[t][h * D + col]) on every output element (gate float32 with rows of ldg floats, or null).
 AIR_API int air_decode_combine_sink(const float* part_o, const float* part_ml, const int* token_seq, void* out, int T,
                                     int H, int D, int splits, const float* sink, const float* gate, int ldg,
+                                    const double* turn_freq, int turn_rot, int turn_pairing, const int* positions,
                                     cudaStream_t stream) {
     using namespace air;
+    const TurnBack turn{turn_freq, turn_rot, turn_pairing, positions};
+    if (turn_freq && (turn_rot < 0 || turn_rot > D || (turn_rot & 1) || !positions)) return AIR_ERR_BAD_ARGUMENT;
     switch (D) {
-        case 64: return launch_combine<64>(part_o, part_ml, token_seq, (__nv_bfloat16*)out, T, H, splits, stream, sink, gate, ldg);
-        case 128: return launch_combine<128>(part_o, part_ml, token_seq, (__nv_bfloat16*)out, T, H, splits, stream, sink, gate, ldg);
-        case 256: return launch_combine<256>(part_o, part_ml, token_seq, (__nv_bfloat16*)out, T, H, splits, stream, sink, gate, ldg);
+        case 64: return launch_combine<64>(part_o, part_ml, token_seq, (__nv_bfloat16*)out, T, H, splits, stream, sink, gate, ldg, turn);
+        case 128: return launch_combine<128>(part_o, part_ml, token_seq, (__nv_bfloat16*)out, T, H, splits, stream, sink, gate, ldg, turn);
+        case 256: return launch_combine<256>(part_o, part_ml, token_seq, (__nv_bfloat16*)out, T, H, splits, stream, sink, gate, ldg, turn);
         default: return AIR_ERR_BAD_ARGUMENT;
     }
 }

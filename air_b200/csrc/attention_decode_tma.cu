@@ -422,6 +422,7 @@ int launch_decode_tma(const CUtensorMap& map, const FreshQkv& fresh, const void*
 // The merge of the splits (attention_decode.cu).
 extern "C" int air_decode_combine_sink(const float* part_o, const float* part_ml, const int* token_seq, void* out, int T,
                                        int H, int D, int splits, const float* sink, const float* gate, int ldg,
+                                       const double* turn_freq, int turn_rot, int turn_pairing, const int* positions,
                                        cudaStream_t stream);
 extern "C" int air_decode_combine(const float* part_o, const float* part_ml, const int* token_seq, void* out, int T,
                                   int H, int D, int splits, cudaStream_t stream);
@@ -432,13 +433,15 @@ static int decode_attention_tma(const FreshQkv& fresh, const void* q, const void
                                 const int* block_table, int max_blocks, const int* token_seq, const int* positions,
                                 void* out, float* part_o, float* part_ml, int T, int H, int K, int D, int P, int window,
                                 float scale, float softcap, int splits, int* status, cudaStream_t stream,
-                                const float* sink = nullptr, const float* gate = nullptr, int ldg = 0) {
+                                const float* sink = nullptr, const float* gate = nullptr, int ldg = 0,
+                                const TurnBack& turn = TurnBack{nullptr, 0, 0, nullptr}) {
     if (T <= 0) return 0;
     if (H <= 0 || K <= 0 || H % K || P % 16 || (P < 64 ? 64 % P : P % 64) || splits < 1 || T > 65535 ||
         (splits > 1 && (!part_o || !part_ml)) || ((uintptr_t)cache & 15))
         return AIR_ERR_BAD_ARGUMENT;
-    // a sink or gates enter where the splits are merged: the keys are then split in two parts at least
-    if ((sink || gate) && splits < 2) return AIR_ERR_BAD_ARGUMENT;
+    // a sink, gates or a turn back enter where the splits are merged: the keys are then split in two parts at least
+    const bool extra = sink || gate || turn.freq;
+    if (extra && splits < 2) return AIR_ERR_BAD_ARGUMENT;
     CUtensorMap map;
     const int map_rc = tensor_map_2d(&map, cache, pages * 2 * K * P, D, P < DT_TILE ? P : DT_TILE);
     if (map_rc) return map_rc;
@@ -460,8 +463,9 @@ static int decode_attention_tma(const FreshQkv& fresh, const void* q, const void
             return AIR_ERR_BAD_ARGUMENT;
     }
     if (rc == 0 && splits > 1)
-        rc = (sink || gate) ? air_decode_combine_sink(part_o, part_ml, token_seq, out, T, H, D, splits, sink, gate, ldg, stream)
-                            : air_decode_combine(part_o, part_ml, token_seq, out, T, H, D, splits, stream);
+        rc = extra ? air_decode_combine_sink(part_o, part_ml, token_seq, out, T, H, D, splits, sink, gate, ldg, turn.freq,
+                                             turn.rot, turn.pairing, positions, stream)
+                   : air_decode_combine(part_o, part_ml, token_seq, out, T, H, D, splits, stream);
     return rc;
 }
 
@@ -479,16 +483,19 @@ AIR_API int air_decode_attention_tma(const void* q, const void* cache, long long
 }
 
 // The same with one more term exp(sink[h]) in every head's softmax denominator (sink float32 [H] or null) and the
-// output multiplied, element by element, by sigmoid(gate[t][h * D + col]) (gate float32, rows of ldg floats, or null);
-// both enter where the key splits are merged, so splits >= 2.
+// output multiplied, element by element, by sigmoid(gate[t][h * D + col]) (gate float32, rows of ldg floats, or null), and
+// ahead of the gate the first turn_rot elements of every head turned back by the token's position (turn_freq float64
+// [turn_rot / 2], or null; see TurnBack); all enter where the key splits are merged, so splits >= 2.
 AIR_API int air_decode_attention_tma_sink(const void* q, const void* cache, long long pages, const int* block_table,
                                           int max_blocks, const int* token_seq, const int* positions, void* out,
                                           float* part_o, float* part_ml, int T, int H, int K, int D, int P, int window,
                                           float scale, float softcap, int splits, int* status, const float* sink,
-                                          const float* gate, int ldg, cudaStream_t stream) {
+                                          const float* gate, int ldg, const double* turn_freq, int turn_rot,
+                                          int turn_pairing, cudaStream_t stream) {
     return air::decode_attention_tma(air::FreshQkv{nullptr, 0, 0, nullptr, nullptr, nullptr}, q, cache, pages,
                                      block_table, max_blocks, token_seq, positions, out, part_o, part_ml, T, H, K, D, P,
-                                     window, scale, softcap, splits, status, stream, sink, gate, ldg);
+                                     window, scale, softcap, splits, status, stream, sink, gate, ldg,
+                                     air::TurnBack{turn_freq, turn_rot, turn_pairing, positions});
 }
 
 // The same from the q/k/v product's output instead of q: qkv float32 [parts][T][(H + 2 K) D] (partial sums that

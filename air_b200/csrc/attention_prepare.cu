@@ -104,7 +104,7 @@ AIR_API int air_trace_set_attention_prepare(unsigned long long* buffer) { return
 //   q and k heads: x <- x / sqrt(mean(x^2) + eps) * w (w [dk], one for all heads of q, one for all heads of k; absent:
 //   no norm); then the first `rot` elements are rotated, pair j by the angle position * freq[j], where pair j is
 //   (2j, 2j + 1) (pairing 1) or (j, j + rot/2) (pairing 0); cos and sin are multiplied by `magnitude`.  The angle is
-//   the product of the position and a 64-bit frequency, and its cos and sin are taken in 64-bit, once per token.
+//   the product of the position and a 64-bit frequency, taken in 64-bit (cos_sin_of), once per token.
 //   v is copied.  Pages as above.  A bias (float32 [(H + G) dk + G dv]) is added to q, k and v first.  With `whole`
 //   the norm is taken over ALL heads of q at once (and all heads of k): x / sqrt(mean over H dk (x^2) + eps) * w with
 //   w of that whole size (q_w [H dk], k_w [G dk]).
@@ -140,19 +140,14 @@ qk_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __
     const float* in = proj + (size_t)t * ld;
     const int half = rot / 2;
     for (int j = threadIdx.x; j < half; j += blockDim.x) {
-        double s, c;
-        sincos((double)pos * freq[j], &s, &c);
-        cs[j] = (float)c * magnitude;
-        sn[j] = (float)s * magnitude;
+        float s, c;
+        cos_sin_of((double)pos, freq[j], c, s);
+        cs[j] = c * magnitude;
+        sn[j] = s * magnitude;
     }
     const int vhalf = v_rot / 2;
     if (write_kv)
-        for (int j = threadIdx.x; j < vhalf; j += blockDim.x) {
-            double s, c;
-            sincos((double)pos * v_freq[j], &s, &c);
-            vcs[j] = (float)c;
-            vsn[j] = (float)s;
-        }
+        for (int j = threadIdx.x; j < vhalf; j += blockDim.x) cos_sin_of((double)pos, v_freq[j], vcs[j], vsn[j]);
     TO* kdst = nullptr;
     TO* vdst = nullptr;
     if (write_kv) {
@@ -268,12 +263,8 @@ turn_heads_kernel(TX* __restrict__ x, const double* __restrict__ freq, int rot, 
     const int t = blockIdx.x;
     if (token_seq[t] < 0) return;
     const int half = rot / 2;
-    for (int j = threadIdx.x; j < half; j += blockDim.x) {
-        double s, c;
-        sincos(sign * (double)positions[t] * freq[j], &s, &c);
-        cs[j] = (float)c;
-        sn[j] = (float)s;
-    }
+    for (int j = threadIdx.x; j < half; j += blockDim.x)
+        cos_sin_of(sign * (double)positions[t], freq[j], cs[j], sn[j]);
     __syncthreads();
     for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
         const int h = idx / half, j = idx % half;

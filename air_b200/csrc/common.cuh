@@ -131,6 +131,33 @@ __device__ __forceinline__ float gated_activation(float g, float u, float alpha,
     return g / (1.f + expf(-alpha * g)) * (u + shift);
 }
 
+// cos and sin of position * freq.  The angle is a 64-bit product; only its fraction of a turn, which 32 bits hold to 2e-7
+// of a radian whatever the position, goes to the 32-bit functions (those of the 64-bit angle take ten times as long).
+__device__ __forceinline__ void cos_sin_of(double position, double freq, float& c, float& s) {
+    double turns = position * freq * 0.15915494309189535;
+    turns -= rint(turns);
+    sincospif(2.f * (float)turns, &s, &c);
+}
+
+// A rotation of a finished row of attention outputs, backwards by the query's position (values that were rotated by their
+// own positions): the first `rot` elements, pair j = (j, j + rot/2) (pairing 0) or (2j, 2j + 1) (pairing 1), by
+// -position * freq[j].  freq null: none.
+struct TurnBack {
+    const double* freq;
+    int rot, pairing;
+    const int* positions;
+};
+__device__ __forceinline__ float turned_back(const float* row, int col, const TurnBack& b, int position) {
+    if (col >= b.rot) return row[col];
+    const int half = b.rot / 2;
+    const bool first = b.pairing == 0 ? col < half : !(col & 1);
+    const int j = b.pairing == 0 ? (first ? col : col - half) : col >> 1;
+    const int other = b.pairing == 0 ? (first ? col + half : col - half) : col ^ 1;
+    float c, s;
+    cos_sin_of(-(double)position, b.freq[j], c, s);
+    return first ? row[col] * c - row[other] * s : row[col] * c + row[other] * s;
+}
+
 // Sum over a block of up to 1024 threads; every thread gets the result.  The order of
 // the additions depends only on the block size, never on the data or the grid.
 __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 32 floats */) {

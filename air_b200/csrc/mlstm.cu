@@ -1,7 +1,7 @@
 // The matrix memory of mLSTM over the step's flat batch: every entry brings the next tokens of one request, rows
 // q_start[e] .. q_start[e + 1], and slots[e] is the request's row of the states (negative: padding, skipped).  32-bit
-// throughout.  proj [T, ld] holds per token the projections q, k (H heads of d), v, g (H heads of dv) and one logit each
-// for the input and the forget gate of every head, each at a column of its own.  Per head and token:
+// throughout.  x holds per token the projections q, k (H heads of d), v, g (H heads of dv), z one logit each for the input
+// and the forget gate of every head, each at a column of its own.  Per head and token:
 //
 //   i = c tanh((zi + bi) / c),  f = log sigmoid(c tanh((zf + bf) / c)),  m' = max(f + m, i),
 //   a = exp(f + m - m'),  b = exp(i - m'),
@@ -20,35 +20,22 @@
 // A_t = a_first .. a_t, a chunk's read-outs are W V + A (Q S_chunk) and n . q = row sum of W + A (q . n_chunk), with S_chunk
 // and n_chunk the states ahead of the chunk: 32-bit products on the CUDA cores, rows of different chunks side by side.
 //
-//   mlstm_gates_kernel   a, b and exp(-m) of every token: block (head, portion); m by a parallel scan of the maps
-//                        m -> max(F + m, M) (64-bit sums), 256 tokens at a time
+//   mlstm_gates_kernel   a, b and exp(-m) of every token, its b P(t, end) and its A: block (head, portion); m by a parallel scan of the maps
+//                        m -> max(F + m, M) (64-bit sums), 512 tokens at a time
 //   mlstm_states_kernel  the states ahead of every chunk: block (tile of 32 x 64 of S, head, portion), the tile in
 //                        registers, chunk after chunk: S <- (product of the chunk's a) S + sum_s b_s P(s, end) k_s v_s^T
 //   mlstm_outputs_kernel block (chunk, head, 128 columns of v): the read-outs; where a head's v fits one block also the norm,
 //                        the weight and the gate, else mlstm_finish_kernel does those
-#include "common.cuh"
+// A bfloat16 engine takes the same steps on the tensor cores (mlstm_tc.cu).
+#include "mlstm.cuh"
 
 namespace air {
-
-constexpr int ML_THREADS = 256;
-
-struct MlstmArgs {
-    const float* proj; int ld;
-    int cq, ck, cv, cg, ci, cf;        // the columns at which the projections start
-    const float* ib; const float* fb;  // [H]
-    const float* w;                    // [H * dv]
-    float* S; float* n; float* m;
-    void* y;                           // [T, H * dv]
-    const int* q_start; const int* slots;
-    int H, d, dv;
-    float cap, q_scale, eps;
-};
 
 __device__ __forceinline__ float ml_log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float ml_capped(float z, float cap) { return cap * tanhf(z / cap); }
 
 // N: columns of S per access (4 where dv and the pointers allow it).
-template <typename TO, int N>
+template <typename TX, typename TO, int N>
 __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(const MlstmArgs p) {
     __shared__ float scratch[32];
     extern __shared__ __align__(16) float smem[];
@@ -65,15 +52,16 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(const MlstmArgs 
     float m = p.m[(size_t)slot * p.H + h];
     const float ib = p.ib[h], fb = p.fb[h];
     for (int t = 0; t < cnt; ++t) {
-        const float* row = p.proj + (size_t)(q0 + t) * p.ld;
-        const float li = ml_capped(row[p.ci + h] + ib, p.cap);
-        const float lf = ml_log_sigmoid(ml_capped(row[p.cf + h] + fb, p.cap));
+        const TX* row = (const TX*)p.x + (size_t)(q0 + t) * p.ldx;
+        const float* zrow = p.z + (size_t)(q0 + t) * p.ldz;
+        const float li = ml_capped(zrow[p.ci + h] + ib, p.cap);
+        const float lf = ml_log_sigmoid(ml_capped(zrow[p.cf + h] + fb, p.cap));
         const float mn = fmaxf(lf + m, li);
         const float a = expf(lf + m - mn), b = expf(li - mn);
         m = mn;
         float nq = 0.f;
         for (int r = tid; r < d; r += ML_THREADS) {
-            const float k = b * row[p.ck + h * d + r], q = row[p.cq + h * d + r] * p.q_scale;
+            const float k = b * to_float(row[p.ck + h * d + r]), q = to_float(row[p.cq + h * d + r]) * p.q_scale;
             sk[r] = k;
             sq[r] = q;
             const float v = fmaf(a, nn[r], k);
@@ -90,7 +78,7 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(const MlstmArgs 
             if (rg < RG && c < cols) {
                 float v[N];
 #pragma unroll
-                for (int j = 0; j < N; ++j) v[j] = row[p.cv + h * dv + c * N + j];
+                for (int j = 0; j < N; ++j) v[j] = to_float(row[p.cv + h * dv + c * N + j]);
                 float* col = S + (size_t)c * N;
                 constexpr int U = 8;                      // rows of a thread under way at once
                 for (int r0 = rg; r0 < d; r0 += U * RG) {
@@ -134,7 +122,7 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(const MlstmArgs 
         const float scale = 1.f / sqrtf(block_sum(ss, scratch) / (float)dv + p.eps);
         TO* y = (TO*)p.y + ((size_t)(q0 + t) * p.H + h) * dv;
         for (int c = tid; c < dv; c += ML_THREADS) {
-            const float g = row[p.cg + h * dv + c];
+            const float g = to_float(row[p.cg + h * dv + c]);
             y[c] = from_float<TO>(so[c] * scale * p.w[h * dv + c] / (1.f + expf(-g)));
         }
     }
@@ -142,40 +130,36 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(const MlstmArgs 
 }
 
 // ------------------------------------------------------------------ longer portions
-constexpr int ML_C = 64;                   // tokens of a chunk
 constexpr int ML_TD = 32, ML_TV = 64;      // the tile of S that a block of mlstm_states_kernel holds
 constexpr int ML_OV = 128;                 // columns of v per block of mlstm_outputs_kernel
 constexpr int ML_KS = 64;                  // key channels staged at a time there
 constexpr int ML_LD = ML_KS + 4, ML_LV = ML_OV + 4;
 
-struct MlstmChunkArgs {
-    MlstmArgs p;
-    const int* portions;                   // [L, 4]: first row, tokens, slot, first chunk
-    const int* chunks;                     // [N, 2]: first row, tokens
-    float* gates;                          // [3, H, T]: a, b, exp(-m)
-    float* chunk_S; float* chunk_n;        // [N, H, d, dv], [N, H, d]: the states ahead of every chunk
-    float* o;                              // [T, H, dv] read-outs where a head's v takes several blocks, else null
-    int T, vec;                            // vec: proj's rows and columns allow 16-byte accesses
-};
+constexpr int ML_GT = 512;                 // threads of mlstm_gates_kernel
 
-__global__ void __launch_bounds__(256) mlstm_gates_kernel(const MlstmChunkArgs c) {
-    __shared__ double wF[8], wM[8], mt[257];
+__global__ void __launch_bounds__(ML_GT) mlstm_gates_kernel(const MlstmChunkArgs c) {
+    __shared__ double wF[ML_GT / 32], wM[ML_GT / 32], mt[ML_GT + 1];
+    __shared__ float wP[ML_GT / 32];
     pdl_enter(TR_MLSTM);
     const MlstmArgs& p = c.p;
     const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int row0 = c.portions[blockIdx.y * 4], cnt = c.portions[blockIdx.y * 4 + 1], slot = c.portions[blockIdx.y * 4 + 2];
     const float ib = p.ib[h], fb = p.fb[h];
     double carry = (double)p.m[(size_t)slot * p.H + h];
-    float *ga = c.gates + (size_t)h * c.T, *gb = ga + (size_t)p.H * c.T, *ge = gb + (size_t)p.H * c.T;
-    for (int t0 = 0; t0 < cnt; t0 += 256) {
+    const size_t plane = (size_t)p.H * c.T;
+    float* g = c.gates + (size_t)h * c.T + row0;
+    auto logit = [&](int t, int col) { return t < cnt ? p.z[(size_t)(row0 + t) * p.ldz + col + h] : 0.f; };
+    float zi = logit(tid, p.ci), zf = logit(tid, p.cf);
+    for (int t0 = 0; t0 < cnt; t0 += ML_GT) {
         const int t = t0 + tid;
         // a place behind the portion's end leaves m as it is: F = 0, M far below
         float lf = 0.f, li = -1e30f;
         if (t < cnt) {
-            const float* row = p.proj + (size_t)(row0 + t) * p.ld;
-            li = ml_capped(row[p.ci + h] + ib, p.cap);
-            lf = ml_log_sigmoid(ml_capped(row[p.cf + h] + fb, p.cap));
+            li = ml_capped(zi + ib, p.cap);
+            lf = ml_log_sigmoid(ml_capped(zf + fb, p.cap));
         }
+        zi = logit(t + ML_GT, p.ci);       // (the next tokens' logits are on their way meanwhile)
+        zf = logit(t + ML_GT, p.cf);
         double F = lf, M = li;
 #pragma unroll
         for (int off = 1; off < 32; off <<= 1) {
@@ -193,15 +177,38 @@ __global__ void __launch_bounds__(256) mlstm_gates_kernel(const MlstmChunkArgs c
         m = fmax(F + m, M);
         mt[tid + 1] = m;
         __syncthreads();
-        if (t < cnt) {
-            ga[row0 + t] = expf((float)((double)lf + mt[tid] - m));
-            gb[row0 + t] = expf((float)((double)li - m));
-            ge[row0 + t] = expf(-(float)m);
+        const float a = t < cnt ? expf((float)((double)lf + mt[tid] - m)) : 1.f;
+        carry = mt[ML_GT];
+        // products over the token's chunk (two warps): of everything up to it, and of everything behind it
+        float upto = a, behind = a;
+#pragma unroll
+        for (int off = 1; off < 32; off <<= 1) {
+            const float u = __shfl_up_sync(0xffffffffu, upto, off), b = __shfl_down_sync(0xffffffffu, behind, off);
+            if (lane >= off) upto *= u;
+            if (lane + off < 32) behind *= b;
         }
-        carry = mt[256];
+        if (lane == 31) wP[warp] = upto;
+        behind = __shfl_down_sync(0xffffffffu, behind, 1);
+        if (lane == 31) behind = 1.f;
+        __syncthreads();
+        if (warp & 1) upto *= wP[warp - 1];
+        else behind *= wP[warp + 1];
+        if (t < cnt) {
+            const float b = expf((float)((double)li - m));
+            g[t] = a;
+            g[plane + t] = b;
+            g[2 * plane + t] = expf(-(float)m);
+            g[3 * plane + t] = b * behind;
+            g[4 * plane + t] = upto;
+        }
         __syncthreads();
     }
     if (tid == 0) p.m[(size_t)slot * p.H + h] = (float)carry;
+}
+
+// The gates of L portions: what every road of portions starts with.
+int launch_mlstm_gates(const MlstmChunkArgs& c, int L, cudaStream_t stream) {
+    return launch(mlstm_gates_kernel, dim3(c.p.H, L), ML_GT, 0, stream, c);
 }
 
 __device__ __forceinline__ void ml_cp16(void* smem, const void* gmem) {
@@ -235,14 +242,12 @@ __device__ __forceinline__ void ml_stage(float* dst, const float* src, size_t ld
     }
 }
 
-constexpr size_t ML_STATES_SMEM = sizeof(float) * (2 * ML_C * (ML_TD + ML_TV) + ML_C + 1);
+constexpr size_t ML_STATES_SMEM = sizeof(float) * 2 * (ML_C * (ML_TD + ML_TV) + ML_C + 4);
 
 // 128 threads, 4 x 4 numbers of the tile each.
 __global__ void __launch_bounds__(128) mlstm_states_kernel(const MlstmChunkArgs c) {
     extern __shared__ __align__(16) float smem[];
-    float* const sk[2] = {smem, smem + ML_C * ML_TD};
-    float* const sv[2] = {smem + 2 * ML_C * ML_TD, smem + 2 * ML_C * ML_TD + ML_C * ML_TV};
-    float* const se = smem + 2 * ML_C * (ML_TD + ML_TV);
+    constexpr int BUF = ML_C * (ML_TD + ML_TV) + ML_C + 4;       // a chunk: k, v, b P(s, end), the product of its a
     pdl_enter(TR_MLSTM);
     const MlstmArgs& p = c.p;
     const int d = p.d, dv = p.dv, tid = threadIdx.x, h = blockIdx.y;
@@ -263,13 +268,21 @@ __global__ void __launch_bounds__(128) mlstm_states_kernel(const MlstmChunkArgs 
         for (int j = 0; j < 4; ++j)
             acc[i][j] = (r0 + ty * 4 + i < d && v0 + tx * 4 + j < dv) ? at(S, i)[j] : 0.f;
     if (has_n) nacc = nn[r0 + tid];
+    const size_t plane = (size_t)p.H * c.T;
+    const float* ga = c.gates + (size_t)h * c.T + row0;
     auto stage = [&](int t0, int b) {
-        const float* src = p.proj + (size_t)(row0 + t0) * p.ld;
-        ml_stage<ML_TD, ML_TD, 128>(sk[b], src + p.ck + h * d + r0, p.ld, ML_C, cnt - t0, d - r0, c.vec);
-        ml_stage<ML_TV, ML_TV, 128>(sv[b], src + p.cv + h * dv + v0, p.ld, ML_C, cnt - t0, dv - v0, c.vec);
+        const float* src = (const float*)p.x + (size_t)(row0 + t0) * p.ldx;
+        float *sk = smem + b * BUF, *sv = sk + ML_C * ML_TD, *se = sv + ML_C * ML_TV;
+        ml_stage<ML_TD, ML_TD, 128>(sk, src + p.ck + h * d + r0, p.ldx, ML_C, cnt - t0, d - r0, c.vec);
+        ml_stage<ML_TV, ML_TV, 128>(sv, src + p.cv + h * dv + v0, p.ldx, ML_C, cnt - t0, dv - v0, c.vec);
+        if (tid < ML_C) {
+            if (t0 + tid < cnt) ml_cp4(se + tid, ga + 3 * plane + t0 + tid);
+            else se[tid] = 0.f;
+        } else if (tid == ML_C) {
+            ml_cp4(se + ML_C, ga + 4 * plane + min(t0 + ML_C, cnt) - 1);
+        }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    const float *ga = c.gates + (size_t)h * c.T + row0, *gb = ga + (size_t)p.H * c.T;
     stage(0, 0);
     int b = 0;
     for (int t0 = 0, ch = chunk0; t0 < cnt; t0 += ML_C, ++ch, b ^= 1) {
@@ -285,27 +298,11 @@ __global__ void __launch_bounds__(128) mlstm_states_kernel(const MlstmChunkArgs 
                     if (v0 + tx * 4 + j < dv) at(cs, i)[j] = acc[i][j];
         }
         if (has_n) c.chunk_n[((size_t)ch * p.H + h) * d + r0 + tid] = nacc;
-        if (tid < 32) {      // b_s P(s, end) for the chunk's tokens and the product of all its a, by one warp, two tokens a lane
-            const int s = t0 + 2 * tid;
-            const float a0 = s < cnt ? ga[s] : 1.f, a1 = s + 1 < cnt ? ga[s + 1] : 1.f;
-            float prod = a0 * a1;                              // becomes the product from this lane's tokens to the end
-#pragma unroll
-            for (int off = 1; off < 32; off <<= 1) {
-                const float up = __shfl_down_sync(0xffffffffu, prod, off);
-                if (tid + off < 32) prod *= up;
-            }
-            float behind = __shfl_down_sync(0xffffffffu, prod, 1);
-            if (tid == 31) behind = 1.f;
-            se[2 * tid] = (s < cnt ? gb[s] : 0.f) * (a1 * behind);
-            se[2 * tid + 1] = (s + 1 < cnt ? gb[s + 1] : 0.f) * behind;
-            if (tid == 0) se[ML_C] = prod;
-        }
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         if (t0 + ML_C < cnt) stage(t0 + ML_C, b ^ 1);
-        for (int i = tid; i < ML_C * ML_TD; i += 128) sk[b][i] *= se[i / ML_TD];
-        const float all = se[ML_C];
-        __syncthreads();
+        const float *sk = smem + b * BUF, *sv = sk + ML_C * ML_TD, *e = sv + ML_C * ML_TV;
+        const float all = e[ML_C];
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -313,8 +310,11 @@ __global__ void __launch_bounds__(128) mlstm_states_kernel(const MlstmChunkArgs 
 #pragma unroll 8
         for (int s = 0; s < ML_C; ++s) {
             float k[4], v[4];
-            load4(&sk[b][s * ML_TD + ty * 4], k);
-            load4(&sv[b][s * ML_TV + tx * 4], v);
+            load4(sk + s * ML_TD + ty * 4, k);
+            load4(sv + s * ML_TV + tx * 4, v);
+            const float weight = e[s];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) k[i] *= weight;
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -325,11 +325,10 @@ __global__ void __launch_bounds__(128) mlstm_states_kernel(const MlstmChunkArgs 
 #pragma unroll 4
             for (int s = 0; s < ML_C; s += 4)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) part[j] += sk[b][(s + j) * ML_TD + tid];
+                for (int j = 0; j < 4; ++j) part[j] = fmaf(e[s + j], sk[(s + j) * ML_TD + tid], part[j]);
             nacc = fmaf(nacc, all, (part[0] + part[1]) + (part[2] + part[3]));
         }
-        // (the next round's barrier stands between these reads and the copies into this buffer after next; se is
-        // written by warp 0 again before that barrier, so everyone must have read `all`: it has, ahead of the second one)
+        // (the next round's barrier stands between these reads and the copies into this buffer after next)
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i)
@@ -375,12 +374,12 @@ __global__ void __launch_bounds__(256, 2) mlstm_outputs_kernel(const MlstmChunkA
     const int row0 = c.chunks[2 * ch], cnt = c.chunks[2 * ch + 1];
     const int ty = tid >> 4, tx = tid & 15;
     const float *ga = c.gates + (size_t)h * c.T + row0, *gb = ga + (size_t)p.H * c.T, *ge = gb + (size_t)p.H * c.T;
-    const float* src = p.proj + (size_t)row0 * p.ld;
+    const float* src = (const float*)p.x + (size_t)row0 * p.ldx;
     const float* S = c.chunk_S + ((size_t)ch * p.H + h) * d * dv;
     const float* nn = c.chunk_n + ((size_t)ch * p.H + h) * d;
     auto stage = [&](int k0) {
-        ml_stage<ML_KS, ML_LD, 256>(sq, src + p.cq + h * d + k0, p.ld, 64, cnt, d - k0, c.vec);
-        ml_stage<ML_KS, ML_LD, 256>(sk, src + p.ck + h * d + k0, p.ld, 64, cnt, d - k0, c.vec);
+        ml_stage<ML_KS, ML_LD, 256>(sq, src + p.cq + h * d + k0, p.ldx, 64, cnt, d - k0, c.vec);
+        ml_stage<ML_KS, ML_LD, 256>(sk, src + p.ck + h * d + k0, p.ldx, 64, cnt, d - k0, c.vec);
         ml_stage<ML_OV, ML_LV, 256>(sb, S + (size_t)k0 * dv + v0, dv, 64, d - k0, dv - v0, dv % 4 == 0);
         asm volatile("cp.async.commit_group;" ::: "memory");
         if (tid < ML_KS) sn[tid] = k0 + tid < d ? nn[k0 + tid] : 0.f;
@@ -394,12 +393,8 @@ __global__ void __launch_bounds__(256, 2) mlstm_outputs_kernel(const MlstmChunkA
             if (t > tid) w *= sa[t];
             sw[t * ML_LD + tid] = t < tid ? 0.f : w;
         }
-    } else if (tid == 64) {  // A_t
-        float w = 1.f;
-        for (int t = 0; t < 64; ++t) {
-            w *= sa[t];
-            sA[t] = w;
-        }
+    } else if (tid < 128) {
+        sA[tid - 64] = tid - 64 < cnt ? ga[4 * (size_t)p.H * c.T + tid - 64] : 0.f;
     }
     float acc[4][8], w[4][4], qn = 0.f;
 #pragma unroll
@@ -440,7 +435,7 @@ __global__ void __launch_bounds__(256, 2) mlstm_outputs_kernel(const MlstmChunkA
     }
     __syncthreads();
     // the values take the last slab's place
-    ml_stage<ML_OV, ML_LV, 256>(sb, src + p.cv + h * dv + v0, p.ld, 64, cnt, dv - v0, c.vec);
+    ml_stage<ML_OV, ML_LV, 256>(sb, src + p.cv + h * dv + v0, p.ldx, 64, cnt, dv - v0, c.vec);
     asm volatile("cp.async.commit_group;" ::: "memory");
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -488,7 +483,7 @@ __global__ void __launch_bounds__(256, 2) mlstm_outputs_kernel(const MlstmChunkA
         for (int off = 1; off < 16; off <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
         if (t >= cnt) continue;
         const float scale = 1.f / sqrtf(ss / (float)dv + p.eps);
-        const float* gr = src + (size_t)t * p.ld + p.cg + h * dv;
+        const float* gr = src + (size_t)t * p.ldx + p.cg + h * dv;
         TO* y = (TO*)p.y + ((size_t)(row0 + t) * p.H + h) * dv;
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
@@ -498,37 +493,20 @@ __global__ void __launch_bounds__(256, 2) mlstm_outputs_kernel(const MlstmChunkA
     }
 }
 
-// One warp per (token of a portion, head): the norm, the weight and the gate.
-template <typename TO>
-__global__ void __launch_bounds__(128) mlstm_finish_kernel(const MlstmChunkArgs c) {
-    pdl_enter(TR_MLSTM);
-    const MlstmArgs& p = c.p;
-    const int row0 = c.chunks[2 * blockIdx.x], cnt = c.chunks[2 * blockIdx.x + 1], h = blockIdx.y, lane = threadIdx.x & 31;
-    for (int t = threadIdx.x >> 5; t < cnt; t += 4) {
-        const size_t at = ((size_t)(row0 + t) * p.H + h) * p.dv;
-        float ss = 0.f;
-        for (int i = lane; i < p.dv; i += 32) ss = fmaf(c.o[at + i], c.o[at + i], ss);
-        const float scale = 1.f / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
-        const float* gr = p.proj + (size_t)(row0 + t) * p.ld + p.cg + h * p.dv;
-        for (int i = lane; i < p.dv; i += 32)
-            ((TO*)p.y)[at + i] = from_float<TO>(c.o[at + i] * scale * p.w[h * p.dv + i] / (1.f + expf(-gr[i])));
-    }
-}
-
 }  // namespace air
 
-AIR_API int air_mlstm_step(const float* proj, int ld, int cq, int ck, int cv, int cg, int ci, int cf, const float* ib,
-                           const float* fb, const float* w, float* S, float* n, float* m, void* y, int out_dtype,
-                           const int* q_start, const int* slots, int entries, int H, int d, int dv, float cap, float q_scale,
-                           float eps, cudaStream_t stream) {
+AIR_API int air_mlstm_step(const void* x, int x_dtype, int ldx, int cq, int ck, int cv, int cg, const float* z, int ldz, int ci,
+                           int cf, const float* ib, const float* fb, const float* w, float* S, float* n, float* m, void* y,
+                           int out_dtype, const int* q_start, const int* slots, int entries, int H, int d, int dv, float cap,
+                           float q_scale, float eps, cudaStream_t stream) {
     if (entries <= 0) return 0;
     if (H <= 0 || d <= 0 || dv <= 0 || entries > 65535 || !(cap > 0.f)) return AIR_ERR_BAD_ARGUMENT;
-    air::MlstmArgs p{proj, ld, cq, ck, cv, cg, ci, cf, ib, fb, w, S, n, m, y, q_start, slots, H, d, dv, cap, q_scale, eps};
+    air::MlstmArgs p{x, ldx, z, ldz, cq, ck, cv, cg, ci, cf, ib, fb, w, S, n, m, y, q_start, slots, H, d, dv, cap, q_scale, eps};
     const bool vec = dv % 4 == 0 && ((uintptr_t)S & 15) == 0;
     const int N = vec ? 4 : 1, cols = dv / N, cw = cols < air::ML_THREADS ? cols : air::ML_THREADS;
     const size_t smem = sizeof(float) * ((size_t)2 * d + dv + (size_t)(air::ML_THREADS / cw) * cw * N);
     if (smem > 200 * 1024) return AIR_ERR_BAD_ARGUMENT;
-    AIR_DISPATCH(out_dtype, TO, {
+    AIR_DISPATCH(x_dtype, TX, AIR_DISPATCH(out_dtype, TO, {
         auto go = [&](auto kernel) {
             if (smem > 44 * 1024) {
                 cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -536,36 +514,49 @@ AIR_API int air_mlstm_step(const float* proj, int ld, int cq, int ck, int cv, in
             }
             return air::launch(kernel, dim3(H, entries), air::ML_THREADS, smem, stream, p);
         };
-        return vec ? go(air::mlstm_step_kernel<TO, 4>) : go(air::mlstm_step_kernel<TO, 1>);
-    });
+        return vec ? go(air::mlstm_step_kernel<TX, TO, 4>) : go(air::mlstm_step_kernel<TX, TO, 1>);
+    }));
     return 0;
 }
 
 // Portions of several tokens (see the file's head): portions int32 [L, 4] = (first row, tokens, slot, first chunk) and
 // chunks int32 [N, 2] = (first row, tokens), a portion's chunks of 64 tokens one after the other.  Scratch: gates float32
-// [3, H, T], chunk_S [N, H, d, dv], chunk_n [N, H, d], and o [T, H, dv] where dv > 128.
-AIR_API int air_mlstm_portions(const float* proj, int ld, int cq, int ck, int cv, int cg, int ci, int cf, const float* ib,
-                               const float* fb, const float* w, float* S, float* n, float* m, void* y, int out_dtype,
-                               const int* portions, int L, const int* chunks, int N, float* gates, float* chunk_S,
-                               float* chunk_n, float* o, int T, int H, int d, int dv, float cap, float q_scale, float eps,
-                               cudaStream_t stream) {
+// [5, H, T], chunk_S [N, H, d, dv], chunk_n [N, H, d], and o [T, H, dv] where dv > 128.
+AIR_API int air_mlstm_portions(const float* x, int ldx, int cq, int ck, int cv, int cg, const float* z, int ldz, int ci, int cf,
+                               const float* ib, const float* fb, const float* w, float* S, float* n, float* m, void* y,
+                               int out_dtype, const int* portions, int L, const int* chunks, int N, float* gates,
+                               float* chunk_S, float* chunk_n, float* o, int T, int H, int d, int dv, float cap,
+                               float q_scale, float eps, cudaStream_t stream) {
     if (L <= 0 || N <= 0) return 0;
     const int v_blocks = (dv + air::ML_OV - 1) / air::ML_OV;
     if (H <= 0 || H > 65535 || d <= 0 || dv <= 0 || L > 65535 || v_blocks > 65535 || !(cap > 0.f) || !gates || !chunk_S ||
         !chunk_n || (v_blocks > 1 && !o) || (((uintptr_t)chunk_S | (uintptr_t)S) & 15))
         return AIR_ERR_BAD_ARGUMENT;
-    const int vec = ((ld | cq | ck | cv | d | dv) & 3) == 0 && ((uintptr_t)proj & 15) == 0;
+    const int vec = ((ldx | cq | ck | cv | d | dv) & 3) == 0 && ((uintptr_t)x & 15) == 0;
     air::MlstmChunkArgs c;
-    c.p = air::MlstmArgs{proj, ld, cq, ck, cv, cg, ci, cf, ib, fb, w, S, n, m, y, nullptr, nullptr, H, d, dv, cap, q_scale, eps};
+    c.p = air::MlstmArgs{x, ldx, z, ldz, cq, ck, cv, cg, ci, cf, ib, fb, w, S, n, m, y, nullptr, nullptr, H, d, dv, cap, q_scale, eps};
     c.portions = portions; c.chunks = chunks; c.gates = gates; c.chunk_S = chunk_S; c.chunk_n = chunk_n;
     c.o = v_blocks > 1 ? o : nullptr; c.T = T; c.vec = vec;
-    int rc = air::launch(air::mlstm_gates_kernel, dim3(H, L), 256, 0, stream, c);
+    int rc = air::launch_mlstm_gates(c, L, stream);
     if (rc) return rc;
     const int tiles = ((d + air::ML_TD - 1) / air::ML_TD) * ((dv + air::ML_TV - 1) / air::ML_TV);
-    cudaError_t err = cudaFuncSetAttribute(air::mlstm_states_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                           (int)air::ML_STATES_SMEM);
+    // A block's time is a chain over its chunks, and blocks that share an SM stretch one another's.  Launched while the
+    // kernel before it is still leaving the SMs they would land several to an SM, so this kernel starts when its
+    // predecessor has ended, and while there are no more blocks than SMs (than twice the SMs) a block asks for so much
+    // shared memory that only one (two) of them fit an SM.
+    int sms = 148, dev = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    const long long blocks = (long long)tiles * H * L;
+    const size_t smem = blocks <= sms ? 120 * 1024 : blocks <= 2ll * sms ? 80 * 1024 : air::ML_STATES_SMEM;
+    cudaError_t err = cudaFuncSetAttribute(air::mlstm_states_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return (int)err;
-    rc = air::launch(air::mlstm_states_kernel, dim3(tiles, H, L), 128, air::ML_STATES_SMEM, stream, c);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(tiles, H, L);
+    cfg.blockDim = dim3(128);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = stream;
+    rc = (int)cudaLaunchKernelEx(&cfg, air::mlstm_states_kernel, c);
     if (rc) return rc;
     AIR_DISPATCH(out_dtype, TO, {
         auto kernel = air::mlstm_outputs_kernel<TO>;
@@ -573,7 +564,7 @@ AIR_API int air_mlstm_portions(const float* proj, int ld, int cq, int ck, int cv
         if (err != cudaSuccess) return (int)err;
         rc = air::launch(kernel, dim3(N, H, v_blocks), 256, air::ML_OUT_SMEM, stream, c);
         if (rc || v_blocks == 1) return rc;
-        return air::launch(air::mlstm_finish_kernel<TO>, dim3(N, H), 128, 0, stream, c);
+        return air::launch(air::mlstm_finish_kernel<float, TO>, dim3(N, H), 128, 0, stream, c);
     });
     return 0;
 }

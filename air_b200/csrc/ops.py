@@ -46,18 +46,19 @@ _SIGNATURES = {
                         c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "air_residual_conv": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                           c_void_p],
-    "air_mlstm_step": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                       c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                       c_float, c_float, c_void_p],
-    "air_mlstm_portions": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                           c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
-                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p],
+    "air_mlstm_step": [c_void_p] + [c_int] * 6 + [c_void_p] + [c_int] * 3 + [c_void_p] * 7 + [c_int] + [c_void_p] * 2 +
+                      [c_int] * 4 + [c_float] * 3 + [c_void_p],
+    "air_mlstm_portions": [c_void_p] + [c_int] * 5 + [c_void_p] + [c_int] * 3 + [c_void_p] * 7 + [c_int] +
+                          [c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 4 + [c_int] * 4 + [c_float] * 3 + [c_void_p],
+    "air_mlstm_portions_tc": [c_void_p] + [c_int] * 5 + [c_void_p] + [c_int] * 3 + [c_void_p] * 7 + [c_int] +
+                             [c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 5 + [c_int] * 4 + [c_float] * 3 +
+                             [c_void_p],
     "air_latent_prepare": [c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                            c_void_p, c_void_p],
     "air_grouped_attention": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_int,
-                              c_float, c_void_p, c_int, c_void_p],
+                              c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
     "air_gather_keys": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                         c_void_p, c_void_p],
     "air_masked_softmax": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
@@ -105,7 +106,7 @@ _SIGNATURES = {
                                  c_void_p],
     "air_decode_attention_tma_sink": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                       c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                      c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                                      c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
     "air_head_gate": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "air_decode_attention_tma_fresh": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int,
                                        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -463,6 +464,17 @@ def paged_attention_ref(q, cache, block_table, token_seq, positions, out, window
     return out
 
 
+def _turn(turn, width):
+    """(pointer, rotated elements, pairing) of a turn back = (freq float64, pairing) or None."""
+    if turn is None:
+        return None, 0, 0
+    freq, pairing = turn
+    _req(freq, "turn freq", (torch.float64,))
+    if 2 * freq.numel() > width or pairing not in ("half", "neighbours"):
+        raise KernelError(f"a turn back of {2 * freq.numel()} of {width} elements, pairing {pairing!r}")
+    return freq.data_ptr(), 2 * freq.numel(), 1 if pairing == "neighbours" else 0
+
+
 def grouped_attention_ok(cache_dtype, d, dv) -> bool:
     """Whether grouped_attention takes keys of d and values of dv elements: rows of whole 16-byte pieces."""
     size = 4 if cache_dtype == torch.float32 else 2
@@ -470,11 +482,12 @@ def grouped_attention_ok(cache_dtype, d, dv) -> bool:
 
 
 def grouped_attention(q, cache, block_table, token_seq, positions, out, window, scale, kv_heads=1, page_tokens=None,
-                      chunk=None, sink=None, latent=False, splits=None, softcap=0.0, gate=None):
+                      chunk=None, sink=None, latent=False, splits=None, softcap=0.0, gate=None, turn=None):
     """paged_attention_ref's arithmetic and arguments (32-bit, any batch, window or chunk, sink, latent rows), by the
     kernel in which a block serves all query heads of a key/value head and the keys of a token are split over
     `splits` blocks (default: enough to fill the device); needs grouped_attention_ok(cache.dtype, d, dv).  gate (float32
-    [T, H * dv], may be a band of columns): out is multiplied, element by element, by sigmoid(gate)."""
+    [T, H * dv], may be a band of columns): out is multiplied, element by element, by sigmoid(gate).  turn = (freq, pairing):
+    ahead of the gate every head's output is turned back as turn_heads(.., back=True) does it."""
     T, H, d = q.shape
     gp, ldg = (None, 0)
     if gate is not None:
@@ -515,7 +528,7 @@ def grouped_attention(q, cache, block_table, token_seq, positions, out, window, 
         q.data_ptr(), 1 if q.dtype == torch.float32 else 0, cache.data_ptr(), _DT[cache.dtype], block_table.data_ptr(),
         block_table.shape[1], token_seq.data_ptr(), positions.data_ptr(), part.data_ptr(), out.data_ptr(), T, H, G, d,
         dv, P, int(chunk or window or 0), float(scale), 1 if chunk else 0, _ptr(sink), 1 if latent else 0, int(splits),
-        float(softcap or 0.0), gp, ldg, _stream()), "grouped_attention")
+        float(softcap or 0.0), gp, ldg, *_turn(turn, dv), _stream()), "grouped_attention")
     global launches
     launches += 1
     return out
@@ -720,12 +733,17 @@ def residual_conv(h, weight, state, out, q_start, slots, max_tokens):
     return out
 
 
-def _mlstm(proj, columns, i_bias, f_bias, weight, S, n, m, out):
+def _mlstm(x, z, columns, i_bias, f_bias, weight, S, n, m, out):
     slots_n, H, d, dv = S.shape
-    pp, ld = _columns(proj, "proj")
-    need = {"q": H * d, "k": H * d, "v": H * dv, "g": H * dv, "i": H, "f": H}
-    for c, width in need.items():
-        if columns[c] + width > proj.shape[1]:
+    T, W = x.shape
+    if not x.is_cuda or x.dtype not in _FLOATS or x.stride(1) != 1:
+        raise KernelError("mlstm: x must be a CUDA matrix with contiguous rows, float32 or bfloat16")
+    zp, ldz = _columns(z, "z")
+    if z.shape[0] != T:
+        raise KernelError("mlstm: x and z have different rows")
+    for c, width, have in (("q", H * d, W), ("k", H * d, W), ("v", H * dv, W), ("g", H * dv, W), ("i", H, z.shape[1]),
+                           ("f", H, z.shape[1])):
+        if columns[c] < 0 or columns[c] + width > have:
             raise KernelError(f"mlstm: projection {c} does not fit")
     _req(i_bias, "i_bias", (torch.float32,), (H,))
     _req(f_bias, "f_bias", (torch.float32,), (H,))
@@ -733,44 +751,54 @@ def _mlstm(proj, columns, i_bias, f_bias, weight, S, n, m, out):
     _req(S, "S", (torch.float32,))
     _req(n, "n", (torch.float32,), (slots_n, H, d))
     _req(m, "m", (torch.float32,), (slots_n, H))
-    _req(out, "out", _FLOATS, (proj.shape[0], H * dv))
-    return (pp, ld, *(int(columns[c]) for c in "qkvgif"), i_bias.data_ptr(), f_bias.data_ptr(), weight.data_ptr(),
-            S.data_ptr(), n.data_ptr(), m.data_ptr(), out.data_ptr(), _DT[out.dtype]), (H, d, dv)
+    _req(out, "out", _FLOATS, (T, H * dv))
+    xs = (x.stride(0), *(int(columns[c]) for c in "qkvg"))
+    rest = (zp, ldz, int(columns["i"]), int(columns["f"]), i_bias.data_ptr(), f_bias.data_ptr(), weight.data_ptr(),
+            S.data_ptr(), n.data_ptr(), m.data_ptr(), out.data_ptr(), _DT[out.dtype])
+    return xs, rest, (H, d, dv)
 
 
-def mlstm_step(proj, columns, i_bias, f_bias, weight, S, n, m, out, q_start, slots, cap, q_scale, eps):
+def mlstm_step(x, z, columns, i_bias, f_bias, weight, S, n, m, out, q_start, slots, cap, q_scale, eps):
     """mLSTM's matrix memory (see mlstm.cu) for every entry of the batch (slots[e] < 0: skipped), token after token, one
-    block per head and entry.  proj float32 [T, W]; columns: where q, k, v, g (the heads side by side), i and f (a logit per
-    head) start in it; i_bias, f_bias float32 [H]; weight float32 [H * dv]; the states S [slots, H, d, dv], n [slots, H, d],
+    block per head and entry.  x [T, W] (float32 or bfloat16, may be a band of columns): q, k, v, g (the heads side by side)
+    start at columns["q"] and so on; z float32 [T, ..]: a logit per head for the input and the forget gate, at columns["i"]
+    and columns["f"]; i_bias, f_bias float32 [H]; weight float32 [H * dv]; the states S [slots, H, d, dv], n [slots, H, d],
     m [slots, H]; out [T, H * dv]: every head's read-out normalised, weighted and gated."""
-    args, (H, d, dv) = _mlstm(proj, columns, i_bias, f_bias, weight, S, n, m, out)
+    xs, rest, (H, d, dv) = _mlstm(x, z, columns, i_bias, f_bias, weight, S, n, m, out)
     _req(q_start, "q_start", _I32)
     _req(slots, "slots", _I32)
-    _check(_get("air_mlstm_step")(*args, q_start.data_ptr(), slots.data_ptr(), slots.shape[0], H, d, dv, float(cap),
-                                  float(q_scale), float(eps), _stream()), "mlstm_step")
+    _check(_get("air_mlstm_step")(x.data_ptr(), _DT[x.dtype], *xs, *rest, q_start.data_ptr(), slots.data_ptr(),
+                                  slots.shape[0], H, d, dv, float(cap), float(q_scale), float(eps), _stream()), "mlstm_step")
     return out
 
 
 MLSTM_CHUNK = 64
 
 
-def mlstm_portions(proj, columns, i_bias, f_bias, weight, S, n, m, out, portions, chunks, cap, q_scale, eps):
+def mlstm_portions(x, z, columns, i_bias, f_bias, weight, S, n, m, out, portions, chunks, cap, q_scale, eps):
     """The same for portions of several tokens, in chunks whose rows are computed side by side: portions int32 [L, 4] =
     (first row, tokens, slot, first chunk), chunks int32 [N, 2] = (first row, tokens), a portion's chunks of MLSTM_CHUNK
-    tokens (the last one shorter) one after the other.  Rows of other entries are left alone."""
+    tokens (the last one shorter) one after the other.  Rows of other entries are left alone.  x in bfloat16 (d, dv, its row
+    stride and columns multiples of 8): the products run on the tensor cores, where 32-bit operands (weighted keys, the
+    chunks' weights, states) enter as the sum of two bfloat16 numbers; float32: on the CUDA cores."""
     global launches
-    args, (H, d, dv) = _mlstm(proj, columns, i_bias, f_bias, weight, S, n, m, out)
-    T, dev = proj.shape[0], proj.device
+    xs, rest, (H, d, dv) = _mlstm(x, z, columns, i_bias, f_bias, weight, S, n, m, out)
+    T, dev = x.shape[0], x.device
     _req(portions, "portions", _I32, (None, 4))
     _req(chunks, "chunks", _I32, (None, 2))
     L, N = portions.shape[0], chunks.shape[0]
-    gates = torch.empty((3, H, T), dtype=torch.float32, device=dev)
+    gates = torch.empty((5, H, T), dtype=torch.float32, device=dev)
     chunk_S = torch.empty((N, H, d, dv), dtype=torch.float32, device=dev)
     chunk_n = torch.empty((N, H, d), dtype=torch.float32, device=dev)
     o = torch.empty((T, H, dv), dtype=torch.float32, device=dev) if dv > 128 else None
-    _check(_get("air_mlstm_portions")(*args, portions.data_ptr(), L, chunks.data_ptr(), N, gates.data_ptr(),
-                                      chunk_S.data_ptr(), chunk_n.data_ptr(), _ptr(o), T, H, d, dv, float(cap),
-                                      float(q_scale), float(eps), _stream()), "mlstm_portions")
+    lists = (portions.data_ptr(), L, chunks.data_ptr(), N, gates.data_ptr(), chunk_S.data_ptr())
+    sizes = (chunk_n.data_ptr(), _ptr(o), T, H, d, dv, float(cap), float(q_scale), float(eps), _stream())
+    if x.dtype == torch.bfloat16:
+        planes = torch.empty((N, H, 2, d, dv), dtype=torch.bfloat16, device=dev)
+        _check(_get("air_mlstm_portions_tc")(x.data_ptr(), *xs, *rest, *lists, planes.data_ptr(), *sizes), "mlstm_portions")
+        launches += 1
+    else:
+        _check(_get("air_mlstm_portions")(x.data_ptr(), *xs, *rest, *lists, *sizes), "mlstm_portions")
     launches += 2 if o is None else 3
     return out
 
@@ -1274,11 +1302,12 @@ def decode_splits(tokens: int, heads: int, kv_heads: int) -> int:
 
 
 def decode_attention(q, cache, block_table, token_seq, positions, out, window, scale, splits=None, scratch=None,
-                     status=None, engine="tma", softcap=0.0, sink=None, gate=None):
+                     status=None, engine="tma", softcap=0.0, sink=None, gate=None, turn=None):
     """bfloat16 attention for one query token per request.  softcap > 0: score = softcap * tanh(scale * q.k /
     softcap) (the copy-engine kernel only).  sink (float32 [H]): one more term exp(sink[h]) in the softmax's
     denominator; gate (float32 [T, H * d] logits, may be a band of columns): out is multiplied by sigmoid(gate) element
-    by element; both enter where the key splits are merged (the copy-engine kernel only, two splits at least).  scratch: (float32 [T*H*splits*D], float32
+    by element; turn = (freq, pairing): ahead of the gate every head's output is turned back as turn_heads(.., back=True)
+    does it; all enter where the key splits are merged (the copy-engine kernel only, two splits at least).  scratch: (float32 [T*H*splits*D], float32
     [T*H*splits*2]) or None to allocate.  engine "tma": keys and values by the copy engine into shared
     memory (attention_decode_tma.cu); "ldg": by the warps' own loads (attention_decode.cu)."""
     T, H, d = q.shape
@@ -1293,11 +1322,11 @@ def decode_attention(q, cache, block_table, token_seq, positions, out, window, s
         raise KernelError(f"decode_attention takes head sizes {DECODE_HEAD_DIMS}, not {d}")
     if splits is None:
         splits = decode_splits(T, H, K)
-    extra = sink is not None or gate is not None
+    extra = sink is not None or gate is not None or turn is not None
     if extra:
         splits = max(2, splits)
         if not (engine == "tma" and tile_pages(P)):
-            raise KernelError("decode_attention: a sink or gates are taken by the copy-engine kernel only")
+            raise KernelError("decode_attention: a sink, gates or a turn back are taken by the copy-engine kernel only")
     po = pm = None
     if splits > 1:
         if scratch is None:
@@ -1321,7 +1350,7 @@ def decode_attention(q, cache, block_table, token_seq, positions, out, window, s
             q.data_ptr(), cache.data_ptr(), cache.shape[0], block_table.data_ptr(), block_table.shape[1],
             token_seq.data_ptr(), positions.data_ptr(), out.data_ptr(), _ptr(po), _ptr(pm), T, H, K, d, P,
             int(window or 0), float(scale), float(softcap or 0.0), splits, _ptr(status), _ptr(sink), gp, ldg,
-            _stream()), "decode_attention_tma")
+            *_turn(turn, d), _stream()), "decode_attention_tma")
     elif engine == "tma" and tile_pages(P):
         _check(_get("air_decode_attention_tma")(
             q.data_ptr(), cache.data_ptr(), cache.shape[0], block_table.data_ptr(), block_table.shape[1],

@@ -143,20 +143,31 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormArgs 
             v[j] = (urow[i + j] - mean) * scale * wv[j];
             if (p.b) v[j] += bv[j];
         }
-        if (slot >= 0) {
+        if (slot >= 0) {      // (four earlier inputs and their weights under way at a time)
             const int keep = p.taps - 1;
             float* st = p.conv_state + (size_t)slot * keep * E + i;
+            const float* cw = p.conv_w + i;
             float acc[N];
+            load_columns<N>(cw + (size_t)keep * E, acc);
 #pragma unroll
-            for (int j = 0; j < N; ++j) acc[j] = v[j];
-            for (int k = 0; k <= keep; ++k) {
+            for (int j = 0; j < N; ++j) acc[j] = fmaf(acc[j], v[j], v[j]);
+            for (int k0 = 0; k0 < keep; k0 += 4) {
+                float in[4][N], wk[4][N];
 #pragma unroll
-                for (int j = 0; j < N; ++j) {
-                    const float in = k < keep ? st[(size_t)k * E + j] : v[j];
-                    acc[j] = fmaf(p.conv_w[(size_t)k * E + i + j], in, acc[j]);
-                    if (k > 0) st[(size_t)(k - 1) * E + j] = in;
-                }
+                for (int u = 0; u < 4; ++u)
+                    if (k0 + u < keep) {
+                        load_columns<N>(st + (size_t)(k0 + u) * E, in[u]);
+                        load_columns<N>(cw + (size_t)(k0 + u) * E, wk[u]);
+                    }
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+                    if (k0 + u < keep) {
+#pragma unroll
+                        for (int j = 0; j < N; ++j) acc[j] = fmaf(wk[u][j], in[u][j], acc[j]);
+                        if (k0 + u > 0) store_columns<N>(st + (size_t)(k0 + u - 1) * E, in[u]);
+                    }
             }
+            if (keep > 0) store_columns<N>(st + (size_t)(keep - 1) * E, v);
 #pragma unroll
             for (int j = 0; j < N; ++j) v[j] = acc[j];
         }
@@ -231,7 +242,7 @@ AIR_API int air_stream_norm(const float* x, long long x_stride, float* h_out, lo
     p.token_seq = token_seq; p.taps = taps;
     auto al = [](const void* q) { return ((uintptr_t)q & 15) == 0; };
     const bool vec = E % 4 == 0 && x_stride % 4 == 0 && h_stride % 4 == 0 && part_stride % 4 == 0 && al(x) && al(h_out) &&
-                     al(y) && al(w) && al(b) && al(out);
+                     al(y) && al(w) && al(b) && al(out) && al(conv_w) && al(conv_state);
     // few rows: one access of a thread per row, all of a row's loads under way at once
     const int items = vec ? E / 4 : E;
     int threads = items >= 256 ? 256 : (items + 31) / 32 * 32;

@@ -53,13 +53,16 @@ class PortionAttention:
             return position - position % self.chunk
         return 0
 
-    def attend(self, q, cache, bt, ctx, out, *, latent=False, kv_heads=1, page_tokens=None, gate=None, pages=None):
+    def attend(self, q, cache, bt, ctx, out, *, latent=False, kv_heads=1, page_tokens=None, gate=None, pages=None,
+               turn=None):
         """out [T, H, dv] = attention of q [T, H, dk] (float32, or the cache's type) over the request's pages.  gate
         (float32 [T, H * dv] logits, may be a band of columns): out is multiplied by sigmoid(gate) element by element,
         in the kernel that merges the key splits where that kernel attends, else by a kernel of its own.  pages: the
         cache as [pages, 2, K, P, d] where keys and values have one size: single tokens and short portions of a bfloat16
         engine then take the copy-engine kernel of the dense decoder (heads of 64, 128 or 256, pages that its tiles fit,
-        no chunks), with the cap in its softmax and the sink and the gates where its key splits are merged."""
+        no chunks), with the cap in its softmax and the sink and the gates where its key splits are merged.  turn = (freq,
+        pairing): every head's output is turned back by the row's position ahead of the gate, in the kernel that merges the
+        key splits where there is one, else by a kernel of its own."""
         sinks = getattr(self, "sinks", None)
         softcap = float(getattr(self, "softcap", 0.0) or 0.0)
         plan = ctx.plans.get((self.PLAN,)) if not self.rt.is_fp32 else None
@@ -69,17 +72,19 @@ class PortionAttention:
                     and out.dtype == torch.bfloat16 and q.shape[2] == out.shape[2]
                     and q.shape[2] in ops.DECODE_HEAD_DIMS and ops.tile_pages(pages.shape[3])):
                 ops.decode_attention(q, pages, bt, token_seq, ctx.positions, out, self.window, self.scale,
-                                     softcap=softcap, sink=sinks, gate=gate, status=ctx.status)
+                                     softcap=softcap, sink=sinks, gate=gate, status=ctx.status, turn=turn)
                 return
             # (the kernel that reads a key once for all heads of its group wants rows of whole 16-byte pieces)
             if ops.grouped_attention_ok(cache.dtype, q.shape[2], out.shape[2]):
                 ops.grouped_attention(q, cache, bt, token_seq, ctx.positions, out, self.window, self.scale,
                                       kv_heads=kv_heads, page_tokens=page_tokens, chunk=self.chunk, sink=sinks,
-                                      latent=latent, softcap=softcap, gate=gate)
+                                      latent=latent, softcap=softcap, gate=gate, turn=turn)
                 return
             ops.paged_attention_ref(q, cache, bt, token_seq, ctx.positions, out, self.window, self.scale,
                                     kv_heads=kv_heads, page_tokens=page_tokens, chunk=self.chunk, sink=sinks,
                                     latent=latent, softcap=softcap)
+            if turn is not None:
+                ops.turn_heads(out, *turn, ctx.positions, token_seq, back=True)
             if gate is not None:
                 ops.sigmoid_gate(out.view(out.shape[0], -1), gate, token_seq)
 
@@ -122,6 +127,8 @@ class PortionAttention:
                     dst.copy_(summed.view(nb, H, dv))
                 else:
                     dst.view(nb, G, J, dv).copy_(summed.view(G, nb, J, dv).permute(1, 0, 2, 3))
+            if turn is not None:
+                ops.turn_heads(out[r0:r0 + n], *turn, ctx.positions[r0:r0 + n], ctx.token_seq[r0:r0 + n], back=True)
             if gate is not None:
                 ops.sigmoid_gate(out[r0:r0 + n].view(n, H * dv), gate[r0:r0 + n], ctx.token_seq[r0:r0 + n])
         return out

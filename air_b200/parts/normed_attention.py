@@ -58,7 +58,8 @@ class NormedAttention(PortionAttention, Mixer):
     values have one size of 64 or 128, the pages fit the tile kernels and there are no chunks, a bfloat16 engine takes
     the dense decoder's roads instead (TiledAttention's plan of a step's tiles): prompt portions the tcgen05 kernel,
     single tokens the copy-engine kernel, both with the cap in their softmax and the sink's term where a row is
-    normalised; the output gates multiply where the decode kernel's key splits are merged, or in a kernel of their own."""
+    normalised; the output gates multiply, and rotated values' sums are turned back, where the decode kernel's key splits
+    are merged, or in kernels of their own."""
 
     graph_safe = True
 
@@ -107,7 +108,7 @@ class NormedAttention(PortionAttention, Mixer):
     def plan(self, batch):
         return TiledAttention.plan(self, batch) if self.tiles_fit() else PortionAttention.plan(self, batch)
 
-    def attend_tiles(self, q, kv, bt, ctx, out, plan, gate):
+    def attend_tiles(self, q, kv, bt, ctx, out, plan, gate, turn=None):
         """The step's attention on the tile kernels: the single next tokens at the head of the batch through the
         copy-engine decode kernel, the other entries through the tcgen05 kernel; kv [pages, 2, K, P, d]."""
         T, H, d = q.shape
@@ -115,13 +116,15 @@ class NormedAttention(PortionAttention, Mixer):
         if n:
             ops.decode_attention(q[:n], kv, bt, ctx.token_seq[:n], ctx.positions[:n], out[:n], self.window, self.scale,
                                  softcap=self.softcap, sink=self.sinks, gate=None if gate is None else gate[:n],
-                                 status=ctx.status)
+                                 status=ctx.status, turn=turn)
         if plan.tiles.shape[0]:
             if plan.slots and getattr(plan, "scratch", None) is None:
                 plan.scratch = ops.prefill_attention_scratch(plan.slots, d, q.device)
             ops.prefill_attention_tc(q, kv, bt, plan.tiles, out, self.window, self.scale, status=ctx.status,
                                      segments=plan.segments, items=plan.items, slots=plan.slots,
                                      scratch=getattr(plan, "scratch", None), softcap=self.softcap, sink=self.sinks)
+            if turn is not None and T > n:
+                ops.turn_heads(out[n:], *turn, ctx.positions[n:], ctx.token_seq[n:], back=True)
             if gate is not None and T > n:
                 ops.sigmoid_gate(out[n:].view(T - n, H * d), gate[n:], ctx.token_seq[n:])
         return out
@@ -223,15 +226,11 @@ class NormedAttention(PortionAttention, Mixer):
                               write_kv=owns_cache)
         out = torch.empty((T, H, dv), dtype=rt.dtype, device=x.device)
         gate = full[:, C:] if self.out_gate else None
-        late_gate, gate = (gate, None) if self.v_freq is not None else (None, gate)      # a gate comes behind the turn back
+        turn = None if self.v_freq is None else (self.v_freq, pos.pairing)
         plan = ctx.plans.get(TiledAttention.plan_key(self)) if self.tiles_fit() and not ctx.all_decode else None
         if plan is not None:
-            self.attend_tiles(q, pages.kv, bt, ctx, out, plan, gate)
+            self.attend_tiles(q, pages.kv, bt, ctx, out, plan, gate, turn)
         else:
             self.attend(q, kv, bt, ctx, out, kv_heads=G, page_tokens=P, gate=gate,
-                        pages=pages.kv if pages.kv.dim() == 5 else None)
-        if self.v_freq is not None:
-            ops.turn_heads(out, self.v_freq, pos.pairing, ctx.positions, ctx.token_seq, back=True)
-            if late_gate is not None:
-                ops.sigmoid_gate(out.view(T, H * dv), late_gate, ctx.token_seq)
+                        pages=pages.kv if pages.kv.dim() == 5 else None, turn=turn)
         return self.o.f32_sums(out.view(T, H * dv))

@@ -361,19 +361,38 @@ class MLSTM(_StateMixer):
         f32 = lambda n: tensors[p + n].to(torch.float32).contiguous()
         self.i_bias, self.f_bias, self.norm_weight = f32("i.b"), f32("f.b"), f32("norm")
         self.o = Linear(tensors[p + "o"], rt.status)
+        # longer portions of a bfloat16 engine: q, k, v and g in 16 bits from one product, the gates' logits in 32 from
+        # another, and the chunks' products on the tensor cores
+        gates = self.columns["i"][0]
+        self.starts = {n: at if at < gates else at - gates for n, (at, _) in self.columns.items()}
+        self.wide = self.narrow = None
+        if self.proj.weight.dtype == torch.bfloat16 and self.head_dim % 8 == 0 and self.v_dim % 8 == 0:
+            self.wide, self.narrow = self.proj.rows(0, gates), self.proj.rows(gates, self.proj.out_features)
 
     def forward(self, x, ctx, cache, owns_cache=True):
         memory, key_sum, level = cache
-        proj = self.proj.f32(x)
-        y = torch.empty((x.shape[0], self.heads * self.v_dim), dtype=self.rt.dtype, device=x.device)
-        args = (proj, {n: at for n, (at, _) in self.columns.items()}, self.i_bias, self.f_bias, self.norm_weight,
-                memory.state, key_sum.state, level.state, y)
-        numbers = (self.cap, self.head_dim ** -0.5, self.eps)
+        gates = self.columns["i"][0]
         plan = ctx.plans.get(self.plan_key())
+        portions = plan is not None and plan.long
+        if portions and self.wide is not None and not self.proj.small(x):
+            qkvg, logits = self.wide(x, torch.bfloat16), self.narrow.f32(x)
+        else:
+            proj = self.proj.f32(x)
+            qkvg, logits = proj[:, :gates], proj[:, gates:]
+        y = torch.empty((x.shape[0], self.heads * self.v_dim), dtype=self.rt.dtype, device=x.device)
+        args = (qkvg, logits, self.starts, self.i_bias, self.f_bias, self.norm_weight, memory.state, key_sum.state,
+                level.state, y)
+        numbers = (self.cap, self.head_dim ** -0.5, self.eps)
+        if not portions or plan.short:
+            ops.mlstm_step(*args, ctx.q_start, plan.short_slots if portions else ctx.slots, *numbers)
+        if portions:
+            ops.mlstm_portions(*args, plan.portions, plan.chunks, *numbers)
+        return self.o.f32_sums(y)
+        proj = self.proj.f32(x)
         if plan is None or not plan.long:
-            ops.mlstm_step(*args, ctx.q_start, ctx.slots, *numbers)
+            ops.mlstm_step(proj, columns, *weights, ctx.q_start, ctx.slots, *numbers)
         else:
             if plan.short:
-                ops.mlstm_step(*args, ctx.q_start, plan.short_slots, *numbers)
-            ops.mlstm_portions(*args, plan.portions, plan.chunks, *numbers)
+                ops.mlstm_step(proj, columns, *weights, ctx.q_start, plan.short_slots, *numbers)
+            ops.mlstm_portions(proj, columns, *weights, plan.portions, plan.chunks, *numbers)
         return self.o.f32_sums(y)

@@ -541,6 +541,25 @@ def _tabopel(width, layers, heads, kv_heads, ff, vocab=32000):
             "layers": [dict(order[i % 4], mlp=moe if i % 2 else dense) for i in range(n)]}
 
 
+# Dafotar beside Bivizen, the closest of the other designs (attention and a recurrence with a matrix state in turn, dense
+# gated feed-forwards), at equal width, depth, heads and ff (`--design dafotar`): four residual streams, convolutions of
+# four taps ahead of the mixers; mLSTM, attention in a window of 1,024, mLSTM, attention that reads the keys and values of
+# the attention layer before it, in turn, heads of 128.
+def _dafotar(width, layers, heads, kv_heads, ff, vocab=32000):
+    memory = {"type": "mlstm", "mixer": {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 15.0}}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128,
+                                          "scale": 128 ** -0.5, "mask": {"size": 1024}, "rot": {"dims": 128, "base": 1e5}}}
+    mlp = {"kind": "dense", "ff": ff}
+    out = []
+    for i in range(layers):
+        layer = att if i % 2 else memory
+        if i % 4 == 3:
+            layer = dict(att, mixer=dict(att["mixer"], kv_from=i - 2))
+        out.append(dict(layer, mlp=mlp))
+    return {"architecture": "Dafotar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": 4,
+            "canon": {"taps": 4}, "layers": out}
+
+
 def _qwen(width, layers, heads, kv_heads, ff, vocab=32000):
     return dict(_QWEN, num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads,
                 num_key_value_heads=kv_heads, intermediate_size=ff, rms_norm_eps=1e-5, max_window_layers=layers,
@@ -1226,13 +1245,176 @@ def tabopel_kernels(width, heads, kv_heads, ff, T, batch, context):
     return rows
 
 
+def kernel_reporter():
+    """(report, rows): report(name, f, nbytes or flops) times f from memory (512 MB written before each launch, the writes'
+    own time subtracted, ten launches replayed as a graph), prints microseconds and the share of the measured copy rate or
+    bf16 rate that the algorithm's bytes or flops make, and appends both to rows."""
+    import torch
+    pk = peaks()
+    big = torch.empty(512 << 20, dtype=torch.uint8, device="cuda")
+
+    def graph_time(calls, reps=5):
+        for c in calls:
+            c()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for _ in range(reps):
+                for c in calls:
+                    c()
+        graph.replay()
+        torch.cuda.synchronize()
+        us = []
+        for _ in range(5):
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            graph.replay()
+            b.record()
+            torch.cuda.synchronize()
+            us.append(a.elapsed_time(b) * 1e3 / reps)
+        return statistics.median(us)
+
+    flush = lambda: big.zero_()
+    t_flush = graph_time([flush])
+    rows = []
+
+    def report(name, f, nbytes=0, flops=0):
+        us = graph_time([flush, f]) - t_flush
+        frac = (nbytes / us / 1e3 / pk["hbm_gbs"]) if nbytes else (flops / us / 1e6 / pk["bf16_tflops"])
+        rows.append({"kernel": name, "us": round(us, 1), "of": "copy rate" if nbytes else "bf16 rate", "frac": round(frac, 3)})
+        print(f"  {name:78s} {us:8.1f} us  {frac:5.2f} of the measured {'copy' if nbytes else 'bf16'} rate", flush=True)
+
+    return report, rows
+
+
+def dafotar_kernels(width, heads, kv_heads, ff, T, batch, context):
+    """Dafotar's kernels alone at the layer's shapes, each beside the like kernel of the other designs."""
+    import torch
+    from air_b200.csrc import ops
+    from air_b200.parts.attention import TiledAttention
+    from air_b200.parts.base import HostBatch
+    from air_b200.parts.recurrent import MLSTM
+    from air_b200.parts.spec import PartSpec
+    report, rows = kernel_reporter()
+    E, H, G, d, P, S4, taps, window = width, heads, kv_heads, 128, 64, 4, 4, 1024
+    dev, bf = "cuda", torch.bfloat16
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    for label, N, entries in (("prompt", T, [(0, T)]), ("decode", batch, [(context - 1, 1)] * batch)):
+        print(f"{label}: {N} rows, width {E}, {S4} streams, {H}/{G} heads of {d}, window {window}")
+        S = len(entries)
+        starts = [0]
+        for _, n in entries:
+            starts.append(starts[-1] + n)
+        q_start, slots = i32(starts), i32(list(range(S)))
+        positions = torch.cat([torch.arange(p, p + n, dtype=torch.int32) for p, n in entries]).to(dev)
+        seq = torch.cat([torch.full((n,), i, dtype=torch.int32) for i, (_, n) in enumerate(entries)]).to(dev)
+        per_request = -(-(max(p + n for p, n in entries)) // P)
+        bt = torch.arange(S * per_request, dtype=torch.int32, device=dev).view(S, per_request).contiguous()
+        longest = max(n for _, n in entries)
+        # ---- streams completed, read and normalised, beside the other designs' sums with their norms
+        h4, h, a = torch.randn(S4, N, E, device=dev), torch.randn(N, E, device=dev), torch.randn(N, E, device=dev)
+        mix, out_w, read = torch.eye(S4, device=dev), torch.ones(S4, device=dev), torch.full((S4,), 0.25, device=dev)
+        w, b = torch.rand(E, device=dev) + 0.5, torch.randn(E, device=dev)
+        wbf = w.to(bf)
+        x, x32 = torch.empty(N, E, dtype=bf, device=dev), torch.empty(N, E, device=dev)
+        streams = lambda out, **kw: ops.stream_norm(h4, S4, w, b, 1e-6, out, term=a, mix=mix, out_weights=out_w, read=read, h_out=h4, **kw)
+        report("stream_norm (4 streams mixed, term added, read, layer norm; bfloat16 rows)", lambda: streams(x), N * E * (8 * S4 + 4 + 2))
+        report("stream_norm, float32 rows for the convolution", lambda: streams(x32), N * E * (8 * S4 + 4 + 4))
+        report("stream_norm of one stream (layer norm)", lambda: ops.stream_norm(h, 1, w, b, 1e-6, x, term=a, h_out=h), N * E * 14)
+        report("  Bivizen: scaled_norm (stream + two scaled terms, norm)", lambda: ops.scaled_norm(h, [(a, w), (x32, w)], wbf, 1e-6, x), N * E * 18)
+        report("  Tabopel: normed_add_norm", lambda: ops.normed_add_norm(h, a, w, 1e-6, w, 1e-6, x), N * E * 14)
+        report("  Qwen2: add_rmsnorm", lambda: ops.add_rmsnorm(h, a, wbf, 1e-6, x), N * E * 14)
+        # ---- the convolution ahead of the mixer
+        cw, cs = torch.randn(taps, E, device=dev), torch.zeros(S, taps - 1, E, device=dev)
+        cwt, tail, y32 = torch.randn(E, taps, device=dev), torch.zeros(S, E, taps - 1, device=dev), torch.empty(N, E, device=dev)
+        report("residual_conv, 4 taps", lambda: ops.residual_conv(x32, cw, cs, x, q_start, slots, longest), N * E * 6)
+        report("  Bivizen: short_conv_silu", lambda: ops.short_conv_silu(x32, cwt, tail, y32, q_start, slots, longest), N * E * 8)
+        if label == "decode":
+            report("stream_norm with the convolution in it", lambda: streams(x, conv=(cw, cs, seq)), N * E * (8 * S4 + 4 + 2 + 8 * (taps - 1)))
+        # ---- norm per head, rotation of q, k and v, page write; the turn back
+        C = (H + 2 * G) * d
+        proj = torch.randn(N, C, device=dev)
+        pages = torch.zeros(S * per_request, G * P * 2 * d, dtype=bf, device=dev)
+        qo = torch.empty(N, H, d, dtype=bf, device=dev)
+        freq = torch.rand(d // 2, dtype=torch.float64, device=dev)
+        qw, kw, temp = torch.rand(d, device=dev), torch.rand(d, device=dev), torch.rand(H, device=dev)
+        report("qk_normed_prepare (norm per head, factor per head, rotation of q, k and v)",
+               lambda: ops.qk_normed_prepare(proj, qw, kw, 1e-6, freq, "half", 1.0, positions, seq, bt, qo, pages, G, d, P, q_scale=temp, v_freq=freq), N * C * 6)
+        report("qk_normed_prepare of a layer that borrows its keys",
+               lambda: ops.qk_normed_prepare(proj[:, :H * d], qw, None, 1e-6, freq, "half", 1.0, positions, seq, bt, qo, pages, G, d, P, q_scale=temp, write_kv=False), N * H * d * 6)
+        report("  Tomodra: qk_normed_prepare (norm per head, neighbouring pairs)",
+               lambda: ops.qk_normed_prepare(proj, qw, kw, 1e-6, freq[:d // 4], "neighbours", 1.0, positions, seq, bt, qo, pages, G, d, P), N * C * 6)
+        lam, gate_h = torch.rand(1, device=dev), torch.empty(N, H, device=dev)
+        pb = torch.randn(N, C + H, device=dev)
+        report("  Bivizen: qkv_prepare (bias, rotation of half a head, values kept, gates)",
+               lambda: ops.qkv_prepare(pb, torch.zeros(C + H, device=dev), torch.rand(d // 4, device=dev), positions, seq, bt, qo, pages, G, d, P, gate_out=gate_h, v_first=torch.empty(N, G * d, device=dev), v_mode=1), N * C * 6 + N * G * d * 4)
+        ao = torch.randn(N, H, d, device=dev).to(bf)
+        report("turn_heads (the turn back of the heads' outputs)", lambda: ops.turn_heads(ao, freq, "half", positions, seq, back=True), N * H * d * 4)
+        report("  Bivizen: head_gate (a gate per head on the heads' outputs)", lambda: ops.head_gate(ao, gate_h, seq), N * H * d * 4)
+        # ---- attention inside the window, heads of 128
+        p5 = pages.view(-1, 2, G, P, d)
+        if label == "prompt":
+            plan = lambda win: i32(type("P", (TiledAttention,), {"heads": H, "window": win})().plan(
+                HostBatch(counts=[T], lengths=[0], slots=[0], q_start=[0, T])).arrays["tiles"].tolist())
+            seen = sum(min(i + 1, window) for i in range(T))
+            tw, ta = plan(window), plan(None)
+            report("prefill_attention_tc, window of 1,024", lambda: ops.prefill_attention_tc(qo, p5, bt, tw, ao, window, d ** -0.5), flops=4 * H * d * seen)
+            report("  Bivizen: prefill_attention_tc with a soft cap, all keys", lambda: ops.prefill_attention_tc(qo, p5, bt, ta, ao, None, d ** -0.5, softcap=30.0), flops=4 * H * d * (T * (T + 1) // 2))
+            report("  Qwen2: prefill_attention_tc, all keys", lambda: ops.prefill_attention_tc(qo, p5, bt, ta, ao, None, d ** -0.5), flops=4 * H * d * (T * (T + 1) // 2))
+        else:
+            kvb = lambda keys: 2 * S * min(keys, context) * G * d * 2
+            report("decode_attention, window of 1,024, the turn back in the merge", lambda: ops.decode_attention(qo, p5, bt, seq, positions, ao, window, d ** -0.5, turn=(freq, "half")), kvb(window))
+            report("  Bivizen: decode_attention with a soft cap, all keys", lambda: ops.decode_attention(qo, p5, bt, seq, positions, ao, None, d ** -0.5, softcap=30.0), kvb(context))
+            report("  Qwen2: decode_attention, all keys", lambda: ops.decode_attention(qo, p5, bt, seq, positions, ao, None, d ** -0.5), kvb(context))
+        # ---- the matrix memory, beside the scans of the other recurrent mixers with the norms behind them
+        # (a prompt's projections come in bfloat16, few rows' in float32)
+        pm, z = torch.randn(N, 4 * H * d, device=dev), torch.randn(N, 2 * H, device=dev)
+        cols = {"q": 0, "k": H * d, "v": 2 * H * d, "g": 3 * H * d, "i": 0, "f": H}
+        mem, ksum, level = torch.zeros(S, H, d, d, device=dev), torch.zeros(S, H, d, device=dev), torch.zeros(S, H, device=dev)
+        ib, fb, wm = torch.zeros(H, device=dev), torch.full((H,), 3.0, device=dev), torch.ones(H * d, device=dev)
+        ym = torch.empty(N, H * d, dtype=bf, device=dev)
+        args = (pm, z, cols, ib, fb, wm, mem, ksum, level, ym)
+        mb = N * H * d * (4 * 4 + 2) + (2 * S * H * d * d * 4 if label == "decode" else 0)
+        if label == "decode":
+            report("mlstm_step (gates, memory, read-out, norm, gate)", lambda: ops.mlstm_step(*args, q_start, slots, 15.0, d ** -0.5, 1e-6), mb)
+        else:
+            pl = MLSTM(PartSpec("mlstm", dict(hidden=E, heads=H, head_dim=d, v_dim=d, gate_cap=15.0, eps=1e-6))).plan(
+                HostBatch(counts=[T], lengths=[0], slots=[0], q_start=[0, T])).arrays
+            po, ch = i32(pl["portions"].tolist()), i32(pl["chunks"].tolist())
+            args16 = (pm.to(bf),) + args[1:]
+            report("mlstm_portions (gates, memory, read-out, norm, gate; tensor cores)", lambda: ops.mlstm_portions(*args16, po, ch, 15.0, d ** -0.5, 1e-6), N * H * d * 10)
+            report("mlstm_portions from float32 projections (CUDA cores)", lambda: ops.mlstm_portions(*args, po, ch, 15.0, d ** -0.5, 1e-6), mb)
+        state, o, dec = torch.zeros(S, H, d, d, device=dev), torch.empty(N, H, d, device=dev), torch.randn(N, H * d, device=dev)
+        alog, dtb = torch.randn(H, device=dev), torch.randn(H, device=dev)
+        bands = [pm[:, i * H * d:(i + 1) * H * d] for i in range(4)]
+        ones = torch.ones(d, device=dev)
+        gla = lambda: (ops.linear_scan(ops.SCAN_GLA, bands[0], bands[1], bands[2], dec, state, o, q_start, slots, seq, q_scale=d ** -0.5, tau=16.0),
+                       ops.gated_rmsnorm(o, bands[3], ones, 1e-6, ym, seq))
+        delta = lambda: (ops.linear_scan(ops.SCAN_DELTA, bands[0], bands[1], bands[2], dec[:, :H], state, o, q_start, slots, seq, q_scale=d ** -0.5, beta=dec[:, H:2 * H], a_log=alog, dt_bias=dtb, unit=True),
+                         ops.gated_rmsnorm(o, bands[3], ones, 1e-6, ym, seq))
+        report("  Bivizen: linear_scan (gated linear attention) and gated_rmsnorm", gla, mb + N * H * d * 4)
+        report("  Bivizen: linear_scan (gated delta rule) and gated_rmsnorm", delta, mb)
+        # ---- the gated feed-forward's activation
+        gu = torch.randn(N, 2 * ff, device=dev).to(bf)
+        act = torch.empty(N, ff, dtype=bf, device=dev)
+        report("max(gate, 0) * up behind the library's product", lambda: ops.silu_mul(gu, act, block=128, relu=True), N * ff * 6)
+        report("  Qwen2: silu_mul", lambda: ops.silu_mul(gu, act, block=128), N * ff * 6)
+        xin, wgu = torch.randn(N, E, device=dev).to(bf), torch.randn(2 * ff, E, device=dev).to(bf) * 0.02
+        kind = dict(flops=4 * N * ff * E) if N > 64 else dict(nbytes=4 * ff * E)
+        report("gemm_tc with max(gate, 0) * up in its epilogue", lambda: ops.gemm_tc(xin, wgu, act, 256, ops.EPI_SILU, act=ops.RELU), **kind)
+        report("  Bivizen: gemm_tc with its limited gate in its epilogue", lambda: ops.gemm_tc(xin, wgu, act, 256, ops.EPI_SILU, act=(1.702, 7.0, 1.0)), **kind)
+        report("  Qwen2: gemm_tc with SiLU(gate) * up in its epilogue", lambda: ops.gemm_tc(xin, wgu, act, 256, ops.EPI_SILU), **kind)
+    return rows
+
+
 def design_bench(args):
     import torch
     from air_b200.engine.batch import Entry, LAST_SAMPLED
     designs = {"bivizen": ("Bivizen", _bivizen), "tomodra": ("Tomodra", _tomodra), "pefivik": ("Pefivik", _pefivik),
-               "tabopel": ("Tabopel", _tabopel)}
+               "tabopel": ("Tabopel", _tabopel), "dafotar": ("Dafotar", _dafotar)}
     # the model that stands beside the design: the Qwen2 decoder, or the closest of the other designs
-    beside = {"pefivik": ("tomodra", "Tomodra", _tomodra), "tabopel": ("tomodra", "Tomodra", _tomodra)} \
+    beside = {"pefivik": ("tomodra", "Tomodra", _tomodra), "tabopel": ("tomodra", "Tomodra", _tomodra),
+              "dafotar": ("bivizen", "Bivizen", _bivizen)} \
         .get(args.design, ("qwen2", "Qwen2ForCausalLM", _qwen))
     if args.design not in designs:
         print(json.dumps({"error": f"--design {args.design}: the designs that are compared are {', '.join(designs)}"}))
@@ -1254,6 +1436,8 @@ def design_bench(args):
             size["kernels"] = pefivik_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
         if not args.skip_kernels and args.design == "tabopel":
             size["kernels"] = tabopel_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
+        if not args.skip_kernels and args.design == "dafotar":
+            size["kernels"] = dafotar_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
         if not args.skip_kernels and args.design == "tomodra":
             size["kernels"] = tomodra_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
         record["sizes"][name] = size
@@ -1335,7 +1519,7 @@ def main():
     ap.add_argument("--skip-decode", action="store_true", help="for profiling the prefill step alone")
     ap.add_argument("--no-graphs", action="store_true", help="launch the decode step's kernels one by one (for ncu)")
     ap.add_argument("--kernel", default="", help="prefill_attention, or prompt_elementwise (at --prefill-tokens rows): time those kernels alone and exit")
-    ap.add_argument("--design", default="", help="bivizen, tomodra, pefivik or tabopel: prefill and decode of that design beside the Qwen2 decoder (pefivik and tabopel: beside Tomodra) at "
+    ap.add_argument("--design", default="", help="bivizen, tomodra, pefivik, tabopel or dafotar: prefill and decode of that design beside the Qwen2 decoder (pefivik and tabopel: beside Tomodra; dafotar: beside Bivizen) at "
                     "equal sizes, and its kernels alone beside the like kernels (another line of output; the default "
                     "workload is not run)")
     ap.add_argument("--design-sizes", default="", help="with --design: which of the sizes 2048,4096 (default: both)")
