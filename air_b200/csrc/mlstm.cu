@@ -21,7 +21,7 @@
 // and n_chunk the states ahead of the chunk: 32-bit products on the CUDA cores, rows of different chunks side by side.
 //
 //   mlstm_gates_kernel   a, b and exp(-m) of every token, its b P(t, end) and its A: block (head, portion); m by a parallel scan of the maps
-//                        m -> max(F + m, M) (64-bit sums), 512 tokens at a time
+//                        m -> max(F + m, M) (64-bit sums), 1,024 tokens at a time
 //   mlstm_states_kernel  the states ahead of every chunk: block (tile of 32 x 64 of S, head, portion), the tile in
 //                        registers, chunk after chunk: S <- (product of the chunk's a) S + sum_s b_s P(s, end) k_s v_s^T
 //   mlstm_outputs_kernel block (chunk, head, 128 columns of v): the read-outs; where a head's v fits one block also the norm,
@@ -135,7 +135,7 @@ constexpr int ML_OV = 128;                 // columns of v per block of mlstm_ou
 constexpr int ML_KS = 64;                  // key channels staged at a time there
 constexpr int ML_LD = ML_KS + 4, ML_LV = ML_OV + 4;
 
-constexpr int ML_GT = 512;                 // threads of mlstm_gates_kernel
+constexpr int ML_GT = 1024;                // threads of mlstm_gates_kernel
 
 __global__ void __launch_bounds__(ML_GT) mlstm_gates_kernel(const MlstmChunkArgs c) {
     __shared__ double wF[ML_GT / 32], wM[ML_GT / 32], mt[ML_GT + 1];
@@ -172,8 +172,21 @@ __global__ void __launch_bounds__(ML_GT) mlstm_gates_kernel(const MlstmChunkArgs
         if (lane == 31) { wF[warp] = F; wM[warp] = M; }
         if (tid == 0) mt[0] = carry;
         __syncthreads();
-        double m = carry;
-        for (int w = 0; w < warp; ++w) m = fmax(wF[w] + m, wM[w]);
+        if (warp == 0) {                   // the maps of all warps before each warp, by one more scan
+            double F1 = wF[lane], M1 = wM[lane];
+#pragma unroll
+            for (int off = 1; off < 32; off <<= 1) {
+                const double F0 = __shfl_up_sync(0xffffffffu, F1, off), M0 = __shfl_up_sync(0xffffffffu, M1, off);
+                if (lane >= off) {
+                    M1 = fmax(M0 + F1, M1);
+                    F1 = F0 + F1;
+                }
+            }
+            wF[lane] = F1;
+            wM[lane] = M1;
+        }
+        __syncthreads();
+        double m = warp == 0 ? carry : fmax(wF[warp - 1] + carry, wM[warp - 1]);
         m = fmax(F + m, M);
         mt[tid + 1] = m;
         __syncthreads();

@@ -24,6 +24,7 @@ struct MlstmTcArgs {
 
 constexpr int MT_LK = 72, MT_LV = 136;     // row lengths in shared memory (64 and 128 numbers; 8 rows on different banks)
 constexpr int MT_LD = 68;
+static_assert(64 * MT_LV <= 2 * 64 * MT_LK, "the gate's rows fit where q and k were");
 
 __device__ __forceinline__ uint32_t mt_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -165,13 +166,13 @@ __global__ void __launch_bounds__(256) mlstm_tc_chain_kernel(const MlstmTcArgs q
     }
 }
 
-constexpr size_t MT_OUT_SMEM = sizeof(float) * (64 * MT_LD + 4 * 64) + 2 * (2 * 64 * MT_LK + 2 * 64 * MT_LV);
+constexpr size_t MT_OUT_SMEM = sizeof(float) * (64 * MT_LD + 4 * 64 + 128) + 2 * (2 * 64 * MT_LK + 2 * 64 * MT_LV);
 
 template <typename TO>
 __global__ void __launch_bounds__(128, 3) mlstm_tc_outputs_kernel(const MlstmTcArgs q) {
     extern __shared__ __align__(16) float smem[];
-    float *sd = smem, *sa = sd + 64 * MT_LD, *sA = sa + 64, *sn = sA + 64, *sfloor = sn + 64;
-    __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(sfloor + 64);
+    float *sd = smem, *sa = sd + 64 * MT_LD, *sA = sa + 64, *sn = sA + 64, *sfloor = sn + 64, *sweight = sfloor + 64;
+    __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(sweight + 128);
     __nv_bfloat16 *sk = sq + 64 * MT_LK, *sh = sk + 64 * MT_LK, *sl = sh + 64 * MT_LV;     // S: high part, rest
     pdl_enter(TR_MLSTM);
     const MlstmArgs& p = q.c.p;
@@ -199,6 +200,7 @@ __global__ void __launch_bounds__(128, 3) mlstm_tc_outputs_kernel(const MlstmTcA
         sA[t] = t < cnt ? ga[4 * plane + t] : 0.f;
         sfloor[t] = t < cnt ? ga[2 * plane + t] : 1.f;
     }
+    sweight[tid] = v0 + tid < dv ? p.w[h * dv + v0 + tid] : 0.f;
     __syncthreads();
     if (tid < 64) {          // b_s P(s, t) for W[t, s]
         float w = tid < cnt ? ga[plane + tid] : 0.f;
@@ -253,7 +255,9 @@ __global__ void __launch_bounds__(128, 3) mlstm_tc_outputs_kernel(const MlstmTcA
         }
     }
     __syncthreads();
-    mt_stage<128, MT_LV>(sh, src + p.cv + h * dv + v0, p.ldx, cnt, dv - v0);      // the values take the states' place
+    mt_stage<128, MT_LV>(sh, src + p.cv + h * dv + v0, p.ldx, cnt, dv - v0);      // the values take the states' place,
+    __nv_bfloat16* sg = sq;                                                        // the gate that of q and k
+    if (!q.c.o) mt_stage<128, MT_LV>(sg, src + p.cg + h * dv + v0, p.ldx, cnt, dv - v0);
     mt_commit();
     const int tr[2] = {16 * warp + g, 16 * warp + g + 8};                          // this thread's two tokens
     float inv[2];
@@ -313,19 +317,22 @@ __global__ void __launch_bounds__(128, 3) mlstm_tc_outputs_kernel(const MlstmTcA
         if (tr[i] >= cnt) continue;
         const size_t at = ((size_t)(row0 + tr[i]) * p.H + h) * dv;
         const float scale = 1.f / sqrtf(ss / (float)dv + p.eps);
-        const __nv_bfloat16* gr = src + (size_t)tr[i] * p.ldx + p.cg + h * dv;
+        const __nv_bfloat16* gr = sg + tr[i] * MT_LV;
 #pragma unroll
         for (int n = 0; n < 16; ++n) {
-            const int c = v0 + 8 * n + t2;
-            if (c >= dv) continue;
+            const int c = 8 * n + t2;
+            if (v0 + c >= dv) continue;
             if (q.c.o) {
-                *reinterpret_cast<float2*>(q.c.o + at + c) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
+                *reinterpret_cast<float2*>(q.c.o + at + v0 + c) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
                 continue;
             }
             const float2 gate = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr + c));
-            TO* y = (TO*)p.y + at + c;
-            y[0] = from_float<TO>(o[n][2 * i] * scale * p.w[h * dv + c] / (1.f + expf(-gate.x)));
-            y[1] = from_float<TO>(o[n][2 * i + 1] * scale * p.w[h * dv + c + 1] / (1.f + expf(-gate.y)));
+            const float2 wv = *reinterpret_cast<const float2*>(sweight + c);
+            const float y0 = o[n][2 * i] * scale * wv.x / (1.f + expf(-gate.x));
+            const float y1 = o[n][2 * i + 1] * scale * wv.y / (1.f + expf(-gate.y));
+            TO* y = (TO*)p.y + at + v0 + c;
+            if constexpr (sizeof(TO) == 2) *reinterpret_cast<__nv_bfloat162*>(y) = __floats2bfloat162_rn(y0, y1);
+            else *reinterpret_cast<float2*>(y) = make_float2(y0, y1);
         }
     }
 }

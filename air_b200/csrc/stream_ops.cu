@@ -90,89 +90,127 @@ __device__ __forceinline__ void stream_columns(const StreamNormArgs& p, size_t s
     }
 }
 
-template <typename TO, int NS, int N>
+// The finished row's columns i .. i + N - 1: weight and bias, the convolution (slot >= 0), the write.
+template <typename TO, int N>
+__device__ __forceinline__ void stream_finish(const StreamNormArgs& p, TO* out, int slot, int i, const float (&u)[N], float mean,
+                                              float scale, const float (&wv)[N], const float (&bv)[N]) {
+    float v[N];
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = (u[j] - mean) * scale * wv[j] + bv[j];
+    if (slot >= 0) {      // (four earlier inputs and their weights under way at a time)
+        const int keep = p.taps - 1, E = p.E;
+        float* st = p.conv_state + (size_t)slot * keep * E + i;
+        const float* cw = p.conv_w + i;
+        float acc[N];
+        load_columns<N>(cw + (size_t)keep * E, acc);
+#pragma unroll
+        for (int j = 0; j < N; ++j) acc[j] = fmaf(acc[j], v[j], v[j]);
+        for (int k0 = 0; k0 < keep; k0 += 4) {
+            float in[4][N], wk[4][N];
+#pragma unroll
+            for (int u2 = 0; u2 < 4; ++u2)
+                if (k0 + u2 < keep) {
+                    load_columns<N>(st + (size_t)(k0 + u2) * E, in[u2]);
+                    load_columns<N>(cw + (size_t)(k0 + u2) * E, wk[u2]);
+                }
+#pragma unroll
+            for (int u2 = 0; u2 < 4; ++u2)
+                if (k0 + u2 < keep) {
+#pragma unroll
+                    for (int j = 0; j < N; ++j) acc[j] = fmaf(wk[u2][j], in[u2][j], acc[j]);
+                    if (k0 + u2 > 0) store_columns<N>(st + (size_t)(k0 + u2 - 1) * E, in[u2]);
+                }
+        }
+        if (keep > 0) store_columns<N>(st + (size_t)(keep - 1) * E, v);
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] = acc[j];
+    }
+    if constexpr (N == 4) store4(out + i, v);
+    else out[i] = from_float<TO>(v[0]);
+}
+
+// A block per row.  ONE: a thread has one piece of N columns at most (few rows: a decode step), which stays in registers, and
+// has its weights before the predecessor's rows are there; else the row waits in shared memory between the passes.
+template <typename TO, int NS, int N, bool ONE>
 __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormArgs p) {
     __shared__ float scratch[32];
     __shared__ float coef[STREAMS_MAX * STREAMS_MAX + 2 * STREAMS_MAX];
     extern __shared__ __align__(16) float urow[];
-    pdl_enter(TR_STREAM_NORM);
-    const int r = blockIdx.x, E = p.E, S = NS ? NS : p.S;
-    const size_t src = (size_t)(p.rows ? p.rows[r] : r) * E;
+    const int E = p.E, S = NS ? NS : p.S, first = threadIdx.x * N;
+    pdl_trigger();
+    // what no kernel writes
     for (int i = threadIdx.x; i < S * S + 2 * S; i += blockDim.x) {
         const int k = i - S * S;
         coef[i] = k < 0 ? (p.mix ? p.mix[i] : 0.f) : k < S ? (p.out_w ? p.out_w[k] : 1.f) : (p.read ? p.read[k - S] : 1.f);
     }
-    __syncthreads();
-    float sum = 0.f;
-    const int step = blockDim.x * N;
-    for (int i = threadIdx.x * N; i < E; i += step) {
-        float u[N];
-        stream_columns<NS, N>(p, src, i, coef, u);
+    float w1[N], b1[N];
 #pragma unroll
-        for (int j = 0; j < N; ++j) {
-            urow[i + j] = u[j];
-            sum += p.center ? u[j] : u[j] * u[j];
+    for (int j = 0; j < N; ++j) w1[j] = b1[j] = 0.f;
+    if (ONE && p.w && first < E) {
+        load_columns<N>(p.w + first, w1);
+        if (p.b) load_columns<N>(p.b + first, b1);
+    }
+    __syncthreads();
+    pdl_wait();
+    trace_point(TR_STREAM_NORM);
+    const int r = blockIdx.x;
+    const size_t src = (size_t)(p.rows ? p.rows[r] : r) * E;
+    const int step = blockDim.x * N;
+    float u1[N], sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < N; ++j) u1[j] = 0.f;
+    if constexpr (ONE) {
+        if (first < E) stream_columns<NS, N>(p, src, first, coef, u1);
+#pragma unroll
+        for (int j = 0; j < N; ++j) sum += p.center ? u1[j] : u1[j] * u1[j];
+    } else {
+        for (int i = first; i < E; i += step) {
+            float u[N];
+            stream_columns<NS, N>(p, src, i, coef, u);
+#pragma unroll
+            for (int j = 0; j < N; ++j) {
+                urow[i + j] = u[j];
+                sum += p.center ? u[j] : u[j] * u[j];
+            }
         }
     }
     if (!p.w) return;
-    float mean = 0.f, var;
+    float mean = 0.f;
     if (p.center) {
         mean = block_sum(sum, scratch) / (float)E;
         sum = 0.f;
-        for (int i = threadIdx.x * N; i < E; i += step)
+        if constexpr (ONE) {
 #pragma unroll
             for (int j = 0; j < N; ++j) {
-                const float d = urow[i + j] - mean;
-                sum = fmaf(d, d, sum);
+                const float d = u1[j] - mean;
+                if (first < E) sum = fmaf(d, d, sum);
             }
+        } else {
+            for (int i = first; i < E; i += step)
+#pragma unroll
+                for (int j = 0; j < N; ++j) {
+                    const float d = urow[i + j] - mean;
+                    sum = fmaf(d, d, sum);
+                }
+        }
     }
-    var = block_sum(sum, scratch) / (float)E;
-    const float scale = 1.f / sqrtf(var + p.eps);
+    const float scale = 1.f / sqrtf(block_sum(sum, scratch) / (float)E + p.eps);
     TO* out = (TO*)p.out + (size_t)r * E;
     const int slot = p.conv_w ? p.token_seq[r] : -1;
-    for (int i = threadIdx.x * N; i < E; i += step) {
-        float v[N], wv[N], bv[N];
-        if constexpr (N == 4) load4(p.w + i, wv);
-        else wv[0] = p.w[i];
-        if (p.b) {
-            if constexpr (N == 4) load4(p.b + i, bv);
-            else bv[0] = p.b[i];
-        }
+    if constexpr (ONE) {
+        if (first < E) stream_finish<TO, N>(p, out, slot, first, u1, mean, scale, w1, b1);
+    } else {
+        for (int i = first; i < E; i += step) {
+            float u[N], wv[N], bv[N];
 #pragma unroll
-        for (int j = 0; j < N; ++j) {
-            v[j] = (urow[i + j] - mean) * scale * wv[j];
-            if (p.b) v[j] += bv[j];
-        }
-        if (slot >= 0) {      // (four earlier inputs and their weights under way at a time)
-            const int keep = p.taps - 1;
-            float* st = p.conv_state + (size_t)slot * keep * E + i;
-            const float* cw = p.conv_w + i;
-            float acc[N];
-            load_columns<N>(cw + (size_t)keep * E, acc);
-#pragma unroll
-            for (int j = 0; j < N; ++j) acc[j] = fmaf(acc[j], v[j], v[j]);
-            for (int k0 = 0; k0 < keep; k0 += 4) {
-                float in[4][N], wk[4][N];
-#pragma unroll
-                for (int u = 0; u < 4; ++u)
-                    if (k0 + u < keep) {
-                        load_columns<N>(st + (size_t)(k0 + u) * E, in[u]);
-                        load_columns<N>(cw + (size_t)(k0 + u) * E, wk[u]);
-                    }
-#pragma unroll
-                for (int u = 0; u < 4; ++u)
-                    if (k0 + u < keep) {
-#pragma unroll
-                        for (int j = 0; j < N; ++j) acc[j] = fmaf(wk[u][j], in[u][j], acc[j]);
-                        if (k0 + u > 0) store_columns<N>(st + (size_t)(k0 + u - 1) * E, in[u]);
-                    }
+            for (int j = 0; j < N; ++j) {
+                u[j] = urow[i + j];
+                bv[j] = 0.f;
             }
-            if (keep > 0) store_columns<N>(st + (size_t)(keep - 1) * E, v);
-#pragma unroll
-            for (int j = 0; j < N; ++j) v[j] = acc[j];
+            load_columns<N>(p.w + i, wv);
+            if (p.b) load_columns<N>(p.b + i, bv);
+            stream_finish<TO, N>(p, out, slot, i, u, mean, scale, wv, bv);
         }
-        if constexpr (N == 4) store4(out + i, v);
-        else out[i] = from_float<TO>(v[0]);
     }
 }
 
@@ -244,24 +282,25 @@ AIR_API int air_stream_norm(const float* x, long long x_stride, float* h_out, lo
     const bool vec = E % 4 == 0 && x_stride % 4 == 0 && h_stride % 4 == 0 && part_stride % 4 == 0 && al(x) && al(h_out) &&
                      al(y) && al(w) && al(b) && al(out) && al(conv_w) && al(conv_state);
     // few rows: one access of a thread per row, all of a row's loads under way at once
-    const int items = vec ? E / 4 : E;
+    const int items = vec && S <= 4 ? E / 4 : E;
     int threads = items >= 256 ? 256 : (items + 31) / 32 * 32;
     if (R <= 256) threads = items >= 1024 ? 1024 : (items + 31) / 32 * 32;
     AIR_DISPATCH(out_dtype, TO, {
-        auto go = [&](auto kernel) {
-            if (smem > 44 * 1024) {
-                cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        auto go = [&](auto kernel, size_t row) {
+            if (row > 44 * 1024) {
+                cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)row);
                 if (err != cudaSuccess) return (int)err;
             }
-            return air::launch(kernel, R, threads, smem, stream, p);
+            return air::launch(kernel, R, threads, row, stream, p);
         };
-        if (!vec) return go(air::stream_norm_kernel<TO, 0, 1>);
+        const bool one = items <= threads;
+        if (!vec || S > 4)
+            return one ? go(air::stream_norm_kernel<TO, 0, 1, true>, 0) : go(air::stream_norm_kernel<TO, 0, 1, false>, smem);
         switch (S) {
-            case 1: return go(air::stream_norm_kernel<TO, 1, 4>);
-            case 2: return go(air::stream_norm_kernel<TO, 2, 4>);
-            case 3: return go(air::stream_norm_kernel<TO, 3, 4>);
-            case 4: return go(air::stream_norm_kernel<TO, 4, 4>);
-            default: return go(air::stream_norm_kernel<TO, 0, 1>);
+            case 1: return one ? go(air::stream_norm_kernel<TO, 1, 4, true>, 0) : go(air::stream_norm_kernel<TO, 1, 4, false>, smem);
+            case 2: return one ? go(air::stream_norm_kernel<TO, 2, 4, true>, 0) : go(air::stream_norm_kernel<TO, 2, 4, false>, smem);
+            case 3: return one ? go(air::stream_norm_kernel<TO, 3, 4, true>, 0) : go(air::stream_norm_kernel<TO, 3, 4, false>, smem);
+            default: return one ? go(air::stream_norm_kernel<TO, 4, 4, true>, 0) : go(air::stream_norm_kernel<TO, 4, 4, false>, smem);
         }
     });
     return 0;
