@@ -1247,7 +1247,7 @@ def tabopel_kernels(width, heads, kv_heads, ff, T, batch, context):
 
 def kernel_reporter():
     """(report, rows): report(name, f, nbytes or flops) times f from memory (512 MB written before each launch, the writes'
-    own time subtracted, ten launches replayed as a graph), prints microseconds and the share of the measured copy rate or
+    own time subtracted, five launches replayed as a graph), prints microseconds and the share of the measured copy rate or
     bf16 rate that the algorithm's bytes or flops make, and appends both to rows."""
     import torch
     pk = peaks()

@@ -77,7 +77,7 @@ def run_in_steps(run, cache, streams, steps):
 
 
 STEPS = [[("a", 3)], [("a", 61), ("b", 1)], [("b", 2), ("a", 1)], [("a", 150), ("b", 40)], [("a", 2)], [("a", 1), ("b", 1)],
-         [("b", 31), ("a", 1)], [("a", 30)], [("a", 70)], [("a", 1)]]          # a: 320 tokens, b: 75
+         [("b", 30), ("a", 1)], [("a", 30)], [("a", 70), ("b", 1)], [("a", 1)]]          # a: 320 tokens, b: 75
 
 
 # ----------------------------------------------------------------------------- mechanisms alone
