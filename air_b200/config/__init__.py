@@ -4,6 +4,7 @@ from .tomodra_config import TomodraConfig
 from .pefivik_config import PefivikConfig
 from .tabopel_config import TabopelConfig
 from .dafotar_config import DafotarConfig
+from .sesulorn_config import SesulornConfig
 from . import architectures  # registers the known architectures
 import json
 import os

@@ -9,6 +9,7 @@ from .bivizen_config import BivizenConfig
 from .dafotar_config import DafotarConfig
 from .model_config import Qwen2Config
 from .pefivik_config import PefivikConfig
+from .sesulorn_config import SesulornConfig
 from .tabopel_config import TabopelConfig
 from .tomodra_config import TomodraConfig
 
@@ -318,3 +319,60 @@ def dafotar_spec(config: DafotarConfig) -> ModelSpec:
 
 
 register_architecture("Dafotar", DafotarConfig, dafotar_spec)
+
+
+def sesulorn_spec(config: SesulornConfig) -> ModelSpec:
+    """Sesulorn: every layer is a parallel block (one layer norm with a bias whose rows the mixer and the feed-forward both
+    read, their outputs added to the stream together).  The mixer is grouped-query attention without positions but for a
+    learned bias per distance and head, with queries and keys over their root mean square ("attention"), the delta rule with a
+    decay per key channel ("channel_delta"), or attention over a compressed latent whose queries come through a latent of
+    their own, with a rotation of neighbouring pairs ("latent_attention").  The feed-forward is a dense gated one, or a
+    mixture of experts with a clamped activation chosen among the groups with the best experts, beside a gated shared expert.
+    A stretch of layers may run several times over with the same weights, every pass with a cache of its own; ahead of every
+    pass the stream is replaced by loop.in [x | x0], x0 being the embedding's output.  Tensors: embed, loop.in, l<i>.norm1,
+    norm1.b, l<i>.mix.*, l<i>.mlp.*, final.norm, final.norm.b, head."""
+    e = config.width
+    norm = PartSpec("layer", {"size": e, "eps": config.eps, "tensor": "", "bias": ".b"})
+    layers = []
+    for l in config.layers:
+        if l.type == "attention":
+            mixer = PartSpec("normed_attention", {
+                "hidden": e, "heads": l.heads, "kv_heads": l.kv_heads, "head_dim": l.dim, "v_dim": l.vdim, "scale": l.scale,
+                "eps": config.eps, "qkv_bias": True, "qk_norm": "bare",
+                "distance_bias": {"rows": l.buckets, "span": l.bias_max},
+                "position": PartSpec("rope_live", {"rotary_dim": 0, "theta": 1.0})})
+        elif l.type == "channel_delta":
+            mixer = PartSpec("channel_delta", {
+                "hidden": e, "heads": l.heads, "kv_heads": l.kv_heads, "head_dim": l.dim, "v_dim": l.vdim, "conv": l.conv,
+                "decay_rank": l.decay_rank, "gate_rank": l.gate_rank, "eps": config.eps})
+        else:
+            params = {"hidden": e, "heads": l.heads, "head_dim": l.dim, "rot_dim": l.rot_dim, "v_dim": l.vdim,
+                      "kv_rank": l.kv_rank, "q_rank": l.q_rank, "scale": l.scale, "window": None, "eps": config.eps}
+            if l.rot_dim:
+                params["position"] = PartSpec("rope_live", {"rotary_dim": l.rot_dim, "theta": l.rot_base,
+                                                            "pairing": "neighbours"})
+            mixer = PartSpec("latent_attention", params)
+        parts = {"norm": norm, "mixer": mixer}
+        f = l.mlp
+        if f is not None and f.kind == "dense":
+            parts["feed_forward"] = PartSpec("swiglu_plain_names", {"hidden": e, "intermediate": f.ff})
+        elif f is not None:
+            parts["feed_forward"] = PartSpec("routed_experts", {
+                "hidden": e, "experts": f.experts, "top": f.top, "intermediate": f.ff, "limit": f.limit,
+                "shared_intermediate": f.shared_ff, "shared_limit": f.shared_limit, "shared_gate": bool(f.shared_ff),
+                "score": "softmax", "renormalize": False, "groups": (f.groups, f.keep) if f.groups > 1 else None,
+                "group_mark": "best", "weight_on": "output", "activation": "clamped_glu"})
+        layers.append(BlockSpec(kind="parallel", prefix=f"l{len(layers)}.", parts=parts,
+                                names={"norm": "norm1", "mixer": "mix.", "feed_forward": "mlp."}))
+    order = [RunStep(i) for i in range(config.loop_start)]
+    if config.loops:
+        order += [RunStep(i, mix_embedding="loop.in" if i == config.loop_start else None)
+                  for _ in range(config.loop_times) for i in range(config.loop_start, config.loop_stop)]
+    order += [RunStep(i) for i in range(config.loop_stop if config.loops else config.loop_start, len(layers))]
+    return ModelSpec(
+        architecture=config.architecture, hidden_size=e, vocab_size=config.vocab, max_positions=config.max_positions,
+        layers=tuple(layers), order=tuple(order), final_norm=norm, embedding_name="embed", final_norm_prefix="final.norm",
+        output_name="head", eos_token_id=config.eos_token_id, stream_mixes=("loop.in",) if config.has_loop else ())
+
+
+register_architecture("Sesulorn", SesulornConfig, sesulorn_spec)

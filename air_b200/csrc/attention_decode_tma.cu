@@ -14,6 +14,9 @@
 // 64 / min(P, 64) boxes of min(P, 64) rows, each found through the block table.
 // Every wait on an mbarrier is bounded (tma.cuh); on giving up the block flags *status = 5.
 //
+// With `bias` a score gets the head's number for its key's distance (DistanceBias); tiles that lie farther back than the
+// table reaches take its last entry from a register.
+//
 // With `fresh.qkv` the kernel also does what qkv_rope_store does for its token (elementwise.cu): it adds up
 // the partial sums of the q/k/v product and the bias, rotates q and k by the table's row of the token's
 // position, keeps q in shared memory, and writes k and v to the page.  The blocks whose tiles hold the
@@ -50,7 +53,7 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const
                             const int* __restrict__ block_table, int max_blocks, const int* __restrict__ token_seq,
                             const int* __restrict__ positions, __nv_bfloat16* __restrict__ out,
                             float* __restrict__ part_o, float* __restrict__ part_ml, int H, int K, int P, int window,
-                            float scale_log2, float cap_log2, float cap_pre, int* status) {
+                            float scale_log2, float cap_log2, float cap_pre, int* status, const DistanceBias bias) {
     // cap_log2 > 0: a score s becomes cap * tanh(s * cap_pre) with cap_pre = scale / cap, in units of log2 e
     constexpr int SUB = D / 64;                 // 64-column sub-tiles of a row
     constexpr int SUB_BYTES = DT_TILE * 128;    // 8 KB
@@ -253,6 +256,15 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const
                 qa[kk][3] = r1 < G ? __ldg(reinterpret_cast<const uint32_t*>(q1 + 8)) : 0u;
             }
         }
+        // the bias' rows of this lane's two heads, and their last entries
+        const float *bias0 = nullptr, *bias1 = nullptr;
+        float far0 = 0.f, far1 = 0.f;
+        if (bias.table) {
+            bias0 = bias.table + (size_t)(kvh * G + min(r0, G - 1)) * bias.n;
+            bias1 = bias.table + (size_t)(kvh * G + min(r1, G - 1)) * bias.n;
+            far0 = bias0[bias.n - 1] * 1.4426950408889634f;
+            far1 = bias1[bias.n - 1] * 1.4426950408889634f;
+        }
         const int mat = lane >> 3, mrow = lane & 7;   // ldmatrix: which 8x8 matrix this lane addresses, which row
         bool alive = true;
         for (int it = 0; it < n_tiles; ++it) {
@@ -288,6 +300,22 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const
                     mma_bf16_16816(s[1], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b[2], b[3]);
                 }
                 float tm0 = -INFINITY, tm1 = -INFINITY;
+                float add[2][4];
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    add[j][0] = add[j][1] = far0;
+                    add[j][2] = add[j][3] = far1;
+                }
+                if (bias.table && pos - (kbase + 15) < bias.n - 1) {
+#pragma unroll
+                    for (int j = 0; j < 2; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) {
+                            const int back = max(0, min(pos - (kbase + 8 * j + 2 * tq + e), bias.n - 1));
+                            add[j][e] = bias0[back] * 1.4426950408889634f;
+                            add[j][2 + e] = bias1[back] * 1.4426950408889634f;
+                        }
+                }
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -295,11 +323,11 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const
                         const int key = kbase + 8 * j + 2 * tq + e;
                         const bool ok = key >= lo && key <= pos;
                         if (cap_log2 > 0.f) {
-                            s[j][e] = ok ? cap_log2 * tanhf(s[j][e] * cap_pre) : -INFINITY;
-                            s[j][2 + e] = ok ? cap_log2 * tanhf(s[j][2 + e] * cap_pre) : -INFINITY;
+                            s[j][e] = ok ? cap_log2 * tanhf(s[j][e] * cap_pre) + add[j][e] : -INFINITY;
+                            s[j][2 + e] = ok ? cap_log2 * tanhf(s[j][2 + e] * cap_pre) + add[j][2 + e] : -INFINITY;
                         } else {
-                            s[j][e] = ok ? s[j][e] * scale_log2 : -INFINITY;
-                            s[j][2 + e] = ok ? s[j][2 + e] * scale_log2 : -INFINITY;
+                            s[j][e] = ok ? fmaf(s[j][e], scale_log2, add[j][e]) : -INFINITY;
+                            s[j][2 + e] = ok ? fmaf(s[j][2 + e], scale_log2, add[j][2 + e]) : -INFINITY;
                         }
                         tm0 = fmaxf(tm0, s[j][e]);
                         tm1 = fmaxf(tm1, s[j][2 + e]);
@@ -403,7 +431,7 @@ template <int D>
 int launch_decode_tma(const CUtensorMap& map, const FreshQkv& fresh, const void* q, const int* block_table, int max_blocks,
                       const int* token_seq, const int* positions, void* out, float* part_o, float* part_ml, int T,
                       int H, int K, int P, int window, float scale, float softcap, int splits, int* status,
-                      cudaStream_t stream) {
+                      const DistanceBias& bias, cudaStream_t stream) {
     const int head_blocks = (H / K + 15) / 16;
     const size_t ring = (size_t)DT_STAGES * 2 * (D / 64) * DT_TILE * 128;
     const size_t merge = (size_t)(DT_CONSUMERS * 16 * D + 2 * DT_CONSUMERS * 16) * sizeof(float);
@@ -414,7 +442,7 @@ int launch_decode_tma(const CUtensorMap& map, const FreshQkv& fresh, const void*
     return launch(kernel, dim3(splits, K * head_blocks, T), DT_THREADS, smem, stream, map, fresh, (const __nv_bfloat16*)q,
                   block_table, max_blocks, token_seq, positions, (__nv_bfloat16*)out, part_o, part_ml, H, K, P, window,
                   scale * 1.4426950408889634f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f,
-                  softcap > 0.f ? scale / softcap : 0.f, status);
+                  softcap > 0.f ? scale / softcap : 0.f, status, bias);
 }
 
 }  // namespace air
@@ -434,8 +462,10 @@ static int decode_attention_tma(const FreshQkv& fresh, const void* q, const void
                                 void* out, float* part_o, float* part_ml, int T, int H, int K, int D, int P, int window,
                                 float scale, float softcap, int splits, int* status, cudaStream_t stream,
                                 const float* sink = nullptr, const float* gate = nullptr, int ldg = 0,
-                                const TurnBack& turn = TurnBack{nullptr, 0, 0, nullptr}) {
+                                const TurnBack& turn = TurnBack{nullptr, 0, 0, nullptr},
+                                const DistanceBias& bias = DistanceBias{nullptr, 0}) {
     if (T <= 0) return 0;
+    if (bias.table && bias.n < 1) return AIR_ERR_BAD_ARGUMENT;
     if (H <= 0 || K <= 0 || H % K || P % 16 || (P < 64 ? 64 % P : P % 64) || splits < 1 || T > 65535 ||
         (splits > 1 && (!part_o || !part_ml)) || ((uintptr_t)cache & 15))
         return AIR_ERR_BAD_ARGUMENT;
@@ -449,15 +479,15 @@ static int decode_attention_tma(const FreshQkv& fresh, const void* q, const void
     switch (D) {
         case 64:
             rc = launch_decode_tma<64>(map, fresh, q, block_table, max_blocks, token_seq, positions, out, part_o, part_ml,
-                                       T, H, K, P, window, scale, softcap, splits, status, stream);
+                                       T, H, K, P, window, scale, softcap, splits, status, bias, stream);
             break;
         case 128:
             rc = launch_decode_tma<128>(map, fresh, q, block_table, max_blocks, token_seq, positions, out, part_o,
-                                        part_ml, T, H, K, P, window, scale, softcap, splits, status, stream);
+                                        part_ml, T, H, K, P, window, scale, softcap, splits, status, bias, stream);
             break;
         case 256:
             rc = launch_decode_tma<256>(map, fresh, q, block_table, max_blocks, token_seq, positions, out, part_o,
-                                        part_ml, T, H, K, P, window, scale, softcap, splits, status, stream);
+                                        part_ml, T, H, K, P, window, scale, softcap, splits, status, bias, stream);
             break;
         default:
             return AIR_ERR_BAD_ARGUMENT;
@@ -485,17 +515,19 @@ AIR_API int air_decode_attention_tma(const void* q, const void* cache, long long
 // The same with one more term exp(sink[h]) in every head's softmax denominator (sink float32 [H] or null) and the
 // output multiplied, element by element, by sigmoid(gate[t][h * D + col]) (gate float32, rows of ldg floats, or null), and
 // ahead of the gate the first turn_rot elements of every head turned back by the token's position (turn_freq float64
-// [turn_rot / 2], or null; see TurnBack); all enter where the key splits are merged, so splits >= 2.
+// [turn_rot / 2], or null; see TurnBack); all enter where the key splits are merged, so splits >= 2 where one of them is
+// given.  bias [H, bias_n] float32 or null: see DistanceBias.
 AIR_API int air_decode_attention_tma_sink(const void* q, const void* cache, long long pages, const int* block_table,
                                           int max_blocks, const int* token_seq, const int* positions, void* out,
                                           float* part_o, float* part_ml, int T, int H, int K, int D, int P, int window,
                                           float scale, float softcap, int splits, int* status, const float* sink,
                                           const float* gate, int ldg, const double* turn_freq, int turn_rot,
-                                          int turn_pairing, cudaStream_t stream) {
+                                          int turn_pairing, const float* bias, int bias_n, cudaStream_t stream) {
     return air::decode_attention_tma(air::FreshQkv{nullptr, 0, 0, nullptr, nullptr, nullptr}, q, cache, pages,
                                      block_table, max_blocks, token_seq, positions, out, part_o, part_ml, T, H, K, D, P,
                                      window, scale, softcap, splits, status, stream, sink, gate, ldg,
-                                     air::TurnBack{turn_freq, turn_rot, turn_pairing, positions});
+                                     air::TurnBack{turn_freq, turn_rot, turn_pairing, positions},
+                                     air::DistanceBias{bias, bias_n});
 }
 
 // The same from the q/k/v product's output instead of q: qkv float32 [parts][T][(H + 2 K) D] (partial sums that

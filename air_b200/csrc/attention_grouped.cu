@@ -51,7 +51,7 @@ __global__ void __launch_bounds__(256)
 grouped_attention_kernel(const void* __restrict__ q_any, int q_f32, const T* __restrict__ cache,
                          const int* __restrict__ block_table, int max_blocks, const int* __restrict__ token_seq,
                          const int* __restrict__ positions, float* __restrict__ part, int H, int G, int d, int dv, int P,
-                         int window, int mask_mode, float scale, float softcap, int latent, int splits) {
+                         int window, int mask_mode, float scale, float softcap, int latent, int splits, const DistanceBias bias) {
     constexpr int JT = JB / 2, PER = Words<T>::per, NI = Words<T>::ni;
     extern __shared__ __align__(16) float smem[];
     pdl_enter(TR_ATT_GROUPED);
@@ -159,8 +159,12 @@ grouped_attention_kernel(const void* __restrict__ q_any, int q_f32, const T* __r
         __syncthreads();
         for (int j = warp; j < JB; j += 8) {
             const bool seen0 = key0 + lane >= lo && key0 + lane <= pos, seen1 = key0 + lane + 32 >= lo && key0 + lane + 32 <= pos;
-            const float s0 = seen0 ? capped((S[lane * JB + j] + S[(GA_KT + lane) * JB + j]) * scale, softcap) : -INFINITY;
-            const float s1 = seen1 ? capped((S[(lane + 32) * JB + j] + S[(GA_KT + lane + 32) * JB + j]) * scale, softcap) : -INFINITY;
+            float s0 = seen0 ? capped((S[lane * JB + j] + S[(GA_KT + lane) * JB + j]) * scale, softcap) : -INFINITY;
+            float s1 = seen1 ? capped((S[(lane + 32) * JB + j] + S[(GA_KT + lane + 32) * JB + j]) * scale, softcap) : -INFINITY;
+            if (bias.table) {
+                s0 += distance_bias(bias, head0 + min(j, nj - 1), pos - key0 - lane);
+                s1 += distance_bias(bias, head0 + min(j, nj - 1), pos - key0 - lane - 32);
+            }
             const float m_old = mrun[j];
             const float m_new = fmaxf(m_old, warp_max(fmaxf(s0, s1)));
             float p0 = 0.f, p1 = 0.f, c = 1.f;
@@ -250,7 +254,8 @@ __global__ void __launch_bounds__(256)
 grouped_attention_tc_kernel(const void* __restrict__ q_any, int q_f32, const __nv_bfloat16* __restrict__ cache,
                             const int* __restrict__ block_table, int max_blocks, const int* __restrict__ token_seq,
                             const int* __restrict__ positions, float* __restrict__ part, int H, int G, int d, int dv,
-                            int P, int window, int mask_mode, float scale, float softcap, int latent, int splits, int stages) {
+                            int P, int window, int mask_mode, float scale, float softcap, int latent, int splits, int stages,
+                            const DistanceBias bias) {
     constexpr int JB = 16, PLD = GA_KT + 8;
     extern __shared__ __align__(16) float smem[];
     pdl_enter(TR_ATT_GROUPED);
@@ -378,8 +383,12 @@ grouped_attention_tc_kernel(const void* __restrict__ q_any, int q_f32, const __n
         __syncthreads();
         for (int j = warp; j < JB; j += 8) {
             const bool seen0 = key0 + lane >= lo && key0 + lane <= pos, seen1 = key0 + lane + 32 >= lo && key0 + lane + 32 <= pos;
-            const float s0 = seen0 ? capped(S[j * GA_KT + lane] * scale, softcap) : -INFINITY;
-            const float s1 = seen1 ? capped(S[j * GA_KT + lane + 32] * scale, softcap) : -INFINITY;
+            float s0 = seen0 ? capped(S[j * GA_KT + lane] * scale, softcap) : -INFINITY;
+            float s1 = seen1 ? capped(S[j * GA_KT + lane + 32] * scale, softcap) : -INFINITY;
+            if (bias.table) {
+                s0 += distance_bias(bias, head0 + min(j, nj - 1), pos - key0 - lane);
+                s1 += distance_bias(bias, head0 + min(j, nj - 1), pos - key0 - lane - 32);
+            }
             const float m_old = mrun[j];
             const float m_new = fmaxf(m_old, warp_max(fmaxf(s0, s1)));
             float p0 = 0.f, p1 = 0.f, c = 1.f;
@@ -489,7 +498,8 @@ grouped_combine_kernel(const float* __restrict__ part, const int* __restrict__ t
 template <typename T, int JB>
 int launch_grouped(const void* q, int q_f32, const void* cache, const int* block_table, int max_blocks,
                    const int* token_seq, const int* positions, float* part, int T_, int H, int G, int d, int dv, int P,
-                   int window, int mask_mode, float scale, float softcap, int latent, int splits, cudaStream_t stream) {
+                   int window, int mask_mode, float scale, float softcap, int latent, int splits, const DistanceBias& bias,
+                   cudaStream_t stream) {
     constexpr int PER = Words<T>::per;
     const int ksw = (d / PER) | 1, vsw = (dv / PER) | 1;
     const size_t smem = sizeof(float) * ((size_t)JB * d + 2 * JB * GA_KT + 3 * JB + GA_KT) +
@@ -500,7 +510,7 @@ int launch_grouped(const void* q, int q_f32, const void* cache, const int* block
     const int J = H / G;
     dim3 grid(T_, G * ((J + JB - 1) / JB), splits);
     return launch(kernel, grid, 256, smem, stream, q, q_f32, (const T*)cache, block_table, max_blocks, token_seq,
-                  positions, part, H, G, d, dv, P, window, mask_mode, scale, softcap, latent, splits);
+                  positions, part, H, G, d, dv, P, window, mask_mode, scale, softcap, latent, splits, bias);
 }
 
 }  // namespace air
@@ -510,8 +520,11 @@ AIR_API int air_grouped_attention(const void* q, int q_f32, const void* cache, i
                                   int max_blocks, const int* token_seq, const int* positions, float* part, void* out,
                                   int T, int H, int G, int d, int dv, int P, int window, float scale, int mask_mode,
                                   const float* sink, int latent, int splits, float softcap, const float* gate, int ldg,
-                                  const double* turn_freq, int turn_rot, int turn_pairing, cudaStream_t stream) {
+                                  const double* turn_freq, int turn_rot, int turn_pairing, const float* bias_table,
+                                  int bias_n, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (bias_table && bias_n < 1) return AIR_ERR_BAD_ARGUMENT;
+    const air::DistanceBias bias{bias_table, bias_n};
     const int bytes = dtype == AIR_F32 ? 4 : 2;
     if (d <= 0 || dv <= 0 || dv > (dtype == AIR_F32 ? 768 : 1024) || (d * bytes) % 16 || (dv * bytes) % 16 || H <= 0 || G <= 0 ||
         H % G || splits <= 0 || splits > 65535 || mask_mode < 0 || mask_mode > 1 || (latent && (dv > d || G != 1)))
@@ -535,7 +548,7 @@ AIR_API int air_grouped_attention(const void* q, int q_f32, const void* cache, i
             dim3 grid(T, G * ((J + 15) / 16), splits);
             rc = air::launch(kernel, grid, 256, smem, stream, q, q_f32, (const __nv_bfloat16*)cache, block_table,
                              max_blocks, token_seq, positions, part, H, G, d, dv, P, window, mask_mode, scale, softcap, latent,
-                             splits, stages);
+                             splits, stages, bias);
             if (rc) return rc;
             return air::launch(air::grouped_combine_kernel<__nv_bfloat16>, dim3(T, H), 128, 0, stream, part, token_seq,
                                sink, (__nv_bfloat16*)out, H, dv, splits, gate, ldg, turn);
@@ -544,10 +557,10 @@ AIR_API int air_grouped_attention(const void* q, int q_f32, const void* cache, i
     AIR_DISPATCH(dtype, TT, {
         if (J > 4)
             rc = air::launch_grouped<TT, 16>(q, q_f32, cache, block_table, max_blocks, token_seq, positions, part, T, H,
-                                             G, d, dv, P, window, mask_mode, scale, softcap, latent, splits, stream);
+                                             G, d, dv, P, window, mask_mode, scale, softcap, latent, splits, bias, stream);
         else
             rc = air::launch_grouped<TT, 4>(q, q_f32, cache, block_table, max_blocks, token_seq, positions, part, T, H,
-                                            G, d, dv, P, window, mask_mode, scale, softcap, latent, splits, stream);
+                                            G, d, dv, P, window, mask_mode, scale, softcap, latent, splits, bias, stream);
         if (rc) return rc;
         return air::launch(air::grouped_combine_kernel<TT>, dim3(T, H), 128, 0, stream, part, token_seq, sink, (TT*)out,
                            H, dv, splits, gate, ldg, turn);

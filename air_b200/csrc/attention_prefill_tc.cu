@@ -32,6 +32,10 @@
 // its reference maximum (in powers of two) and its sum of probabilities part_ml[slot][256] (0 where the row saw no
 // key); prefill_combine_kernel then merges an item's slots, in their order, into the output rows.
 //
+// With BIAS a score gets the head's number for its key's distance (DistanceBias).  Where all of a warp's rows stand farther
+// from a tile's keys than the table reaches, that is one number more in the exponent's multiply-add; in the tiles near the
+// diagonal a lane looks up its row's numbers one key after the other, 32 neighbours per access.
+//
 // tiles, q, out, cache, block_table, window as in attention_prefill.cu; the list pads every request
 // to whole pairs of groups.  Head size 64 or 128; pages of a divisor or a multiple of 64 tokens.
 // Every wait on an mbarrier is bounded (tma.cuh); on giving up the block flags *status = 7.  A list
@@ -111,14 +115,14 @@ struct RowTile {
     int n;           // key tiles it takes
 };
 
-template <int D>
+template <int D, bool BIAS>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_cache,
                             const int* __restrict__ block_table, int max_blocks, const int* __restrict__ tiles,
                             int n_pairs, const int* __restrict__ segments, int n_slots, float* __restrict__ part_o,
                             float2* __restrict__ part_ml, __nv_bfloat16* __restrict__ out, int H, int K, int P,
                             int window, float scale_log2, float cap, float cap_pre, int* __restrict__ status,
-                            const float* __restrict__ sink) {
+                            const float* __restrict__ sink, const DistanceBias bias) {
     // sink (or null): float32 [H]; one more term exp(sink[h]) in the softmax's denominator, which has no key and no
     // value: it joins a row's sum where the row is normalised (here, or where its segments are merged)
     // cap > 0: a score s becomes cap * tanh(s * cap_pre) (cap_pre = scale / cap) and scale_log2 is log2(e) alone
@@ -348,6 +352,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t my_s = tmem_base + lane_addr + 2 * x * AT_BN;
         const uint32_t my_o = tmem_base + lane_addr + O_COL + x * D;
         float m = -INFINITY, l = 0.f;
+        const float* bias_row = BIAS ? bias.table + (size_t)h * bias.n : nullptr;
+        const float bias_far = BIAS ? bias_row[bias.n - 1] * 1.4426950408889634f : 0.f;
         bool ok = true;
         for (int it = 0; it < me.n && ok; ++it) {
             const int b = it & 1;
@@ -364,6 +370,19 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // Scores stay as the product left them; the scale goes into the exponent's multiply-add.
             // Only tiles on the diagonal or at a window's edge need the mask (the same for the warp).
             const int warp_first = me.pos0 + quarter * 32;
+            float sc = scale_log2, shift = 0.f;      // a score's exponent is sv * sc + shift
+            if constexpr (BIAS) {
+                if (warp_first - (kbase + AT_BN - 1) >= bias.n - 1) {
+                    shift = bias_far;
+                } else {
+#pragma unroll
+                    for (int c = 0; c < AT_BN; ++c) {
+                        const float b = __ldg(bias_row + max(0, min(pos - kbase - c, bias.n - 1)));
+                        sv[c] = __float_as_uint(fmaf(b, 1.4426950408889634f, __uint_as_float(sv[c]) * scale_log2));
+                    }
+                    sc = 1.f;
+                }
+            }
             const bool full_tile = kbase + AT_BN - 1 <= warp_first && (window <= 0 || kbase > warp_first + 31 - window);
             // (four running maxima and, below, two pairs of running sums: independent chains)
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -382,7 +401,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 }
             }
             // the scale is positive: the maximum of the scaled scores
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * sc + shift;
             // The reference maximum m of the row moves only when the tile's maximum exceeds it by more
             // than 2^8 (or the row had seen no key): probabilities up to 256 are harmless in bfloat16 and
             // in the 32-bit sums, and a row of O that is not rescaled does not have to wait for the
@@ -394,7 +413,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             m = m_new;
             float2 sum2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
             uint32_t pk[AT_BN / 2];
-            const float2 scale2 = make_float2(scale_log2, scale_log2), nbase2 = make_float2(-base, -base);
+            const float2 scale2 = make_float2(sc, sc), nbase2 = make_float2(shift - base, shift - base);
             if (full_tile) {
 #pragma unroll
                 for (int c = 0; c < AT_BN; c += 2) {
@@ -608,12 +627,12 @@ template <int D>
 int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mc, const int* block_table, int max_blocks,
                       const int* tiles, int n_tiles, const int* segments, int n_segments, const int* items, int n_items,
                       int n_slots, float* part_o, float* part_ml, void* out, int H, int K, int P, int window, float scale,
-                      float softcap, int* status, cudaStream_t stream, const float* sink = nullptr) {
+                      float softcap, int* status, cudaStream_t stream, const float* sink, const DistanceBias& bias) {
     // (more than half of an SM's shared memory, so that two blocks never share its tensor memory)
     size_t smem = 1024 + (size_t)AT_ROW_TILES * (D / 64) * AT_BM * 128 +
                   (size_t)AT_STAGES * 2 * (D / 64) * AT_BN * 128 + 256;
     if (smem < 120 * 1024) smem = 120 * 1024;
-    auto kernel = prefill_attention_tc_kernel<D>;
+    auto kernel = bias.table ? prefill_attention_tc_kernel<D, true> : prefill_attention_tc_kernel<D, false>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     const int n_pairs = n_tiles / (AT_GROUP * AT_ROW_TILES);
@@ -621,7 +640,7 @@ int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mc, const int* b
     int rc = launch(kernel, grid, AT_THREADS, smem, stream, mq, mc, block_table, max_blocks, tiles, n_pairs, segments,
                     n_slots, part_o, (float2*)part_ml, (__nv_bfloat16*)out, H, K, P, window,
                     (softcap > 0.f ? 1.f : scale) * 1.4426950408889634f, softcap > 0.f ? softcap : 0.f,
-                    softcap > 0.f ? scale / softcap : 0.f, status, sink);
+                    softcap > 0.f ? scale / softcap : 0.f, status, sink, bias);
     if (rc || !segments || n_items <= 0) return rc;
     return launch(prefill_combine_kernel<D>, dim3(n_items, AT_ROW_TILES * AT_BM / 8), 256, 0, stream, tiles, n_pairs,
                   items, n_slots, (const float*)part_o, (const float2*)part_ml, (__nv_bfloat16*)out, H, status, sink);
@@ -637,9 +656,10 @@ static int prefill_attention_tc_any(const void* q, int T, const void* cache, lon
                                     int max_blocks, const int* tiles, int n_tiles, const int* segments, int n_segments,
                                     const int* items, int n_items, int n_slots, float* part_o, float* part_ml,
                                     void* out, int H, int K, int D, int P, int window, float scale, float softcap,
-                                    int* status, const float* sink, cudaStream_t stream) {
+                                    int* status, const float* sink, const air::DistanceBias& bias, cudaStream_t stream) {
     using namespace air;
     if (n_tiles <= 0) return 0;
+    if (bias.table && bias.n < 1) return AIR_ERR_BAD_ARGUMENT;
     if (segments && (n_segments <= 0 || n_items < 0 || n_slots < 0 || (n_items > 0 && !items) ||
                      (n_slots > 0 && (!part_o || !part_ml || ((uintptr_t)part_o & 15) || ((uintptr_t)part_ml & 7)))))
         return AIR_ERR_BAD_ARGUMENT;
@@ -654,9 +674,9 @@ static int prefill_attention_tc_any(const void* q, int T, const void* cache, lon
     if (rc) return rc;
     if (D == 64)
         return launch_prefill_tc<64>(mq, mc, block_table, max_blocks, tiles, n_tiles, segments, n_segments, items, n_items,
-                                     n_slots, part_o, part_ml, out, H, K, P, window, scale, softcap, status, stream, sink);
+                                     n_slots, part_o, part_ml, out, H, K, P, window, scale, softcap, status, stream, sink, bias);
     return launch_prefill_tc<128>(mq, mc, block_table, max_blocks, tiles, n_tiles, segments, n_segments, items, n_items,
-                                  n_slots, part_o, part_ml, out, H, K, P, window, scale, softcap, status, stream, sink);
+                                  n_slots, part_o, part_ml, out, H, K, P, window, scale, softcap, status, stream, sink, bias);
 }
 
 AIR_API int air_prefill_attention_tc(const void* q, int T, const void* cache, long long pages, const int* block_table,
@@ -666,19 +686,20 @@ AIR_API int air_prefill_attention_tc(const void* q, int T, const void* cache, lo
                                      int* status, cudaStream_t stream) {
     return prefill_attention_tc_any(q, T, cache, pages, block_table, max_blocks, tiles, n_tiles, segments, n_segments,
                                     items, n_items, n_slots, part_o, part_ml, out, H, K, D, P, window, scale, softcap,
-                                    status, nullptr, stream);
+                                    status, nullptr, air::DistanceBias{nullptr, 0}, stream);
 }
 
-// The same with one more term exp(sink[h]) in every head's softmax denominator (sink float32 [H]).
+// The same with one more term exp(sink[h]) in every head's softmax denominator (sink float32 [H] or null), and a number per
+// head and distance on the scores (bias float32 [H, bias_n] or null, see DistanceBias).
 AIR_API int air_prefill_attention_tc_sink(const void* q, int T, const void* cache, long long pages,
                                           const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                                           const int* segments, int n_segments, const int* items, int n_items,
                                           int n_slots, float* part_o, float* part_ml, void* out, int H, int K, int D,
                                           int P, int window, float scale, float softcap, int* status,
-                                          const float* sink, cudaStream_t stream) {
+                                          const float* sink, const float* bias, int bias_n, cudaStream_t stream) {
     return prefill_attention_tc_any(q, T, cache, pages, block_table, max_blocks, tiles, n_tiles, segments, n_segments,
                                     items, n_items, n_slots, part_o, part_ml, out, H, K, D, P, window, scale, softcap,
-                                    status, sink, stream);
+                                    status, sink, air::DistanceBias{bias, bias_n}, stream);
 }
 
 AIR_API int air_trace_set_attention_prefill_tc(unsigned long long* buffer) { return air::set_trace_here(buffer); }

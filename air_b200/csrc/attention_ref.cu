@@ -18,7 +18,8 @@
 // a bare logit that `scale` does not touch and that brings nothing to the output.  With `latent` a page is [P, d] (one row per token, no heads): every
 // query head reads the same row as its key, and the row's first dv elements as its value.  q is float32 if q_f32,
 // else of the cache's type.
-// score = scale * q.k, and with softcap > 0 then softcap * tanh(score / softcap).  With `gate` [T, H] (float32) a
+// score = scale * q.k, and with softcap > 0 then softcap * tanh(score / softcap); then, where `bias` is given, plus the
+// head's number for the distance (DistanceBias).  With `gate` [T, H] (float32) a
 // head's output is multiplied by its token's gate.
 #include "common.cuh"
 
@@ -33,7 +34,7 @@ paged_attention_ref_kernel(const void* __restrict__ q_any, int q_f32, const T* _
                            const int* __restrict__ token_seq, const int* __restrict__ positions,
                            T* __restrict__ out, const float* __restrict__ gate, int H, int K, int d, int dv, int P,
                            int window, float scale, float softcap, int mask_mode, const float* __restrict__ sink,
-                           int latent) {
+                           int latent, const DistanceBias bias) {
     __shared__ float sq[ATT_MAX_D];
     __shared__ float sm[ATT_WARPS], sl[ATT_WARPS];
     __shared__ float sacc[ATT_WARPS][ATT_MAX_D];
@@ -75,6 +76,7 @@ paged_attention_ref_kernel(const void* __restrict__ q_any, int q_f32, const T* _
             for (int i = 0; i < d; ++i) dot = fmaf(sq[i], to_float(kp[i]), dot);
             s = dot * scale;
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+            s += distance_bias(bias, h, pos - key);
         }
         const float bm = warp_max(s);
         if (bm == -INFINITY) continue;  // the whole block is outside the window
@@ -126,8 +128,10 @@ AIR_API int air_paged_attention_ref(const void* q, int q_f32, const void* cache,
                                     int max_blocks, const int* token_seq, const int* positions, void* out,
                                     const float* gate, int T, int H, int K, int d, int dv, int P, int window,
                                     float scale, float softcap, int mask_mode, const float* sink, int latent,
-                                    cudaStream_t stream) {
+                                    const float* bias, int bias_n, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (bias && bias_n < 1) return AIR_ERR_BAD_ARGUMENT;
+    const air::DistanceBias db{bias, bias_n};
     if (d <= 0 || d > 640 || dv <= 0 || dv > 640 || H <= 0 || K <= 0 || H > 65535 || mask_mode < 0 || mask_mode > 1 ||
         (latent && (dv > d || K != 1)))
         return AIR_ERR_BAD_ARGUMENT;
@@ -136,10 +140,10 @@ AIR_API int air_paged_attention_ref(const void* q, int q_f32, const void* cache,
         if (d <= 256 && dv <= 256)
             return air::launch(air::paged_attention_ref_kernel<TT, 256>, grid, air::ATT_WARPS * 32, 0, stream, q, q_f32,
                                (const TT*)cache, block_table, max_blocks, token_seq, positions, (TT*)out, gate, H, K,
-                               d, dv, P, window, scale, softcap, mask_mode, sink, latent);
+                               d, dv, P, window, scale, softcap, mask_mode, sink, latent, db);
         return air::launch(air::paged_attention_ref_kernel<TT, 640>, grid, air::ATT_WARPS * 32, 0, stream, q, q_f32,
                            (const TT*)cache, block_table, max_blocks, token_seq, positions, (TT*)out, gate, H, K, d,
-                           dv, P, window, scale, softcap, mask_mode, sink, latent);
+                           dv, P, window, scale, softcap, mask_mode, sink, latent, db);
     });
     return 0;
 }

@@ -139,6 +139,16 @@ __device__ __forceinline__ void cos_sin_of(double position, double freq, float& 
     sincospif(2.f * (float)turns, &s, &c);
 }
 
+// A learned number that a score of head h gets for how many positions back its key stands (behind scale and cap): entry
+// min(distance, n - 1) of the head's row of table [heads, n].  table null: none.
+struct DistanceBias {
+    const float* table;
+    int n;
+};
+__device__ __forceinline__ float distance_bias(const DistanceBias& b, int h, int distance) {
+    return b.table ? b.table[(size_t)h * b.n + max(0, min(distance, b.n - 1))] : 0.f;
+}
+
 // A rotation of a finished row of attention outputs, backwards by the query's position (values that were rotated by their
 // own positions): the first `rot` elements, pair j = (j, j + rot/2) (pairing 0) or (2j, 2j + 1) (pairing 1), by
 // -position * freq[j].  freq null: none.

@@ -2,7 +2,7 @@
 //
 //   glu_kernel          out[t, i] = g' * sigmoid(alpha * g') * (u' + shift), with g' = min(gate, limit) and
 //                       u' = clamp(up, -limit, limit) where limit > 0 (else gate and up as they are).  alpha = 1,
-//                       shift = 0, limit = 0 is SiLU(gate) * up.  The input [T, 2I] holds blocks of `block` gate
+//                       shift = 0, limit = 0 is SiLU(gate) * up (gated_activation, common.cuh).  The input [T, 2I] holds blocks of `block` gate
 //                       columns and `block` up columns in turn.
 //   head_gate_kernel    x[t, h, :] *= gate[t, h], for attention kernels that do not multiply by a gate as they write
 //   scaled_norm_kernel  x = h + sa * a + sb * b (float32; a scale per column, each term optional; a term may come as
@@ -200,13 +200,26 @@ __global__ void glu_kernel(const TI* __restrict__ in, TO* __restrict__ out, int 
         const size_t t = idx / I;
         const int i = (int)(idx % I);
         const TI* row = in + t * 2 * (size_t)I + (size_t)(i / block) * 2 * block;
-        float g = to_float(row[i % block]), u = to_float(row[block + i % block]);
-        if (limit > 0.f) {
-            g = fminf(g, limit);
-            u = fminf(fmaxf(u, -limit), limit);
-        }
-        out[idx] = from_float<TO>(g / (1.f + expf(-alpha * g)) * (u + shift));
+        out[idx] = from_float<TO>(gated_activation(to_float(row[i % block]), to_float(row[block + i % block]), alpha, limit, shift));
     }
+}
+
+// The same four columns at a time (block a multiple of 4, the tensors on boundaries of four elements).
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256)
+glu_vec4_kernel(const TI* __restrict__ in, TO* __restrict__ out, int I, int block, unsigned total4, float alpha, float limit,
+                float shift) {
+    pdl_enter(TR_GLU);
+    const unsigned idx = blockIdx.x * 256u + threadIdx.x;
+    if (idx >= total4) return;
+    const unsigned per_row = (unsigned)I / 4, t = idx / per_row, i = (idx % per_row) * 4;
+    const TI* row = in + (size_t)t * 2 * I + (size_t)(i / block) * 2 * block + i % block;
+    float g[4], u[4];
+    load4(row, g);
+    load4(row + block, u);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) g[j] = gated_activation(g[j], u[j], alpha, limit, shift);
+    store4(out + (size_t)t * I + i, g);
 }
 
 // x [T, H, d] *= gate[T, H] in place (one gate per token and head); rows whose token_seq is negative are padding.
@@ -313,7 +326,11 @@ AIR_API int air_glu(const void* in, int in_dtype, void* out, int out_dtype, int 
     if (total == 0) return 0;
     if (block <= 0 || I % block) return AIR_ERR_BAD_ARGUMENT;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+    const bool vec = I % 4 == 0 && block % 4 == 0 && total / 4 < 0xffffff00ull && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
     AIR_DISPATCH(in_dtype, TI, AIR_DISPATCH(out_dtype, TO, {
+        if (vec)
+            return air::launch(air::glu_vec4_kernel<TI, TO>, (unsigned)((total / 4 + 255) / 256), 256, 0, stream,
+                               (const TI*)in, (TO*)out, I, block, (unsigned)(total / 4), alpha, limit, shift);
         return air::launch(air::glu_kernel<TI, TO>, blocks, 256, 0, stream, (const TI*)in, (TO*)out, I, block, total,
                            alpha, limit, shift);
     }));

@@ -16,7 +16,8 @@
 //   o_scale[row * o_scale_ld + g] (a gate per token and head behind a product per head).
 //   Epilogue 0: C as float32 or in A's type.  Epilogue 1: W_g is [2 F, K], blocks of gate_block rows of the gate and
 //   as many of the linear branch in turn (gate_block = F: all gate rows, then all linear rows), the arrangement that
-//   the dense gated feed-forward uses; C [rows, F] = silu(gate) * linear in A's type.  Epilogue 2: C = max(x, 0)^2 of the
+//   the dense gated feed-forward uses; C [rows, F] = gated_activation(gate, linear) (common.cuh; SiLU(gate) * linear with
+//   alpha 1, no limit and no shift) in A's type.  Epilogue 2: C = max(x, 0)^2 of the
 //   plain product x, in A's type (the hidden layer of an expert without a gate).
 //
 // Arithmetic.  float32 operands (and bfloat16 ones whose strides are not multiples of 8 elements): 32-bit multiply-adds
@@ -39,6 +40,7 @@ struct GroupedArgs {
     int N, K;
     int gate_block;      // epilogue 1: rows of W_g come in blocks of gate_block gate rows and as many linear rows in turn
     const float* o_scale; int o_scale_ld;
+    float alpha, limit, shift;      // epilogue 1: the gated activation
 };
 
 constexpr int GG_BM = 64, GG_BN = 64, GG_BK = 16;
@@ -156,7 +158,7 @@ grouped_gemm_kernel(const GroupedArgs p) {
             if (n >= N) continue;
             if (EPI == 1) {
                 const float gate = acc[0][i][j], lin = acc[EPI == 1 ? 1 : 0][i][j];
-                ((T*)p.out)[o + n] = from_float<T>(gate / (1.f + expf(-gate)) * lin);
+                ((T*)p.out)[o + n] = from_float<T>(gated_activation(gate, lin, p.alpha, p.limit, p.shift));
             } else if (EPI == 2) {
                 const float r = fmaxf(acc[0][i][j], 0.f);
                 ((T*)p.out)[o + n] = from_float<T>(r * r);
@@ -332,7 +334,7 @@ grouped_gemm_tc_kernel(const GroupedArgs p) {
                 const float v = acc[0][j][2 * half + i] * (EPI == 0 ? om : 1.f);
                 if (EPI == 1) {
                     const float lin = acc[NW - 1][j][2 * half + i];
-                    ((__nv_bfloat16*)p.out)[o + n] = __float2bfloat16_rn(v / (1.f + expf(-v)) * lin);
+                    ((__nv_bfloat16*)p.out)[o + n] = __float2bfloat16_rn(gated_activation(v, lin, p.alpha, p.limit, p.shift));
                 } else if (EPI == 2) {
                     const float r = fmaxf(acc[0][j][2 * half + i], 0.f);
                     ((__nv_bfloat16*)p.out)[o + n] = __float2bfloat16_rn(r * r);
@@ -352,8 +354,8 @@ AIR_API int air_grouped_gemm(const void* A, long long lda, long long a_group_str
                              long long ldo, long long o_group_stride, const int* o_index, int o_div,
                              long long o_part_stride, int o_local, int out_f32, const int* start, int rows_per_group,
                              const int* tiles, const int* num_tiles, int max_tiles, int groups, int N, int K,
-                             int dtype, int epi, int gate_block, const float* o_scale, int o_scale_ld,
-                             cudaStream_t stream) {
+                             int dtype, int epi, int gate_block, const float* o_scale, int o_scale_ld, float alpha,
+                             float limit, float shift, cudaStream_t stream) {
     if (N <= 0 || K <= 0 || groups <= 0) return 0;
     if ((start != nullptr) != (tiles != nullptr) || (start && !num_tiles) || epi < 0 || epi > 2 ||
         (a_index && a_div <= 0) || (o_index && o_div <= 0) || (a_scale && !a_index) || (o_scale && epi))
@@ -362,7 +364,7 @@ AIR_API int air_grouped_gemm(const void* A, long long lda, long long a_group_str
     if (epi == 1 && N % gate_block) return AIR_ERR_BAD_ARGUMENT;
     air::GroupedArgs p{A, lda, a_group_stride, a_index, a_div, a_local, a_scale, W, w_group_stride, out, ldo,
                        o_group_stride, o_index, o_div, o_part_stride, o_local, out_f32, start, rows_per_group, tiles,
-                       num_tiles, N, K, gate_block, o_scale, o_scale_ld};
+                       num_tiles, N, K, gate_block, o_scale, o_scale_ld, alpha, limit, shift};
     const int row_tiles = start ? max_tiles : (rows_per_group + air::GG_BM - 1) / air::GG_BM;
     if (row_tiles <= 0) return 0;
     if (row_tiles > 65535 || groups > 65535) return AIR_ERR_BAD_ARGUMENT;

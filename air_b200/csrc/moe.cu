@@ -6,8 +6,8 @@
 //   score 0 is sigmoid(z), score 1 the softmax over the n logits; the weights are the chosen scores as they are, or
 //   (renormalize) divided by their sum (+ norm_eps), and then times route_scale.  Equal scores: the lower index wins.
 //   With groups > 1 experts g * (n / groups) .. (g + 1) * (n / groups) - 1 make group g; a group's mark is its best score
-//   plus its second best (its only score where a group is one expert), and only the experts of the `keep` groups with the
-//   largest marks (of equal marks the lower group) can be chosen.  One warp per token.
+//   plus its second best (its only score where a group is one expert), or with mark 1 its best score alone, and only the
+//   experts of the `keep` groups with the largest marks (of equal marks the lower group) can be chosen.  One warp per token.
 //   With a bias (float32 [n]) the experts are chosen by score + bias, while the weights stay the scores themselves.
 //   Writes expert [T, top] int32, weight [T, top] float32 and gate [T] = sigmoid(z[n]).
 //
@@ -29,7 +29,7 @@ constexpr int MOE_MAX_PER_LANE = 16;      // up to 512 experts
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ z, int ld, int T, int n, int top, int score, int renormalize,
                  int has_gate, int* __restrict__ expert, float* __restrict__ weight, float* __restrict__ gate,
-                 int groups, int keep, float route_scale, float norm_eps, const float* __restrict__ bias) {
+                 int groups, int keep, int mark, float route_scale, float norm_eps, const float* __restrict__ bias) {
     __shared__ float held[4][32 * MOE_MAX_PER_LANE], marks[4][32 * MOE_MAX_PER_LANE];
     pdl_enter(TR_MOE_ROUTE);
     const int lane = threadIdx.x & 31;
@@ -87,7 +87,7 @@ moe_route_kernel(const float* __restrict__ z, int ld, int T, int n, int top, int
                 if (v > a) { b = a; a = v; }
                 else if (v > b) b = v;
             }
-            mk[g] = size > 1 ? a + b : a;
+            mk[g] = size > 1 && mark == 0 ? a + b : a;
         }
         __syncwarp();
         // a group takes part if fewer than `keep` groups come before it (a larger mark, or an equal one and a lower
@@ -250,15 +250,15 @@ AIR_API int air_planes_by_index(const void* rows, int dtype, const int* index, i
 }
 
 AIR_API int air_moe_route(const float* z, int ld, int T, int n, int top, int score, int renormalize, int has_gate,
-                          int* expert, float* weight, float* gate, int groups, int keep, float route_scale,
+                          int* expert, float* weight, float* gate, int groups, int keep, int mark, float route_scale,
                           float norm_eps, const float* bias, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (n <= 0 || n > 32 * air::MOE_MAX_PER_LANE || top <= 0 || top > n || top > 32 || ld < n + (has_gate ? 1 : 0) ||
-        score < 0 || score > 1)
+        score < 0 || score > 1 || mark < 0 || mark > 1)
         return AIR_ERR_BAD_ARGUMENT;
     if (groups > 1 && (n % groups || keep <= 0 || keep > groups || top > keep * (n / groups))) return AIR_ERR_BAD_ARGUMENT;
     return air::launch(air::moe_route_kernel, (T + 3) / 4, 128, 0, stream, z, ld, T, n, top, score, renormalize,
-                       has_gate, expert, weight, gate, groups, keep, route_scale, norm_eps, bias);
+                       has_gate, expert, weight, gate, groups, keep, mark, route_scale, norm_eps, bias);
 }
 
 AIR_API int air_moe_identity(const void* x, int dtype, const int* expert, const float* weight, int n_real, int top,

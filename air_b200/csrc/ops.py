@@ -34,7 +34,7 @@ _SIGNATURES = {
     "air_gemm_f32": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "air_paged_attention_ref": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                 c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p,
-                                c_int, c_void_p],
+                                c_int, c_void_p, c_int, c_void_p],
     "air_post_norm": [c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int,
                       c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "air_qk_normed_prepare": [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_float, c_void_p,
@@ -43,7 +43,8 @@ _SIGNATURES = {
     "air_turn_heads": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "air_stream_norm": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_void_p, c_void_p,
                         c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float,
-                        c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                        c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p,
+                        c_void_p, c_void_p],
     "air_residual_conv": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                           c_void_p],
     "air_mlstm_step": [c_void_p] + [c_int] * 6 + [c_void_p] + [c_int] * 3 + [c_void_p] * 7 + [c_int] + [c_void_p] * 2 +
@@ -53,18 +54,20 @@ _SIGNATURES = {
     "air_mlstm_portions_tc": [c_void_p] + [c_int] * 5 + [c_void_p] + [c_int] * 3 + [c_void_p] * 7 + [c_int] +
                              [c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 5 + [c_int] * 4 + [c_float] * 3 +
                              [c_void_p],
-    "air_latent_prepare": [c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-                           c_void_p, c_void_p],
+    "air_latent_prepare": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p,
+                           c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                           c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    "air_band_rmsnorm": [c_void_p, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "air_split_bands": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p],
     "air_grouped_attention": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_int,
-                              c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
+                              c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p],
     "air_gather_keys": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                         c_void_p, c_void_p],
     "air_masked_softmax": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                           c_void_p, c_float, c_void_p],
+                           c_void_p, c_float, c_void_p, c_int, c_void_p],
     "air_moe_route": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                      c_int, c_float, c_float, c_void_p, c_void_p],
+                      c_int, c_int, c_float, c_float, c_void_p, c_void_p],
     "air_moe_identity": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "air_normed_add_norm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_float, c_void_p, c_void_p, c_int,
                             c_void_p, c_int, c_int, c_float, c_void_p],
@@ -73,7 +76,8 @@ _SIGNATURES = {
     "air_moe_sort": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     "air_grouped_gemm": [c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_int, c_void_p, c_void_p, c_longlong,
                          c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_int,
-                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
+                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float,
+                         c_float, c_float, c_void_p],
     "air_rows_by_index": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "air_planes_by_index": [c_void_p, c_int, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "air_qkv_prepare": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
@@ -86,7 +90,7 @@ _SIGNATURES = {
                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_float, c_void_p,
                         c_void_p, c_int, c_float, c_void_p],
     "air_gated_rmsnorm": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float,
-                          c_void_p],
+                          c_int, c_void_p],
     "air_polynorm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float,
                      c_float, c_void_p],
     "air_glu": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p],
@@ -106,7 +110,8 @@ _SIGNATURES = {
                                  c_void_p],
     "air_decode_attention_tma_sink": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                       c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                      c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
+                                      c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
+                                      c_int, c_void_p],
     "air_head_gate": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "air_decode_attention_tma_fresh": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int,
                                        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -116,7 +121,8 @@ _SIGNATURES = {
                                  c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p],
     "air_prefill_attention_tc_sink": [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p,
                                       c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                      c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p],
+                                      c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int,
+                                      c_void_p],
     "air_sample": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                    c_void_p, c_void_p],
 }
@@ -415,7 +421,7 @@ def gemm_f32(a, w, bias, out):
 
 
 def paged_attention_ref(q, cache, block_table, token_seq, positions, out, window, scale, softcap=0.0, gate=None,
-                        kv_heads=None, page_tokens=None, chunk=None, sink=None, latent=False):
+                        kv_heads=None, page_tokens=None, chunk=None, sink=None, latent=False, bias=None):
     """Causal attention over the pages with 32-bit arithmetic, for any batch.  q [T, H, d], out [T, H, dv].
     cache [page, 2, K, P, d] where dv == d; where keys and values differ in size a page is flat: the keys
     [K, P, d], then the values [K, P, dv], and kv_heads and page_tokens say what K and P are.  score = scale * q.k,
@@ -423,7 +429,8 @@ def paged_attention_ref(q, cache, block_table, token_seq, positions, out, window
     Which keys a query at position p sees: all up to its own; with `window` the last `window` of them; with `chunk`
     those from p - p % chunk on.  sink (float32 [H]): one more term exp(sink[h]) in the softmax's denominator.
     latent: cache [page, P, d] holds one row per token that every head reads as its key and whose first dv elements
-    it reads as its value; q may then be float32 whatever the cache's type."""
+    it reads as its value; q may then be float32 whatever the cache's type.  bias (float32 [H, n]): a score gets
+    bias[h, min(p - key's position, n - 1)]."""
     T, H, d = q.shape
     dv = out.shape[2]
     _req(q, "q", _FLOATS)
@@ -460,7 +467,7 @@ def paged_attention_ref(q, cache, block_table, token_seq, positions, out, window
         q.data_ptr(), 1 if q.dtype == torch.float32 else 0, cache.data_ptr(), _DT[cache.dtype], block_table.data_ptr(),
         block_table.shape[1], token_seq.data_ptr(), positions.data_ptr(), out.data_ptr(), _ptr(gate), T, H, K, d, dv, P,
         int(chunk or window or 0), float(scale), float(softcap or 0.0), 1 if chunk else 0, _ptr(sink),
-        1 if latent else 0, _stream()), "paged_attention_ref")
+        1 if latent else 0, *_distance_bias(bias, H), _stream()), "paged_attention_ref")
     return out
 
 
@@ -475,6 +482,14 @@ def _turn(turn, width):
     return freq.data_ptr(), 2 * freq.numel(), 1 if pairing == "neighbours" else 0
 
 
+def _distance_bias(bias, heads):
+    """(pointer, entries per head) of a bias per head and distance (float32 [H, n]) or None."""
+    if bias is None:
+        return None, 0
+    _req(bias, "bias", (torch.float32,), (heads, None))
+    return bias.data_ptr(), bias.shape[1]
+
+
 def grouped_attention_ok(cache_dtype, d, dv) -> bool:
     """Whether grouped_attention takes keys of d and values of dv elements: rows of whole 16-byte pieces."""
     size = 4 if cache_dtype == torch.float32 else 2
@@ -482,8 +497,8 @@ def grouped_attention_ok(cache_dtype, d, dv) -> bool:
 
 
 def grouped_attention(q, cache, block_table, token_seq, positions, out, window, scale, kv_heads=1, page_tokens=None,
-                      chunk=None, sink=None, latent=False, splits=None, softcap=0.0, gate=None, turn=None):
-    """paged_attention_ref's arithmetic and arguments (32-bit, any batch, window or chunk, sink, latent rows), by the
+                      chunk=None, sink=None, latent=False, splits=None, softcap=0.0, gate=None, turn=None, bias=None):
+    """paged_attention_ref's arithmetic and arguments (32-bit, any batch, window or chunk, sink, latent rows, bias), by the
     kernel in which a block serves all query heads of a key/value head and the keys of a token are split over
     `splits` blocks (default: enough to fill the device); needs grouped_attention_ok(cache.dtype, d, dv).  gate (float32
     [T, H * dv], may be a band of columns): out is multiplied, element by element, by sigmoid(gate).  turn = (freq, pairing):
@@ -528,7 +543,7 @@ def grouped_attention(q, cache, block_table, token_seq, positions, out, window, 
         q.data_ptr(), 1 if q.dtype == torch.float32 else 0, cache.data_ptr(), _DT[cache.dtype], block_table.data_ptr(),
         block_table.shape[1], token_seq.data_ptr(), positions.data_ptr(), part.data_ptr(), out.data_ptr(), T, H, G, d,
         dv, P, int(chunk or window or 0), float(scale), 1 if chunk else 0, _ptr(sink), 1 if latent else 0, int(splits),
-        float(softcap or 0.0), gp, ldg, *_turn(turn, dv), _stream()), "grouped_attention")
+        float(softcap or 0.0), gp, ldg, *_turn(turn, dv), *_distance_bias(bias, H), _stream()), "grouped_attention")
     global launches
     launches += 1
     return out
@@ -554,11 +569,12 @@ def gather_keys(cache, table_row, lo, count, keys, values, kv_heads=1, page_toke
 
 
 def masked_softmax(scores, weights, heads_per_group, lo, count, pos0, scale, window=None, chunk=None, sink=None,
-                   softcap=0.0):
+                   softcap=0.0, bias=None):
     """scores float32 [G, n * J, Lp] -> weights bfloat16 of the same shape: the softmax of scale * scores over the keys
     that each row's query sees (column c = key lo + c, c < count; row (t, j) = the query at pos0 + t of head g * J + j),
     with exp(sink[h]) in the denominator where sink (float32 [G * J]) is given; with softcap > 0 a score is
-    softcap * tanh(scale * score / softcap)."""
+    softcap * tanh(scale * score / softcap).  bias (float32 [G * J, n]): behind that a score gets bias[h, min(distance,
+    n - 1)]."""
     G, rows, Lp = scores.shape
     J = int(heads_per_group)
     _req(scores, "scores", (torch.float32,))
@@ -569,7 +585,7 @@ def masked_softmax(scores, weights, heads_per_group, lo, count, pos0, scale, win
         raise KernelError("masked_softmax: a window or a chunk, not both")
     _check(_get("air_masked_softmax")(scores.data_ptr(), weights.data_ptr(), G, rows // J, J, int(count), Lp, int(lo),
                                       int(pos0), int(chunk or window or 0), 1 if chunk else 0, float(scale), _ptr(sink),
-                                      float(softcap or 0.0), _stream()), "masked_softmax")
+                                      float(softcap or 0.0), *_distance_bias(bias, G * J), _stream()), "masked_softmax")
 
 
 def post_norm(h, alpha, a, b, b_row_scale, weight, eps, out):
@@ -666,14 +682,17 @@ STREAMS_MAX = 16
 
 
 def stream_norm(h, streams, weight, bias, eps, out, term=None, mix=None, out_weights=None, read=None, h_out=None, rows=None,
-                center=True, conv=None):
+                center=True, conv=None, more=(), again=None):
     """Residual streams x_0 .. x_(S-1): h float32 [S, T, E], or [T, E] where all streams are still equal (or S = 1).
     x'_t = sum_s mix[s, t] x_s + out_weights[t] * term (mix None: x_t; term None: nothing is added; term [T, E] or partial
     sums [parts, T, E]); written to h_out [S, T, E] (which may be h) where given.  u = sum_t read[t] x'_t (read None: the
     plain sum); out = norm(u) * weight + bias with norm(u) = (u - mean) / sqrt(var + eps), or u / sqrt(mean(u^2) + eps)
     without center; bias may be None; weight None (and out None): only the streams are completed.  rows: out[r] is that of
     row rows[r].  conv = (weight [taps, E], state [slots, taps - 1, E] or None, token_seq [T]): every row is its request's
-    only token of the step, and a causal convolution over time is added to the row (see residual_conv)."""
+    only token of the step, and a causal convolution over time is added to the row (see residual_conv).
+    more (one stream only): up to two further terms (float32 [T, E] or [parts, T, E], factor per row float32 [T] or None),
+    added to `term`.  With out but without weight the row u is written as it is, and behind it the row of again (float32
+    [T, E]) where that is given: out [R, E] or [R, 2 E]."""
     S, E = int(streams), h.shape[-1]
     T = h.shape[-2]
     _req(h, "h", (torch.float32,), (T, E) if h.dim() == 2 else (S, T, E))
@@ -694,8 +713,21 @@ def stream_norm(h, streams, weight, bias, eps, out, term=None, mix=None, out_wei
     R = T if rows is None else rows.shape[0]
     if rows is not None:
         _req(rows, "rows", _I32)
-    if weight is not None:
-        _req(out, "out", _FLOATS, (R, E))
+    if out is not None:
+        _req(out, "out", _FLOATS, (R, E if again is None else 2 * E))
+    extra = []
+    if more and (S != 1 or term is None or len(more) > 2):
+        raise KernelError("stream_norm: up to three terms, the first of them `term`, on one stream")
+    for t, gate in tuple(more) + ((None, None),) * (2 - len(more)):
+        n = 1
+        if t is not None:
+            n = 1 if t.dim() == 2 else t.shape[0]
+            _req(t, "term", (torch.float32,), (T, E) if t.dim() == 2 else (n, T, E))
+        if gate is not None:
+            _req(gate, "gate", (torch.float32,), (T,))
+        extra += [_ptr(t), n, _ptr(gate)]
+    if again is not None:
+        _req(again, "again", (torch.float32,), (T, E))
     cw = cs = ct = None
     taps = 0
     if conv is not None:
@@ -707,9 +739,9 @@ def stream_norm(h, streams, weight, bias, eps, out, term=None, mix=None, out_wei
         _req(ct, "token_seq", _I32, (T,))
     _check(_get("air_stream_norm")(
         h.data_ptr(), 0 if h.dim() == 2 else T * E, _ptr(h_out), T * E, _ptr(term), parts, T * E, _ptr(mix),
-        _ptr(out_weights), _ptr(read), S, _ptr(weight), _ptr(bias), _ptr(out) if weight is not None else None,
-        _DT[out.dtype] if weight is not None else 0, _ptr(rows), R, E, 1 if center else 0, float(eps), _ptr(cw),
-        _ptr(cs) if taps > 1 else None, _ptr(ct), taps, _stream()), "stream_norm")
+        _ptr(out_weights), _ptr(read), S, _ptr(weight), _ptr(bias), _ptr(out),
+        _DT[out.dtype] if out is not None else 0, _ptr(rows), R, E, 1 if center else 0, float(eps), _ptr(cw),
+        _ptr(cs) if taps > 1 else None, _ptr(ct), taps, *extra, _ptr(again), _stream()), "stream_norm")
     return out
 
 
@@ -803,24 +835,35 @@ def mlstm_portions(x, z, columns, i_bias, f_bias, weight, S, n, m, out, portions
     return out
 
 
-def latent_prepare(proj, c_weight, eps, freq, positions, token_seq, block_table, q_plain, q_full, cache, owns,
-                   status=None, gate_out=None, gate_column=0):
-    """From the first projection of a latent-attention layer (float32 [T, H (d + rot) (+ R + rot where owns) (+ more)])
-    to q_plain [T, H, d] (the cache's type), the rotated parts in q_full[:, :, R:] (float32 [T, H, R + rot]) and, where
-    owns, the row [rms(c) * c_weight | rotated kr] in the pages (cache [pages, P, R + rot]).  freq None: nothing is
-    rotated (rot = 0).  gate_out float32 [T, H] = sigmoid of the H columns of proj from gate_column on."""
+def latent_prepare(q, c, c_weight, eps, freq, positions, token_seq, block_table, q_plain, q_full, cache, owns,
+                   status=None, gate=None, gate_out=None, pairing="half"):
+    """From the projections of a latent-attention layer, q float32 [T, H (d + rot)] and (where owns) c float32
+    [T, R + rot] (both may be bands of columns), to q_plain [T, H, d] (the cache's type), the rotated parts in
+    q_full[:, :, R:] (float32 [T, H, R + rot]) and, where owns, the row [rms(c) * c_weight | rotated kr] in the pages
+    (cache [pages, P, R + rot]).  freq None: nothing is rotated (rot = 0); pairing "half": element i turns with i + rot/2,
+    "neighbours": 2i with 2i + 1.  gate_out float32 [T, H] = sigmoid(gate), gate float32 [T, H] (may be a band)."""
     T, H, d = q_plain.shape
     P, width = cache.shape[1], cache.shape[2]
     rot = 2 * freq.numel() if freq is not None else 0
     R = width - rot
-    ld = proj.shape[1]
-    _req(proj, "proj", (torch.float32,), (T, None))
-    if ld < H * (d + rot) + (width if owns else 0):
-        raise KernelError(f"latent_prepare: proj has {ld} columns, too few")
+    qp, ldq = _columns(q, "q")
+    if tuple(q.shape) != (T, H * (d + rot)):
+        raise KernelError(f"latent_prepare: q {tuple(q.shape)}, wanted {(T, H * (d + rot))}")
+    cp, ldc = (None, 0)
+    if owns:
+        cp, ldc = _columns(c, "c")
+        if tuple(c.shape) != (T, width):
+            raise KernelError(f"latent_prepare: c {tuple(c.shape)}, wanted {(T, width)}")
+    gp, ldg = (None, 0)
     if gate_out is not None:
+        gp, ldg = _columns(gate, "gate")
         _req(gate_out, "gate_out", (torch.float32,), (T, H))
+        if tuple(gate.shape) != (T, H):
+            raise KernelError("latent_prepare: the gate does not fit")
     if freq is not None:
         _req(freq, "freq", (torch.float64,))
+    if pairing not in ("half", "neighbours"):
+        raise KernelError(f"latent_prepare: pairing {pairing!r}")
     if owns:
         _req(c_weight, "c_weight", (torch.float32,), (R,))
     _req(positions, "positions", _I32, (T,))
@@ -830,19 +873,20 @@ def latent_prepare(proj, c_weight, eps, freq, positions, token_seq, block_table,
     _req(q_full, "q_full", (torch.float32,), (T, H, width))
     _req(cache, "cache", (q_plain.dtype,))
     _check(_get("air_latent_prepare")(
-        proj.data_ptr(), ld, _ptr(c_weight), float(eps), _ptr(freq), positions.data_ptr(), token_seq.data_ptr(),
-        block_table.data_ptr(), block_table.shape[1], q_plain.data_ptr(), q_full.data_ptr(), cache.data_ptr(),
-        _DT[q_plain.dtype], 1 if owns else 0, T, H, d, rot, R, P, _ptr(gate_out), int(gate_column), _ptr(status),
-        _stream()), "latent_prepare")
+        qp, ldq, cp, ldc, gp, ldg, _ptr(c_weight), float(eps), _ptr(freq), 1 if pairing == "neighbours" else 0,
+        positions.data_ptr(), token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1], q_plain.data_ptr(),
+        q_full.data_ptr(), cache.data_ptr(), _DT[q_plain.dtype], 1 if owns else 0, T, H, d, rot, R, P, _ptr(gate_out),
+        _ptr(status), _stream()), "latent_prepare")
 
 
 def moe_route(z, experts, top, expert_out, weight_out, gate_out=None, has_gate=False, score="sigmoid",
-              renormalize=False, groups=0, keep=0, route_scale=1.0, norm_eps=0.0, choice_bias=None):
+              renormalize=False, groups=0, keep=0, route_scale=1.0, norm_eps=0.0, choice_bias=None, mark="two"):
     """z float32 [T, >= experts (+ 1)]: router logits.  expert_out int32 [T, top], weight_out float32 [T, top]: the
     experts with the largest scores (sigmoid(z), or softmax(z)) and those scores (divided by their sum + norm_eps where
     renormalize), times route_scale; gate_out float32 [T] = sigmoid(z[:, experts]) where has_gate, else 1.  groups > 1:
     the experts are cut into `groups` runs of experts / groups consecutive indices, a run's mark is its best score plus
-    its second best, and only experts of the `keep` runs with the highest marks can be chosen.  choice_bias (float32
+    its second best (mark "two"; "best": its best score alone), and only experts of the `keep` runs with the highest marks
+    can be chosen.  choice_bias (float32
     [experts]): the experts are chosen by score + choice_bias; the weights stay the scores."""
     T = z.shape[0]
     if choice_bias is not None:
@@ -854,9 +898,12 @@ def moe_route(z, experts, top, expert_out, weight_out, gate_out=None, has_gate=F
         _req(gate_out, "gate_out", (torch.float32,), (T,))
     if score not in ("sigmoid", "softmax"):
         raise KernelError(f"moe_route: score {score!r}")
+    if mark not in ("two", "best"):
+        raise KernelError(f"moe_route: mark {mark!r}")
     _check(_get("air_moe_route")(z.data_ptr(), z.shape[1], T, int(experts), int(top), 1 if score == "softmax" else 0,
                                  1 if renormalize else 0, 1 if has_gate else 0, expert_out.data_ptr(),
-                                 weight_out.data_ptr(), _ptr(gate_out), int(groups), int(keep), float(route_scale),
+                                 weight_out.data_ptr(), _ptr(gate_out), int(groups), int(keep),
+                                 1 if mark == "best" else 0, float(route_scale),
                                  float(norm_eps), _ptr(choice_bias), _stream()), "moe_route")
 
 
@@ -896,10 +943,11 @@ def moe_sort(expert, experts, start, pair_of_slot, tiles, num_tiles):
 def grouped_gemm(a, w, out, n, k, *, lda, ldo, groups, a_group_stride=0, o_group_stride=0, a_index=None, a_div=1,
                  a_scale=None, a_local=False, o_index=None, o_div=1, o_part_stride=0, o_local=False, start=None,
                  rows_per_group=0, tiles=None, num_tiles=None, silu_mul=False, gate_block=0, o_scale=None, o_scale_ld=0,
-                 relu2=False):
+                 relu2=False, act=(1.0, 0.0, 0.0)):
     """out rows = a rows @ w[g]^T for every group g (w [groups, n (2n with silu_mul), k]); see grouped_gemm.cu for how
     rows are found.  Strides in elements.  out is float32 or of a's type; with silu_mul out = silu(gate) * linear, the
-    rows of w[g] being blocks of gate_block gate rows and as many linear rows in turn (0: all gate rows first).
+    rows of w[g] being blocks of gate_block gate rows and as many linear rows in turn (0: all gate rows first); act =
+    (alpha, limit, shift) is then the gated activation as gemm_tc describes it (default: SiLU).
     o_scale float32: the row written for slot s is multiplied, in 32-bit, by o_scale[o_index[s]], or without o_index by
     o_scale[row * o_scale_ld + g] (row: the row of out, inside the group where o_local).  relu2: out = max(product, 0)^2
     in a's type."""
@@ -923,7 +971,8 @@ def grouped_gemm(a, w, out, n, k, *, lda, ldo, groups, a_group_stride=0, o_group
         w.data_ptr(), w.shape[1] * w.shape[2], out.data_ptr(), int(ldo), int(o_group_stride), _ptr(o_index), int(o_div),
         int(o_part_stride), 1 if o_local else 0, 1 if out.dtype == torch.float32 else 0, _ptr(start),
         int(rows_per_group), _ptr(tiles), _ptr(num_tiles), tiles.shape[0] if tiles is not None else 0, int(groups),
-        int(n), int(k), _DT[a.dtype], 2 if relu2 else (1 if silu_mul else 0), int(gate_block), _ptr(o_scale), int(o_scale_ld), _stream()), "grouped_gemm")
+        int(n), int(k), _DT[a.dtype], 2 if relu2 else (1 if silu_mul else 0), int(gate_block), _ptr(o_scale), int(o_scale_ld), float(act[0]),
+        float(act[1]), float(act[2]), _stream()), "grouped_gemm")
     return out
 
 
@@ -1027,7 +1076,7 @@ def short_conv_silu(x, weight, state, y, q_start, slots, max_tokens, act=True):
     return y
 
 
-SCAN_DELTA, SCAN_GLA, SCAN_HGRN, SCAN_RETENTION = 0, 1, 2, 3
+SCAN_DELTA, SCAN_GLA, SCAN_HGRN, SCAN_RETENTION, SCAN_CHANNEL_DELTA = 0, 1, 2, 3, 4
 
 
 def linear_scan(mode, q, k, v, decay, state, out, q_start, slots, token_seq, q_scale=1.0, beta=None, a_log=None,
@@ -1041,6 +1090,7 @@ def linear_scan(mode, q, k, v, decay, state, out, q_start, slots, token_seq, q_s
     SCAN_DELTA: decay, beta [T, H] logits; g = exp(-exp(a_log[h]) * softplus(decay + dt_bias[h])), b = sigmoid(beta);
       with unit, q and k are first divided by sqrt(sum of squares + unit_eps), q then multiplied by q_scale;
       S = g S; u = b (v - S^T k); S += k u^T; o = S^T q.
+    SCAN_CHANNEL_DELTA: as SCAN_DELTA with a decay per key channel: decay [T, H * d], dt_bias [H * d], S = diag(g) S.
     SCAN_GLA: decay [T, H * d] logits; alpha = sigmoid(decay)^(1 / tau); q is multiplied by q_scale;
       S = diag(alpha) S + k v^T; o = S^T q.
     SCAN_HGRN: decay [T, H * d] logits, lower and gate_bias float32 [H * d]; alpha = lower + (1 - lower) *
@@ -1068,12 +1118,14 @@ def linear_scan(mode, q, k, v, decay, state, out, q_start, slots, token_seq, q_s
     if G == 0 or H % G:
         raise KernelError(f"linear_scan: {H} heads over {G} heads of q and k")
     bp, ldb = (None, 0)
-    if mode == SCAN_DELTA:
+    if mode in (SCAN_DELTA, SCAN_CHANNEL_DELTA):
+        per_head = 1 if mode == SCAN_DELTA else d
         bp, ldb = _columns(beta, "beta")
         _req(a_log, "a_log", (torch.float32,), (H,))
-        _req(dt_bias, "dt_bias", (torch.float32,), (H,))
-        if decay.shape[1] != H or beta.shape[1] != H:
-            raise KernelError("linear_scan: the delta rule takes one decay and one beta per head")
+        _req(dt_bias, "dt_bias", (torch.float32,), (H * per_head,))
+        if decay.shape[1] != H * per_head or beta.shape[1] != H:
+            raise KernelError("linear_scan: the delta rule takes one beta per head, and one decay per head or per key "
+                              "channel of every head")
     elif mode == SCAN_GLA:
         if decay.shape[1] != H * d or G != H:
             raise KernelError("linear_scan: gated linear attention takes a decay per key channel of every head")
@@ -1105,7 +1157,7 @@ def linear_scan(mode, q, k, v, decay, state, out, q_start, slots, token_seq, q_s
         lanes *= 2
     kq = torch.empty((T, G, 2, lanes * rows), dtype=torch.float32, device=out.device)
     dec = None if mode == SCAN_RETENTION else \
-        torch.empty((T, H, 2 if mode == SCAN_DELTA else lanes * rows), dtype=torch.float32, device=out.device)
+        torch.empty((T, H, {SCAN_DELTA: 2, SCAN_CHANNEL_DELTA: lanes * rows + 4}.get(mode, lanes * rows)), dtype=torch.float32, device=out.device)
     _check(_get("air_linear_scan")(
         int(mode), qp, ldq, kp, ldk, vp, ldv, dp, ldd, bp, ldb, _ptr(a_log), _ptr(dt_bias), state.data_ptr(),
         out.data_ptr(), q_start.data_ptr(), slots.data_ptr(), token_seq.data_ptr(), kq.data_ptr(), _ptr(dec),
@@ -1117,8 +1169,8 @@ def linear_scan(mode, q, k, v, decay, state, out, q_start, slots, token_seq, q_s
     return out
 
 
-def gated_rmsnorm(o, gate, weight, eps, out, token_seq):
-    """out[t, h, :] = o[t, h, :] / sqrt(mean(o^2) + eps) * weight * silu(gate[t, h, :]).  o float32 [T, H, dv]; gate
+def gated_rmsnorm(o, gate, weight, eps, out, token_seq, sigmoid=False):
+    """out[t, h, :] = o[t, h, :] / sqrt(mean(o^2) + eps) * weight * act(gate[t, h, :]), act SiLU or (sigmoid) the sigmoid.  o float32 [T, H, dv]; gate
     float32 [T, H * dv] (may be a band of columns) or None (no gate); weight float32 [dv]; out [T, H * dv]."""
     T, H, dv = o.shape
     _req(o, "o", (torch.float32,))
@@ -1129,7 +1181,34 @@ def gated_rmsnorm(o, gate, weight, eps, out, token_seq):
     _req(out, "out", _FLOATS, (T, H * dv))
     _req(token_seq, "token_seq", _I32, (T,))
     _check(_get("air_gated_rmsnorm")(o.data_ptr(), gp, ldg, weight.data_ptr(), out.data_ptr(), _DT[out.dtype],
-                                     token_seq.data_ptr(), T, H, dv, float(eps), _stream()), "gated_rmsnorm")
+                                     token_seq.data_ptr(), T, H, dv, float(eps), 1 if sigmoid else 0, _stream()),
+           "gated_rmsnorm")
+    return out
+
+
+def split_bands(x, first, second):
+    """The first `first` columns of x (float32, may be a band of a wider matrix) and the `second` ones behind them as
+    bfloat16 rows [hi | lo] with hi + lo the number to 16 bits: ([T, 2 first], [T, 2 second]).  A product with a matrix
+    [W | W] then has the exactness of a 32-bit operand."""
+    T = x.shape[0]
+    xp, ld = _columns(x, "x")
+    if x.shape[1] != first + second:
+        raise KernelError(f"split_bands: {x.shape[1]} columns, not {first} + {second}")
+    a = torch.empty((T, 2 * first), dtype=torch.bfloat16, device=x.device)
+    b = torch.empty((T, 2 * second), dtype=torch.bfloat16, device=x.device)
+    _check(_get("air_split_bands")(xp, ld, int(first), int(second), a.data_ptr(), b.data_ptr(), T, _stream()), "split_bands")
+    return a, b
+
+
+def band_rmsnorm(x, weight, eps, out):
+    """out = x / sqrt(mean(x^2) + eps) * weight per row; x float32 [T, n], may be a band of columns; weight float32 [n];
+    out [T, >= n] gets zeros behind the n columns."""
+    T, n = x.shape
+    xp, ld = _columns(x, "x")
+    _req(weight, "weight", (torch.float32,), (n,))
+    _req(out, "out", _FLOATS, (T, None))
+    _check(_get("air_band_rmsnorm")(xp, ld, weight.data_ptr(), float(eps), out.data_ptr(), _DT[out.dtype], out.shape[1], T, n,
+                                    _stream()), "band_rmsnorm")
     return out
 
 
@@ -1302,12 +1381,13 @@ def decode_splits(tokens: int, heads: int, kv_heads: int) -> int:
 
 
 def decode_attention(q, cache, block_table, token_seq, positions, out, window, scale, splits=None, scratch=None,
-                     status=None, engine="tma", softcap=0.0, sink=None, gate=None, turn=None):
+                     status=None, engine="tma", softcap=0.0, sink=None, gate=None, turn=None, bias=None):
     """bfloat16 attention for one query token per request.  softcap > 0: score = softcap * tanh(scale * q.k /
     softcap) (the copy-engine kernel only).  sink (float32 [H]): one more term exp(sink[h]) in the softmax's
     denominator; gate (float32 [T, H * d] logits, may be a band of columns): out is multiplied by sigmoid(gate) element
     by element; turn = (freq, pairing): ahead of the gate every head's output is turned back as turn_heads(.., back=True)
-    does it; all enter where the key splits are merged (the copy-engine kernel only, two splits at least).  scratch: (float32 [T*H*splits*D], float32
+    does it; all enter where the key splits are merged (the copy-engine kernel only, two splits at least).  bias (float32
+    [H, n]): a score gets bias[h, min(distance, n - 1)] (the copy-engine kernel only).  scratch: (float32 [T*H*splits*D], float32
     [T*H*splits*2]) or None to allocate.  engine "tma": keys and values by the copy engine into shared
     memory (attention_decode_tma.cu); "ldg": by the warps' own loads (attention_decode.cu)."""
     T, H, d = q.shape
@@ -1325,8 +1405,8 @@ def decode_attention(q, cache, block_table, token_seq, positions, out, window, s
     extra = sink is not None or gate is not None or turn is not None
     if extra:
         splits = max(2, splits)
-        if not (engine == "tma" and tile_pages(P)):
-            raise KernelError("decode_attention: a sink, gates or a turn back are taken by the copy-engine kernel only")
+    if (extra or bias is not None) and not (engine == "tma" and tile_pages(P)):
+        raise KernelError("decode_attention: a sink, gates, a turn back or a bias are taken by the copy-engine kernel only")
     po = pm = None
     if splits > 1:
         if scratch is None:
@@ -1338,7 +1418,7 @@ def decode_attention(q, cache, block_table, token_seq, positions, out, window, s
         if po.numel() < T * H * splits * d or pm.numel() < T * H * splits * 2:
             raise KernelError("decode_attention: scratch is too small")
     global launches
-    if extra:
+    if extra or bias is not None:
         gp, ldg = (None, 0)
         if sink is not None:
             _req(sink, "sink", (torch.float32,), (H,))
@@ -1350,7 +1430,7 @@ def decode_attention(q, cache, block_table, token_seq, positions, out, window, s
             q.data_ptr(), cache.data_ptr(), cache.shape[0], block_table.data_ptr(), block_table.shape[1],
             token_seq.data_ptr(), positions.data_ptr(), out.data_ptr(), _ptr(po), _ptr(pm), T, H, K, d, P,
             int(window or 0), float(scale), float(softcap or 0.0), splits, _ptr(status), _ptr(sink), gp, ldg,
-            *_turn(turn, d), _stream()), "decode_attention_tma")
+            *_turn(turn, d), *_distance_bias(bias, H), _stream()), "decode_attention_tma")
     elif engine == "tma" and tile_pages(P):
         _check(_get("air_decode_attention_tma")(
             q.data_ptr(), cache.data_ptr(), cache.shape[0], block_table.data_ptr(), block_table.shape[1],
@@ -1520,10 +1600,11 @@ def prefill_attention_scratch(slots: int, head_dim: int, device):
 
 
 def prefill_attention_tc(q, cache, block_table, tiles, out, window, scale, status=None, segments=None, items=None,
-                         slots=0, scratch=None, softcap=0.0, sink=None):
+                         slots=0, scratch=None, softcap=0.0, sink=None, bias=None):
     """bfloat16 causal attention with both products on the tcgen05 tensor cores (see
     attention_prefill_tc.cu); arguments as prefill_attention; head size 64 or 128.  softcap > 0: score = softcap *
     tanh(scale * q.k / softcap).  sink (float32 [H]): one more term exp(sink[h]) in the softmax's denominator.
+    bias (float32 [H, n]): a score gets bias[h, min(distance, n - 1)].
     segments [n, 5] int32 (pair of the list, head, first key tile, key tiles, slot or -1): which block takes which
     part of which pair's stream of keys, instead of one block per pair and head; items [m, 4] int32 (pair, head,
     first slot, slots): the (pair, head)s whose segments write partial sums into `slots` slots, merged here.
@@ -1560,9 +1641,11 @@ def prefill_attention_tc(q, cache, block_table, tiles, out, window, scale, statu
             _ptr(items) if n_items else None, n_items, int(slots) if segments is not None else 0, _ptr(part_o),
             _ptr(part_ml), out.data_ptr(), H, K, d, P, int(window or 0), float(scale), float(softcap or 0.0),
             _ptr(status))
-    if sink is not None:
-        _req(sink, "sink", (torch.float32,), (H,))
-        _check(_get("air_prefill_attention_tc_sink")(*args, sink.data_ptr(), _stream()), "prefill_attention_tc")
+    if sink is not None or bias is not None:
+        if sink is not None:
+            _req(sink, "sink", (torch.float32,), (H,))
+        _check(_get("air_prefill_attention_tc_sink")(*args, _ptr(sink), *_distance_bias(bias, H), _stream()),
+               "prefill_attention_tc")
     else:
         _check(_get("air_prefill_attention_tc")(*args, _stream()), "prefill_attention_tc")
     return out

@@ -13,13 +13,16 @@
 //                              HGRN   the same recurrence with k = 1 - alpha (the complement of the decay stands where
 //                                     a key would); alpha = l + (1 - l) sigmoid(z + bias) with a lower bound l per
 //                                     channel, q = silu(q)
+//                              CDELTA the delta rule with a decay per key channel: S = diag(g) S, then as DELTA
 //                              RET    S = g_h S + k v^T;  o = S^T q with one constant g_h per head (retention); q and k
 //                                     are first rotated by the token's position, k then multiplied by a constant
 //                            Columns of S do not depend on one another, so a block takes a few of them and a column is
 //                            held in the registers of L lanes of one warp; the tokens of a portion are taken in order.
 //                            What a token's output is depends on the state and the tokens before it only, not on how
 //                            the request was cut into steps or on the rest of the batch.
-//   gated_rmsnorm_kernel     out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate[t, h, :]) (without a gate: * w)
+//   gated_rmsnorm_kernel     out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, h, :]), act SiLU or the sigmoid
+//                            (without a gate: * w)
+//   split_bands_kernel       two bands of columns as bfloat16 rows [hi | lo] with hi + lo the 32-bit number (to 16 bits)
 #include "common.cuh"
 
 namespace air {
@@ -87,7 +90,9 @@ short_conv_silu_kernel(const float* __restrict__ x, int ld, const float* __restr
     }
 }
 
-enum { SCAN_DELTA = 0, SCAN_GLA = 1, SCAN_HGRN = 2, SCAN_RET = 3 };
+enum { SCAN_DELTA = 0, SCAN_GLA = 1, SCAN_HGRN = 2, SCAN_RET = 3, SCAN_CDELTA = 4 };
+// CDELTA: floats per token and head behind the dpad decays: beta, and three to the next 16 bytes
+constexpr int CDELTA_TAIL = 4;
 constexpr int SCAN_THREADS = 128;
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -108,6 +113,8 @@ __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wai
 //                        GLA   [T, H, dpad]: alpha = sigmoid(decay)^(1 / tau) per key channel, zeros from d on
 //                        HGRN  [T, H, dpad]: alpha = l + (1 - l) sigmoid(decay + bias); kq's k is 1 - alpha (no k is
 //                              read) and its q is silu(q) * q_scale
+//                        CDELTA [T, H, dpad + 4]: g = exp(-exp(a_log) softplus(decay + dt_bias)) per key channel of every
+//                              head, zeros from d on, then b = sigmoid(beta)
 //                        RET   nothing: the decay is one constant per head, read by the scan from decay [H]; kq's q and
 //                              k have their first `rot` elements rotated (element i with i + rot / 2, angle position *
 //                              freq[i] as a 64-bit product, its cos and sin taken in 64-bit), q times q_scale, k times
@@ -115,10 +122,10 @@ __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wai
 struct ScanPrepArgs {
     const float* q; int ldq;         // [T, ldq]: head g's d elements at column g * d
     const float* k; int ldk;
-    const float* decay; int ldd;     // DELTA: [T, ldd] one logit per head;  GLA: [T, ldd] d logits per head
-    const float* beta; int ldb;      // DELTA: [T, ldb] one logit per head
-    const float* a_log;              // DELTA: [H];  HGRN: the lower bounds l [H * d]
-    const float* dt_bias;            // DELTA: [H];  HGRN: the gate's bias [H * d]
+    const float* decay; int ldd;     // DELTA: [T, ldd] one logit per head;  GLA, CDELTA: [T, ldd] d logits per head
+    const float* beta; int ldb;      // DELTA, CDELTA: [T, ldb] one logit per head
+    const float* a_log;              // DELTA, CDELTA: [H];  HGRN: the lower bounds l [H * d]
+    const float* dt_bias;            // DELTA: [H];  CDELTA: [H * d];  HGRN: the gate's bias [H * d]
     const int* token_seq;
     float* kq;
     float* dec;
@@ -202,6 +209,15 @@ __global__ void __launch_bounds__(128) scan_prepare_kernel(const ScanPrepArgs p)
         float* a = p.dec + ((size_t)t * p.H + g) * p.dpad;
         for (int r = threadIdx.x; r < p.dpad; r += blockDim.x)
             a[r] = r < p.d ? expf(p.inv_tau * log_sigmoid_f(z[r])) : 0.f;
+    } else if (MODE == SCAN_CDELTA) {
+        for (int h = g * (p.H / p.G); h < (g + 1) * (p.H / p.G); ++h) {      // the heads that read this head of q and k
+            const float* z = p.decay + (size_t)t * p.ldd + h * p.d;
+            float* a = p.dec + ((size_t)t * p.H + h) * (p.dpad + CDELTA_TAIL);
+            const float rate = -expf(p.a_log[h]);
+            for (int r = threadIdx.x; r < p.dpad; r += blockDim.x)
+                a[r] = r < p.d ? expf(rate * softplus_f(z[r] + p.dt_bias[h * p.d + r])) : 0.f;
+            if (threadIdx.x == 0) a[p.dpad] = 1.f / (1.f + expf(-p.beta[(size_t)t * p.ldb + h]));
+        }
     } else if (g == 0) {
         for (int h = threadIdx.x; h < p.H; h += blockDim.x) {
             p.dec[((size_t)t * p.H + h) * 2] =
@@ -213,7 +229,7 @@ __global__ void __launch_bounds__(128) scan_prepare_kernel(const ScanPrepArgs p)
 
 struct ScanArgs {
     const float* kq;                 // [T, G, 2, dpad] (scan_prepare_kernel)
-    const float* dec;                // DELTA [T, H, 2];  GLA [T, H, dpad]
+    const float* dec;                // DELTA [T, H, 2];  GLA [T, H, dpad];  CDELTA [T, H, dpad + 4]
     const float* v; int ldv;         // [T, ldv]: head h's dv elements at column h * dv
     float* state;                    // [slots, H, d, dv]
     float* out;                      // [T, H, dv]
@@ -245,8 +261,10 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
     const bool live = col < p.dv;
     const int g = h / (p.H / p.G);
 
-    // a buffer: kq [TK][2][dpad], then (GLA) alpha [TK][dpad] or (DELTA) g, b [TK][2], then v [TK][CB]
-    const int dec_floats = MODE == SCAN_GLA ? TK * dpad : (MODE == SCAN_RET ? 0 : ((2 * TK + 3) & ~3));
+    // a buffer: kq [TK][2][dpad], then (GLA) alpha [TK][dpad] or (CDELTA) g and b [TK][dpad + 4] or (DELTA) g, b [TK][2],
+    // then v [TK][CB]
+    constexpr int per_dec = MODE == SCAN_GLA ? dpad : MODE == SCAN_CDELTA ? dpad + CDELTA_TAIL : 0;
+    const int dec_floats = per_dec ? TK * per_dec : (MODE == SCAN_RET ? 0 : ((2 * TK + 3) & ~3));
     const int buf_floats = TK * 2 * dpad + dec_floats + TK * CB;
     float* so = smem + 2 * buf_floats;                           // [TK][CB][L]: the lanes' partial read-outs
 
@@ -260,11 +278,11 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
             const int tt = idx / per_token, c = idx % per_token;
             cp_async16(bkq + tt * 2 * dpad + 4 * c, p.kq + ((size_t)(q0 + t0 + tt) * p.G + g) * 2 * dpad + 4 * c);
         }
-        if (MODE == SCAN_GLA) {
-            constexpr int per = dpad / 4;
+        if constexpr (per_dec > 0) {
+            constexpr int per = per_dec / 4;
             for (int idx = threadIdx.x; idx < cnt * per; idx += SCAN_THREADS) {
                 const int tt = idx / per, c = idx % per;
-                cp_async16(bdec + tt * dpad + 4 * c, p.dec + ((size_t)(q0 + t0 + tt) * p.H + h) * dpad + 4 * c);
+                cp_async16(bdec + tt * per_dec + 4 * c, p.dec + ((size_t)(q0 + t0 + tt) * p.H + h) * per_dec + 4 * c);
             }
         } else if (MODE == SCAN_DELTA) {
             for (int idx = threadIdx.x; idx < cnt * 2; idx += SCAN_THREADS)
@@ -302,13 +320,15 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
             const float vv = live ? bv[tt * CB + cc] : 0.f;
             // (four partial sums each: the chain of dependent additions is a quarter as long)
             float orr[4] = {0.f, 0.f, 0.f, 0.f};
-            if (MODE == SCAN_DELTA) {
-                const float gv = bdec[2 * tt], bb = bdec[2 * tt + 1];
+            if (MODE == SCAN_DELTA || MODE == SCAN_CDELTA) {
+                const float* aa = bdec + tt * per_dec + l;       // CDELTA: a decay per row of the column
+                const float gv = MODE == SCAN_DELTA ? bdec[2 * tt] : 0.f;
+                const float bb = MODE == SCAN_DELTA ? bdec[2 * tt + 1] : bdec[tt * per_dec + dpad];
                 float kr[R], pr[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int i = 0; i < R; ++i) {
                     kr[i] = kk[i * L];
-                    S[i] *= gv;
+                    S[i] *= MODE == SCAN_DELTA ? gv : aa[i * L];
                     pr[i & 3] = fmaf(S[i], kr[i], pr[i & 3]);
                 }
                 float pred = (pr[0] + pr[1]) + (pr[2] + pr[3]);
@@ -353,12 +373,13 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
 }
 
 // o [T, H, dv] float32; gate [T, ldg] float32 (head h at column h * dv) or null (no gate); w [dv]; out [T, H * dv].
-// One warp per (token, head).
+// sigmoid: the gate multiplies by its sigmoid instead of its SiLU.  One warp per (token, head).
 template <typename TO>
 __global__ void __launch_bounds__(128)
 gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int ldg, const float* __restrict__ w,
-                     TO* __restrict__ out, const int* __restrict__ token_seq, int T, int H, int dv, float eps, int vec) {
+                     TO* __restrict__ out, const int* __restrict__ token_seq, int T, int H, int dv, float eps, int vec, int sigmoid) {
     pdl_enter(TR_GATED);
+    auto opened = [&](float z) { return (sigmoid ? 1.f : z) / (1.f + expf(-z)); };
     const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (item >= T * H) return;
     const int t = item / H, h = item % H;
@@ -381,7 +402,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate
             load4(w + i, wv);
             if (gr) load4(gr + i, g);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) x[j] = x[j] * scale * wv[j] * (gr ? silu_f(g[j]) : 1.f);
+            for (int j = 0; j < 4; ++j) x[j] = x[j] * scale * wv[j] * (gr ? opened(g[j]) : 1.f);
             store4(out + (size_t)item * dv + i, x);
         }
         return;
@@ -391,7 +412,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate
     const float scale = rsqrtf(ss / (float)dv + eps);
     const float* gr = gate ? gate + (size_t)t * ldg + h * dv : nullptr;
     for (int i = lane; i < dv; i += 32)
-        out[(size_t)item * dv + i] = from_float<TO>(row[i] * scale * w[i] * (gr ? silu_f(gr[i]) : 1.f));
+        out[(size_t)item * dv + i] = from_float<TO>(row[i] * scale * w[i] * (gr ? opened(gr[i]) : 1.f));
 }
 
 // rows of a column per lane: 16 up to 512 key channels, 32 beyond
@@ -410,7 +431,9 @@ static int launch_scan(const ScanPrepArgs& prep, const ScanArgs& a, int T, int S
     const int CB = SCAN_THREADS / L;
     // two buffers of `tokens` tokens each, and their partial read-outs, within 96 KB
     auto bytes = [&](int tk) {
-        const size_t dec = MODE == SCAN_GLA ? (size_t)tk * dpad : (MODE == SCAN_RET ? 0 : (size_t)((2 * tk + 3) & ~3));
+        const size_t dec = MODE == SCAN_GLA ? (size_t)tk * dpad
+                         : MODE == SCAN_CDELTA ? (size_t)tk * (dpad + CDELTA_TAIL)
+                         : MODE == SCAN_RET ? 0 : (size_t)((2 * tk + 3) & ~3);
         return sizeof(float) * (2 * ((size_t)tk * 2 * dpad + dec + (size_t)tk * CB) + (size_t)tk * SCAN_THREADS);
     };
     int tk = 16;
@@ -468,7 +491,8 @@ AIR_API int air_short_conv_silu(const float* x, int ld, const float* w, float* s
                        slots, C, taps, chunk, act);
 }
 
-// kq: float32 workspace [T, G, 2, L * R] and dec: [T, H, 2] (mode 0) or [T, H, L * R] (modes 1, 2), with R = 16 up to
+// kq: float32 workspace [T, G, 2, L * R] and dec: [T, H, 2] (mode 0), [T, H, L * R] (modes 1, 2) or [T, H, L * R + 4] (mode
+// 4), with R = 16 up to
 // 512 key channels and 32 beyond, L the power of two with L * R >= d.  Mode 3 (retention): decay is [H], the heads'
 // constants, and no dec is needed; positions [T], freq float64 [rot / 2], k_scale as ScanPrepArgs says.
 AIR_API int air_linear_scan(int mode, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv,
@@ -491,6 +515,10 @@ AIR_API int air_linear_scan(int mode, const float* q, int ldq, const float* k, i
     a.H = H; a.G = G; a.d = d; a.dv = dv; a.L = L; a.tokens = 0;
     if (mode == air::SCAN_DELTA) return air::launch_scan<air::SCAN_DELTA>(pr, a, T, S, stream);
     if (mode == air::SCAN_GLA) return air::launch_scan<air::SCAN_GLA>(pr, a, T, S, stream);
+    if (mode == air::SCAN_CDELTA) {
+        if (!decay || !beta || !a_log || !dt_bias) return AIR_ERR_BAD_ARGUMENT;
+        return air::launch_scan<air::SCAN_CDELTA>(pr, a, T, S, stream);
+    }
     if (mode == air::SCAN_HGRN) {
         if (G != H || !a_log || !dt_bias) return AIR_ERR_BAD_ARGUMENT;
         return air::launch_scan<air::SCAN_HGRN>(pr, a, T, S, stream);
@@ -505,14 +533,41 @@ AIR_API int air_linear_scan(int mode, const float* q, int ldq, const float* k, i
 }
 
 AIR_API int air_gated_rmsnorm(const float* o, const float* gate, int ldg, const float* w, void* out, int out_dtype,
-                              const int* token_seq, int T, int H, int dv, float eps, cudaStream_t stream) {
+                              const int* token_seq, int T, int H, int dv, float eps, int sigmoid, cudaStream_t stream) {
     if (T <= 0) return 0;
     const int blocks = (T * H + 3) / 4;
     const int vec = dv % 4 == 0 && (!gate || ldg % 4 == 0) &&
                     (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
     AIR_DISPATCH(out_dtype, TO, return air::launch(air::gated_rmsnorm_kernel<TO>, blocks, 128, 0, stream, o, gate, ldg, w,
-                                                   (TO*)out, token_seq, T, H, dv, eps, vec));
+                                                   (TO*)out, token_seq, T, H, dv, eps, vec, sigmoid));
     return 0;
+}
+
+// x [T, ldx] float32: the columns 0 .. na - 1 and na .. na + nb - 1 -> a [T, 2 na], b [T, 2 nb] bfloat16, rows [hi | lo].
+namespace air {
+__global__ void __launch_bounds__(256)
+split_bands_kernel(const float* __restrict__ x, int ldx, int na, int nb, __nv_bfloat16* __restrict__ a,
+                   __nv_bfloat16* __restrict__ b, int T) {
+    pdl_enter(TR_CONVERT);
+    const int n = na + nb;
+    for (long long idx = (long long)blockIdx.x * 256 + threadIdx.x; idx < (long long)T * n; idx += (long long)gridDim.x * 256) {
+        const int t = (int)(idx / n), c = (int)(idx % n);
+        const float v = x[(size_t)t * ldx + c];
+        const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+        const __nv_bfloat16 lo = __float2bfloat16_rn(v - __bfloat162float(hi));
+        __nv_bfloat16* row = c < na ? a + (size_t)t * 2 * na + c : b + (size_t)t * 2 * nb + (c - na);
+        row[0] = hi;
+        row[c < na ? na : nb] = lo;
+    }
+}
+}  // namespace air
+
+AIR_API int air_split_bands(const float* x, int ldx, int na, int nb, void* a, void* b, int T, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (na < 0 || nb < 0 || na + nb <= 0 || ldx < na + nb || (na && !a) || (nb && !b)) return AIR_ERR_BAD_ARGUMENT;
+    const long long blocks = ((long long)T * (na + nb) + 255) / 256;
+    return air::launch(air::split_bands_kernel, (unsigned)(blocks < 148 * 8 ? blocks : 148 * 8), 256, 0, stream, x, ldx, na,
+                       nb, (__nv_bfloat16*)a, (__nv_bfloat16*)b, T);
 }
 
 AIR_API int air_trace_set_recurrent(unsigned long long* buffer) { return air::set_trace_here(buffer); }

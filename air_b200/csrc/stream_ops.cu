@@ -11,6 +11,11 @@
 //                         u / sqrt(mean(u^2) + eps), and b may be absent.  x' is written when h_out is given; with `rows` the
 //                         kernel reads row rows[r] of everything and writes row r.  The streams may all be one tensor
 //                         (stream stride 0: they start out equal).  Everything is 32-bit; the row is written in its own type.
+//                         More terms than y may join the one stream of an ordinary layer (S = 1) in the same pass: up to
+//                         two, each a tensor or partial sums, each with a factor per row (the sub-layers of a layer that
+//                         stand side by side, one of them with a gate per token).  Without w but with `out` the row
+//                         is written as it is, no norm, ahead of the row of a second tensor where one is given: [u | again],
+//                         2 E columns.
 //                         With conv (a step in which every row is its request's only token) the row becomes
 //                         row + sum_j cw[j] in_(t - taps + 1 + j) before it is written, the earlier inputs coming from
 //                         the request's state, which is moved on by one token.
@@ -22,6 +27,12 @@
 #include "common.cuh"
 
 namespace air {
+
+// One more term of the sum into an ordinary residual stream: partial sums [parts, T, E], times a factor per row (or 1).
+struct StreamTerm {
+    const float* y; int parts; const float* gate;
+};
+constexpr int STREAM_MORE = 2;
 
 struct StreamNormArgs {
     const float* x; size_t x_stride;       // stream s at x + s * x_stride
@@ -36,6 +47,8 @@ struct StreamNormArgs {
     const float* conv_w; float* conv_state; const int* token_seq; int taps;
     int S, E, center;
     float eps;
+    StreamTerm more[STREAM_MORE];          // (S = 1)
+    const float* again;                    // [T, E], written behind the row where there is no norm
 };
 
 constexpr int STREAMS_MAX = 16;
@@ -52,7 +65,8 @@ template <int N> __device__ __forceinline__ void store_columns(float* q, const f
 // N columns of all streams of a row: mixed, written, and folded into u.  NS: the number of streams, all at compile-time
 // indices; 0: p.S of them, in a loop.
 template <int NS, int N>
-__device__ __forceinline__ void stream_columns(const StreamNormArgs& p, size_t src, int i, const float* coef, float (&u)[N]) {
+__device__ __forceinline__ void stream_columns(const StreamNormArgs& p, int row, int i, const float* coef, float (&u)[N]) {
+    const size_t src = (size_t)row * p.E;
     const int S = NS ? NS : p.S;
     constexpr int UN = NS ? NS : 1;
     float x[NS ? NS : STREAMS_MAX][N], y[N];
@@ -66,6 +80,25 @@ __device__ __forceinline__ void stream_columns(const StreamNormArgs& p, size_t s
             load_columns<N>(p.y + q * p.part_stride + src + i, t);
 #pragma unroll
             for (int j = 0; j < N; ++j) y[j] += t[j];
+        }
+        if constexpr (NS <= 1) {
+#pragma unroll
+            for (int m = 0; m < STREAM_MORE; ++m) {
+                const StreamTerm& term = p.more[m];
+                if (!term.y) continue;
+                float z[N];
+                load_columns<N>(term.y + src + i, z);
+#pragma unroll 4
+                for (int q = 1; q < term.parts; ++q) {
+                    float t[N];
+                    load_columns<N>(term.y + q * p.part_stride + src + i, t);
+#pragma unroll
+                    for (int j = 0; j < N; ++j) z[j] += t[j];
+                }
+                const float g = term.gate ? term.gate[row] : 1.f;
+#pragma unroll
+                for (int j = 0; j < N; ++j) y[j] = fmaf(g, z[j], y[j]);
+            }
         }
     }
     const float *mix = coef, *out_w = coef + S * S, *read = out_w + S;
@@ -154,19 +187,20 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormArgs 
     pdl_wait();
     trace_point(TR_STREAM_NORM);
     const int r = blockIdx.x;
-    const size_t src = (size_t)(p.rows ? p.rows[r] : r) * E;
+    const int row = p.rows ? p.rows[r] : r;
+    const size_t src = (size_t)row * E;
     const int step = blockDim.x * N;
     float u1[N], sum = 0.f;
 #pragma unroll
     for (int j = 0; j < N; ++j) u1[j] = 0.f;
     if constexpr (ONE) {
-        if (first < E) stream_columns<NS, N>(p, src, first, coef, u1);
+        if (first < E) stream_columns<NS, N>(p, row, first, coef, u1);
 #pragma unroll
         for (int j = 0; j < N; ++j) sum += p.center ? u1[j] : u1[j] * u1[j];
     } else {
         for (int i = first; i < E; i += step) {
             float u[N];
-            stream_columns<NS, N>(p, src, i, coef, u);
+            stream_columns<NS, N>(p, row, i, coef, u);
 #pragma unroll
             for (int j = 0; j < N; ++j) {
                 urow[i + j] = u[j];
@@ -174,7 +208,24 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormArgs 
             }
         }
     }
-    if (!p.w) return;
+    if (!p.w) {
+        if (!p.out) return;
+        // the row as it is, and the second tensor's row behind it
+        const int width = p.again ? 2 * E : E;
+        TO* out = (TO*)p.out + (size_t)r * width;
+        for (int i = first; i < E; i += step) {
+            float u[N], a[N];
+#pragma unroll
+            for (int j = 0; j < N; ++j) u[j] = ONE ? u1[j] : urow[i + j];
+            if constexpr (N == 4) store4(out + i, u);
+            else out[i] = from_float<TO>(u[0]);
+            if (!p.again) continue;
+            load_columns<N>(p.again + src + i, a);
+            if constexpr (N == 4) store4(out + E + i, a);
+            else out[E + i] = from_float<TO>(a[0]);
+        }
+        return;
+    }
     float mean = 0.f;
     if (p.center) {
         mean = block_sum(sum, scratch) / (float)E;
@@ -266,8 +317,12 @@ AIR_API int air_stream_norm(const float* x, long long x_stride, float* h_out, lo
                             long long part_stride, const float* mix, const float* out_w, const float* read, int S,
                             const float* w, const float* b, void* out, int out_dtype, const int* rows, int R, int E,
                             int center, float eps, const float* conv_w, float* conv_state, const int* token_seq, int taps,
-                            cudaStream_t stream) {
+                            const float* more1, int more1_parts, const float* gate1, const float* more2, int more2_parts,
+                            const float* gate2, const float* again, cudaStream_t stream) {
     if (R <= 0) return 0;
+    if ((more1 || more2) && (S != 1 || !y || (more1 && more1_parts < 1) || (more2 && more2_parts < 1)))
+        return AIR_ERR_BAD_ARGUMENT;
+    if (again && (w || !out)) return AIR_ERR_BAD_ARGUMENT;
     if (!x || S < 1 || S > air::STREAMS_MAX || E <= 0 || (y && y_parts < 1) || (w && !out) || (conv_w && (taps < 1 || rows || !token_seq)) ||
         (conv_w && taps > 1 && !conv_state))
         return AIR_ERR_BAD_ARGUMENT;
@@ -278,9 +333,11 @@ AIR_API int air_stream_norm(const float* x, long long x_stride, float* h_out, lo
     p.part_stride = (size_t)part_stride; p.mix = mix; p.out_w = out_w; p.read = read; p.S = S; p.w = w; p.b = b; p.out = out;
     p.rows = rows; p.E = E; p.center = center; p.eps = eps; p.conv_w = conv_w; p.conv_state = conv_state;
     p.token_seq = token_seq; p.taps = taps;
+    p.more[0] = air::StreamTerm{more1, more1_parts, gate1}; p.more[1] = air::StreamTerm{more2, more2_parts, gate2};
+    p.again = again;
     auto al = [](const void* q) { return ((uintptr_t)q & 15) == 0; };
     const bool vec = E % 4 == 0 && x_stride % 4 == 0 && h_stride % 4 == 0 && part_stride % 4 == 0 && al(x) && al(h_out) &&
-                     al(y) && al(w) && al(b) && al(out) && al(conv_w) && al(conv_state);
+                     al(y) && al(w) && al(b) && al(out) && al(conv_w) && al(conv_state) && al(more1) && al(more2) && al(again);
     // few rows: one access of a thread per row, all of a row's loads under way at once
     const int items = vec && S <= 4 ? E / 4 : E;
     int threads = items >= 256 ? 256 : (items + 31) / 32 * 32;

@@ -11,7 +11,7 @@ import torch
 
 from ..csrc import ops
 from ..parts import registry
-from ..parts.base import Norm, Runtime
+from ..parts.base import Norm, Runtime, row_terms
 from ..parts.linear import Linear
 from ..parts.spec import ModelSpec, PartSpec
 from ..weights.loader import TensorSpec
@@ -26,14 +26,15 @@ class Model:
         emb = spec.embedding or PartSpec("tokens", {"vocab": spec.vocab_size, "hidden": spec.hidden_size,
                                                     "multiplier": spec.embedding_multiplier})
         self.embedder = registry.EMBEDDINGS.get(emb.kind)(emb, spec.embedding_name)
-        # runs that add the embedding's output to the stream again need a second copy of it
-        self.embedding_copies = 2 if any(run.add_embedding for run in spec.order) else 1
+        # runs that take the embedding's output into the stream again need a second copy of it
+        self.embedding_copies = 2 if any(run.add_embedding or run.mix_embedding for run in spec.order) else 1
 
     # ------------------------------------------------------------------ tensors
     def tensor_specs(self) -> List[TensorSpec]:
         s = self.spec
         specs = list(self.embedder.tensor_specs())
         specs += [TensorSpec(name, (rows, s.hidden_size), wide=True) for name, rows in s.stream_tables]
+        specs += [TensorSpec(name, (s.hidden_size, 2 * s.hidden_size)) for name in s.stream_mixes]
         for b in self.blocks:
             specs += b.tensor_specs()
         specs += self.final_norm.tensor_specs()
@@ -53,6 +54,7 @@ class Model:
         self.embedder.load(tensors, rt)
         self.embedding = self.embedder.table
         self.stream_tables = {name: tensors[name].to(torch.float32).contiguous() for name, _ in self.spec.stream_tables}
+        self.stream_mixes = {name: Linear(tensors[name], rt.status) for name in self.spec.stream_mixes}
         for b in self.blocks:
             b.load(tensors, rt)
         self.final_norm.load(tensors, rt)
@@ -108,11 +110,27 @@ class Model:
                         add(v.weight)
                     else:
                         add(v)
+        for mix in self.stream_mixes.values():
+            add(mix.weight)
         add(self.output.weight)
         add(self.final_norm.weight)
         return total
 
     # ------------------------------------------------------------------ computing
+    def _mixed(self, h, pending, x0, mix):
+        """(stream, pending) of W [x | x0]: one kernel completes x and writes the rows [x | x0] in the compute dtype; the
+        product's partial sums (few rows) are the new stream and what is still to be added to it."""
+        T, E = h.shape
+        terms = row_terms(pending)
+        if terms is None:
+            h, terms = Norm.add_delta(h, pending), []
+        rows = torch.empty((T, 2 * E), dtype=self.rt.dtype, device=h.device)
+        ops.stream_norm(h, 1, None, None, 0.0, rows, term=terms[0][0] if terms else None, more=terms[1:], again=x0)
+        y = mix.f32_sums(rows)
+        if y.dim() == 2:
+            return y, None
+        return y[0], y[1:] if y.shape[0] > 1 else None
+
     def forward(self, ctx, cache) -> torch.Tensor:
         """Runs the batch's tokens through every run of the order list, writing the caches,
         and returns float32 logits [wanted rows, vocab]."""
@@ -122,6 +140,8 @@ class Model:
         pending = None
         for i, run in enumerate(self.spec.order):
             owner = i if run.cache_from is None else run.cache_from
+            if run.mix_embedding is not None:
+                h, pending = self._mixed(h, pending, again[0], self.stream_mixes[run.mix_embedding])
             if run.add_embedding or run.add_row is not None:
                 # what the run adds to the stream ahead of its layer: the stream is completed first
                 h = Norm.add_delta(h, pending)

@@ -231,9 +231,9 @@ class PreNormed:
 
 @dataclass
 class ScaledSum:
-    """What parts that stand side by side add to the stream together: the sum of scale * term over `terms`, a list
+    """What parts that stand side by side add to the stream together: the sum of scale * gate * term over `terms`, a list
     of (float32 [T, hidden], or [parts, T, hidden] partial sums of a split product; float32 [hidden] or None: a scale
-    per column).  A form of a norm's `delta`: the norm
+    per column; optionally float32 [T] or None: a gate per row).  A form of a norm's `delta`: the norm
     that follows completes the stream with it (Norm.add_delta, or a kernel of its own that also normalises)."""
     terms: list
 
@@ -257,6 +257,28 @@ class NormedSum:
     term: torch.Tensor
     weight: torch.Tensor
     eps: float
+
+
+def row_terms(delta) -> Optional[list]:
+    """A delta as a list of (float32 [T, hidden] or [parts, T, hidden], gate per row float32 [T] or None) to be added up, for
+    kernels that take that form; None where it has no such form (scales per column, a norm behind the sub-layer, several
+    streams, 16-bit tensors, more than three terms)."""
+    if delta is None:
+        return []
+    if isinstance(delta, torch.Tensor):
+        terms = [(delta, None)]
+    elif isinstance(delta, GatedSum):
+        terms = [(t, g) for t, g in ((delta.a, None), (delta.b, delta.gate)) if t is not None]
+    elif isinstance(delta, ScaledSum):
+        if any(t[1] is not None for t in delta.terms):
+            return None
+        # (the kernels take a gate on every term but the first)
+        terms = sorted(((t[0], t[2] if len(t) > 2 else None) for t in delta.terms), key=lambda t: t[1] is not None)
+    else:
+        return None
+    if len(terms) > 3 or any(t.dtype != torch.float32 for t, _ in terms) or (terms and terms[0][1] is not None):
+        return None
+    return terms
 
 
 @dataclass
@@ -315,7 +337,12 @@ class Norm(Part):
                 ops.stream_norm(h, S, None, None, 0.0, None, term=delta.term, mix=delta.mix, out_weights=delta.out,
                                 h_out=full)
                 return full
-            if isinstance(delta, ScaledSum):
+            if isinstance(delta, ScaledSum) and (len(delta.terms) > 2 or any(len(t) > 2 for t in delta.terms)):
+                terms = row_terms(delta)
+                if terms is None:
+                    raise ops.KernelError("a sum of more than two terms, or with a gate per row, takes no scales per column")
+                ops.stream_norm(h, 1, None, None, 0.0, None, term=terms[0][0], more=terms[1:], h_out=h)
+            elif isinstance(delta, ScaledSum):
                 ops.scaled_norm(h, delta.terms, None, 0.0, None)
             elif isinstance(delta, GatedSum):
                 ops.post_norm(h, 1.0, delta.a, delta.b, delta.gate, None, 0.0, None)

@@ -196,7 +196,7 @@ class ParallelBlock(Block):
     "mixer_scale" and "feed_forward_scale", what follows the layer's prefix in the names of the two scale vectors
     [hidden]; a scale that is not named is 1.
 
-    The block hands its two outputs on as a ScaledSum: the next block's norm (or the model's last one) completes the
+    The block hands its outputs on as a ScaledSum (a feed-forward with a gated branch makes two terms): the next block's norm (or the model's last one) completes the
     stream with them in 32-bit in the kernel that normalises."""
 
     def __init__(self, spec: BlockSpec):
@@ -236,10 +236,18 @@ class ParallelBlock(Block):
         from .base import ScaledSum
         ctx.residual = None          # the sub-layers' outputs are scaled before they are added: they return them
         x = self.norm.forward(h, pending)
-        terms = [(self.mixer.forward(x, ctx, cache, owns_cache), self.scales.get("mixer"))]
+        terms = self._terms(self.mixer.forward(x, ctx, cache, owns_cache), self.scales.get("mixer"))
         if self.feed_forward is not None:
-            terms.append((self.feed_forward.forward(x, ctx), self.scales.get("feed_forward")))
+            terms += self._terms(self.feed_forward.forward(x, ctx), self.scales.get("feed_forward"))
         return h, ScaledSum(terms)
+
+    @staticmethod
+    def _terms(delta, scale):
+        """What a sub-layer returned as terms of the sum; a branch with a gate per row is a term of its own."""
+        from .base import GatedSum
+        if not isinstance(delta, GatedSum):
+            return [(delta, scale)]
+        return [(delta.a, scale)] * (delta.a is not None) + [(delta.b, scale, delta.gate)] * (delta.b is not None)
 
 
 @register_block("post_norm")

@@ -8,7 +8,7 @@ from ..csrc import ops
 from ..weights.loader import TensorSpec
 from .base import FeedForward, GatedSum
 from .linear import Linear
-from .mlp import SwiGLU
+from .mlp import ClampedGLU, SwiGLU
 from .registry import register_feed_forward
 from .spec import PartSpec
 
@@ -26,12 +26,16 @@ class RoutedExperts(FeedForward):
     Router: z = Wr x in 32-bit; scores s = sigmoid(z) (score "sigmoid") or softmax(z); the `top` largest are chosen
     (of equal scores the lower index); the weights are the chosen scores, divided by their sum (+ norm_eps) where
     renormalize, times route_scale.  With groups = (count, keep) experts g * (experts / count) .. (g + 1) * (experts /
-    count) - 1 make group g, a group's mark is its best score plus its second best, and only experts of the `keep`
+    count) - 1 make group g, a group's mark is its best score plus its second best (group_mark "two", the default) or its best
+    score alone ("best"), and only experts of the `keep`
     groups with the highest marks can be chosen.  With weight_on "input" (the default) the weight multiplies the expert's INPUT (the
     scaled row is rounded to the compute dtype like any input of a product), which is not the same as weighting its
     output, since an expert is not linear; with "output" it multiplies the expert's output, in 32-bit.  expert(u) = Wdown (silu(Wgate u) *
     (Wup u)).  The shared expert (shared_intermediate > 0) has the same form and runs for every token; with shared_gate
     its output is multiplied by g = sigmoid(w_sg . x), one number per token, else g = 1.
+
+    With activation "clamped_glu" an expert, and the shared one, is expert(u) = Wdown (a sigmoid(1.702 a) (b + 1)), a = min(Wgate
+    u, limit), b = clamp(Wup u, -limit, limit); the shared expert has a limit of its own (shared_limit).
 
     With gated False an expert has no gate: expert(u) = Wdown act(Wup u) with act the square of the rectifier
     (activation "relu2").  With choice_bias the experts are chosen by score + bias (a learned number per expert, the
@@ -40,7 +44,7 @@ class RoutedExperts(FeedForward):
     take part in the softmax and in the choice like the others.
 
     params: hidden, experts, top, intermediate, shared_intermediate, shared_gate, score, renormalize, norm_eps,
-    route_scale, groups, weight_on, gated, activation, choice_bias, identity.
+    route_scale, groups, group_mark, weight_on, gated, activation, limit, shared_limit, choice_bias, identity.
     Tensors: <prefix>router [experts + identity, hidden], e<i>.gate, e<i>.up [intermediate, hidden], e<i>.down [hidden,
     intermediate], shared.gate, shared.up, shared.down, shared.sg [1, hidden], correction [experts + identity].
 
@@ -74,9 +78,12 @@ class RoutedExperts(FeedForward):
         self.gated, self.activation = bool(p.get("gated", True)), p.get("activation", "silu")
         self.choice_bias, self.identity = bool(p.get("choice_bias", False)), int(p.get("identity") or 0)
         self.outputs = self.experts + self.identity          # what the router chooses among
-        if (self.gated, self.activation) not in ((True, "silu"), (False, "relu2")):
-            raise ConfigError("unsupported", "routed experts: gated experts with SiLU, or plain ones with the squared "
-                                             "rectifier")
+        if (self.gated, self.activation) not in ((True, "silu"), (True, "clamped_glu"), (False, "relu2")):
+            raise ConfigError("unsupported", "routed experts: gated experts with SiLU or the clamped activation, or plain ones "
+                                             "with the squared rectifier")
+        self.act, self.group_mark = ops.SILU, p.get("group_mark", "two")
+        if self.activation == "clamped_glu":
+            self.act = (1.702, float(p["limit"]), 1.0)      # alpha, limit, shift
         if self.identity < 0 or (self.identity and (self.weight_on != "output" or self.groups > 1)):
             raise ConfigError("unsupported", "routed experts: identity experts take their weight on the output, and "
                                              "no groups")
@@ -85,7 +92,11 @@ class RoutedExperts(FeedForward):
         if self.outputs > 512 or self.top > 32:
             raise ConfigError("unsupported", "routed experts: up to 512 experts and 32 choices per token")
         self.shared = None
-        if self.shared_inter:
+        if self.shared_inter and self.activation == "clamped_glu":
+            self.shared = ClampedGLU(PartSpec("clamped_glu", {"hidden": self.hidden, "intermediate": self.shared_inter,
+                                                              "limit": float(p["shared_limit"]), "alpha": 1.702}),
+                                     prefix + "shared.")
+        elif self.shared_inter:
             self.shared = PlainNamesSwiGLU(PartSpec("swiglu_plain_names", {"hidden": self.hidden,
                                                                            "intermediate": self.shared_inter}),
                                            prefix + "shared.")
@@ -148,7 +159,7 @@ class RoutedExperts(FeedForward):
         gate = torch.empty((T,), dtype=torch.float32, device=dev) if self.shared_gate else None
         ops.moe_route(z, self.outputs, top, expert, weight, gate, has_gate=self.shared_gate, score=self.score,
                       renormalize=self.renormalize, groups=self.groups, keep=self.keep, route_scale=self.route_scale,
-                      norm_eps=self.norm_eps, choice_bias=self.correction)
+                      norm_eps=self.norm_eps, choice_bias=self.correction, mark=self.group_mark)
         on_input = self.weight_on == "input"
         pairs = T * top
         ints = torch.empty(n + 1 + pairs + 2 * (pairs // ops.GROUP_TILE + n) + 1, dtype=torch.int32, device=dev)
@@ -166,7 +177,7 @@ class RoutedExperts(FeedForward):
             ops.grouped_gemm(x, self.gate_up, act, F, E, lda=E, ldo=F, groups=n, a_index=pair_of_slot, a_div=top,
                              a_scale=weight.view(-1) if on_input else None, start=start, tiles=tiles,
                              num_tiles=num_tiles, silu_mul=self.gated, gate_block=self.block if self.gated else 0,
-                             relu2=not self.gated)
+                             relu2=not self.gated, act=self.act)
             ops.grouped_gemm(act, self.down, y, E, F, lda=F, ldo=E, groups=n, o_index=pair_of_slot, o_div=top,
                              o_part_stride=T * E, start=start, tiles=tiles, num_tiles=num_tiles,
                              o_scale=None if on_input else weight.view(-1))
@@ -186,7 +197,9 @@ class RoutedExperts(FeedForward):
         ends = start[1:].clone()
         act = torch.empty((pairs, self.inter), dtype=x.dtype, device=x.device)
         hidden = torch._grouped_mm(rows, self.gate_up.transpose(1, 2), offs=ends)
-        if self.gated:
+        if self.activation == "clamped_glu":
+            ops.glu(hidden, act, block=self.block, alpha=self.act[0], limit=self.act[1], shift=self.act[2])
+        elif self.gated:
             ops.silu_mul(hidden, act, block=self.block)
         else:
             ops.relu2(hidden, act)

@@ -22,7 +22,8 @@ class PortionAttention:
     16-byte pieces, the one with a block per head.
 
     The mixer offers: rt, heads, kv_heads (1 for a latent), scale, window, chunk, sinks (float32 [heads] or None) and
-    optionally softcap (> 0: a score s becomes softcap * tanh(s / softcap))."""
+    optionally softcap (> 0: a score s becomes softcap * tanh(s / softcap)) and bias_table (float32 [heads, n]: a score gets
+    the head's number for its key's distance, the last one from n - 1 on)."""
 
     PORTION = 32
     BLOCK = 1024
@@ -65,6 +66,7 @@ class PortionAttention:
         key splits where there is one, else by a kernel of its own."""
         sinks = getattr(self, "sinks", None)
         softcap = float(getattr(self, "softcap", 0.0) or 0.0)
+        bias = getattr(self, "bias_table", None)
         plan = ctx.plans.get((self.PLAN,)) if not self.rt.is_fp32 else None
 
         def through_the_pages(token_seq):
@@ -72,17 +74,17 @@ class PortionAttention:
                     and out.dtype == torch.bfloat16 and q.shape[2] == out.shape[2]
                     and q.shape[2] in ops.DECODE_HEAD_DIMS and ops.tile_pages(pages.shape[3])):
                 ops.decode_attention(q, pages, bt, token_seq, ctx.positions, out, self.window, self.scale,
-                                     softcap=softcap, sink=sinks, gate=gate, status=ctx.status, turn=turn)
+                                     softcap=softcap, sink=sinks, gate=gate, status=ctx.status, turn=turn, bias=bias)
                 return
             # (the kernel that reads a key once for all heads of its group wants rows of whole 16-byte pieces)
             if ops.grouped_attention_ok(cache.dtype, q.shape[2], out.shape[2]):
                 ops.grouped_attention(q, cache, bt, token_seq, ctx.positions, out, self.window, self.scale,
                                       kv_heads=kv_heads, page_tokens=page_tokens, chunk=self.chunk, sink=sinks,
-                                      latent=latent, softcap=softcap, gate=gate, turn=turn)
+                                      latent=latent, softcap=softcap, gate=gate, turn=turn, bias=bias)
                 return
             ops.paged_attention_ref(q, cache, bt, token_seq, ctx.positions, out, self.window, self.scale,
                                     kv_heads=kv_heads, page_tokens=page_tokens, chunk=self.chunk, sink=sinks,
-                                    latent=latent, softcap=softcap)
+                                    latent=latent, softcap=softcap, bias=bias)
             if turn is not None:
                 ops.turn_heads(out, *turn, ctx.positions, token_seq, back=True)
             if gate is not None:
@@ -118,7 +120,7 @@ class PortionAttention:
                     torch.mm(rows[g], keys[g].t(), out_dtype=torch.float32, out=scores[g])
                 weights = torch.empty(scores.shape, dtype=torch.bfloat16, device=dev)
                 ops.masked_softmax(scores, weights, J, lo, L, p0, self.scale, window=self.window, chunk=self.chunk,
-                                   sink=sinks, softcap=softcap)
+                                   sink=sinks, softcap=softcap, bias=bias)
                 summed = torch.empty((G, nb * J, dv), dtype=torch.bfloat16, device=dev)
                 for g in range(G):
                     torch.mm(weights[g], keys[g, :, :dv] if latent else values[g], out=summed[g])

@@ -5,7 +5,7 @@ import torch
 
 from ..csrc import ops
 from ..weights.loader import TensorSpec
-from .base import GatedSum, Norm, NormedSum, PreNormed, ScaledSum, StreamSum
+from .base import GatedSum, Norm, NormedSum, PreNormed, ScaledSum, StreamSum, row_terms
 from .registry import register_norm
 
 
@@ -60,6 +60,13 @@ class RMSNorm(Norm):
             # and normalises it
             return ops.normed_add_norm(h, delta.term, delta.weight, delta.eps, self.weight_f32(), self.eps, out,
                                        rows=rows)
+        if isinstance(delta, ScaledSum) and (len(delta.terms) > 2 or any(len(t) > 2 for t in delta.terms)):
+            # more sub-layers' outputs than two, or a gate per row among them
+            terms = row_terms(delta)
+            if terms is None:
+                raise ops.KernelError("rms: a sum of more than two terms, or with a gate per row, takes no scales per column")
+            return ops.stream_norm(h, 1, self.weight_f32(), None, self.eps, out, term=terms[0][0], more=terms[1:],
+                                   h_out=h if rows is None else None, rows=rows, center=False)
         if isinstance(delta, ScaledSum):
             # the outputs of sub-layers that stand side by side, each with its scale per column: one kernel
             # completes the stream with them and normalises
@@ -156,13 +163,14 @@ class LayerNorm(Norm):
             return self.forward_streams(h, delta, None, rows=rows)[1]
         n = h.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, h.shape[1]), dtype=self.rt.dtype, device=h.device)
-        if isinstance(delta, (ScaledSum, GatedSum, NormedSum)) or (delta is not None and delta.dtype != torch.float32):
+        terms = row_terms(delta)
+        if terms is None:
             if rows is not None:
                 h = h.clone()
             self.add_delta(h, delta)
-            delta = None
-        return ops.stream_norm(h, 1, self.weight, self.bias, self.eps, out, term=delta,
-                               h_out=h if delta is not None and rows is None else None, rows=rows)
+            terms = []
+        return ops.stream_norm(h, 1, self.weight, self.bias, self.eps, out, term=terms[0][0] if terms else None,
+                               more=terms[1:], h_out=h if terms and rows is None else None, rows=rows)
 
     def forward_streams(self, h, delta, read, rows=None, dtype=None, conv=None):
         """(the streams, the normalised rows): delta is a StreamSum (or None), read float32 [S] the weights with which the

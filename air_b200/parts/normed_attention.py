@@ -1,6 +1,8 @@
 """Grouped-query attention with normalised queries and keys, chunks or a window, and a sink in the softmax."""
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..config.model_config import ConfigError
@@ -11,6 +13,16 @@ from .base import Mixer, PagedKV, SlotState
 from .gathered_attention import PortionAttention
 from .linear import Linear
 from .registry import register_mixer, POSITION_ENCODINGS
+
+
+def distance_rows(rows: int, span: float):
+    """The row of a distance bias for the distances 0, 1, .. up to the first one that takes the last row (all larger ones
+    take it too): see NormedAttention.  The logarithms are 64-bit."""
+    low, out, n = rows // 2, [], 0
+    while not out or out[-1] < rows - 1:
+        out.append(n if n < low else min(rows - 1, low + math.floor(math.log(n / low) / math.log(span / low) * (rows - low))))
+        n += 1
+    return out
 
 
 @register_mixer("normed_attention")
@@ -40,17 +52,21 @@ class NormedAttention(PortionAttention, Mixer):
       * value_position rotates the values by their position before they are kept (an encoding of kind rope_live over the
         first part of a value) and turns every head's sum over values back by the query's position, ahead of the gate:
         what a head returns then depends on how far away the values stand;
+      * distance_bias = {"rows": B, "span": D} adds to head h's score a learned number that depends on how many positions n
+        the key stands back, B rows for all distances: row n for n < L = B // 2, behind that row min(B - 1, L +
+        floor(ln(n / L) / ln(D / L) * (B - L))); the scale does not multiply it;
       * a layer that borrows reads the keys and values that another layer's run keeps (RunStep.cache_from): it has no
         projections or norms of keys and values; `keep` is the widest window among the layers that read one layer's
         pages, which live as long.
 
     params: hidden, heads, kv_heads, head_dim, v_dim, scale, window, chunk (at most one of the two), qk_norm (False,
-    True or "head", "whole"), sink (False, True or "learned", "zero"), eps, position, qkv_bias, conv, softcap, out_gate,
-    head_temp, value_position, borrows, keep.
+    True or "head", "whole", "bare": per head, without a weight), sink (False, True or "learned", "zero"), eps, position, qkv_bias, conv, softcap, out_gate,
+    head_temp, value_position, distance_bias, borrows, keep.
     Tensors: <prefix>q [heads*head_dim, hidden], k [kv_heads*head_dim, hidden], v [kv_heads*v_dim, hidden],
     q.norm, k.norm [head_dim] where qk_norm ([heads*head_dim] and [kv_heads*head_dim] where "whole"), sink [heads] where
     the sink is learned, o [hidden, heads*v_dim]; q.b, k.b, v.b where qkv_bias; q.conv, k.conv, v.conv [channels, conv]
-    where conv; g [heads*v_dim, hidden] where out_gate; temp [heads] where head_temp.
+    where conv; g [heads*v_dim, hidden] where out_gate; temp [heads] where head_temp; rel [B, heads] where
+    distance_bias.
 
     q, k and v are one product; one kernel then normalises, rotates and writes keys and values to the pages; pages of a
     chunk that no later query can see go back to the pool.  Prompt portions attend through matrix products over their
@@ -72,15 +88,20 @@ class NormedAttention(PortionAttention, Mixer):
         self.window, self.chunk = p.get("window"), p.get("chunk")
         norm, sink = p.get("qk_norm", False), p.get("sink", False)
         self.qk_norm = bool(norm)
-        self.norm_whole = norm == "whole"
+        self.norm_whole, self.norm_bare = norm == "whole", norm == "bare"
         self.sink = bool(sink)
         self.sink_learned = self.sink and sink != "zero"
-        if norm not in (False, True, None, "head", "whole") or sink not in (False, True, None, "learned", "zero"):
+        if norm not in (False, True, None, "head", "whole", "bare") or sink not in (False, True, None, "learned", "zero"):
             raise ConfigError("data_error", f"normed_attention: qk_norm {norm!r}, sink {sink!r}")
         self.head_temp, self.borrows = bool(p.get("head_temp", False)), bool(p.get("borrows", False))
         self.keep = p.get("keep", self.window) if self.window else None
         self.qkv_bias, self.out_gate = bool(p.get("qkv_bias", False)), bool(p.get("out_gate", False))
         self.taps, self.softcap = int(p.get("conv") or 0), float(p.get("softcap") or 0.0)
+        self.distance = p.get("distance_bias")
+        if self.distance is not None:
+            rows, span = int(self.distance["rows"]), float(self.distance["span"])
+            if rows < 2 or span <= rows // 2:
+                raise ConfigError("data_error", f"normed_attention: a distance bias of {rows} rows over {span} positions")
         if self.taps > 16:
             raise ConfigError("unsupported", f"normed_attention: a convolution of {self.taps} taps (up to 16)")
         if self.window and self.chunk:
@@ -116,13 +137,14 @@ class NormedAttention(PortionAttention, Mixer):
         if n:
             ops.decode_attention(q[:n], kv, bt, ctx.token_seq[:n], ctx.positions[:n], out[:n], self.window, self.scale,
                                  softcap=self.softcap, sink=self.sinks, gate=None if gate is None else gate[:n],
-                                 status=ctx.status, turn=turn)
+                                 status=ctx.status, turn=turn, bias=self.bias_table)
         if plan.tiles.shape[0]:
             if plan.slots and getattr(plan, "scratch", None) is None:
                 plan.scratch = ops.prefill_attention_scratch(plan.slots, d, q.device)
             ops.prefill_attention_tc(q, kv, bt, plan.tiles, out, self.window, self.scale, status=ctx.status,
                                      segments=plan.segments, items=plan.items, slots=plan.slots,
-                                     scratch=getattr(plan, "scratch", None), softcap=self.softcap, sink=self.sinks)
+                                     scratch=getattr(plan, "scratch", None), softcap=self.softcap, sink=self.sinks,
+                                     bias=self.bias_table)
             if turn is not None and T > n:
                 ops.turn_heads(out[n:], *turn, ctx.positions[n:], ctx.token_seq[n:], back=True)
             if gate is not None and T > n:
@@ -148,11 +170,13 @@ class NormedAttention(PortionAttention, Mixer):
             specs += [TensorSpec(p + n + ".b", (rows[n],), wide=True) for n in "qkv"]
         if self.taps:
             specs += [TensorSpec(p + n + ".conv", (rows[n], self.taps), wide=True, std=0.3) for n in "qkv"]
-        if self.qk_norm:
+        if self.qk_norm and not self.norm_bare:
             specs += [TensorSpec(p + n + ".norm", (rows[n] if self.norm_whole else self.head_dim,),
                                  init="one_plus_normal", wide=True) for n in ("q" if self.borrows else "qk")]
         if self.head_temp:
             specs.append(TensorSpec(p + "temp", (self.heads,), init="one_plus_normal", wide=True))
+        if self.distance is not None:
+            specs.append(TensorSpec(p + "rel", (int(self.distance["rows"]), self.heads), std=0.5, wide=True))
         if self.sink_learned:
             specs.append(TensorSpec(p + "sink", (self.heads,), std=1.0, wide=True))
         if self.out_gate:
@@ -169,7 +193,10 @@ class NormedAttention(PortionAttention, Mixer):
         self.proj = Linear(torch.cat(ws, dim=0).contiguous(), rt.status)
         self.o = Linear(tensors[p + "o"], rt.status)
         self.q_weight = self.k_weight = self.sinks = None
-        if self.qk_norm:
+        if self.norm_bare:
+            self.q_weight = torch.ones(self.head_dim, dtype=torch.float32, device=rt.device)
+            self.k_weight = None if self.borrows else self.q_weight
+        elif self.qk_norm:
             self.q_weight = tensors[p + "q.norm"].to(torch.float32).contiguous()
             self.k_weight = None if self.borrows else tensors[p + "k.norm"].to(torch.float32).contiguous()
         self.temp = tensors[p + "temp"].to(torch.float32).contiguous() if self.head_temp else None
@@ -177,7 +204,12 @@ class NormedAttention(PortionAttention, Mixer):
             self.sinks = tensors[p + "sink"].to(torch.float32).contiguous()
         elif self.sink:
             self.sinks = torch.zeros(self.heads, dtype=torch.float32, device=rt.device)
-        self.bias = self.conv_weight = None
+        self.bias = self.conv_weight = self.bias_table = None
+        if self.distance is not None:
+            # the table's rows spread over the distances, head by head, as far as the last row's first distance
+            rows = distance_rows(int(self.distance["rows"]), float(self.distance["span"]))
+            rel = tensors[p + "rel"].to(torch.float32)
+            self.bias_table = rel[torch.tensor(rows, device=rel.device)].t().contiguous()
         if self.qkv_bias:
             self.bias = torch.cat([tensors[p + n + ".b"].to(torch.float32) for n in "qkv"]).contiguous()
         if self.taps:

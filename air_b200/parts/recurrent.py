@@ -33,12 +33,18 @@ class _StateMixer(Mixer):
         lo, hi = self.columns[name]
         return proj[:, lo:hi]
 
-    def _finish(self, o, proj, ctx):
-        """norm over each head's read-out, times the weight and silu(gate), then the output projection"""
+    def _finish(self, o, gate, ctx, sigmoid=False):
+        """norm over each head's read-out, times the weight and silu(gate) (or sigmoid(gate)), then the output projection"""
         T = o.shape[0]
         y = torch.empty((T, self.heads * self.v_dim), dtype=self.rt.dtype, device=o.device)
-        ops.gated_rmsnorm(o, self._band(proj, "g"), self.norm_weight, self.eps, y, ctx.token_seq)
+        ops.gated_rmsnorm(o, gate, self.norm_weight, self.eps, y, ctx.token_seq, sigmoid=sigmoid)
         return self.o.f32_sums(y)
+
+    def _convolved(self, proj, tail, ctx):
+        """The first `channels` columns of proj behind the short convolution and SiLU; tail: the state of its last inputs."""
+        y = torch.empty((proj.shape[0], self.channels), dtype=torch.float32, device=proj.device)
+        state = tail.state if self.taps > 1 else tail.state[:, :, :0].contiguous()
+        return ops.short_conv_silu(proj[:, :self.channels], self.conv_weight, state, y, ctx.q_start, ctx.slots, ctx.max_q_len)
 
 
 @register_mixer("gated_delta")
@@ -100,18 +106,122 @@ class GatedDeltaRule(_StateMixer):
         state, tail = cache
         T, H, G, d, dv = x.shape[0], self.heads, self.kv_heads, self.head_dim, self.v_dim
         proj = self.proj.f32(x)
-        y = torch.empty((T, self.channels), dtype=torch.float32, device=x.device)
-        if self.taps > 1:
-            ops.short_conv_silu(proj[:, :self.channels], self.conv_weight, tail.state, y, ctx.q_start, ctx.slots,
-                                ctx.max_q_len)
-        else:
-            ops.short_conv_silu(proj[:, :self.channels], self.conv_weight, tail.state[:, :, :0].contiguous(), y,
-                                ctx.q_start, ctx.slots, ctx.max_q_len)
+        y = self._convolved(proj, tail, ctx)
         o = torch.empty((T, H, dv), dtype=torch.float32, device=x.device)
         ops.linear_scan(ops.SCAN_DELTA, y[:, :G * d], y[:, G * d:2 * G * d], y[:, 2 * G * d:],
                         self._band(proj, "a"), state.state, o, ctx.q_start, ctx.slots, ctx.token_seq, q_scale=d ** -0.5,
                         beta=self._band(proj, "b"), a_log=self.a_log, dt_bias=self.dt_bias, unit=True, unit_eps=1e-6)
-        return self._finish(o, proj, ctx)
+        return self._finish(o, self._band(proj, "g"), ctx)
+
+
+@register_mixer("channel_delta")
+class ChannelDeltaRule(_StateMixer):
+    """The delta rule with a decay per key channel.  q, k, v, their convolutions, unit lengths and b as in GatedDeltaRule; the
+    decay of channel c of head h is g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 x) + dt_bias)), a product through a narrow
+    middle laid out heads x head_dim, and scales row c of the head's state:
+
+        S = diag(g) S;   u = b (v - S^T k);   S = S + k u^T;   o = S^T q
+
+    then o / sqrt(mean(o^2) + eps) * norm, times sigmoid(W_g2 (W_g1 x)) (laid out heads x v_dim), and the output
+    projection.  S and the convolutions' last conv - 1 inputs are the request's state, 32-bit, zero at its start.
+
+    The two products out of a narrow middle take its numbers as they left the first product: a float32 engine in 32-bit,
+    a bfloat16 engine as two bfloat16 halves side by side, against the matrix twice (ops.split_bands), so that the
+    decays are 32-bit but for the weights' own precision.
+
+    params: hidden, heads, kv_heads, head_dim, v_dim, conv, decay_rank, gate_rank (the narrow middles), eps.  Tensors:
+    <prefix>q, k, v, each with <name>.conv [channels, conv]; b [heads, hidden]; A_log [heads]; dt_bias [heads*head_dim];
+    a1 [decay_rank, hidden]; a2 [heads*head_dim, decay_rank]; g1 [gate_rank, hidden]; g2 [heads*v_dim, gate_rank]; norm
+    [v_dim]; o [hidden, heads*v_dim]."""
+
+    def __init__(self, spec, prefix=""):
+        super().__init__(spec, prefix)
+        p = spec.params
+        self.hidden, self.heads, self.kv_heads = p["hidden"], p["heads"], p["kv_heads"]
+        self.head_dim, self.v_dim, self.taps, self.eps = p["head_dim"], p["v_dim"], int(p["conv"]), float(p["eps"])
+        self.decay_rank, self.gate_rank = int(p["decay_rank"]), int(p["gate_rank"])
+        if self.heads % self.kv_heads:
+            raise ConfigError("data_error", "channel_delta: heads must be a multiple of kv_heads")
+        if not (1 <= self.taps <= 16):
+            raise ConfigError("unsupported", f"channel_delta: a convolution of {self.taps} taps (the kernel takes 1 to 16)")
+        if self.head_dim > 1024:
+            raise ConfigError("unsupported", f"channel_delta: {self.head_dim} key channels per head (up to 1,024)")
+        self.channels = 2 * self.kv_heads * self.head_dim + self.heads * self.v_dim
+
+    def cache_needs(self):
+        return (SlotState((self.heads, self.head_dim, self.v_dim)),
+                SlotState((self.channels, max(self.taps - 1, 1))))
+
+    def tensor_specs(self):
+        p, e, H, G, d, dv = self.prefix, self.hidden, self.heads, self.kv_heads, self.head_dim, self.v_dim
+        rows = {"q": G * d, "k": G * d, "v": H * dv}
+        specs = []
+        for n in "qkv":
+            specs += [TensorSpec(p + n, (rows[n], e)), TensorSpec(p + n + ".conv", (rows[n], self.taps), wide=True, std=0.3)]
+        return specs + [
+            TensorSpec(p + "b", (H, e)), TensorSpec(p + "A_log", (H,), wide=True), TensorSpec(p + "dt_bias", (H * d,), wide=True),
+            TensorSpec(p + "a1", (self.decay_rank, e)), TensorSpec(p + "a2", (H * d, self.decay_rank), std=0.3),
+            TensorSpec(p + "g1", (self.gate_rank, e)), TensorSpec(p + "g2", (H * dv, self.gate_rank), std=0.3),
+            TensorSpec(p + "norm", (dv,), init="one_plus_normal", wide=True), TensorSpec(p + "o", (e, H * dv))]
+
+    def load(self, tensors, rt):
+        super().load(tensors, rt)
+        p, w = self.prefix, tensors[self.prefix + "q"]
+        # rows of zeros: the narrow middles are filled up to multiples of 4 numbers (the second products' inner size, two
+        # halves each, is then one of 8), the matrix up to a multiple of 8 rows, which the tensor-core kernels want
+        tensors = dict(tensors)
+
+        def zeros(name, rows):
+            if rows:
+                tensors[p + name] = torch.zeros((rows, self.hidden), dtype=w.dtype, device=w.device)
+            return [name] * (rows > 0)
+
+        self.middle = tuple(r + (-r % 4) for r in (self.decay_rank, self.gate_rank))
+        bands = ["q", "k", "v", "b"]
+        bands += zeros("pad.b", -sum(tensors[p + n].shape[0] for n in bands) % 4)
+        bands += ["a1"] + zeros("pad.a", self.middle[0] - self.decay_rank)
+        bands += ["g1"] + zeros("pad.g", self.middle[1] - self.gate_rank)
+        bands += zeros("pad", -sum(tensors[p + n].shape[0] for n in bands) % 8)
+        self._project(tensors, bands, rt)
+        f32 = lambda n: tensors[p + n].to(torch.float32).contiguous()
+        self.conv_weight = torch.cat([f32(n + ".conv") for n in "qkv"], dim=0).contiguous()
+        self.a_log, self.dt_bias, self.norm_weight = f32("A_log"), f32("dt_bias"), f32("norm")
+        self.a2, self.g2 = (self._out_of_the_middle(tensors[p + n], r, rt) for n, r in zip(("a2", "g2"), self.middle))
+        self.o = Linear(tensors[p + "o"], rt.status)
+
+    @staticmethod
+    def _out_of_the_middle(m, width, rt):
+        """The second product as a Linear: its inner size filled up with zeros, and in a bfloat16 engine the matrix twice; its
+        rows filled up to a multiple of 4."""
+        rows, rank = m.shape
+        twice = 1 if m.dtype == torch.float32 else 2
+        full = torch.zeros((rows + (-rows % 4), twice * width), dtype=m.dtype, device=m.device)
+        for i in range(twice):
+            full[:rows, i * width:i * width + rank] = m
+        return Linear(full, rt.status)
+
+    def _narrow(self, proj):
+        """(decay logits [T, heads*head_dim], gate logits [T, heads*v_dim]), float32."""
+        at, (ra, rg) = self.columns["a1"][0], self.middle
+        if self.a2.weight.dtype == torch.float32:
+            za, zg = (lin(proj[:, lo:lo + r].contiguous(), torch.float32)
+                      for lin, lo, r in ((self.a2, at, ra), (self.g2, at + ra, rg)))
+        else:
+            a, g = ops.split_bands(proj[:, at:at + ra + rg], ra, rg)
+            za, zg = self.a2.f32(a), self.g2.f32(g)
+        return za[:, :self.heads * self.head_dim], zg[:, :self.heads * self.v_dim]
+
+    def forward(self, x, ctx, cache, owns_cache=True):
+        state, tail = cache
+        T, H, G, d, dv = x.shape[0], self.heads, self.kv_heads, self.head_dim, self.v_dim
+        proj = self.proj.f32(x)
+        y = self._convolved(proj, tail, ctx)
+        decay, gate = self._narrow(proj)
+        o = torch.empty((T, H, dv), dtype=torch.float32, device=x.device)
+        ops.linear_scan(ops.SCAN_CHANNEL_DELTA, y[:, :G * d], y[:, G * d:2 * G * d], y[:, 2 * G * d:], decay, state.state, o,
+                        ctx.q_start, ctx.slots, ctx.token_seq, q_scale=d ** -0.5, beta=self._band(proj, "b"),
+                        a_log=self.a_log, dt_bias=self.dt_bias, unit=True, unit_eps=1e-6)
+        return self._finish(o, gate, ctx, sigmoid=True)
 
 
 @register_mixer("gla")
@@ -166,7 +276,7 @@ class GatedLinearAttention(_StateMixer):
         o = torch.empty((T, H, dv), dtype=torch.float32, device=x.device)
         ops.linear_scan(ops.SCAN_GLA, self._band(proj, "q"), self._band(proj, "k"), self._band(proj, "v"), z,
                         state.state, o, ctx.q_start, ctx.slots, ctx.token_seq, q_scale=d ** -0.5, tau=self.tau)
-        return self._finish(o, proj, ctx)
+        return self._finish(o, self._band(proj, "g"), ctx)
 
 
 @register_mixer("hgrn2")
@@ -286,7 +396,7 @@ class Retention(_StateMixer):
         ops.linear_scan(ops.SCAN_RETENTION, self._band(proj, "q"), self._band(proj, "k"), self._band(proj, "v"),
                         self.decays, state.state, o, ctx.q_start, ctx.slots, ctx.token_seq, positions=ctx.positions,
                         freq=self.freq, k_scale=d ** -0.5)
-        return self._finish(o, proj, ctx)
+        return self._finish(o, self._band(proj, "g"), ctx)
 
 
 @register_mixer("mlstm")
@@ -387,12 +497,4 @@ class MLSTM(_StateMixer):
             ops.mlstm_step(*args, ctx.q_start, plan.short_slots if portions else ctx.slots, *numbers)
         if portions:
             ops.mlstm_portions(*args, plan.portions, plan.chunks, *numbers)
-        return self.o.f32_sums(y)
-        proj = self.proj.f32(x)
-        if plan is None or not plan.long:
-            ops.mlstm_step(proj, columns, *weights, ctx.q_start, ctx.slots, *numbers)
-        else:
-            if plan.short:
-                ops.mlstm_step(proj, columns, *weights, ctx.q_start, plan.short_slots, *numbers)
-            ops.mlstm_portions(proj, columns, *weights, plan.portions, plan.chunks, *numbers)
         return self.o.f32_sums(y)

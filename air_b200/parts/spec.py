@@ -58,14 +58,16 @@ class RunStep:
     the index (in the order list) of the earlier run whose cache this run reads.
 
     What the stream receives right before the run, after everything that earlier runs left pending has been
-    added: add_embedding, the embedding's output of this step once more (x += x0); add_row = (name, r), row r of
-    the model's table `name` (ModelSpec.stream_tables), the same vector for every token.  A stretch of layers that
+    added: mix_embedding, the name of a matrix W [hidden, 2 hidden] (ModelSpec.stream_mixes) that replaces the stream by
+    W [x | x0], x0 being the embedding's output of this step; add_embedding, that output once more (x += x0); add_row =
+    (name, r), row r of the model's table `name` (ModelSpec.stream_tables), the same vector for every token.  A stretch of layers that
     runs several times over with the same weights is written as its runs, one after the other, each with a cache
     of its own, and the first run of each pass carries what the pass adds."""
     layer: int
     cache_from: Optional[int] = None
     add_embedding: bool = False
     add_row: Optional[Tuple[str, int]] = None
+    mix_embedding: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -91,6 +93,8 @@ class ModelSpec:
     embedding: Optional[PartSpec] = None
     # (name, rows): tables [rows, hidden] whose rows runs add to the stream (RunStep.add_row)
     stream_tables: Tuple[Tuple[str, int], ...] = ()
+    # names of the matrices [hidden, 2 hidden] through which runs take the stream (RunStep.mix_embedding)
+    stream_mixes: Tuple[str, ...] = ()
 
     def validate(self) -> None:
         for i, run in enumerate(self.order):
@@ -101,6 +105,8 @@ class ModelSpec:
                     raise ValueError(f"order[{i}] reads the cache of run {run.cache_from}, which is not earlier")
                 if self.order[run.cache_from].cache_from is not None:
                     raise ValueError(f"order[{i}] reads the cache of run {run.cache_from}, which has none of its own")
+            if run.mix_embedding is not None and run.mix_embedding not in self.stream_mixes:
+                raise ValueError(f"order[{i}] takes the stream through '{run.mix_embedding}', which the model does not have")
             if run.add_row is not None:
                 rows = dict(self.stream_tables).get(run.add_row[0])
                 if rows is None or not (0 <= run.add_row[1] < rows):

@@ -799,7 +799,7 @@ def tomodra_kernels(width, heads, kv_heads, ff, T, batch, context):
         cw = torch.ones(R, device=dev)
         rows_ = torch.zeros(S * per_request, P, R + rot, device=dev, dtype=bf).normal_(0, 0.5)
         q_plain, q_full = torch.empty(N, H, d, device=dev, dtype=bf), torch.empty(N, H, R + rot, device=dev)
-        report("latent_prepare (norm of the latent, rotation, page write)", lambda: ops.latent_prepare(proj, cw, 1e-5, freq, positions, seq, bt, q_plain, q_full, rows_, True),
+        report("latent_prepare (norm of the latent, rotation, page write)", lambda: ops.latent_prepare(proj[:, :H * (d + rot)], proj[:, H * (d + rot):], cw, 1e-5, freq, positions, seq, bt, q_plain, q_full, rows_, True),
                N * (proj.shape[1] * 4 + H * d * 2 + H * rot * 4 + (R + rot) * 2))
         Wq = (H + 2 * G) * d
         qkv = torch.randn(N, Wq, device=dev)
@@ -969,14 +969,15 @@ def pefivik_kernels(width, heads, kv_heads, ff, T, batch, context):
         q_plain, q_full = torch.empty(N, H, d, device=dev, dtype=bf), torch.empty(N, H, R, device=dev)
         gate = torch.empty(N, H, device=dev)
         report("latent_prepare (norm of the latent, gates, page write; no rotation)",
-               lambda: ops.latent_prepare(proj, cw, 1e-5, None, positions, seq, bt, q_plain, q_full, rows_, True, gate_out=gate, gate_column=H * d + R),
+               lambda: ops.latent_prepare(proj[:, :H * d], proj[:, H * d:H * d + R], cw, 1e-5, None, positions, seq, bt, q_plain, q_full, rows_, True,
+                                          gate=proj[:, H * d + R:H * d + R + H], gate_out=gate),
                N * (cols * 4 + H * d * 2 + R * 2 + H * 4))
         freq = torch.rand(32, device=dev, dtype=torch.float64)
         proj_t = torch.randn(N, H * (d + 64) + R + 64, device=dev)
         rows_t = torch.zeros(S * per_request, P, R + 64, device=dev, dtype=bf).normal_(0, 0.5)
         q_full_t = torch.empty(N, H, R + 64, device=dev)
         report("  Tomodra: latent_prepare (norm, rotation of 64, page write)",
-               lambda: ops.latent_prepare(proj_t, cw, 1e-5, freq, positions, seq, bt, q_plain, q_full_t, rows_t, True),
+               lambda: ops.latent_prepare(proj_t[:, :H * (d + 64)], proj_t[:, H * (d + 64):], cw, 1e-5, freq, positions, seq, bt, q_plain, q_full_t, rows_t, True),
                N * (proj_t.shape[1] * 4 + H * d * 2 + H * 64 * 4 + (R + 64) * 2))
         out16 = torch.empty(N, H, d, device=dev, dtype=bf)
         sums16, uv = torch.randn(N, H, R, device=dev).to(bf), torch.randn(H, d, R, device=dev, dtype=bf) * 0.05

@@ -229,7 +229,9 @@ def test_latent_attention_through_its_kernels(H, d, rot, R, dv, window, dtype):
         pos, seq = i32(range(at, at + cut)), i32([2] * cut)
         q_plain = torch.empty((cut, H, d), dtype=dtype, device=DEV)
         q_full = torch.empty((cut, H, R + rot), device=DEV)
-        ops.latent_prepare(dev(proj[at:at + cut]), dev(cw), eps, freq, pos, seq, table, q_plain, q_full, rows, True)
+        p = dev(proj[at:at + cut])
+        ops.latent_prepare(p[:, :H * (d + rot)], p[:, H * (d + rot):], dev(cw), eps, freq, pos, seq, table, q_plain, q_full, rows,
+                           True)
         ops.grouped_gemm(q_plain, uk_t, q_full, R, d, lda=H * d, ldo=H * (R + rot), groups=H, a_group_stride=d,
                          o_group_stride=R + rot, a_local=True, o_local=True, rows_per_group=cut)
         summed = torch.empty((cut, H, R), dtype=dtype, device=DEV)
