@@ -113,7 +113,9 @@ AIR_API int air_trace_set_attention_prepare(unsigned long long* buffer) { return
 //   rotates the first v_rot elements of every head of v as well, in the same pairing, before it is written (no magnitude).
 //   Without write_kv proj holds q alone and nothing is written to the pages (a layer that reads another layer's keys).
 //
-// One block per token, one warp per head of q or k; a lane holds up to QKN_PAIRS pairs of its head.
+// One block per token, one warp per head of q or k; a lane holds up to QKN_PAIRS pairs of its head.  Without any rotation
+// and with a norm per head or none (qk_normed_rows_kernel) nothing pairs up: a lane holds four neighbours, as many lanes as a
+// head needs (a power of two) take it, and the heads of a token are spread over the blocks of a row of the grid.
 //
 // turn_heads_kernel  rotates the first `rot` elements of every head of x [T, H, n] by sign * position * freq[j], in place:
 //                    values that were rotated by their own positions and summed over positions are turned back by the
@@ -254,6 +256,82 @@ qk_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __
     }
 }
 
+template <typename TO>
+__global__ void __launch_bounds__(256)
+qk_normed_rows_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ q_w, const float* __restrict__ k_w,
+                      float eps, const int* __restrict__ positions, const int* __restrict__ token_seq,
+                      const int* __restrict__ block_table, int max_blocks, TO* __restrict__ q_out, TO* __restrict__ cache,
+                      int H, int G, int dk, int dv, int P, int* status, const float* __restrict__ bias,
+                      const float* __restrict__ q_scale, int write_kv, int lanes) {
+    pdl_enter(TR_QK_NORMED_PREPARE);
+    const int t = blockIdx.x;
+    const int slot = token_seq[t];
+    if (slot < 0) return;
+    const int pos = positions[t];
+    const float* in = proj + (size_t)t * ld;
+    TO* kdst = nullptr;
+    TO* vdst = nullptr;
+    if (write_kv) {
+        const int page = block_table[(size_t)slot * max_blocks + pos / P];
+        if (page < 0) {
+            if (threadIdx.x == 0 && status) atomicExch(status, 2);
+        } else {
+            TO* base = cache + (size_t)page * G * P * (dk + dv);
+            kdst = base + (size_t)(pos % P) * dk;
+            vdst = base + (size_t)G * P * dk + (size_t)(pos % P) * dv;
+        }
+    }
+    const int heads = write_kv ? H + G : H;
+    const int head = blockIdx.y * (256 / lanes) + threadIdx.x / lanes, l = threadIdx.x % lanes;
+    const bool live = head < heads;
+    constexpr int M = QKN_PAIRS / 2;      // pieces of four per lane
+    float x[M][4], ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < M; ++c) {
+        const int i = (l + c * lanes) * 4;
+        if (live && i < dk) {
+            load4(in + (size_t)head * dk + i, x[c]);
+            if (bias) {
+                float b[4];
+                load4(bias + (size_t)head * dk + i, b);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) x[c][j] += b[j];
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) ss = fmaf(x[c][j], x[c][j], ss);
+        }
+    }
+    for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (live) {
+        const float* w = head < H ? q_w : k_w;
+        const float scale = (w ? 1.f / sqrtf(ss / (float)dk + eps) : 1.f), more = q_scale && head < H ? q_scale[head] : 1.f;
+        TO* dst = head < H ? q_out + ((size_t)t * H + head) * dk : (kdst ? kdst + (size_t)(head - H) * P * dk : nullptr);
+#pragma unroll
+        for (int c = 0; c < M; ++c) {
+            const int i = (l + c * lanes) * 4;
+            if (i >= dk || !dst) continue;
+            float wv[4] = {1.f, 1.f, 1.f, 1.f};
+            if (w) load4(w + i, wv);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) x[c][j] = x[c][j] * scale * wv[j] * more;
+            store4(dst + i, x[c]);
+        }
+    }
+    if (!vdst) return;
+    const int vcol = (H + G) * dk;
+    for (int i = (blockIdx.y * 256 + threadIdx.x) * 4; i < G * dv; i += gridDim.y * 1024) {
+        float v[4];
+        load4(in + vcol + i, v);
+        if (bias) {
+            float b[4];
+            load4(bias + vcol + i, b);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[j] += b[j];
+        }
+        store4(vdst + (size_t)(i / dv) * P * dv + i % dv, v);
+    }
+}
+
 template <typename TX>
 __global__ void __launch_bounds__(256)
 turn_heads_kernel(TX* __restrict__ x, const double* __restrict__ freq, int rot, int pairing, double sign,
@@ -289,6 +367,17 @@ AIR_API int air_qk_normed_prepare(const float* proj, int ld, const float* q_w, c
     if (rot < 0 || rot > dk || (rot & 1) || (dk & 1) || rot > 256 || dk > 64 * air::QKN_PAIRS || (rot > 0 && !freq) ||
         pairing < 0 || pairing > 1 || (write_kv && (!q_w) != (!k_w)))
         return AIR_ERR_BAD_ARGUMENT;
+    auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    if (rot == 0 && v_rot == 0 && !whole && dk % 4 == 0 && (!write_kv || dv % 4 == 0) && ld % 4 == 0 && al(proj) && al(q_w) &&
+        al(k_w) && al(q_out) && al(cache) && al(bias)) {
+        int lanes = 1;
+        while (lanes < 32 && lanes * 4 < dk) lanes *= 2;
+        const int heads = write_kv ? H + G : H, per_block = 256 / lanes;
+        const dim3 grid(T, (heads + per_block - 1) / per_block);
+        AIR_DISPATCH(out_dtype, TO, return air::launch(air::qk_normed_rows_kernel<TO>, grid, 256, 0, stream, proj, ld, q_w, k_w,
+                                                       eps, positions, token_seq, block_table, max_blocks, (TO*)q_out,
+                                                       (TO*)cache, H, G, dk, dv, P, status, bias, q_scale, write_kv, lanes));
+    }
     AIR_DISPATCH(out_dtype, TO, return air::launch(air::qk_normed_prepare_kernel<TO>, T, 256, 0, stream, proj, ld, q_w,
                                                    k_w, eps, freq, rot, pairing, magnitude, positions, token_seq,
                                                    block_table, max_blocks, (TO*)q_out, (TO*)cache, H, G, dk, dv, P,

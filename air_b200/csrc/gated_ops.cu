@@ -210,16 +210,17 @@ __global__ void __launch_bounds__(256)
 glu_vec4_kernel(const TI* __restrict__ in, TO* __restrict__ out, int I, int block, unsigned total4, float alpha, float limit,
                 float shift) {
     pdl_enter(TR_GLU);
-    const unsigned idx = blockIdx.x * 256u + threadIdx.x;
-    if (idx >= total4) return;
-    const unsigned per_row = (unsigned)I / 4, t = idx / per_row, i = (idx % per_row) * 4;
-    const TI* row = in + (size_t)t * 2 * I + (size_t)(i / block) * 2 * block + i % block;
-    float g[4], u[4];
-    load4(row, g);
-    load4(row + block, u);
+    const unsigned per_row = (unsigned)I / 4;
+    for (unsigned idx = blockIdx.x * 256u + threadIdx.x; idx < total4; idx += gridDim.x * 256u) {
+        const unsigned t = idx / per_row, i = (idx % per_row) * 4;
+        const TI* row = in + (size_t)t * 2 * I + (size_t)(i / block) * 2 * block + i % block;
+        float g[4], u[4];
+        load4(row, g);
+        load4(row + block, u);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) g[j] = gated_activation(g[j], u[j], alpha, limit, shift);
-    store4(out + (size_t)t * I + i, g);
+        for (int j = 0; j < 4; ++j) g[j] = gated_activation(g[j], u[j], alpha, limit, shift);
+        store4(out + (size_t)t * I + i, g);
+    }
 }
 
 // x [T, H, d] *= gate[T, H] in place (one gate per token and head); rows whose token_seq is negative are padding.
@@ -326,10 +327,10 @@ AIR_API int air_glu(const void* in, int in_dtype, void* out, int out_dtype, int 
     if (total == 0) return 0;
     if (block <= 0 || I % block) return AIR_ERR_BAD_ARGUMENT;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-    const bool vec = I % 4 == 0 && block % 4 == 0 && total / 4 < 0xffffff00ull && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
+    const bool vec = I % 4 == 0 && block % 4 == 0 && total / 4 < 0x7fffffffull && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
     AIR_DISPATCH(in_dtype, TI, AIR_DISPATCH(out_dtype, TO, {
         if (vec)
-            return air::launch(air::glu_vec4_kernel<TI, TO>, (unsigned)((total / 4 + 255) / 256), 256, 0, stream,
+            return air::launch(air::glu_vec4_kernel<TI, TO>, (unsigned)((total / 4 + 255) / 256 < 148 * 32 ? (total / 4 + 255) / 256 : 148 * 32), 256, 0, stream,
                                (const TI*)in, (TO*)out, I, block, (unsigned)(total / 4), alpha, limit, shift);
         return air::launch(air::glu_kernel<TI, TO>, blocks, 256, 0, stream, (const TI*)in, (TO*)out, I, block, total,
                            alpha, limit, shift);

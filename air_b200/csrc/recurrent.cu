@@ -255,7 +255,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
     if (slot < 0) return;
     const int q0 = p.q_start[e], n = p.q_start[e + 1] - q0;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int l = lane / cpw;                                    // which rows of the column: l, l + L, l + 2L, ...
+    const int l = lane / cpw;                                    // which rows of the column: see row_of
     const int cc = warp * cpw + lane % cpw;                      // column within the block
     const int col = blockIdx.x * CB + cc;
     const bool live = col < p.dv;
@@ -297,11 +297,13 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
 
     stage(0, 0);
     const float ghead = MODE == SCAN_RET ? p.dec[h] : 0.f;      // the head's constant decay
+    // the rows of the column that this lane holds: four neighbours at a time, the lanes' quadruples side by side
+    auto row_of = [&](int i) { return (i / 4) * 4 * L + 4 * l + i % 4; };
     float S[R];
     float* st = p.state + ((size_t)slot * p.H + h) * p.d * p.dv;
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-        const int r = i * L + l;
+        const int r = row_of(i);
         S[i] = (live && r < p.d) ? st[(size_t)r * p.dv + col] : 0.f;
     }
 
@@ -314,47 +316,68 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
         const float* bkq = smem + b * buf_floats;
         const float* bdec = bkq + TK * 2 * dpad;
         const float* bv = bdec + dec_floats;
-        for (int tt = 0; tt < cnt; ++tt) {
-            const float* kk = bkq + tt * 2 * dpad + l;
-            const float* qq = kk + dpad;
-            const float vv = live ? bv[tt * CB + cc] : 0.f;
+        // What a token brings, fetched from shared memory one token ahead of its use: the store of a token's partial
+        // read-outs stands between the fetches of two tokens, and nothing may be moved across it.
+        struct Token {
+            float k[R], q[R], a[per_dec ? R : 1], v, g, beta;
+        };
+        auto fetch = [&](Token& w, int tt) {
+            const float* kk = bkq + tt * 2 * dpad + 4 * l;
+#pragma unroll
+            for (int i = 0; i < R; i += 4) {
+                load4(kk + i * L, reinterpret_cast<float(&)[4]>(w.k[i]));
+                load4(kk + dpad + i * L, reinterpret_cast<float(&)[4]>(w.q[i]));
+                if constexpr (per_dec > 0)
+                    load4(bdec + tt * per_dec + 4 * l + i * L, reinterpret_cast<float(&)[4]>(w.a[i]));
+            }
+            w.v = live ? bv[tt * CB + cc] : 0.f;
+            if (MODE == SCAN_DELTA) { w.g = bdec[2 * tt]; w.beta = bdec[2 * tt + 1]; }
+            if (MODE == SCAN_CDELTA) w.beta = bdec[tt * per_dec + dpad];
+        };
+        auto take = [&](const Token& w, int tt) {
             // (four partial sums each: the chain of dependent additions is a quarter as long)
             float orr[4] = {0.f, 0.f, 0.f, 0.f};
             if (MODE == SCAN_DELTA || MODE == SCAN_CDELTA) {
-                const float* aa = bdec + tt * per_dec + l;       // CDELTA: a decay per row of the column
-                const float gv = MODE == SCAN_DELTA ? bdec[2 * tt] : 0.f;
-                const float bb = MODE == SCAN_DELTA ? bdec[2 * tt + 1] : bdec[tt * per_dec + dpad];
-                float kr[R], pr[4] = {0.f, 0.f, 0.f, 0.f};
+                float pr[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int i = 0; i < R; ++i) {
-                    kr[i] = kk[i * L];
-                    S[i] *= MODE == SCAN_DELTA ? gv : aa[i * L];
-                    pr[i & 3] = fmaf(S[i], kr[i], pr[i & 3]);
+                    S[i] *= MODE == SCAN_DELTA ? w.g : w.a[per_dec ? i : 0];
+                    pr[i & 3] = fmaf(S[i], w.k[i], pr[i & 3]);
                 }
                 float pred = (pr[0] + pr[1]) + (pr[2] + pr[3]);
 #pragma unroll
                 for (int off = 16; off >= cpw; off >>= 1) pred += __shfl_xor_sync(0xffffffffu, pred, off);
-                const float u = bb * (vv - pred);
+                const float u = w.beta * (w.v - pred);
 #pragma unroll
                 for (int i = 0; i < R; ++i) {
-                    S[i] = fmaf(kr[i], u, S[i]);
-                    orr[i & 3] = fmaf(S[i], qq[i * L], orr[i & 3]);
-                }
-            } else if (MODE == SCAN_RET) {
-#pragma unroll
-                for (int i = 0; i < R; ++i) {
-                    S[i] = fmaf(ghead, S[i], kk[i * L] * vv);
-                    orr[i & 3] = fmaf(S[i], qq[i * L], orr[i & 3]);
+                    S[i] = fmaf(w.k[i], u, S[i]);
+                    orr[i & 3] = fmaf(S[i], w.q[i], orr[i & 3]);
                 }
             } else {
-                const float* aa = bdec + tt * dpad + l;
 #pragma unroll
                 for (int i = 0; i < R; ++i) {
-                    S[i] = fmaf(aa[i * L], S[i], kk[i * L] * vv);
-                    orr[i & 3] = fmaf(S[i], qq[i * L], orr[i & 3]);
+                    S[i] = fmaf(MODE == SCAN_RET ? ghead : w.a[per_dec ? i : 0], S[i], w.k[i] * w.v);
+                    orr[i & 3] = fmaf(S[i], w.q[i], orr[i & 3]);
                 }
             }
             so[(tt * CB + cc) * L + l] = (orr[0] + orr[1]) + (orr[2] + orr[3]);
+        };
+        if constexpr (R <= 16) {
+            Token x, y;
+            fetch(x, 0);
+            for (int tt = 0; tt < cnt; tt += 2) {
+                fetch(y, min(tt + 1, cnt - 1));
+                take(x, tt);
+                if (tt + 1 == cnt) break;
+                fetch(x, min(tt + 2, cnt - 1));
+                take(y, tt + 1);
+            }
+        } else {
+            for (int tt = 0; tt < cnt; ++tt) {
+                Token x;
+                fetch(x, tt);
+                take(x, tt);
+            }
         }
         __syncthreads();
         for (int idx = threadIdx.x; idx < cnt * CB; idx += SCAN_THREADS) {
@@ -367,7 +390,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) linear_scan_kernel(const ScanArg
     }
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-        const int r = i * L + l;
+        const int r = row_of(i);
         if (live && r < p.d) st[(size_t)r * p.dv + col] = S[i];
     }
 }

@@ -560,6 +560,31 @@ def _dafotar(width, layers, heads, kv_heads, ff, vocab=32000):
             "canon": {"taps": 4}, "layers": out}
 
 
+# Sesulorn beside Pefivik, the closest of the other designs (attention over a latent, a recurrence with a matrix state, dense
+# feed-forwards and mixtures of experts among groups in turn, a repeated stretch), at equal width, heads, feed-forward and
+# number of runs (`--design sesulorn`): latent attention (a latent of 512 + 64 per token, queries through a latent of 1,536),
+# attention with a distance table of 32 rows that reaches 128 positions, the channel-wise delta rule behind convolutions of
+# four taps (narrow middles of 128), attention, in turn, heads of 128; mixtures of 16 experts of ff / 4 in 4 groups (2 take
+# part, a token takes 2) with a shared expert of ff / 2; two of its layers run twice, so `layers` runs are layers - 2
+# layers' weights.
+def _sesulorn(width, layers, heads, kv_heads, ff, vocab=32000):
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 0.2,
+                                          "bias_max": 128, "buckets": 32}}
+    delta = {"type": "channel_delta", "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4,
+                                                "decay_rank": 128, "gate_rank": 128}}
+    latent = {"type": "latent_attention", "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512,
+                                                    "q_rank": 1536, "scale": 192 ** -0.5, "rot": {"base": 1e4, "dims": 64}}}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 2}},
+           "shared": {"ff": ff // 2, "limit": 7.0}}
+    n = max(2, layers - 2)
+    start = min(1, n - 2)
+    order = [latent, att, delta, att]
+    return {"architecture": "Sesulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "loop": {"start": start, "stop": start + 2, "times": 2},
+            "layers": [dict(order[i % 4], mlp=moe if i % 2 else dense) for i in range(n)]}
+
+
 def _qwen(width, layers, heads, kv_heads, ff, vocab=32000):
     return dict(_QWEN, num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads,
                 num_key_value_heads=kv_heads, intermediate_size=ff, rms_norm_eps=1e-5, max_window_layers=layers,
@@ -1408,14 +1433,146 @@ def dafotar_kernels(width, heads, kv_heads, ff, T, batch, context):
     return rows
 
 
+def sesulorn_kernels(width, heads, kv_heads, ff, T, batch, context):
+    """Sesulorn's kernels alone at the layer's shapes, each beside the like kernel of the other designs."""
+    import torch
+    from air_b200.csrc import ops
+    from air_b200.parts.attention import TiledAttention
+    from air_b200.parts.base import HostBatch
+    from air_b200.parts.normed_attention import distance_rows
+    report, rows = kernel_reporter()
+    E, H, G, d, P, R, rot, Q = width, heads, kv_heads, 128, 64, 512, 64, 1536
+    dev, bf = "cuda", torch.bfloat16
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    for label, N, entries in (("prompt", T, [(0, T)]), ("decode", batch, [(context - 1, 1)] * batch)):
+        print(f"{label}: {N} rows, width {E}, {H}/{G} heads of {d}, latents of {R} + {rot} and {Q}")
+        S = len(entries)
+        starts = [0]
+        for _, n in entries:
+            starts.append(starts[-1] + n)
+        q_start, slots = i32(starts), i32(list(range(S)))
+        positions = torch.cat([torch.arange(p, p + n, dtype=torch.int32) for p, n in entries]).to(dev)
+        seq = torch.cat([torch.full((n,), i, dtype=torch.int32) for i, (_, n) in enumerate(entries)]).to(dev)
+        per_request = -(-(max(p + n for p, n in entries)) // P)
+        bt = torch.arange(S * per_request, dtype=torch.int32, device=dev).view(S, per_request).contiguous()
+        longest = max(n for _, n in entries)
+        # ---- the stream completed with a layer's terms and normalised, and written beside the embedding's output
+        parts = 1 if label == "prompt" else 4
+        h, x0, gate = torch.randn(N, E, device=dev), torch.randn(N, E, device=dev), torch.rand(N, device=dev)
+        mix = torch.randn(parts, N, E, device=dev) if parts > 1 else torch.randn(N, E, device=dev)
+        planes, shared = torch.randn(2, N, E, device=dev), torch.randn_like(mix)
+        w, b = torch.rand(E, device=dev) + 0.5, torch.randn(E, device=dev)
+        wbf, x, two = w.to(bf), torch.empty(N, E, dtype=bf, device=dev), torch.empty(N, 2 * E, dtype=bf, device=dev)
+        one = N * E * 4 * parts
+        report("stream_norm (stream + mixer + experts' planes + gated shared expert, layer norm)",
+               lambda: ops.stream_norm(h, 1, w, b, 1e-6, x, term=mix, more=[(planes, None), (shared, gate)], h_out=h), N * E * 18 + 2 * one)
+        report("  Tomodra: post_norm (stream + planes + gated shared expert)", lambda: ops.post_norm(h, 3.0, planes, shared, gate, wbf, 1e-6, x), N * E * 18 + one)
+        report("  Pefivik: scaled_norm (stream + m x (planes + shared expert))", lambda: ops.scaled_norm(h, [(planes, w), (shared, w)], wbf, 1e-6, x), N * E * 18 + one)
+        report("stream_norm (stream + mixer + feed-forward, layer norm)",
+               lambda: ops.stream_norm(h, 1, w, b, 1e-6, x, term=mix, more=[(shared, None)], h_out=h), N * E * 10 + 2 * one)
+        report("  Bivizen: scaled_norm (stream + two scaled terms)", lambda: ops.scaled_norm(h, [(mix, w), (shared, w)], wbf, 1e-6, x), N * E * 10 + 2 * one)
+        report("stream_norm as rows [x | x0] (three terms)",
+               lambda: ops.stream_norm(h, 1, None, None, 0.0, two, term=mix, more=[(planes, None), (shared, gate)], again=x0), N * E * 20 + 2 * one)
+        report("  Pefivik: stream_add (the embedding's output again and a row)", lambda: ops.stream_add(h, x0, b), N * E * 12)
+        # ---- attention: biases, norm per head, page write; the bias per distance
+        C = (H + 2 * G) * d
+        proj, bias = torch.randn(N, C, device=dev), torch.randn(C, device=dev)
+        pages = torch.zeros(S * per_request, G * P * 2 * d, dtype=bf, device=dev)
+        qo, ao = torch.empty(N, H, d, dtype=bf, device=dev), torch.empty(N, H, d, dtype=bf, device=dev)
+        ones = torch.ones(d, device=dev)
+        freq = torch.rand(d // 2, dtype=torch.float64, device=dev)
+        report("qk_normed_prepare (biases, norm per head, no rotation)",
+               lambda: ops.qk_normed_prepare(proj, ones, ones, 1e-6, None, "half", 1.0, positions, seq, bt, qo, pages, G, d, P, bias=bias), N * C * 6)
+        report("  Tomodra: qk_normed_prepare (norm per head, neighbouring pairs)",
+               lambda: ops.qk_normed_prepare(proj, ones, ones, 1e-6, freq[:d // 4], "neighbours", 1.0, positions, seq, bt, qo, pages, G, d, P), N * C * 6)
+        p5 = pages.view(-1, 2, G, P, d)
+        table = lambda reach: torch.randn(H, len(distance_rows(32, reach)), device=dev)
+        near, wide = table(128), table(8192)
+        if label == "prompt":
+            tiles = i32(type("P", (TiledAttention,), {"heads": H, "window": None})().plan(
+                HostBatch(counts=[T], lengths=[0], slots=[0], q_start=[0, T])).arrays["tiles"].tolist())
+            fl = 4 * H * d * (T * (T + 1) // 2)
+            for name, tab in (("128", near), ("8,192", wide)):
+                report(f"prefill_attention_tc with a distance table that reaches {name}", lambda: ops.prefill_attention_tc(qo, p5, bt, tiles, ao, None, 0.2, bias=tab), flops=fl)
+            report("  Bivizen: prefill_attention_tc with a soft cap", lambda: ops.prefill_attention_tc(qo, p5, bt, tiles, ao, None, 0.2, softcap=30.0), flops=fl)
+            report("  Qwen2: prefill_attention_tc", lambda: ops.prefill_attention_tc(qo, p5, bt, tiles, ao, None, 0.2), flops=fl)
+        else:
+            kvb = 2 * S * context * G * d * 2
+            for name, tab in (("128", near), ("8,192", wide)):
+                report(f"decode_attention with a distance table that reaches {name}", lambda: ops.decode_attention(qo, p5, bt, seq, positions, ao, None, 0.2, bias=tab), kvb)
+            report("  Bivizen: decode_attention with a soft cap", lambda: ops.decode_attention(qo, p5, bt, seq, positions, ao, None, 0.2, softcap=30.0), kvb)
+            report("  Qwen2: decode_attention", lambda: ops.decode_attention(qo, p5, bt, seq, positions, ao, None, 0.2), kvb)
+        # ---- latent attention: the query's latent, the heads, the row in the pages
+        first = torch.randn(N, Q + R + rot, device=dev)
+        cq, cw, qw = torch.empty(N, Q, dtype=bf, device=dev), torch.ones(R, device=dev), torch.ones(Q, device=dev)
+        heads = torch.randn(N, Q // d, d, device=dev)
+        report("band_rmsnorm (the query's latent)", lambda: ops.band_rmsnorm(first[:, :Q], qw, 1e-6, cq), N * Q * 6)
+        report("  Bivizen: gated_rmsnorm (heads of 128 with a gate, as wide)",
+               lambda: ops.gated_rmsnorm(heads, first[:, :Q], ones, 1e-6, cq, seq), N * Q * 10)
+        qf = torch.randn(N, H * (d + rot), device=dev)
+        q_plain, q_full = torch.empty(N, H, d, device=dev, dtype=bf), torch.empty(N, H, R + rot, device=dev)
+        lrows = torch.zeros(S * per_request, P, R + rot, device=dev, dtype=bf).normal_(0, 0.5)
+        lb = N * ((H * (d + rot) + R + rot) * 4 + H * d * 2 + H * rot * 4 + (R + rot) * 2)
+        for name, pairing in (("latent_prepare (queries of their own product, neighbouring pairs)", "neighbours"),
+                              ("  Tomodra: latent_prepare (in halves)", "half")):
+            report(name, lambda: ops.latent_prepare(qf, first[:, Q:], cw, 1e-6, freq[:rot // 2], positions, seq, bt, q_plain, q_full, lrows, True, pairing=pairing), lb)
+        if label == "decode":
+            summed = torch.empty(N, H, R, device=dev, dtype=bf)
+            report("grouped_attention, latent rows of 576, all keys", lambda: ops.grouped_attention(q_full, lrows, bt, seq, positions, summed, None, 0.07, latent=True), S * context * (R + rot) * 2)
+            r512 = torch.zeros(S * per_request, P, R, device=dev, dtype=bf).normal_(0, 0.5)
+            q512 = torch.randn(N, H, R, device=dev)
+            report("  Pefivik: grouped_attention, latent rows of 512, all keys, sink", lambda: ops.grouped_attention(q512, r512, bt, seq, positions, summed, None, 0.09, latent=True, sink=torch.zeros(H, device=dev)), S * context * R * 2)
+        # ---- the delta rule
+        pm, z = torch.randn(N, 4 * H * d, device=dev), torch.randn(N, H * d, device=dev)
+        state, o, ym = torch.zeros(S, H, d, d, device=dev), torch.empty(N, H, d, device=dev), torch.empty(N, H * d, dtype=bf, device=dev)
+        alog, dtb, dtc = torch.randn(H, device=dev), torch.randn(H, device=dev), torch.randn(H * d, device=dev)
+        bands = [pm[:, i * H * d:(i + 1) * H * d] for i in range(4)]
+        beta = pm[:, 3 * H * d:3 * H * d + H]
+        sb = N * H * d * 16 + 2 * S * H * d * d * 4
+        report("linear_scan (delta rule, a decay per key channel)",
+               lambda: ops.linear_scan(ops.SCAN_CHANNEL_DELTA, bands[0], bands[1], bands[2], z, state, o, q_start, slots, seq, q_scale=d ** -0.5, beta=beta, a_log=alog, dt_bias=dtc, unit=True), sb + N * H * d * 4)
+        report("  Bivizen: linear_scan (delta rule, a decay per head)",
+               lambda: ops.linear_scan(ops.SCAN_DELTA, bands[0], bands[1], bands[2], z[:, :H], state, o, q_start, slots, seq, q_scale=d ** -0.5, beta=beta, a_log=alog, dt_bias=dtb, unit=True), sb)
+        report("  Bivizen: linear_scan (gated linear attention)",
+               lambda: ops.linear_scan(ops.SCAN_GLA, bands[0], bands[1], bands[2], z, state, o, q_start, slots, seq, q_scale=d ** -0.5, tau=16.0), sb + N * H * d * 4)
+        report("gated_rmsnorm with the sigmoid", lambda: ops.gated_rmsnorm(o, bands[3], ones, 1e-6, ym, seq, sigmoid=True), N * H * d * 10)
+        report("  Bivizen: gated_rmsnorm", lambda: ops.gated_rmsnorm(o, bands[3], ones, 1e-6, ym, seq), N * H * d * 10)
+        report("split_bands (two narrow middles of 128)", lambda: ops.split_bands(pm[:, :256], 128, 128), N * 256 * 8)
+        report("  Qwen2: convert", lambda: ops.convert(first, two.view(-1)[:first.numel()].view(first.shape)) if first.numel() <= two.numel() else ops.convert(h, x), (first if first.numel() <= two.numel() else h).numel() * 6)
+        # ---- experts
+        n_exp, top, F = 16, 2, ff // 4
+        zr = torch.randn(N, 24, device=dev)
+        expert, weight, g2 = torch.empty(N, top, dtype=torch.int32, device=dev), torch.empty(N, top, device=dev), torch.empty(N, device=dev)
+        report("moe_route (softmax, groups by their best expert, shared gate)",
+               lambda: ops.moe_route(zr, n_exp, top, expert, weight, g2, has_gate=True, score="softmax", groups=4, keep=2, mark="best"), N * 24 * 4 + N * top * 8)
+        report("  Pefivik: moe_route (sigmoid, groups by their two best)",
+               lambda: ops.moe_route(zr, n_exp, top, expert, weight, None, renormalize=True, groups=4, keep=2, norm_eps=1e-20), N * 24 * 4 + N * top * 8)
+        pairs = N * top
+        act, xin = torch.empty(pairs, F, dtype=bf, device=dev), torch.randn(N, E, device=dev).to(bf)
+        if label == "prompt":
+            gu = torch.randn(pairs, 2 * F, device=dev).to(bf)
+            report("glu (clamped) behind the experts' library product", lambda: ops.glu(gu, act, block=128, alpha=1.702, limit=7.0, shift=1.0), pairs * F * 6)
+            report("  Pefivik: silu_mul", lambda: ops.silu_mul(gu, act, block=128), pairs * F * 6)
+        else:
+            start, pos = torch.empty(n_exp + 1, dtype=torch.int32, device=dev), torch.empty(pairs, dtype=torch.int32, device=dev)
+            tl, nt = torch.empty(pairs // ops.GROUP_TILE + n_exp, 2, dtype=torch.int32, device=dev), torch.empty(1, dtype=torch.int32, device=dev)
+            ops.moe_sort(expert, n_exp, start, pos, tl, nt)
+            torch.cuda.synchronize()
+            used = len(set(expert.view(-1).tolist()))
+            gate_up = torch.randn(n_exp, 2 * F, E, device=dev).to(bf) * 0.02
+            for name, how in (("grouped product: gate, up and the clamped activation", (1.702, 7.0, 1.0)), ("  Pefivik: grouped product with SiLU", ops.SILU)):
+                report(f"{name} of {used} experts", lambda: ops.grouped_gemm(xin, gate_up, act, F, E, lda=E, ldo=F, groups=n_exp, a_index=pos, a_div=top, start=start, tiles=tl, num_tiles=nt, silu_mul=True, gate_block=128, act=how), nbytes=used * 2 * F * E * 2)
+    return rows
+
+
 def design_bench(args):
     import torch
     from air_b200.engine.batch import Entry, LAST_SAMPLED
     designs = {"bivizen": ("Bivizen", _bivizen), "tomodra": ("Tomodra", _tomodra), "pefivik": ("Pefivik", _pefivik),
-               "tabopel": ("Tabopel", _tabopel), "dafotar": ("Dafotar", _dafotar)}
+               "tabopel": ("Tabopel", _tabopel), "dafotar": ("Dafotar", _dafotar), "sesulorn": ("Sesulorn", _sesulorn)}
     # the model that stands beside the design: the Qwen2 decoder, or the closest of the other designs
     beside = {"pefivik": ("tomodra", "Tomodra", _tomodra), "tabopel": ("tomodra", "Tomodra", _tomodra),
-              "dafotar": ("bivizen", "Bivizen", _bivizen)} \
+              "dafotar": ("bivizen", "Bivizen", _bivizen), "sesulorn": ("pefivik", "Pefivik", _pefivik)} \
         .get(args.design, ("qwen2", "Qwen2ForCausalLM", _qwen))
     if args.design not in designs:
         print(json.dumps({"error": f"--design {args.design}: the designs that are compared are {', '.join(designs)}"}))
@@ -1439,6 +1596,8 @@ def design_bench(args):
             size["kernels"] = tabopel_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
         if not args.skip_kernels and args.design == "dafotar":
             size["kernels"] = dafotar_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
+        if not args.skip_kernels and args.design == "sesulorn":
+            size["kernels"] = sesulorn_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
         if not args.skip_kernels and args.design == "tomodra":
             size["kernels"] = tomodra_kernels(width, heads, kv_heads, ff, args.prefill_tokens, args.batch, context)
         record["sizes"][name] = size
@@ -1520,7 +1679,7 @@ def main():
     ap.add_argument("--skip-decode", action="store_true", help="for profiling the prefill step alone")
     ap.add_argument("--no-graphs", action="store_true", help="launch the decode step's kernels one by one (for ncu)")
     ap.add_argument("--kernel", default="", help="prefill_attention, or prompt_elementwise (at --prefill-tokens rows): time those kernels alone and exit")
-    ap.add_argument("--design", default="", help="bivizen, tomodra, pefivik, tabopel or dafotar: prefill and decode of that design beside the Qwen2 decoder (pefivik and tabopel: beside Tomodra; dafotar: beside Bivizen) at "
+    ap.add_argument("--design", default="", help="bivizen, tomodra, pefivik, tabopel, dafotar or sesulorn: prefill and decode of that design beside the Qwen2 decoder (pefivik and tabopel: beside Tomodra; dafotar: beside Bivizen; sesulorn: beside Pefivik) at "
                     "equal sizes, and its kernels alone beside the like kernels (another line of output; the default "
                     "workload is not run)")
     ap.add_argument("--design-sizes", default="", help="with --design: which of the sizes 2048,4096 (default: both)")
