@@ -89,6 +89,9 @@ _SIGNATURES = {
                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_float, c_void_p,
                         c_void_p, c_int, c_float, c_void_p],
+    "air_delta_portions": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
+                           c_int, c_float, c_float, c_void_p],
     "air_gated_rmsnorm": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float,
                           c_int, c_void_p],
     "air_polynorm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float,
@@ -1164,6 +1167,41 @@ def linear_scan(mode, q, k, v, decay, state, out, q_start, slots, token_seq, q_s
         T, slots.shape[0], H, G, d, dv, lanes, float(q_scale), 1.0 / float(tau), 1 if unit else 0, float(unit_eps),
         _ptr(positions), _ptr(freq), 2 * freq.numel() if (mode == SCAN_RETENTION and freq is not None) else 0,
         float(k_scale), _stream()), "linear_scan")
+    global launches
+    launches += 1
+    return out
+
+
+DELTA_CHUNK = 16         # tokens of a chunk of delta_portions
+DELTA_MAX_D = 256        # key channels per head that it takes
+
+
+def delta_portions(q, k, v, decay, state, out, portions, chunks, q_scale, beta, a_log, dt_bias, unit_eps=1e-6):
+    """linear_scan's SCAN_CHANNEL_DELTA with unit lengths, for whole portions: the tokens of a chunk are computed side by side
+    from the state ahead of it (delta_chunks.cu).  portions int32 [L, 4] = (first row, tokens, slot, first chunk), chunks
+    int32 [N, 2] = (first row, tokens): a portion's tokens cut into chunks of DELTA_CHUNK.  32-bit throughout."""
+    _, H, d, dv = state.shape
+    _req(state, "state", (torch.float32,))
+    T = out.shape[0]
+    _req(out, "out", (torch.float32,), (T, H, dv))
+    (qp, ldq), (kp, ldk), (vp, ldv) = _columns(q, "q"), _columns(k, "k"), _columns(v, "v")
+    (dp, ldd), (bp, ldb) = _columns(decay, "decay"), _columns(beta, "beta")
+    if q.shape[1] % d or k.shape != q.shape or v.shape[1] != H * dv or decay.shape[1] != H * d or beta.shape[1] != H:
+        raise KernelError("delta_portions: q, k, v, decay or beta do not fit the state's shape")
+    G = q.shape[1] // d
+    if G == 0 or H % G or d > DELTA_MAX_D:
+        raise KernelError(f"delta_portions: {H} heads over {G} heads of q and k, of {d} channels (up to {DELTA_MAX_D})")
+    _req(a_log, "a_log", (torch.float32,), (H,))
+    _req(dt_bias, "dt_bias", (torch.float32,), (H * d,))
+    _req(portions, "portions", _I32, (None, 4))
+    _req(chunks, "chunks", _I32, (None, 2))
+    N = chunks.shape[0]
+    stride = 3 * DELTA_CHUNK * (-(-d // 8) * 8) + -(-d // 8) * 8 + DELTA_CHUNK ** 2 + DELTA_CHUNK * (-(-dv // 4) * 4)
+    scratch = torch.empty(N * H * stride, dtype=torch.float32, device=out.device)
+    _check(_get("air_delta_portions")(
+        qp, ldq, kp, ldk, vp, ldv, dp, ldd, bp, ldb, a_log.data_ptr(), dt_bias.data_ptr(), state.data_ptr(), out.data_ptr(),
+        portions.data_ptr(), portions.shape[0], chunks.data_ptr(), N, scratch.data_ptr(), H, G, d, dv, float(q_scale),
+        float(unit_eps), _stream()), "delta_portions")
     global launches
     launches += 1
     return out

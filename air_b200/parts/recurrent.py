@@ -125,6 +125,9 @@ class ChannelDeltaRule(_StateMixer):
     then o / sqrt(mean(o^2) + eps) * norm, times sigmoid(W_g2 (W_g1 x)) (laid out heads x v_dim), and the output
     projection.  S and the convolutions' last conv - 1 inputs are the request's state, 32-bit, zero at its start.
 
+    Portions of PORTION tokens or more are taken in chunks whose rows are computed side by side (ops.delta_portions), single
+    tokens and shorter portions token by token (ops.linear_scan); both are 32-bit.
+
     The two products out of a narrow middle take its numbers as they left the first product: a float32 engine in 32-bit,
     a bfloat16 engine as two bfloat16 halves side by side, against the matrix twice (ops.split_bands), so that the
     decays are 32-bit but for the weights' own precision.
@@ -200,6 +203,30 @@ class ChannelDeltaRule(_StateMixer):
             full[:rows, i * width:i * width + rank] = m
         return Linear(full, rt.status)
 
+    PORTION = 24
+
+    def plan_key(self):
+        return ("channel_delta.chunks", self.PORTION) if self.head_dim <= ops.DELTA_MAX_D else None
+
+    def plan(self, batch: HostBatch) -> Plan:
+        """portions [L, 4] = (first row, tokens, slot, first chunk) of the entries of at least PORTION tokens, chunks [N, 2] =
+        (first row, tokens) of theirs; short_slots: the slot of every other entry, short_seq: of their rows, -1 elsewhere."""
+        portions, chunks, short_slots = [], [], []
+        short_seq = np.full(batch.q_start[-1], -1, dtype=np.int32)
+        for i, n in enumerate(batch.counts):
+            first = batch.q_start[i]
+            if n < self.PORTION:
+                short_slots.append(batch.slots[i])
+                short_seq[first:first + n] = batch.slots[i]
+                continue
+            short_slots.append(-1)
+            portions.append((first, n, batch.slots[i], len(chunks)))
+            chunks += [(first + at, min(ops.DELTA_CHUNK, n - at)) for at in range(0, n, ops.DELTA_CHUNK)]
+        return Plan(arrays={"portions": np.asarray(portions, dtype=np.int32).reshape(-1, 4),
+                            "chunks": np.asarray(chunks, dtype=np.int32).reshape(-1, 2),
+                            "short_slots": np.asarray(short_slots, dtype=np.int32), "short_seq": short_seq},
+                    values={"long": bool(portions), "short": len(portions) < len(batch.counts)})
+
     def _narrow(self, proj):
         """(decay logits [T, heads*head_dim], gate logits [T, heads*v_dim]), float32."""
         at, (ra, rg) = self.columns["a1"][0], self.middle
@@ -218,9 +245,16 @@ class ChannelDeltaRule(_StateMixer):
         y = self._convolved(proj, tail, ctx)
         decay, gate = self._narrow(proj)
         o = torch.empty((T, H, dv), dtype=torch.float32, device=x.device)
-        ops.linear_scan(ops.SCAN_CHANNEL_DELTA, y[:, :G * d], y[:, G * d:2 * G * d], y[:, 2 * G * d:], decay, state.state, o,
-                        ctx.q_start, ctx.slots, ctx.token_seq, q_scale=d ** -0.5, beta=self._band(proj, "b"),
-                        a_log=self.a_log, dt_bias=self.dt_bias, unit=True, unit_eps=1e-6)
+        bands = (y[:, :G * d], y[:, G * d:2 * G * d], y[:, 2 * G * d:], decay, state.state, o)
+        numbers = dict(q_scale=d ** -0.5, beta=self._band(proj, "b"), a_log=self.a_log, dt_bias=self.dt_bias, unit_eps=1e-6)
+        plan = ctx.plans.get(self.plan_key()) if self.plan_key() is not None else None
+        if plan is None or not plan.long:
+            ops.linear_scan(ops.SCAN_CHANNEL_DELTA, *bands, ctx.q_start, ctx.slots, ctx.token_seq, unit=True, **numbers)
+        else:
+            if plan.short:
+                ops.linear_scan(ops.SCAN_CHANNEL_DELTA, *bands, ctx.q_start, plan.short_slots, plan.short_seq, unit=True,
+                                **numbers)
+            ops.delta_portions(*bands, plan.portions, plan.chunks, **numbers)
         return self._finish(o, gate, ctx, sigmoid=True)
 
 

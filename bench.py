@@ -563,8 +563,8 @@ def _dafotar(width, layers, heads, kv_heads, ff, vocab=32000):
 # Sesulorn beside Pefivik, the closest of the other designs (attention over a latent, a recurrence with a matrix state, dense
 # feed-forwards and mixtures of experts among groups in turn, a repeated stretch), at equal width, heads, feed-forward and
 # number of runs (`--design sesulorn`): latent attention (a latent of 512 + 64 per token, queries through a latent of 1,536),
-# attention with a distance table of 32 rows that reaches 128 positions, the channel-wise delta rule behind convolutions of
-# four taps (narrow middles of 128), attention, in turn, heads of 128; mixtures of 16 experts of ff / 4 in 4 groups (2 take
+# the channel-wise delta rule behind convolutions of four taps (narrow middles of 128), attention with a distance table of
+# 32 rows that reaches 128 positions, in turn, heads of 128; mixtures of 16 experts of ff / 4 in 4 groups (2 take
 # part, a token takes 2) with a shared expert of ff / 2; two of its layers run twice, so `layers` runs are layers - 2
 # layers' weights.
 def _sesulorn(width, layers, heads, kv_heads, ff, vocab=32000):
@@ -579,10 +579,10 @@ def _sesulorn(width, layers, heads, kv_heads, ff, vocab=32000):
            "shared": {"ff": ff // 2, "limit": 7.0}}
     n = max(2, layers - 2)
     start = min(1, n - 2)
-    order = [latent, att, delta, att]
+    order = [latent, delta, att]
     return {"architecture": "Sesulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
             "loop": {"start": start, "stop": start + 2, "times": 2},
-            "layers": [dict(order[i % 4], mlp=moe if i % 2 else dense) for i in range(n)]}
+            "layers": [dict(order[i % 3], mlp=moe if i % 2 else dense) for i in range(n)]}
 
 
 def _qwen(width, layers, heads, kv_heads, ff, vocab=32000):
@@ -1529,6 +1529,15 @@ def sesulorn_kernels(width, heads, kv_heads, ff, T, batch, context):
         bands = [pm[:, i * H * d:(i + 1) * H * d] for i in range(4)]
         beta = pm[:, 3 * H * d:3 * H * d + H]
         sb = N * H * d * 16 + 2 * S * H * d * d * 4
+        if label == "prompt":
+            por, chk = i32([[0, T, 0, 0]]), i32([[a, min(ops.DELTA_CHUNK, T - a)] for a in range(0, T, ops.DELTA_CHUNK)])
+            report("delta_portions (delta rule, a decay per key channel, chunks of 16)",
+                   lambda: ops.delta_portions(bands[0], bands[1], bands[2], z, state, o, por, chk, q_scale=d ** -0.5, beta=beta, a_log=alog, dt_bias=dtc), sb + N * H * d * 4)
+            mcols = {"q": 0, "k": H * d, "v": 2 * H * d, "g": 3 * H * d, "i": 0, "f": H}
+            pm16, zl, mch = pm.to(bf), torch.randn(N, 2 * H, device=dev), i32([[a, min(ops.MLSTM_CHUNK, T - a)] for a in range(0, T, ops.MLSTM_CHUNK)])
+            report("  Dafotar: mlstm_portions (bfloat16 projections, tensor cores; norm and gate in it)",
+                   lambda: ops.mlstm_portions(pm16, zl, mcols, torch.zeros(H, device=dev), torch.full((H,), 3.0, device=dev), torch.ones(H * d, device=dev), state, torch.zeros(S, H, d, device=dev),
+                                              torch.zeros(S, H, device=dev), ym, por, mch, 15.0, d ** -0.5, 1e-6), N * H * d * 10)
         report("linear_scan (delta rule, a decay per key channel)",
                lambda: ops.linear_scan(ops.SCAN_CHANNEL_DELTA, bands[0], bands[1], bands[2], z, state, o, q_start, slots, seq, q_scale=d ** -0.5, beta=beta, a_log=alog, dt_bias=dtc, unit=True), sb + N * H * d * 4)
         report("  Bivizen: linear_scan (delta rule, a decay per head)",

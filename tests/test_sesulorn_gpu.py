@@ -319,6 +319,58 @@ def test_channel_delta_scan(H, G, d, dv):
             at += n
 
 
+@pytest.mark.parametrize("H,G,d,dv", [(4, 2, 24, 20), (1, 1, 64, 33), (2, 2, 130, 8), (3, 1, 16, 128), (2, 1, 256, 5), (1, 1, 1, 1),
+                                      (2, 2, 128, 128), (6, 3, 12, 18)])
+@pytest.mark.parametrize("decays", ["mixed", "slow", "fast"])
+def test_delta_rule_in_chunks_against_token_by_token(decays, H, G, d, dv):
+    """Both roads of the channel-wise delta rule and the plain recurrence, from states that are not empty, the states they
+    leave behind among the results: portions of every length around a chunk's in one batch, channels that keep everything,
+    that forget at once, and that change from one to the other from token to token; keys that repeat."""
+    from air_b200.csrc import ops
+    rng = np.random.default_rng(d + dv)
+    for counts in ([15, 16, 17], [1, 32, 200], [48, 31, 2]):
+        T = sum(counts)
+        start = np.concatenate([[0], np.cumsum(counts)])
+        a_log = rng.uniform(-2, 0.5, size=H)
+        dt = {"mixed": rng.choice([-9.0, -2.0, 1.0, 6.0], size=H * d), "slow": np.full(H * d, -8.0), "fast": np.full(H * d, 9.0)}[decays]
+        q, k, v = rng.normal(size=(T, G * d)), rng.normal(size=(T, G * d)), rng.normal(size=(T, H * dv))
+        k[T // 3:T // 3 + 6] = k[T // 3]                 # the same key several times
+        z, b = rng.normal(size=(T, H * d)) * 2, rng.normal(size=(T, H)) * 3
+        z[::5] += 30.0 * (rng.random(size=(len(z[::5]), H * d)) < 0.2)
+        S0 = rng.normal(size=(4, H, d, dv))
+        slots = [2, 0, 3]
+        chunks, portions = [], []
+        for i, n in enumerate(counts):
+            portions.append((start[i], n, slots[i], len(chunks)))
+            chunks += [(start[i] + a, min(ops.DELTA_CHUNK, n - a)) for a in range(0, n, ops.DELTA_CHUNK)]
+        wide = dev(np.concatenate([q, k, v], axis=1))          # bands of a wider matrix
+        bands = (wide[:, :G * d], wide[:, G * d:2 * G * d], wide[:, 2 * G * d:], dev(z))
+        kw = dict(q_scale=d ** -0.5, beta=dev(b), a_log=dev(a_log), dt_bias=dev(dt))
+        got = []
+        for road in ("tokens", "chunks"):
+            S, o = dev(S0), torch.full((T, H, dv), 9.0, device=DEV)
+            if road == "tokens":
+                ops.linear_scan(ops.SCAN_CHANNEL_DELTA, *bands, S, o, i32(start), i32(slots),
+                                i32(np.repeat(slots, counts)), unit=True, **kw)
+            else:
+                ops.delta_portions(*bands, S, o, torch.tensor(np.array(portions), dtype=torch.int32, device=DEV),
+                                   torch.tensor(np.array(chunks), dtype=torch.int32, device=DEV), **kw)
+            got.append((o.cpu().numpy(), S.cpu().numpy()))
+        assert np.array_equal(got[1][1][1], S0[1].astype(np.float32)), "another request's state is not touched"
+        g = np.exp(-np.exp(a_log)[:, None] * plain.softplus(z + dt).reshape(T, H, d))
+        kk, qq = plain.unit(k.reshape(T, G, d)), plain.unit(q.reshape(T, G, d)) * d ** -0.5
+        for i, n in enumerate(counts):
+            for h in range(H):
+                S = S0[slots[i], h].copy()
+                for t in range(start[i], start[i] + n):
+                    S = g[t, h][:, None] * S
+                    S = S + np.outer(kk[t, h // (H // G)], plain.sigmoid(b[t, h]) * (v[t, h * dv:(h + 1) * dv] - S.T @ kk[t, h // (H // G)]))
+                    for road in range(2):
+                        assert np.abs(got[road][0][t, h] - S.T @ qq[t, h // (H // G)]).max() < 5e-5, (road, i, t)
+                for road in range(2):
+                    assert np.abs(got[road][1][slots[i], h] - S).max() < 5e-5 * max(1.0, np.abs(S).max()), (road, i)
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,G,d,dv,taps,ra,rg", [(4, 2, 20, 12, 4, 6, 10), (1, 1, 24, 40, 1, 1, 1), (3, 1, 10, 6, 6, 3, 7),
                                                  (2, 2, 64, 64, 3, 16, 8), (2, 1, 136, 72, 2, 32, 40), (6, 3, 8, 8, 16, 5, 2),
