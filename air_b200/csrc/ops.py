@@ -1179,7 +1179,8 @@ DELTA_MAX_D = 256        # key channels per head that it takes
 def delta_portions(q, k, v, decay, state, out, portions, chunks, q_scale, beta, a_log, dt_bias, unit_eps=1e-6):
     """linear_scan's SCAN_CHANNEL_DELTA with unit lengths, for whole portions: the tokens of a chunk are computed side by side
     from the state ahead of it (delta_chunks.cu).  portions int32 [L, 4] = (first row, tokens, slot, first chunk), chunks
-    int32 [N, 2] = (first row, tokens): a portion's tokens cut into chunks of DELTA_CHUNK.  32-bit throughout."""
+    int32 [N, 2] = (first row, tokens): a portion's tokens cut into chunks of DELTA_CHUNK.  State, decays and sums
+    are 32-bit; the products with the state run on the tensor cores, their 32-bit operands as two TF32 numbers each."""
     _, H, d, dv = state.shape
     _req(state, "state", (torch.float32,))
     T = out.shape[0]
@@ -1196,7 +1197,8 @@ def delta_portions(q, k, v, decay, state, out, portions, chunks, q_scale, beta, 
     _req(portions, "portions", _I32, (None, 4))
     _req(chunks, "chunks", _I32, (None, 2))
     N = chunks.shape[0]
-    stride = 3 * DELTA_CHUNK * (-(-d // 8) * 8) + -(-d // 8) * 8 + DELTA_CHUNK ** 2 + DELTA_CHUNK * (-(-dv // 4) * 4)
+    wide = -(-d // 16) * 16
+    stride = 3 * DELTA_CHUNK * wide + wide + DELTA_CHUNK ** 2 + DELTA_CHUNK * (-(-dv // 4) * 4)
     scratch = torch.empty(N * H * stride, dtype=torch.float32, device=out.device)
     _check(_get("air_delta_portions")(
         qp, ldq, kp, ldk, vp, ldv, dp, ldd, bp, ldb, a_log.data_ptr(), dt_bias.data_ptr(), state.data_ptr(), out.data_ptr(),

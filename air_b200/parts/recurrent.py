@@ -125,8 +125,8 @@ class ChannelDeltaRule(_StateMixer):
     then o / sqrt(mean(o^2) + eps) * norm, times sigmoid(W_g2 (W_g1 x)) (laid out heads x v_dim), and the output
     projection.  S and the convolutions' last conv - 1 inputs are the request's state, 32-bit, zero at its start.
 
-    Portions of PORTION tokens or more are taken in chunks whose rows are computed side by side (ops.delta_portions), single
-    tokens and shorter portions token by token (ops.linear_scan); both are 32-bit.
+    In a bfloat16 engine portions of PORTION tokens or more are taken in chunks whose rows are computed side by side
+    (ops.delta_portions); everything else goes token by token (ops.linear_scan).
 
     The two products out of a narrow middle take its numbers as they left the first product: a float32 engine in 32-bit,
     a bfloat16 engine as two bfloat16 halves side by side, against the matrix twice (ops.split_bands), so that the
@@ -206,7 +206,8 @@ class ChannelDeltaRule(_StateMixer):
     PORTION = 24
 
     def plan_key(self):
-        return ("channel_delta.chunks", self.PORTION) if self.head_dim <= ops.DELTA_MAX_D else None
+        chunks = self.rt.dtype == torch.bfloat16 and self.head_dim <= ops.DELTA_MAX_D
+        return ("channel_delta.chunks", self.PORTION) if chunks else None
 
     def plan(self, batch: HostBatch) -> Plan:
         """portions [L, 4] = (first row, tokens, slot, first chunk) of the entries of at least PORTION tokens, chunks [N, 2] =
