@@ -19,19 +19,32 @@
 //                              channels lie across the warps and stay in accumulators from the first chunk to the last:
 //                              as a result of one product they are the left operand of the next without a move (the
 //                              instruction's k may run in any order that both operands share).  Every 32-bit operand enters as
-//                              two TF32 numbers, hi + lo, and every product as lo hi + hi lo + hi hi, which keeps 22 bits of
+//                              two TF32 numbers, hi + lo, and every product as lo hi + hi lo + hi hi, which keeps 21 bits of
 //                              the operands: what is left out is of the order of 32-bit rounding.  The next chunk's
-//                              numbers arrive (cp.async) while this one's are used.
+//                              numbers arrive by the copy engine, in two runs of bytes, while this one's are used.
 //
 // What a row is depends on the state and the portion's tokens only.
 #include "common.cuh"
+#include "tma.cuh"
 
 namespace air {
 
 constexpr int DC = 16;              // tokens of a chunk, and columns of a block of the scan
-constexpr int DC_MAX_D = 256;
-constexpr int DC_KLD = 24, DC_RLD = 40, DC_ULD = 24;      // staged rows' strides: four rows fall into different banks
+constexpr int DC_RLD = 40, DC_ULD = 24;      // strides of rows in shared memory: four rows fall into different banks
 constexpr float DC_FLOOR = -60.f;   // a decay of 2^-60 is none: the logarithms' sums stay small enough to be exact
+
+// What a chunk and head leave in the scratch memory, DP the channels filled up to 32, 64, 128 or 256 (zeros), in floats:
+//   rows [32][DP]     W and q exp b; the eight channels from 8 i on of row t stand at 8 (i ^ (t & 3))
+//   keys [DP][16]     (k exp(b_last - b))^T; the eight tokens from 8 i on of channel c stand at 8 (i ^ (c / 2 & 1))
+//   last [DP]         exp b_last
+//   p    [16][16]     swizzled as the keys are
+//   Y^T  [dvp][16]    dvp: dv filled up to a multiple of 16 (zeros)
+// (in this arrangement four rows that a warp reads eight bytes at a time fall into different banks)
+template <int DP> struct DeltaChunk {
+    static constexpr int KEYS = 32 * DP, LAST = KEYS + DC * DP, P = LAST + DP, Y = P + DC * DC;
+};
+__device__ __forceinline__ int dc_row_place(int t, int c) { return c ^ ((t & 3) << 3); }
+__device__ __forceinline__ int dc_key_place(int c, int t) { return t ^ (((c >> 1) & 1) << 3); }
 
 struct DeltaChunkArgs {
     const float* q; int ldq;        // [T, ldq]: head g's d numbers at column g * d, before their unit length and scale
@@ -46,10 +59,10 @@ struct DeltaChunkArgs {
     float* scratch;                 // [N, H, stride]
     float* state;                   // [slots, H, d, dv]
     float* out;                     // [T, H, dv]
-    int H, G, d, dv, dp, dvp;       // dp: d filled up to a multiple of 16, dvp: dv to one of 4
+    int H, G, d, dv, dvp;
     float q_scale, unit_eps;
-    long long stride;               // of a chunk and head: W, q exp b [16, dp] each, (k exp(b_last - b))^T [dp, 16],
-                                    // exp b_last [dp], p [16, 16], Y [16, dvp]
+    long long stride;
+    int* status;
 };
 
 __device__ __forceinline__ float softplus_1(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -60,65 +73,70 @@ __device__ __forceinline__ float power_of_2(float x) {
     return y;
 }
 
+template <int DP>
 __global__ void __launch_bounds__(256, 2) delta_chunk_prepare_kernel(const DeltaChunkArgs p) {
+    constexpr int ld = DP + 4, PER = DP / 32;
     extern __shared__ __align__(16) float smem[];
     __shared__ __align__(16) float sa[DC][DC];
     __shared__ float sbeta[DC];
     pdl_enter(TR_SCAN);
     const int h = blockIdx.y, g = h / (p.H / p.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int q0 = p.chunks[2 * blockIdx.x], n = p.chunks[2 * blockIdx.x + 1];
-    const int d = p.d, dp = p.dp, ld = dp + 4;
+    const int d = p.d;
     float* sk = smem;                       // [16][ld]
     float* sq = sk + DC * ld;
     float* sb = sq + DC * ld;               // the decays' logarithms to the base 2, then their sums
     const float rate = -expf(p.a_log[h]) * 1.4426950408889634f;
-    for (int t = warp; t < DC; t += 8) {    // a warp per token: unit lengths, logarithms
-        const float* kin = p.k + (size_t)(q0 + t) * p.ldk + g * d;
-        const float* qin = p.q + (size_t)(q0 + t) * p.ldq + g * d;
-        const float* zin = p.decay + (size_t)(q0 + t) * p.ldd + h * d;
-        float x[DC_MAX_D / 32], y[DC_MAX_D / 32], ss = 0.f, qs = 0.f;
+    {   // a warp per two tokens: unit lengths, logarithms (both tokens' loads under way at once)
+        float x[2][PER], y[2][PER], z[2][PER];
 #pragma unroll
-        for (int i = 0; i < DC_MAX_D / 32; ++i) {
-            const int c = lane + 32 * i;
-            const bool in = t < n && c < d;
-            x[i] = in ? kin[c] : 0.f;
-            y[i] = in ? qin[c] : 0.f;
-            ss = fmaf(x[i], x[i], ss);
-            qs = fmaf(y[i], y[i], qs);
-            if (c < dp) sb[t * ld + c] = in ? fmaxf(rate * softplus_1(zin[c] + p.dt_bias[h * d + c]), DC_FLOOR) : 0.f;
-        }
-        const float kf = 1.f / sqrtf(warp_sum(ss) + p.unit_eps), qf = p.q_scale / sqrtf(warp_sum(qs) + p.unit_eps);
+        for (int r = 0; r < 2; ++r) {
+            const int t = warp + 8 * r;
 #pragma unroll
-        for (int i = 0; i < DC_MAX_D / 32; ++i) {
-            const int c = lane + 32 * i;
-            if (c < dp) {
-                sk[t * ld + c] = x[i] * kf;
-                sq[t * ld + c] = y[i] * qf;
+            for (int i = 0; i < PER; ++i) {
+                const int c = lane + 32 * i;
+                const bool in = t < n && c < d;
+                x[r][i] = in ? p.k[(size_t)(q0 + t) * p.ldk + g * d + c] : 0.f;
+                y[r][i] = in ? p.q[(size_t)(q0 + t) * p.ldq + g * d + c] : 0.f;
+                z[r][i] = in ? p.decay[(size_t)(q0 + t) * p.ldd + h * d + c] + p.dt_bias[h * d + c] : 0.f;
             }
         }
-        if (lane == 0) sbeta[t] = t < n ? 1.f / (1.f + expf(-p.beta[(size_t)(q0 + t) * p.ldb + h])) : 0.f;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int t = warp + 8 * r;
+            float ss = 0.f, qs = 0.f;
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                ss = fmaf(x[r][i], x[r][i], ss);
+                qs = fmaf(y[r][i], y[r][i], qs);
+                sb[t * ld + lane + 32 * i] = t < n && lane + 32 * i < d ? fmaxf(rate * softplus_1(z[r][i]), DC_FLOOR) : 0.f;
+            }
+            const float kf = 1.f / sqrtf(warp_sum(ss) + p.unit_eps), qf = p.q_scale / sqrtf(warp_sum(qs) + p.unit_eps);
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                sk[t * ld + lane + 32 * i] = x[r][i] * kf;
+                sq[t * ld + lane + 32 * i] = y[r][i] * qf;
+            }
+            if (lane == 0) sbeta[t] = t < n ? 1.f / (1.f + expf(-p.beta[(size_t)(q0 + t) * p.ldb + h])) : 0.f;
+        }
     }
     __syncthreads();
-    for (int c = tid; c < dp; c += 256) {
+    if (tid < DP) {
         float sum = 0.f;
 #pragma unroll
         for (int t = 0; t < DC; ++t) {
-            sum += sb[t * ld + c];
-            sb[t * ld + c] = sum;
+            sum += sb[t * ld + tid];
+            sb[t * ld + tid] = sum;
         }
     }
+    using Place = DeltaChunk<DP>;
     float* base = p.scratch + ((size_t)blockIdx.x * p.H + h) * p.stride;
-    float* W = base;
-    float* Qe = W + (size_t)dp * DC;
-    float* Kt = Qe + (size_t)dp * DC;
-    float* E = Kt + (size_t)DC * dp;
-    float* Pm = E + dp;
-    float* Y = Pm + DC * DC;
+    float* Pm = base + Place::P;
     {
         const int t = tid / DC, s = tid % DC;
         if (s > t) {
             sa[t][s] = 0.f;
-            Pm[tid] = 0.f;
+            Pm[t * DC + dc_key_place(t, s)] = 0.f;
         }
     }
     __syncthreads();
@@ -129,7 +147,8 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_prepare_kernel(const Delta
         while ((i + 1) * (i + 2) / 2 <= square) ++i;
         const int j = square - i * (i + 1) / 2;          // tokens 2 i, 2 i + 1 against 2 j, 2 j + 1
         float a[2][2] = {{0.f, 0.f}, {0.f, 0.f}}, pq[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
-        for (int c = part * 4; c < dp; c += 16) {
+#pragma unroll 2
+        for (int c = part * 4; c < DP; c += 16) {
             float xk[2][4], xq[2][4], xb[2][4], yk[2][4], yb[2][4];
 #pragma unroll
             for (int r = 0; r < 2; ++r) {
@@ -144,8 +163,10 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_prepare_kernel(const Delta
 #pragma unroll
                 for (int s = 0; s < 2; ++s)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {      // (a pair above the diagonal is not kept; its power may not overflow)
-                        const float w = yk[s][e] * power_of_2(fminf(xb[r][e] - yb[s][e], 0.f));
+                    for (int e = 0; e < 4; ++e) {
+                        float x = xb[r][e] - yb[s][e];
+                        if (r < s) x = fminf(x, 0.f);      // (above the diagonal where i = j: not kept, but it may not overflow)
+                        const float w = yk[s][e] * power_of_2(x);
                         a[r][s] = fmaf(xk[r][e], w, a[r][s]);
                         pq[r][s] = fmaf(xq[r][e], w, pq[r][s]);
                     }
@@ -161,16 +182,17 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_prepare_kernel(const Delta
                 const int t = 2 * i + r, u = 2 * j + s;
                 if (part == 0 && tid < 144 && u <= t) {
                     sa[t][u] = u < t ? sbeta[t] * a[r][s] : 0.f;
-                    Pm[t * DC + u] = pq[r][s];
+                    Pm[t * DC + dc_key_place(t, u)] = pq[r][s];
                 }
             }
     }
     __syncthreads();
     // W and Y, a thread per column; what else the scan reads of a channel
-    for (int j = tid; j < dp + p.dvp; j += 256) {
+    for (int j = tid; j < DP + p.dvp; j += 256) {
         float x[DC];
-        if (j < dp) {
+        if (j < DP) {
             const float last = sb[(DC - 1) * ld + j];
+            float* keys = base + Place::KEYS + j * DC;
 #pragma unroll
             for (int t = 0; t < DC; t += 4) {
                 float kv[4];
@@ -178,14 +200,14 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_prepare_kernel(const Delta
                 for (int i = 0; i < 4; ++i) {
                     const float b = sb[(t + i) * ld + j], k = sk[(t + i) * ld + j], e = power_of_2(b);
                     x[t + i] = k * e;
-                    Qe[(size_t)(t + i) * dp + j] = sq[(t + i) * ld + j] * e;
+                    base[(DC + t + i) * DP + dc_row_place(t + i, j)] = sq[(t + i) * ld + j] * e;
                     kv[i] = k * power_of_2(last - b);
                 }
-                store4(Kt + (size_t)j * DC + t, kv);
+                store4(keys + dc_key_place(j, t), kv);
             }
-            E[j] = power_of_2(last);
+            base[Place::LAST + j] = power_of_2(last);
         } else {
-            const int c = j - dp;
+            const int c = j - DP;
 #pragma unroll
             for (int t = 0; t < DC; ++t) x[t] = t < n && c < p.dv ? p.v[(size_t)(q0 + t) * p.ldv + h * p.dv + c] : 0.f;
         }
@@ -202,26 +224,25 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_prepare_kernel(const Delta
             }
             x[t] = sum;
         }
-        float* dst = j < dp ? W + j : Y + (j - dp);
-        const int step = j < dp ? dp : p.dvp;
+        if (j < DP) {
 #pragma unroll
-        for (int t = 0; t < DC; ++t) dst[(size_t)t * step] = x[t];
+            for (int t = 0; t < DC; ++t) base[t * DP + dc_row_place(t, j)] = x[t];
+        } else {
+            float* dst = base + Place::Y + (j - DP) * DC;
+#pragma unroll
+            for (int t = 0; t < DC; t += 4) {
+                const float y[4] = {x[t], x[t + 1], x[t + 2], x[t + 3]};
+                store4(dst + t, y);
+            }
+        }
     }
 }
 
-__device__ __forceinline__ void dc_copy16(void* dst, const void* src, bool valid = true) {
-    const int bytes = valid ? 16 : 0;      // 0: zeros, nothing is read
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src),
-                 "r"(bytes) : "memory");
-}
-
-// A 32-bit number as two TF32 numbers.
+// A 32-bit number as two TF32 numbers: the instruction reads the upper 19 bits of an operand.
 struct Two { uint32_t hi, lo; };
 __device__ __forceinline__ Two two_of(float x) {
-    Two r;
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r.hi) : "f"(x));
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r.lo) : "f"(x - __uint_as_float(r.hi)));
-    return r;
+    const uint32_t hi = __float_as_uint(x) & 0xffffe000u;
+    return Two{hi, __float_as_uint(x - __uint_as_float(hi))};
 }
 __device__ __forceinline__ void mma_tf32(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
                                          uint32_t b1) {
@@ -242,102 +263,107 @@ __device__ __forceinline__ void two_pair(Two (&b)[2], const float* p) {
     b[1] = two_of(v.y);
 }
 
-__host__ __device__ inline int dc_row(int dp) { return dp + (40 - dp % 32) % 32; }      // stride of a staged row of dp numbers
-
-// Eight warps; a warp holds 16 NG channels of the state (dp <= 128 NG), transposed: S[j] is (column g or g + 8 of the block) x
-// (channels 8 j + 2 t, 8 j + 2 t + 1), g = lane / 4, t = lane % 4.
-template <int NG>
+// Eight warps; DP / 16 of them (all, with twice as many each, for DP = 256) hold NJ times 8 channels of the state, transposed:
+// S[j] is (column g or g + 8 of the block) x (channels 8 j + 2 t, 8 j + 2 t + 1), g = lane / 4, t = lane % 4.
+template <int DP>
 __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkArgs p) {
+    constexpr int NJ = DP <= 128 ? 2 : 4, HOLD = DP / (8 * NJ);      // 8-channel tiles per warp, warps that hold channels
+    constexpr int BUF = DeltaChunk<DP>::Y + DC * DC;                 // floats of a buffer: the chunk's, and 16 columns of Y
+    using Place = DeltaChunk<DP>;
     extern __shared__ __align__(16) float smem[];
-    pdl_enter(TR_SCAN);
+    __shared__ __align__(8) uint64_t full[2];
+    __shared__ int gave_up;
+    float* red = smem + 2 * BUF;            // [HOLD warps][16 columns][DC_RLD]: 32 sums over a warp's channels
+    float* UT = red + 8 * DC * DC_RLD;      // [16 columns][DC_ULD]: U transposed
+    float* OT = UT + DC * DC_ULD;           // the same of o's first part
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t2 = 2 * (lane & 3);
+    if (tid == 0) {
+        mbar_init(&full[0], 1);
+        mbar_init(&full[1], 1);
+        gave_up = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    pdl_enter(TR_SCAN);
     const int h = blockIdx.y, col0 = blockIdx.x * DC;
     const int* por = p.portions + 4 * blockIdx.z;
     const int row0 = por[0], tokens = por[1], slot = por[2], chunk0 = por[3];
     if (slot < 0) return;
-    const int dp = p.dp, ldw = dc_row(dp), chunks = (tokens + DC - 1) / DC;
-    const int buf_floats = 2 * DC * ldw + dp * DC_KLD + dp + 2 * DC * DC;
-    float* red = smem + 2 * buf_floats;     // [8 warps][16 columns][DC_RLD]: 32 sums over a warp's channels
-    float* UT = red + 8 * DC * DC_RLD;      // [16 columns][DC_ULD]: U transposed
-    float* OT = UT + DC * DC_ULD;           // the same of o's first part
-    auto stage = [&](int i, int b) {
+    const int chunks = (tokens + DC - 1) / DC;
+    auto stage = [&](int i) {               // (one thread)
         const float* src = p.scratch + ((size_t)(chunk0 + i) * p.H + h) * p.stride;
-        float* dst = smem + b * buf_floats;
-        const int per = dp / 4;             // pieces of a row
-        for (int x = tid; x < 2 * DC * per; x += 256) dc_copy16(dst + (x / per) * ldw + 4 * (x % per), src + 4 * (size_t)x);
-        src += 2 * (size_t)DC * dp;
-        dst += 2 * DC * ldw;
-        for (int x = tid; x < dp * 4; x += 256) dc_copy16(dst + (x >> 2) * DC_KLD + 4 * (x & 3), src + 4 * (size_t)x);
-        src += (size_t)dp * DC;
-        dst += dp * DC_KLD;
-        const int rest = (dp + DC * DC) / 4;
-        for (int x = tid; x < rest; x += 256) dc_copy16(dst + 4 * x, src + 4 * (size_t)x);
-        src += 4 * (size_t)rest;
-        dst += 4 * rest;
-        if (tid < DC * 4) {                 // this block's columns of Y
-            const int t = tid >> 2, c = col0 + 4 * (tid & 3);
-            const bool in = c < p.dvp;
-            dc_copy16(dst + t * DC + 4 * (tid & 3), src + (size_t)t * p.dvp + (in ? c : 0), in);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        float* dst = smem + (i & 1) * BUF;
+        mbar_expect_tx(&full[i & 1], BUF * 4);
+        bulk_load(dst, src, Place::Y * 4, &full[i & 1]);
+        bulk_load(dst + Place::Y, src + Place::Y + col0 * DC, DC * DC * 4, &full[i & 1]);
     };
-    stage(0, 0);
-    const int r0 = warp * 16 * NG;
+    if (tid == 0) stage(0);
+    const int r0 = warp * 8 * NJ;
     float* st = p.state + ((size_t)slot * p.H + h) * p.d * p.dv;
-    float S[2 * NG][4];
+    float S[NJ][4];
 #pragma unroll
-    for (int j = 0; j < 2 * NG; ++j)
+    for (int j = 0; j < NJ; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int r = r0 + 8 * j + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
             S[j][e] = r < p.d && c < p.dv ? st[(size_t)r * p.dv + c] : 0.f;
         }
     for (int i = 0; i < chunks; ++i) {
-        const float* W = smem + (i & 1) * buf_floats;      // [32][ldw]: W, then q exp b
-        const float* Kt = W + 2 * DC * ldw;
-        const float* E = Kt + dp * DC_KLD;
-        const float* Pm = E + dp;
-        const float* Y = Pm + DC * DC;
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();                     // this chunk's numbers are there; the other buffer is free
-        if (i + 1 < chunks) stage(i + 1, (i + 1) & 1);
-        if (r0 < dp) {
+        const float* buf = smem + (i & 1) * BUF;
+        const bool ok = mbar_wait(&full[i & 1], (i >> 1) & 1, &gave_up);
+        // this chunk's numbers are there and everybody is done with the other buffer
+        if (__syncthreads_or(!ok)) {
+            for (int x = 0; x < 32; ++x) __nanosleep(2000);      // (a copy on its way may still land)
+            if (tid == 0 && p.status) atomicExch(p.status, 9);
+            return;
+        }
+        if (tid == 0 && i + 1 < chunks) stage(i + 1);
+        if (warp < HOLD) {
             float acc[4][4];
 #pragma unroll
             for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+            const float* rows = buf + g * DP;
 #pragma unroll
-            for (int j = 0; j < 2 * NG; ++j) {
-                if (r0 + 8 * j >= dp) break;
+            for (int j = 0; j < NJ; ++j) {
                 const Two a[4] = {two_of(S[j][0]), two_of(S[j][2]), two_of(S[j][1]), two_of(S[j][3])};
+                const float* at = rows + dc_row_place(g, r0 + 8 * j) + t2;
+                Two b[4][2];
 #pragma unroll
-                for (int x = 0; x < 4; ++x) {
-                    Two b[2];
-                    two_pair(b, W + (8 * x + g) * ldw + r0 + 8 * j + t2);
-                    mma_32(acc[x], a, b);
-                }
+                for (int x = 0; x < 4; ++x) two_pair(b[x], at + 8 * x * DP);
+                // (the four sums in turn: a product does not wait for the one before it)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].lo, a[1].lo, a[2].lo, a[3].lo, b[x][0].hi, b[x][1].hi);
+#pragma unroll
+                for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].lo, b[x][1].lo);
+#pragma unroll
+                for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].hi, b[x][1].hi);
             }
-            float* mine = red + warp * DC * DC_RLD;
+            float* mine = red + (warp * DC + g) * DC_RLD + t2;
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
-                *reinterpret_cast<float2*>(mine + g * DC_RLD + 8 * x + t2) = make_float2(acc[x][0], acc[x][1]);
-                *reinterpret_cast<float2*>(mine + (g + 8) * DC_RLD + 8 * x + t2) = make_float2(acc[x][2], acc[x][3]);
+                *reinterpret_cast<float2*>(mine + 8 * x) = make_float2(acc[x][0], acc[x][1]);
+                *reinterpret_cast<float2*>(mine + 8 * DC_RLD + 8 * x) = make_float2(acc[x][2], acc[x][3]);
             }
         }
         __syncthreads();
         {   // the warps' sums in order: U = Y - W S (tokens 0 .. 15 of 32), o's first part (the others)
             const int c = tid >> 4, t = 2 * (tid & 15);
-            float2 sum = make_float2(0.f, 0.f);
+            const float* from = red + c * DC_RLD + t;
+            float2 v[HOLD];
 #pragma unroll
-            for (int w = 0; w < 8; ++w) {
-                if (w * 16 * NG >= dp) break;
-                const float2 v = *reinterpret_cast<const float2*>(red + w * DC * DC_RLD + c * DC_RLD + t);
-                sum.x += v.x;
-                sum.y += v.y;
+            for (int w = 0; w < HOLD; ++w) v[w] = *reinterpret_cast<const float2*>(from + w * DC * DC_RLD);
+            float2 sum = v[0];
+#pragma unroll
+            for (int w = 1; w < HOLD; ++w) {
+                sum.x += v[w].x;
+                sum.y += v[w].y;
             }
-            if (t < DC)
-                *reinterpret_cast<float2*>(UT + c * DC_ULD + t) = make_float2(Y[t * DC + c] - sum.x, Y[(t + 1) * DC + c] - sum.y);
-            else
+            if (t < DC) {
+                const float2 y = *reinterpret_cast<const float2*>(buf + Place::Y + c * DC + t);
+                *reinterpret_cast<float2*>(UT + c * DC_ULD + t) = make_float2(y.x - sum.x, y.y - sum.y);
+            } else {
                 *reinterpret_cast<float2*>(OT + c * DC_ULD + t - DC) = sum;
+            }
         }
         __syncthreads();
         Two u[2][4];                         // U transposed, tokens 0 .. 7 and 8 .. 15
@@ -348,27 +374,39 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
             two_pair(hi, UT + (g + 8) * DC_ULD + 8 * x + t2);
             u[x][0] = lo[0]; u[x][1] = hi[0]; u[x][2] = lo[1]; u[x][3] = hi[1];
         }
+        const int swap = dc_key_place(g, 0);      // (rows 8 j + g: the tile does not matter)
+        if (warp < HOLD) {
+            Two b[NJ][2][2];
 #pragma unroll
-        for (int j = 0; j < 2 * NG; ++j) {
-            if (r0 + 8 * j >= dp) break;
-            const float2 e = *reinterpret_cast<const float2*>(E + r0 + 8 * j + t2);
-            S[j][0] *= e.x; S[j][1] *= e.y; S[j][2] *= e.x; S[j][3] *= e.y;
+            for (int j = 0; j < NJ; ++j) {
+                const float2 e = *reinterpret_cast<const float2*>(buf + Place::LAST + r0 + 8 * j + t2);
+                S[j][0] *= e.x; S[j][1] *= e.y; S[j][2] *= e.x; S[j][3] *= e.y;
 #pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                Two b[2];
-                two_pair(b, Kt + (r0 + 8 * j + g) * DC_KLD + 8 * x + t2);
-                mma_32(S[j], u[x], b);
+                for (int x = 0; x < 2; ++x)
+                    two_pair(b[j][x], buf + Place::KEYS + (r0 + 8 * j + g) * DC + ((8 * x) ^ swap) + t2);
             }
+#pragma unroll
+            for (int x = 0; x < 2; ++x)
+#pragma unroll
+                for (int part = 0; part < 3; ++part)
+#pragma unroll
+                    for (int j = 0; j < NJ; ++j) {
+                        const Two(&a)[4] = u[x];
+                        const Two(&k)[2] = b[j][x];
+                        if (part == 0) mma_tf32(S[j], a[0].lo, a[1].lo, a[2].lo, a[3].lo, k[0].hi, k[1].hi);
+                        if (part == 1) mma_tf32(S[j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].lo, k[1].lo);
+                        if (part == 2) mma_tf32(S[j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].hi, k[1].hi);
+                    }
         }
         if (warp >= 6) {                     // o: tokens 0 .. 7 and 8 .. 15
             const int t0 = 8 * (warp - 6);
-            float2 lo = *reinterpret_cast<const float2*>(OT + g * DC_ULD + t0 + t2);
-            float2 hi = *reinterpret_cast<const float2*>(OT + (g + 8) * DC_ULD + t0 + t2);
+            const float2 lo = *reinterpret_cast<const float2*>(OT + g * DC_ULD + t0 + t2);
+            const float2 hi = *reinterpret_cast<const float2*>(OT + (g + 8) * DC_ULD + t0 + t2);
             float o[4] = {lo.x, lo.y, hi.x, hi.y};
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
                 Two b[2];
-                two_pair(b, Pm + (t0 + g) * DC + 8 * x + t2);
+                two_pair(b, buf + Place::P + (t0 + g) * DC + ((8 * x) ^ swap) + t2);
                 mma_32(o, u[x], b);
             }
 #pragma unroll
@@ -378,59 +416,68 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
             }
         }
     }
+    if (warp < HOLD)
 #pragma unroll
-    for (int j = 0; j < 2 * NG; ++j)
+        for (int j = 0; j < NJ; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int r = r0 + 8 * j + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
-            if (r < p.d && c < p.dv) st[(size_t)r * p.dv + c] = S[j][e];
-        }
+            for (int e = 0; e < 4; ++e) {
+                const int r = r0 + 8 * j + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
+                if (r < p.d && c < p.dv) st[(size_t)r * p.dv + c] = S[j][e];
+            }
 }
 
-}  // namespace air
-
-// scratch: float32 [N, H, 3 * 16 dp + dp + 256 + 16 dvp] with dp = d filled up to a multiple of 16, dvp = dv to one of 4.
-// Rows and slots as the lists say; d up to 256.
-AIR_API int air_delta_portions(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* decay,
-                               int ldd, const float* beta, int ldb, const float* a_log, const float* dt_bias, float* state,
-                               float* out, const int* portions, int L, const int* chunks, int N, float* scratch, int H, int G,
-                               int d, int dv, float q_scale, float unit_eps, cudaStream_t stream) {
-    using namespace air;
-    if (L <= 0 || N <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || d <= 0 || d > DC_MAX_D || dv <= 0 || H > 65535 || L > 65535 || !scratch ||
-        ((uintptr_t)scratch & 15))
-        return AIR_ERR_BAD_ARGUMENT;
-    DeltaChunkArgs a;
-    a.q = q; a.ldq = ldq; a.k = k; a.ldk = ldk; a.v = v; a.ldv = ldv; a.decay = decay; a.ldd = ldd; a.beta = beta; a.ldb = ldb;
-    a.a_log = a_log; a.dt_bias = dt_bias; a.chunks = chunks; a.portions = portions; a.scratch = scratch; a.state = state;
-    a.out = out; a.H = H; a.G = G; a.d = d; a.dv = dv; a.dp = (d + 15) / 16 * 16; a.dvp = (dv + 3) / 4 * 4;
-    a.q_scale = q_scale; a.unit_eps = unit_eps;
-    a.stride = 3ll * a.dp * DC + a.dp + DC * DC + (long long)DC * a.dvp;
-    const size_t smem1 = sizeof(float) * 3 * DC * (size_t)(a.dp + 4);
+template <int DP>
+static int launch_delta_chunks(const DeltaChunkArgs& args, int N, int L, cudaStream_t stream) {
+    DeltaChunkArgs a = args;
+    a.dvp = (a.dv + 15) / 16 * 16;
+    a.stride = DeltaChunk<DP>::Y + (long long)DC * a.dvp;
+    const size_t smem1 = sizeof(float) * 3 * DC * (DP + 4);
     if (smem1 > 44 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        cudaError_t e = cudaFuncSetAttribute(delta_chunk_prepare_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
         if (e != cudaSuccess) return (int)e;
     }
-    int rc = launch(delta_chunk_prepare_kernel, dim3(N, H), 256, smem1, stream, a);
+    int rc = launch(delta_chunk_prepare_kernel<DP>, dim3(N, a.H), 256, smem1, stream, a);
     if (rc) return rc;
-    size_t smem2 = sizeof(float) * (2 * (size_t)(2 * DC * dc_row(a.dp) + a.dp * DC_KLD + a.dp + 2 * DC * DC) +
-                                    8 * DC * DC_RLD + 2 * DC * DC_ULD);
-    const dim3 grid((dv + DC - 1) / DC, H, L);
+    size_t smem2 = sizeof(float) * (2 * (DeltaChunk<DP>::Y + DC * DC) + 8 * DC * DC_RLD + 2 * DC * DC_ULD);
+    const dim3 grid(a.dvp / DC, a.H, L);
     // (as for the scan token by token: the blocks start when their predecessor has ended, and spread over the SMs)
     int sms = 148, dev = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     const long long blocks = (long long)grid.x * grid.y * grid.z;
     if (blocks <= sms && smem2 < 120 * 1024) smem2 = 120 * 1024;
-    auto kernel = a.dp <= 128 ? delta_chunk_scan_kernel<1> : delta_chunk_scan_kernel<2>;
-    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
+    cudaError_t e = cudaFuncSetAttribute(delta_chunk_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
     if (e != cudaSuccess) return (int)e;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = dim3(256);
     cfg.dynamicSmemBytes = smem2;
     cfg.stream = stream;
-    return (int)cudaLaunchKernelEx(&cfg, kernel, a);
+    return (int)cudaLaunchKernelEx(&cfg, delta_chunk_scan_kernel<DP>, a);
+}
+
+}  // namespace air
+
+// scratch: float32 [N, H, 49 DP + 256 + 16 dvp] with DP = d filled up to 32, 64, 128 or 256, dvp = dv to a multiple of 16.
+// Rows and slots as the lists say; d up to 256.
+AIR_API int air_delta_portions(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* decay,
+                               int ldd, const float* beta, int ldb, const float* a_log, const float* dt_bias, float* state,
+                               float* out, const int* portions, int L, const int* chunks, int N, float* scratch, int H, int G,
+                               int d, int dv, float q_scale, float unit_eps, int* status, cudaStream_t stream) {
+    using namespace air;
+    if (L <= 0 || N <= 0) return 0;
+    if (H <= 0 || G <= 0 || H % G || d <= 0 || d > 256 || dv <= 0 || H > 65535 || L > 65535 || !scratch ||
+        ((uintptr_t)scratch & 15))
+        return AIR_ERR_BAD_ARGUMENT;
+    DeltaChunkArgs a;
+    a.q = q; a.ldq = ldq; a.k = k; a.ldk = ldk; a.v = v; a.ldv = ldv; a.decay = decay; a.ldd = ldd; a.beta = beta; a.ldb = ldb;
+    a.a_log = a_log; a.dt_bias = dt_bias; a.chunks = chunks; a.portions = portions; a.scratch = scratch; a.state = state;
+    a.out = out; a.H = H; a.G = G; a.d = d; a.dv = dv; a.dvp = 0; a.q_scale = q_scale; a.unit_eps = unit_eps; a.stride = 0;
+    a.status = status;
+    if (d <= 32) return launch_delta_chunks<32>(a, N, L, stream);
+    if (d <= 64) return launch_delta_chunks<64>(a, N, L, stream);
+    if (d <= 128) return launch_delta_chunks<128>(a, N, L, stream);
+    return launch_delta_chunks<256>(a, N, L, stream);
 }
 
 AIR_API int air_trace_set_delta_chunks(unsigned long long* buffer) { return air::set_trace_here(buffer); }

@@ -91,7 +91,7 @@ _SIGNATURES = {
                         c_void_p, c_int, c_float, c_void_p],
     "air_delta_portions": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                           c_int, c_float, c_float, c_void_p],
+                           c_int, c_float, c_float, c_void_p, c_void_p],
     "air_gated_rmsnorm": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float,
                           c_int, c_void_p],
     "air_polynorm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float,
@@ -1176,7 +1176,8 @@ DELTA_CHUNK = 16         # tokens of a chunk of delta_portions
 DELTA_MAX_D = 256        # key channels per head that it takes
 
 
-def delta_portions(q, k, v, decay, state, out, portions, chunks, q_scale, beta, a_log, dt_bias, unit_eps=1e-6):
+def delta_portions(q, k, v, decay, state, out, portions, chunks, q_scale, beta, a_log, dt_bias, unit_eps=1e-6,
+                   status=None):
     """linear_scan's SCAN_CHANNEL_DELTA with unit lengths, for whole portions: the tokens of a chunk are computed side by side
     from the state ahead of it (delta_chunks.cu).  portions int32 [L, 4] = (first row, tokens, slot, first chunk), chunks
     int32 [N, 2] = (first row, tokens): a portion's tokens cut into chunks of DELTA_CHUNK.  State, decays and sums
@@ -1197,13 +1198,13 @@ def delta_portions(q, k, v, decay, state, out, portions, chunks, q_scale, beta, 
     _req(portions, "portions", _I32, (None, 4))
     _req(chunks, "chunks", _I32, (None, 2))
     N = chunks.shape[0]
-    wide = -(-d // 16) * 16
-    stride = 3 * DELTA_CHUNK * wide + wide + DELTA_CHUNK ** 2 + DELTA_CHUNK * (-(-dv // 4) * 4)
+    wide = next(w for w in (32, 64, 128, 256) if d <= w)
+    stride = 49 * wide + 256 + 16 * (-(-dv // 16) * 16)
     scratch = torch.empty(N * H * stride, dtype=torch.float32, device=out.device)
     _check(_get("air_delta_portions")(
         qp, ldq, kp, ldk, vp, ldv, dp, ldd, bp, ldb, a_log.data_ptr(), dt_bias.data_ptr(), state.data_ptr(), out.data_ptr(),
         portions.data_ptr(), portions.shape[0], chunks.data_ptr(), N, scratch.data_ptr(), H, G, d, dv, float(q_scale),
-        float(unit_eps), _stream()), "delta_portions")
+        float(unit_eps), _ptr(status), _stream()), "delta_portions")
     global launches
     launches += 1
     return out

@@ -305,7 +305,8 @@ class Engine:
                    5: "a wait inside the decode attention kernel ran out",
                    6: "a wait inside the prefill attention kernel ran out",
                    7: "a wait inside the tcgen05 prefill attention kernel ran out",
-                   8: "the tile list of the tcgen05 prefill attention kernel is not in pairs of one request"}
+                   8: "the tile list of the tcgen05 prefill attention kernel is not in pairs of one request",
+                   9: "a wait inside the delta rule's chunk kernel ran out"}
 
     def read_status(self) -> int:
         """The device's error word (a synchronisation): 0, or the code of what a kernel could not do."""

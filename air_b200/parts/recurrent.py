@@ -255,7 +255,7 @@ class ChannelDeltaRule(_StateMixer):
             if plan.short:
                 ops.linear_scan(ops.SCAN_CHANNEL_DELTA, *bands, ctx.q_start, plan.short_slots, plan.short_seq, unit=True,
                                 **numbers)
-            ops.delta_portions(*bands, plan.portions, plan.chunks, **numbers)
+            ops.delta_portions(*bands, plan.portions, plan.chunks, status=ctx.status, **numbers)
         return self._finish(o, gate, ctx, sigmoid=True)
 
 
