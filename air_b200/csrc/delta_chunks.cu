@@ -74,7 +74,7 @@ __device__ __forceinline__ float power_of_2(float x) {
 }
 
 template <int DP>
-__global__ void __launch_bounds__(256, 2) delta_chunk_prepare_kernel(const DeltaChunkArgs p) {
+__global__ void __launch_bounds__(256, DP <= 128 ? 3 : 2) delta_chunk_prepare_kernel(const DeltaChunkArgs p) {
     constexpr int ld = DP + 4, PER = DP / 32;
     extern __shared__ __align__(16) float smem[];
     __shared__ __align__(16) float sa[DC][DC];
@@ -244,18 +244,14 @@ __device__ __forceinline__ Two two_of(float x) {
     const uint32_t hi = __float_as_uint(x) & 0xffffe000u;
     return Two{hi, __float_as_uint(x - __uint_as_float(hi))};
 }
+// c += a b; with k in the order that the accumulators have: a holds (row g, k 2t), (g + 8, 2t), (g, 2t + 1), (g + 8, 2t + 1), b
+// holds (k 2t, column g), (2t + 1, g)
 __device__ __forceinline__ void mma_tf32(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
                                          uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
                  "{%0, %1, %2, %3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-// c += a b with both operands 32-bit; a: (row g, k 2t), (g + 8, 2t), (g, 2t + 1), (g + 8, 2t + 1); b: (k 2t, column g), (2t + 1, g)
-__device__ __forceinline__ void mma_32(float (&c)[4], const Two (&a)[4], const Two (&b)[2]) {
-    mma_tf32(c, a[0].lo, a[1].lo, a[2].lo, a[3].lo, b[0].hi, b[1].hi);
-    mma_tf32(c, a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[0].lo, b[1].lo);
-    mma_tf32(c, a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[0].hi, b[1].hi);
 }
 __device__ __forceinline__ void two_pair(Two (&b)[2], const float* p) {
     const float2 v = *reinterpret_cast<const float2*>(p);
@@ -319,9 +315,12 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
         }
         if (tid == 0 && i + 1 < chunks) stage(i + 1);
         if (warp < HOLD) {
-            float acc[4][4];
+            // (a sum per kind of product: the chain of products that wait for one another is a third as long)
+            float acc[4][4], part[2][4][4];
 #pragma unroll
-            for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+            for (int x = 0; x < 4; ++x)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[x][e] = part[0][x][e] = part[1][x][e] = 0.f;
             const float* rows = buf + g * DP;
 #pragma unroll
             for (int j = 0; j < NJ; ++j) {
@@ -330,14 +329,17 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
                 Two b[4][2];
 #pragma unroll
                 for (int x = 0; x < 4; ++x) two_pair(b[x], at + 8 * x * DP);
-                // (the four sums in turn: a product does not wait for the one before it)
 #pragma unroll
-                for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].lo, a[1].lo, a[2].lo, a[3].lo, b[x][0].hi, b[x][1].hi);
-#pragma unroll
-                for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].lo, b[x][1].lo);
-#pragma unroll
-                for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].hi, b[x][1].hi);
+                for (int x = 0; x < 4; ++x) {
+                    mma_tf32(part[0][x], a[0].lo, a[1].lo, a[2].lo, a[3].lo, b[x][0].hi, b[x][1].hi);
+                    mma_tf32(part[1][x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].lo, b[x][1].lo);
+                    mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].hi, b[x][1].hi);
+                }
             }
+#pragma unroll
+            for (int x = 0; x < 4; ++x)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[x][e] += part[0][x][e] + part[1][x][e];
             float* mine = red + (warp * DC + g) * DC_RLD + t2;
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
@@ -375,12 +377,31 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
             u[x][0] = lo[0]; u[x][1] = hi[0]; u[x][2] = lo[1]; u[x][3] = hi[1];
         }
         const int swap = dc_key_place(g, 0);      // (rows 8 j + g: the tile does not matter)
+        // o of tokens 0 .. 7 (warp 6) and 8 .. 15 (warp 7), ahead of the state's products, which do not wait for it
+        const int t0 = 8 * (warp & 1);
+        float o[4] = {0.f, 0.f, 0.f, 0.f}, o_part[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        if (warp >= 6) {
+            const float2 lo = *reinterpret_cast<const float2*>(OT + g * DC_ULD + t0 + t2);
+            const float2 hi = *reinterpret_cast<const float2*>(OT + (g + 8) * DC_ULD + t0 + t2);
+            o[0] = lo.x; o[1] = lo.y; o[2] = hi.x; o[3] = hi.y;
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                Two b[2];
+                two_pair(b, buf + Place::P + (t0 + g) * DC + ((8 * x) ^ swap) + t2);
+                mma_tf32(o_part[0], u[x][0].lo, u[x][1].lo, u[x][2].lo, u[x][3].lo, b[0].hi, b[1].hi);
+                mma_tf32(o_part[1], u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, b[0].lo, b[1].lo);
+                mma_tf32(o, u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, b[0].hi, b[1].hi);
+            }
+        }
         if (warp < HOLD) {
             Two b[NJ][2][2];
+            float part[2][NJ][4];
 #pragma unroll
             for (int j = 0; j < NJ; ++j) {
                 const float2 e = *reinterpret_cast<const float2*>(buf + Place::LAST + r0 + 8 * j + t2);
                 S[j][0] *= e.x; S[j][1] *= e.y; S[j][2] *= e.x; S[j][3] *= e.y;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) part[0][j][k] = part[1][j][k] = 0.f;
 #pragma unroll
                 for (int x = 0; x < 2; ++x)
                     two_pair(b[j][x], buf + Place::KEYS + (r0 + 8 * j + g) * DC + ((8 * x) ^ swap) + t2);
@@ -388,31 +409,24 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
 #pragma unroll
             for (int x = 0; x < 2; ++x)
 #pragma unroll
-                for (int part = 0; part < 3; ++part)
+                for (int j = 0; j < NJ; ++j) {
+                    const Two(&a)[4] = u[x];
+                    const Two(&k)[2] = b[j][x];
+                    mma_tf32(part[0][j], a[0].lo, a[1].lo, a[2].lo, a[3].lo, k[0].hi, k[1].hi);
+                    mma_tf32(part[1][j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].lo, k[1].lo);
+                    mma_tf32(S[j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].hi, k[1].hi);
+                }
 #pragma unroll
-                    for (int j = 0; j < NJ; ++j) {
-                        const Two(&a)[4] = u[x];
-                        const Two(&k)[2] = b[j][x];
-                        if (part == 0) mma_tf32(S[j], a[0].lo, a[1].lo, a[2].lo, a[3].lo, k[0].hi, k[1].hi);
-                        if (part == 1) mma_tf32(S[j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].lo, k[1].lo);
-                        if (part == 2) mma_tf32(S[j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].hi, k[1].hi);
-                    }
+            for (int j = 0; j < NJ; ++j)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) S[j][k] += part[0][j][k] + part[1][j][k];
         }
-        if (warp >= 6) {                     // o: tokens 0 .. 7 and 8 .. 15
-            const int t0 = 8 * (warp - 6);
-            const float2 lo = *reinterpret_cast<const float2*>(OT + g * DC_ULD + t0 + t2);
-            const float2 hi = *reinterpret_cast<const float2*>(OT + (g + 8) * DC_ULD + t0 + t2);
-            float o[4] = {lo.x, lo.y, hi.x, hi.y};
-#pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                Two b[2];
-                two_pair(b, buf + Place::P + (t0 + g) * DC + ((8 * x) ^ swap) + t2);
-                mma_32(o, u[x], b);
-            }
+        if (warp >= 6) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int t = i * DC + t0 + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
-                if (t < tokens && c < p.dv) p.out[((size_t)(row0 + t) * p.H + h) * p.dv + c] = o[e];
+                if (t < tokens && c < p.dv)
+                    p.out[((size_t)(row0 + t) * p.H + h) * p.dv + c] = o[e] + (o_part[0][e] + o_part[1][e]);
             }
         }
     }
