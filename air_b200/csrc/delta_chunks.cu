@@ -259,23 +259,26 @@ __device__ __forceinline__ void two_pair(Two (&b)[2], const float* p) {
     b[1] = two_of(v.y);
 }
 
-// Eight warps; DP / 16 of them (all, with twice as many each, for DP = 256) hold NJ times 8 channels of the state, transposed:
-// S[j] is (column g or g + 8 of the block) x (channels 8 j + 2 t, 8 j + 2 t + 1), g = lane / 4, t = lane % 4.
+constexpr int DC_WARPS = 4;         // one per scheduler: the products follow one another in the tensor pipe as fast as it takes them,
+                                    // and the fewer warps share the channels, the fewer sums cross between them
+constexpr int DC_STAGES = 2;
+
+// A warp holds NJ tiles of 8 channels of the state, transposed: S[j] is (column g or g + 8 of the block) x (channels 8 j + 2 t,
+// 8 j + 2 t + 1), g = lane / 4, t = lane % 4.
 template <int DP>
-__global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkArgs p) {
-    constexpr int NJ = DP <= 128 ? 2 : 4, HOLD = DP / (8 * NJ);      // 8-channel tiles per warp, warps that hold channels
-    constexpr int BUF = DeltaChunk<DP>::Y + DC * DC;                 // floats of a buffer: the chunk's, and 16 columns of Y
+__global__ void __launch_bounds__(DC_WARPS * 32) delta_chunk_scan_kernel(const DeltaChunkArgs p) {
+    constexpr int NJ = DP / (8 * DC_WARPS);
+    constexpr int STAGES = DC_STAGES, BUF = DeltaChunk<DP>::Y + DC * DC;      // floats of a buffer: the chunk's, and 16 columns of Y
     using Place = DeltaChunk<DP>;
     extern __shared__ __align__(16) float smem[];
-    __shared__ __align__(8) uint64_t full[2];
+    __shared__ __align__(8) uint64_t full[STAGES];
     __shared__ int gave_up;
-    float* red = smem + 2 * BUF;            // [HOLD warps][16 columns][DC_RLD]: 32 sums over a warp's channels
-    float* UT = red + 8 * DC * DC_RLD;      // [16 columns][DC_ULD]: U transposed
+    float* red = smem + STAGES * BUF;       // [warps][16 columns][DC_RLD]: 32 sums over a warp's channels
+    float* UT = red + DC_WARPS * DC * DC_RLD;   // [16 columns][DC_ULD]: U transposed
     float* OT = UT + DC * DC_ULD;           // the same of o's first part
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t2 = 2 * (lane & 3);
     if (tid == 0) {
-        mbar_init(&full[0], 1);
-        mbar_init(&full[1], 1);
+        for (int i = 0; i < STAGES; ++i) mbar_init(&full[i], 1);
         gave_up = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -288,12 +291,14 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
     const int chunks = (tokens + DC - 1) / DC;
     auto stage = [&](int i) {               // (one thread)
         const float* src = p.scratch + ((size_t)(chunk0 + i) * p.H + h) * p.stride;
-        float* dst = smem + (i & 1) * BUF;
-        mbar_expect_tx(&full[i & 1], BUF * 4);
-        bulk_load(dst, src, Place::Y * 4, &full[i & 1]);
-        bulk_load(dst + Place::Y, src + Place::Y + col0 * DC, DC * DC * 4, &full[i & 1]);
+        float* dst = smem + (i % STAGES) * BUF;
+        uint64_t* bar = &full[i % STAGES];
+        mbar_expect_tx(bar, BUF * 4);
+        bulk_load(dst, src, Place::Y * 4, bar);
+        bulk_load(dst + Place::Y, src + Place::Y + col0 * DC, DC * DC * 4, bar);
     };
-    if (tid == 0) stage(0);
+    if (tid == 0)
+        for (int i = 0; i < min(STAGES - 1, chunks); ++i) stage(i);
     const int r0 = warp * 8 * NJ;
     float* st = p.state + ((size_t)slot * p.H + h) * p.d * p.dv;
     float S[NJ][4];
@@ -304,68 +309,61 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
             const int r = r0 + 8 * j + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
             S[j][e] = r < p.d && c < p.dv ? st[(size_t)r * p.dv + c] : 0.f;
         }
+    // places that do not change from chunk to chunk
+    const int rows_at = g * DP + t2, swap = dc_key_place(g, 0);      // (of rows 8 j + g: the tile does not matter)
+    float* mine = red + (warp * DC + g) * DC_RLD + t2;
+    const int sum_c = tid >> 3, sum_t = 4 * (tid & 7);               // the four sums that this thread completes: column, rows
+    const float* sum_from = red + sum_c * DC_RLD + sum_t;
+    float* sum_to = (sum_t < DC ? UT : OT - DC) + sum_c * DC_ULD + sum_t;
+    const int t0 = 8 * (warp & 1);                                   // warps 0 and 1: the tokens whose o they finish
+    float* out = p.out + ((size_t)(row0 + t0 + t2) * p.H + h) * p.dv + col0 + g;
+    const size_t out_row = (size_t)p.H * p.dv;
     for (int i = 0; i < chunks; ++i) {
-        const float* buf = smem + (i & 1) * BUF;
-        const bool ok = mbar_wait(&full[i & 1], (i >> 1) & 1, &gave_up);
-        // this chunk's numbers are there and everybody is done with the other buffer
+        const float* buf = smem + (i % STAGES) * BUF;
+        const bool ok = mbar_wait(&full[i % STAGES], (i / STAGES) & 1, &gave_up);
+        // this chunk's numbers are there and everybody is done with the chunk before it
         if (__syncthreads_or(!ok)) {
             for (int x = 0; x < 32; ++x) __nanosleep(2000);      // (a copy on its way may still land)
             if (tid == 0 && p.status) atomicExch(p.status, 9);
             return;
         }
-        if (tid == 0 && i + 1 < chunks) stage(i + 1);
-        if (warp < HOLD) {
-            // (a sum per kind of product: the chain of products that wait for one another is a third as long)
-            float acc[4][4], part[2][4][4];
+        if (tid == 0 && i + STAGES - 1 < chunks) stage(i + STAGES - 1);
+        float acc[4][4];
 #pragma unroll
-            for (int x = 0; x < 4; ++x)
+        for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
 #pragma unroll
-                for (int e = 0; e < 4; ++e) acc[x][e] = part[0][x][e] = part[1][x][e] = 0.f;
-            const float* rows = buf + g * DP;
+        for (int j = 0; j < NJ; ++j) {
+            const Two a[4] = {two_of(S[j][0]), two_of(S[j][2]), two_of(S[j][1]), two_of(S[j][3])};
+            const float* at = buf + rows_at + dc_row_place(g, r0 + 8 * j);
+            Two b[4][2];
 #pragma unroll
-            for (int j = 0; j < NJ; ++j) {
-                const Two a[4] = {two_of(S[j][0]), two_of(S[j][2]), two_of(S[j][1]), two_of(S[j][3])};
-                const float* at = rows + dc_row_place(g, r0 + 8 * j) + t2;
-                Two b[4][2];
+            for (int x = 0; x < 4; ++x) two_pair(b[x], at + 8 * x * DP);
+            // (the four sums in turn: a product does not wait for the one before it)
 #pragma unroll
-                for (int x = 0; x < 4; ++x) two_pair(b[x], at + 8 * x * DP);
+            for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].lo, a[1].lo, a[2].lo, a[3].lo, b[x][0].hi, b[x][1].hi);
 #pragma unroll
-                for (int x = 0; x < 4; ++x) {
-                    mma_tf32(part[0][x], a[0].lo, a[1].lo, a[2].lo, a[3].lo, b[x][0].hi, b[x][1].hi);
-                    mma_tf32(part[1][x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].lo, b[x][1].lo);
-                    mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].hi, b[x][1].hi);
-                }
-            }
+            for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].lo, b[x][1].lo);
 #pragma unroll
-            for (int x = 0; x < 4; ++x)
+            for (int x = 0; x < 4; ++x) mma_tf32(acc[x], a[0].hi, a[1].hi, a[2].hi, a[3].hi, b[x][0].hi, b[x][1].hi);
+        }
 #pragma unroll
-                for (int e = 0; e < 4; ++e) acc[x][e] += part[0][x][e] + part[1][x][e];
-            float* mine = red + (warp * DC + g) * DC_RLD + t2;
-#pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                *reinterpret_cast<float2*>(mine + 8 * x) = make_float2(acc[x][0], acc[x][1]);
-                *reinterpret_cast<float2*>(mine + 8 * DC_RLD + 8 * x) = make_float2(acc[x][2], acc[x][3]);
-            }
+        for (int x = 0; x < 4; ++x) {
+            *reinterpret_cast<float2*>(mine + 8 * x) = make_float2(acc[x][0], acc[x][1]);
+            *reinterpret_cast<float2*>(mine + 8 * DC_RLD + 8 * x) = make_float2(acc[x][2], acc[x][3]);
         }
         __syncthreads();
-        {   // the warps' sums in order: U = Y - W S (tokens 0 .. 15 of 32), o's first part (the others)
-            const int c = tid >> 4, t = 2 * (tid & 15);
-            const float* from = red + c * DC_RLD + t;
-            float2 v[HOLD];
+        {   // the warps' sums in order: U = Y - W S (rows 0 .. 15 of 32), o's first part (the others)
+            float v[DC_WARPS][4];
 #pragma unroll
-            for (int w = 0; w < HOLD; ++w) v[w] = *reinterpret_cast<const float2*>(from + w * DC * DC_RLD);
-            float2 sum = v[0];
+            for (int w = 0; w < DC_WARPS; ++w) load4(sum_from + w * DC * DC_RLD, v[w]);
+            float y[4] = {0.f, 0.f, 0.f, 0.f};
+            if (sum_t < DC) load4(buf + Place::Y + sum_c * DC + sum_t, y);
 #pragma unroll
-            for (int w = 1; w < HOLD; ++w) {
-                sum.x += v[w].x;
-                sum.y += v[w].y;
+            for (int e = 0; e < 4; ++e) {
+                const float sum = (v[0][e] + v[1][e]) + (v[2][e] + v[3][e]);
+                y[e] = sum_t < DC ? y[e] - sum : sum;
             }
-            if (t < DC) {
-                const float2 y = *reinterpret_cast<const float2*>(buf + Place::Y + c * DC + t);
-                *reinterpret_cast<float2*>(UT + c * DC_ULD + t) = make_float2(y.x - sum.x, y.y - sum.y);
-            } else {
-                *reinterpret_cast<float2*>(OT + c * DC_ULD + t - DC) = sum;
-            }
+            store4(sum_to, y);
         }
         __syncthreads();
         Two u[2][4];                         // U transposed, tokens 0 .. 7 and 8 .. 15
@@ -376,68 +374,51 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
             two_pair(hi, UT + (g + 8) * DC_ULD + 8 * x + t2);
             u[x][0] = lo[0]; u[x][1] = hi[0]; u[x][2] = lo[1]; u[x][3] = hi[1];
         }
-        const int swap = dc_key_place(g, 0);      // (rows 8 j + g: the tile does not matter)
-        // o of tokens 0 .. 7 (warp 6) and 8 .. 15 (warp 7), ahead of the state's products, which do not wait for it
-        const int t0 = 8 * (warp & 1);
-        float o[4] = {0.f, 0.f, 0.f, 0.f}, o_part[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-        if (warp >= 6) {
-            const float2 lo = *reinterpret_cast<const float2*>(OT + g * DC_ULD + t0 + t2);
-            const float2 hi = *reinterpret_cast<const float2*>(OT + (g + 8) * DC_ULD + t0 + t2);
-            o[0] = lo.x; o[1] = lo.y; o[2] = hi.x; o[3] = hi.y;
 #pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                Two b[2];
-                two_pair(b, buf + Place::P + (t0 + g) * DC + ((8 * x) ^ swap) + t2);
-                mma_tf32(o_part[0], u[x][0].lo, u[x][1].lo, u[x][2].lo, u[x][3].lo, b[0].hi, b[1].hi);
-                mma_tf32(o_part[1], u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, b[0].lo, b[1].lo);
-                mma_tf32(o, u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, b[0].hi, b[1].hi);
-            }
+        for (int j = 0; j < NJ; ++j) {
+            const float2 e = *reinterpret_cast<const float2*>(buf + Place::LAST + r0 + 8 * j + t2);
+            S[j][0] *= e.x; S[j][1] *= e.y; S[j][2] *= e.x; S[j][3] *= e.y;
         }
-        if (warp < HOLD) {
-            Two b[NJ][2][2];
-            float part[2][NJ][4];
+        float o[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-            for (int j = 0; j < NJ; ++j) {
-                const float2 e = *reinterpret_cast<const float2*>(buf + Place::LAST + r0 + 8 * j + t2);
-                S[j][0] *= e.x; S[j][1] *= e.y; S[j][2] *= e.x; S[j][3] *= e.y;
-#pragma unroll
-                for (int k = 0; k < 4; ++k) part[0][j][k] = part[1][j][k] = 0.f;
-#pragma unroll
-                for (int x = 0; x < 2; ++x)
-                    two_pair(b[j][x], buf + Place::KEYS + (r0 + 8 * j + g) * DC + ((8 * x) ^ swap) + t2);
-            }
-#pragma unroll
-            for (int x = 0; x < 2; ++x)
-#pragma unroll
-                for (int j = 0; j < NJ; ++j) {
-                    const Two(&a)[4] = u[x];
-                    const Two(&k)[2] = b[j][x];
-                    mma_tf32(part[0][j], a[0].lo, a[1].lo, a[2].lo, a[3].lo, k[0].hi, k[1].hi);
-                    mma_tf32(part[1][j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].lo, k[1].lo);
-                    mma_tf32(S[j], a[0].hi, a[1].hi, a[2].hi, a[3].hi, k[0].hi, k[1].hi);
-                }
+        for (int x = 0; x < 2; ++x) {
+            Two k[NJ][2], w[2];
 #pragma unroll
             for (int j = 0; j < NJ; ++j)
-#pragma unroll
-                for (int k = 0; k < 4; ++k) S[j][k] += part[0][j][k] + part[1][j][k];
-        }
-        if (warp >= 6) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int t = i * DC + t0 + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
-                if (t < tokens && c < p.dv)
-                    p.out[((size_t)(row0 + t) * p.H + h) * p.dv + c] = o[e] + (o_part[0][e] + o_part[1][e]);
+                two_pair(k[j], buf + Place::KEYS + (r0 + 8 * j + g) * DC + ((8 * x) ^ swap) + t2);
+            if (warp < 2) {                  // o: its products stand among the state's, which do not wait for them
+                if (x == 0) {
+                    const float2 lo = *reinterpret_cast<const float2*>(OT + g * DC_ULD + t0 + t2);
+                    const float2 hi = *reinterpret_cast<const float2*>(OT + (g + 8) * DC_ULD + t0 + t2);
+                    o[0] = lo.x; o[1] = lo.y; o[2] = hi.x; o[3] = hi.y;
+                }
+                two_pair(w, buf + Place::P + (t0 + g) * DC + ((8 * x) ^ swap) + t2);
+                mma_tf32(o, u[x][0].lo, u[x][1].lo, u[x][2].lo, u[x][3].lo, w[0].hi, w[1].hi);
             }
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) mma_tf32(S[j], u[x][0].lo, u[x][1].lo, u[x][2].lo, u[x][3].lo, k[j][0].hi, k[j][1].hi);
+            if (warp < 2) mma_tf32(o, u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, w[0].lo, w[1].lo);
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) mma_tf32(S[j], u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, k[j][0].lo, k[j][1].lo);
+            if (warp < 2) mma_tf32(o, u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, w[0].hi, w[1].hi);
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) mma_tf32(S[j], u[x][0].hi, u[x][1].hi, u[x][2].hi, u[x][3].hi, k[j][0].hi, k[j][1].hi);
+        }
+        if (warp < 2) {
+            float* to = out + (size_t)i * DC * out_row;
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (i * DC + t0 + t2 + (e & 1) < tokens && col0 + g + 8 * (e >> 1) < p.dv)
+                    to[(e & 1) * out_row + 8 * (e >> 1)] = o[e];
         }
     }
-    if (warp < HOLD)
 #pragma unroll
-        for (int j = 0; j < NJ; ++j)
+    for (int j = 0; j < NJ; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int r = r0 + 8 * j + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
-                if (r < p.d && c < p.dv) st[(size_t)r * p.dv + c] = S[j][e];
-            }
+        for (int e = 0; e < 4; ++e) {
+            const int r = r0 + 8 * j + t2 + (e & 1), c = col0 + g + 8 * (e >> 1);
+            if (r < p.d && c < p.dv) st[(size_t)r * p.dv + c] = S[j][e];
+        }
 }
 
 template <int DP>
@@ -452,7 +433,7 @@ static int launch_delta_chunks(const DeltaChunkArgs& args, int N, int L, cudaStr
     }
     int rc = launch(delta_chunk_prepare_kernel<DP>, dim3(N, a.H), 256, smem1, stream, a);
     if (rc) return rc;
-    size_t smem2 = sizeof(float) * (2 * (DeltaChunk<DP>::Y + DC * DC) + 8 * DC * DC_RLD + 2 * DC * DC_ULD);
+    size_t smem2 = sizeof(float) * (DC_STAGES * (DeltaChunk<DP>::Y + DC * DC) + DC_WARPS * DC * DC_RLD + 2 * DC * DC_ULD);
     const dim3 grid(a.dvp / DC, a.H, L);
     // (as for the scan token by token: the blocks start when their predecessor has ended, and spread over the SMs)
     int sms = 148, dev = 0;
@@ -464,7 +445,7 @@ static int launch_delta_chunks(const DeltaChunkArgs& args, int N, int L, cudaStr
     if (e != cudaSuccess) return (int)e;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
-    cfg.blockDim = dim3(256);
+    cfg.blockDim = dim3(DC_WARPS * 32);
     cfg.dynamicSmemBytes = smem2;
     cfg.stream = stream;
     return (int)cudaLaunchKernelEx(&cfg, delta_chunk_scan_kernel<DP>, a);
