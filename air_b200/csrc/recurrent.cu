@@ -37,6 +37,8 @@ __device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) -
 // x [T, ld] (the first C columns), w [C, taps], state [slots, C, taps - 1] (oldest first), y [T, C].
 // grid (channel blocks, entries, chunks of `chunk` tokens); the thread of a channel in the first chunk of an
 // entry is the only one that reads or writes the channel's state.
+// M: places for the taps (4, or CONV_MAX_TAPS), so that short convolutions carry a short window.
+template <int M>
 __global__ void __launch_bounds__(CONV_THREADS)
 short_conv_silu_kernel(const float* __restrict__ x, int ld, const float* __restrict__ w, float* __restrict__ state,
                        float* __restrict__ y, const int* __restrict__ q_start, const int* __restrict__ slots,
@@ -51,10 +53,9 @@ short_conv_silu_kernel(const float* __restrict__ x, int ld, const float* __restr
     if (t0 >= n && blockIdx.z > 0) return;
     const int t1 = min(n, t0 + chunk);
     const int keep = taps - 1;
-    // Weights and window are held right-aligned in arrays of the largest size, so that every index is a
+    // Weights and window are held right-aligned in arrays of M places, so that every index is a
     // compile-time number (registers): wv[M - 1] is the current token's weight, win[j] the input M - 1 - j tokens
     // before the next one; the places in front of the taps hold zeros.
-    constexpr int M = CONV_MAX_TAPS;
     const int lead = M - 1 - keep;            // unused places in front
     float wv[M], win[M - 1];
     float* st = state + ((size_t)slot * C + c) * keep;
@@ -510,8 +511,8 @@ AIR_API int air_short_conv_silu(const float* x, int ld, const float* w, float* s
     if (chunks < 1) chunks = 1;
     if (chunks > 65535) return AIR_ERR_BAD_ARGUMENT;
     dim3 grid((C + air::CONV_THREADS - 1) / air::CONV_THREADS, S, chunks);
-    return air::launch(air::short_conv_silu_kernel, grid, air::CONV_THREADS, 0, stream, x, ld, w, state, y, q_start,
-                       slots, C, taps, chunk, act);
+    auto kernel = taps <= 4 ? air::short_conv_silu_kernel<4> : air::short_conv_silu_kernel<air::CONV_MAX_TAPS>;
+    return air::launch(kernel, grid, air::CONV_THREADS, 0, stream, x, ld, w, state, y, q_start, slots, C, taps, chunk, act);
 }
 
 // kq: float32 workspace [T, G, 2, L * R] and dec: [T, H, 2] (mode 0), [T, H, L * R] (modes 1, 2) or [T, H, L * R + 4] (mode
