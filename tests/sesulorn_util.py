@@ -317,10 +317,10 @@ def plain_greedy(name, prompt, n):
 # float32: sums in another order than the 64-bit oracle.  bfloat16: activations rounded to 8 bits at the inputs of the
 # products and in the cache, through sharp attention and gates; a request's rows must all be within the row limits, and
 # their median within the tighter one.
-FP32_TOL = 1e-4
-BF16_MAX_TOL = 0.15
-BF16_MEAN_TOL = 6e-2
-BF16_MEDIAN_TOL = 1e-2
+FP32_TOL = 2e-5
+BF16_MAX_TOL = 0.1
+BF16_MEAN_TOL = 3e-2
+BF16_MEDIAN_TOL = 8e-3
 
 
 def check(got, name, streams, dtype):
