@@ -14,7 +14,7 @@
 // 64 / min(P, 64) boxes of min(P, 64) rows, each found through the block table.
 // Every wait on an mbarrier is bounded (tma.cuh); on giving up the block flags *status = 5.
 //
-// With `bias` a score gets the head's number for its key's distance (DistanceBias); tiles that lie farther back than the
+// With BIAS a score gets the head's number for its key's distance (DistanceBias); tiles that lie farther back than the
 // table reaches take its last entry from a register.
 //
 // With `fresh.qkv` the kernel also does what qkv_rope_store does for its token (elementwise.cu): it adds up
@@ -46,7 +46,7 @@ struct FreshQkv {
     __nv_bfloat16* cache;    // where k and v are written (nullptr: another run has written them)
 };
 
-template <int D>
+template <int D, bool BIAS>
 __global__ void __launch_bounds__(DT_THREADS)
 decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const FreshQkv fresh,
                             const __nv_bfloat16* __restrict__ q,
@@ -259,7 +259,7 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const
         // the bias' rows of this lane's two heads, and their last entries
         const float *bias0 = nullptr, *bias1 = nullptr;
         float far0 = 0.f, far1 = 0.f;
-        if (bias.table) {
+        if constexpr (BIAS) {
             bias0 = bias.table + (size_t)(kvh * G + min(r0, G - 1)) * bias.n;
             bias1 = bias.table + (size_t)(kvh * G + min(r1, G - 1)) * bias.n;
             far0 = bias0[bias.n - 1] * 1.4426950408889634f;
@@ -301,20 +301,22 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const
                 }
                 float tm0 = -INFINITY, tm1 = -INFINITY;
                 float add[2][4];
+                if constexpr (BIAS) {
 #pragma unroll
-                for (int j = 0; j < 2; ++j) {
-                    add[j][0] = add[j][1] = far0;
-                    add[j][2] = add[j][3] = far1;
-                }
-                if (bias.table && pos - (kbase + 15) < bias.n - 1) {
+                    for (int j = 0; j < 2; ++j) {
+                        add[j][0] = add[j][1] = far0;
+                        add[j][2] = add[j][3] = far1;
+                    }
+                    if (pos - (kbase + 15) < bias.n - 1) {
 #pragma unroll
-                    for (int j = 0; j < 2; ++j)
+                        for (int j = 0; j < 2; ++j)
 #pragma unroll
-                        for (int e = 0; e < 2; ++e) {
-                            const int back = max(0, min(pos - (kbase + 8 * j + 2 * tq + e), bias.n - 1));
-                            add[j][e] = bias0[back] * 1.4426950408889634f;
-                            add[j][2 + e] = bias1[back] * 1.4426950408889634f;
-                        }
+                            for (int e = 0; e < 2; ++e) {
+                                const int back = max(0, min(pos - (kbase + 8 * j + 2 * tq + e), bias.n - 1));
+                                add[j][e] = bias0[back] * 1.4426950408889634f;
+                                add[j][2 + e] = bias1[back] * 1.4426950408889634f;
+                            }
+                    }
                 }
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
@@ -323,11 +325,15 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const
                         const int key = kbase + 8 * j + 2 * tq + e;
                         const bool ok = key >= lo && key <= pos;
                         if (cap_log2 > 0.f) {
-                            s[j][e] = ok ? cap_log2 * tanhf(s[j][e] * cap_pre) + add[j][e] : -INFINITY;
-                            s[j][2 + e] = ok ? cap_log2 * tanhf(s[j][2 + e] * cap_pre) + add[j][2 + e] : -INFINITY;
+                            s[j][e] = ok ? cap_log2 * tanhf(s[j][e] * cap_pre) : -INFINITY;
+                            s[j][2 + e] = ok ? cap_log2 * tanhf(s[j][2 + e] * cap_pre) : -INFINITY;
                         } else {
-                            s[j][e] = ok ? fmaf(s[j][e], scale_log2, add[j][e]) : -INFINITY;
-                            s[j][2 + e] = ok ? fmaf(s[j][2 + e], scale_log2, add[j][2 + e]) : -INFINITY;
+                            s[j][e] = ok ? s[j][e] * scale_log2 : -INFINITY;
+                            s[j][2 + e] = ok ? s[j][2 + e] * scale_log2 : -INFINITY;
+                        }
+                        if constexpr (BIAS) {
+                            s[j][e] += add[j][e];
+                            s[j][2 + e] += add[j][2 + e];
                         }
                         tm0 = fmaxf(tm0, s[j][e]);
                         tm1 = fmaxf(tm1, s[j][2 + e]);
@@ -436,7 +442,7 @@ int launch_decode_tma(const CUtensorMap& map, const FreshQkv& fresh, const void*
     const size_t ring = (size_t)DT_STAGES * 2 * (D / 64) * DT_TILE * 128;
     const size_t merge = (size_t)(DT_CONSUMERS * 16 * D + 2 * DT_CONSUMERS * 16) * sizeof(float);
     const size_t smem = 1024 + (ring > merge ? ring : merge) + 128 + (fresh.qkv ? (size_t)18 * D * 2 : 0);
-    auto kernel = decode_attention_tma_kernel<D>;
+    auto kernel = bias.table ? decode_attention_tma_kernel<D, true> : decode_attention_tma_kernel<D, false>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     return launch(kernel, dim3(splits, K * head_blocks, T), DT_THREADS, smem, stream, map, fresh, (const __nv_bfloat16*)q,
